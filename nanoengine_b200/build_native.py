@@ -32,14 +32,20 @@ REPO = PKG.parent
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 CXX = os.environ.get("CXX", "g++")
 GENCODE = ["-gencode", "arch=compute_100a,code=sm_100a"]
-NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
+NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
               "-Xptxas", "-v", "-DNDEBUG", "-rdc=true"] + GENCODE
+# translation units whose 32-bit results are held to 32-bit accuracy (gates of a recurrence, tanh): no approximate functions there
+PRECISE = {"delta", "residual", "gemm_simt"}
+
+
+def nvcc_flags(stem: str):
+    return NVCC_FLAGS + ([] if stem in PRECISE else ["--use_fast_math"])
 
 
 def _stamp(paths, extra=""):
     h = hashlib.sha256(extra.encode())
     for p in sorted(paths):
-        h.update(str(p).encode())
+        h.update(Path(p).name.encode())       # not the full path: a copied tree keeps its build
         h.update(Path(p).read_bytes())
     return h.hexdigest()
 
@@ -87,30 +93,36 @@ def build_core(force=False) -> Path:
     return target
 
 
-def build_kernels(force=False, debug_bounds=False) -> Path:
+def build_kernels(force=False, debug_bounds=False, only=None, tag="") -> Path:
     """`debug_bounds`: the same sources with -DNE_DEBUG_BOUNDS into libne_kernels_dbg.so (kernels compare the cache rows, pages,
-    state slots and expert ids they take from tables with the bounds the worker registers; loaded when NE_DEBUG_BOUNDS=1)."""
-    target = OUT / ("libne_kernels_dbg.so" if debug_bounds else "libne_kernels.so")
+    state slots and expert ids they take from tables with the bounds the worker registers; loaded when NE_DEBUG_BOUNDS=1).
+    `only` (stems of .cu files) with `tag`: just those sources into libne_kernels_<tag>.so, for a process that serves one model
+    from a tree that has not been built; the objects are shared with the full build."""
+    target = OUT / ("libne_kernels_dbg.so" if debug_bounds else f"libne_kernels_{tag}.so" if only else "libne_kernels.so")
     OBJ = OUT / ("obj_dbg" if debug_bounds else "obj")
-    NVCC_FLAGS = globals()["NVCC_FLAGS"] + (["-DNE_DEBUG_BOUNDS"] if debug_bounds else [])
+    extra = ["-DNE_DEBUG_BOUNDS"] if debug_bounds else []
     kdir = CSRC / "kernels"
     cus = sorted(kdir.glob("*.cu")) + sorted((CSRC / "comm").glob("*.cu"))
+    if only:
+        missing = set(only) - {c.stem for c in cus}
+        if missing:
+            raise ValueError(f"no such kernel sources: {sorted(missing)}")
+        cus = [c for c in cus if c.stem in set(only)]
     hdrs = sorted(kdir.glob("*.cuh")) + sorted(kdir.glob("*.h")) + sorted((CSRC / "comm").glob("*.cuh")) + sorted((CSRC / "comm").glob("*.h"))
     if not cus:
         return target
     OBJ.mkdir(parents=True, exist_ok=True)
-    hstamp = _stamp(hdrs, " ".join(NVCC_FLAGS))
     objs, jobs = [], []
     for cu in cus:
         obj = OBJ / (cu.stem + ".o")
         objs.append(obj)
-        st = _stamp([cu], hstamp)
+        st = _stamp([cu], _stamp(hdrs, " ".join(nvcc_flags(cu.stem) + extra)))
         if _needs(obj, st, force):
             jobs.append((cu, obj, st))
 
     def one(job):
         cu, obj, st = job
-        _run([NVCC, *NVCC_FLAGS, f"-I{kdir}", f"-I{CSRC / 'comm'}", "-c", str(cu), "-o", str(obj)],
+        _run([NVCC, *nvcc_flags(cu.stem), *extra, f"-I{kdir}", f"-I{CSRC / 'comm'}", "-c", str(cu), "-o", str(obj)],
              log=OBJ / (cu.stem + ".ptxas.log"))
         _mark(obj, st)
 
@@ -170,6 +182,19 @@ def build_sanitized(kind: str = "address,undefined", force=False) -> dict:
         compile_(sorted(gdir.glob("*.cpp")), gateway)
         _mark(gateway, st)
     return {"selftest": selftest, "gateway": gateway}
+
+
+def build_for(architecture: str) -> Path:
+    """The C++ core and the kernels one architecture needs, for a process that serves nothing else.  Returns the kernel library to
+    load: the full one when it is there, the architecture's own otherwise."""
+    from .models.registry import kernel_sources
+    OUT.mkdir(parents=True, exist_ok=True)
+    build_core()
+    full = OUT / "libne_kernels.so"
+    only = kernel_sources(architecture)
+    if only is None or full.exists():
+        return build_kernels()
+    return build_kernels(only=only, tag=architecture.lower())
 
 
 def build_all(force=False):

@@ -200,6 +200,11 @@ class Config:
                 raise ValueError("NVFP4 experts need hidden and moe_intermediate sizes in multiples of 256")
         if self.max_model_len is None:
             self.max_model_len = mc.max_position_embeddings
+        if mc.layer_specs:
+            if self.attention_tp != 1 or self.pp != 1:
+                raise ValueError("models with listed layers run with attention_tp = pp = 1")
+            # the design has no context limit: the rotary tables follow the engine's
+            mc.max_position_embeddings = max(mc.max_position_embeddings, self.max_model_len)
         if self.max_num_seqs < 1 or self.max_num_batched_tokens < 1:
             raise ValueError("max_num_seqs and max_num_batched_tokens must be positive")
         if not (0.0 < self.gpu_memory_utilization <= 1.0):

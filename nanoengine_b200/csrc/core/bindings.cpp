@@ -279,6 +279,10 @@ PYBIND11_MODULE(_core, m) {
       .def("add_migration", &Scheduler::add_migration)
       .def("add_request_bytes", [](Scheduler& s, const std::string& b) { return s.add_request_bytes(b); })
       .def("schedule", [](Scheduler& s) { return s.schedule(); })
+      .def("schedule_fed", [](Scheduler& s, const std::vector<std::pair<uint64_t, std::vector<int32_t>>>& e) { return s.schedule_fed(e); },
+           py::arg("entries"))
+      .def("release_fed", &Scheduler::release_fed, py::arg("seq_ids"))
+      .def("num_fed", &Scheduler::num_fed)
       .def("serialize_run_batches", [](Scheduler& s) {
         py::list out; for (auto& b : s.serialize_run_batches()) out.append(py::bytes(b)); return out; })
       .def("serialize_migrate_batches", [](Scheduler& s) {

@@ -147,7 +147,7 @@ class Scheduler {
         placed = try_swap_in(s, batches);
       } else {
         for (int d : route_candidates(s)) {
-          if ((int)(running_[d].size() + prefilling_[d].size()) >= cfg_.max_num_seqs) continue;
+          if ((int)(running_[d].size() + prefilling_[d].size() + fed_.size()) >= cfg_.max_num_seqs) continue;
           if (budget[d] <= 0) continue;
           int remaining_hint = (int)s.tokens.size();
           if (!cfg_.enable_chunked_prefill && remaining_hint > budget[d] && budget[d] < cfg_.max_num_batched_tokens) continue;
@@ -246,6 +246,80 @@ class Scheduler {
     }
   }
 
+  // ---- fed steps -------------------------------------------------------------------------
+  // A step whose sequences and tokens the caller names (scoring, replaying a recorded schedule) instead of the queues: every entry
+  // brings the next tokens of its sequence, prompt portions and single tokens in one batch.  A sequence is admitted at its first
+  // entry - pages as its tokens arrive, a state slot for the plans that keep one - and holds them until `release_fed`.  Nothing is
+  // sampled.  A step that does not fit (pages, slots, max_num_seqs, max_model_len) throws and changes nothing.
+  const ScheduleResult& schedule_fed(const std::vector<std::pair<uint64_t, std::vector<int32_t>>>& entries) {
+    if (cfg_.attention_dp != 1 || spec() > 0) throw std::invalid_argument("fed steps run with attention_dp = 1 and without speculative decoding");
+    if (entries.empty()) throw std::invalid_argument("a fed step needs at least one entry");
+    const int d = 0;
+    std::set<uint64_t> ids;
+    int need = 0, fresh = 0;
+    for (auto& e : entries) {
+      if (e.second.empty()) throw std::invalid_argument("a fed entry needs at least one token");
+      if (!ids.insert(e.first).second) throw std::invalid_argument("a sequence may appear once in a fed step");
+      auto it = seqs_.find(e.first);
+      if (it != seqs_.end() && !fed_.count(e.first)) throw std::invalid_argument("the sequence belongs to the queues");
+      const int have = it == seqs_.end() ? 0 : (int)it->second->tokens.size();
+      const int held = it == seqs_.end() ? 0 : (int)it->second->block_table.size();
+      if (have + (int)e.second.size() > cfg_.max_model_len) throw std::invalid_argument("a fed sequence exceeds max_model_len");
+      need += std::max(0, blocks_for(have + (int)e.second.size()) - held);
+      if (it == seqs_.end()) fresh++;
+    }
+    if ((int)(fed_.size() + running_[d].size() + prefilling_[d].size()) + fresh > cfg_.max_num_seqs) throw std::runtime_error("fed step: no sequence left (max_num_seqs)");
+    if (!pools_[d].can_allocate(need)) throw std::runtime_error("fed step: no cache pages left");
+    if (cfg_.needs_state_slots() && state_slots_[d].num_free() < fresh) throw std::runtime_error("fed step: no state slots left");
+    step_++;
+    last_ = ScheduleResult{};
+    last_.step = step_; last_.has_work = true;
+    Batch b;
+    b.dp_idx = d; b.step = step_; b.block_offsets.push_back(0);
+    for (auto& e : entries) {
+      auto it = seqs_.find(e.first);
+      if (it == seqs_.end()) {
+        auto n = std::make_unique<Sequence>();
+        n->seq_id = e.first; n->dp_idx = d; n->status = RUNNING; n->t_arrival = now_seconds();
+        it = seqs_.emplace(e.first, std::move(n)).first;
+        fed_.insert(e.first);
+        if (!acquire_slots(*it->second, d)) throw std::runtime_error("fed step: no slots left");
+      }
+      Sequence& s = *it->second;
+      const int start = (int)s.tokens.size(), n = (int)e.second.size();
+      s.tokens.insert(s.tokens.end(), e.second.begin(), e.second.end());
+      s.prompt_len = (int)s.tokens.size();
+      std::vector<int32_t> pages;
+      const int more = blocks_for(start + n) - (int)s.block_table.size();
+      if (more > 0) { pools_[d].allocate(more, &pages); s.block_table.insert(s.block_table.end(), pages.begin(), pages.end()); }
+      b.seq_ids.push_back(e.first);
+      for (int i = 0; i < n; i++) { b.input_ids.push_back(e.second[i]); b.positions.push_back(start + i); }
+      b.q_lens.push_back(n); b.seq_lens.push_back(start + n);
+      push_common(b, s);
+      b.sample_mask.push_back(0);
+      if (n > 1) b.is_prefill = true;
+      s.num_computed = start + n; s.last_scheduled_step = step_;
+      last_.num_tokens += n; last_.num_seqs++;
+    }
+    last_.is_prefill = b.is_prefill;
+    last_.batches.push_back(std::move(b));
+    return last_;
+  }
+
+  // Give back what fed sequences hold; returns how many there were.
+  int release_fed(const std::vector<uint64_t>& ids) {
+    int n = 0;
+    for (uint64_t id : ids) {
+      if (!fed_.erase(id)) continue;
+      auto it = seqs_.find(id);
+      release_resources(*it->second);
+      seqs_.erase(it);
+      n++;
+    }
+    return n;
+  }
+  int num_fed() const { return (int)fed_.size(); }
+
   // ---- post-processing -------------------------------------------------------------------
   std::vector<StepOut> postprocess(const std::vector<RunResult>& results, double latency_ms = -1.0) {
     std::vector<StepOut> outs;
@@ -314,7 +388,7 @@ class Scheduler {
     Sequence& s = *it->second;
     remove_from_deque(waiting_, id); remove_from_deque(waiting_migration_, id);
     if (s.dp_idx >= 0) { remove_from(running_[s.dp_idx], id); remove_from(prefilling_[s.dp_idx], id); }
-    to_be_migrated_.erase(id);
+    to_be_migrated_.erase(id); fed_.erase(id);
     release_resources(s);
     itl_.erase(id); affinity_wait_.erase(id);
     metrics_.on_abort();
@@ -640,7 +714,7 @@ class Scheduler {
   std::unordered_map<uint64_t, std::unique_ptr<Sequence>> seqs_;
   std::deque<uint64_t> waiting_, waiting_migration_;
   std::vector<std::vector<uint64_t>> running_, prefilling_;
-  std::set<uint64_t> to_be_migrated_, exported_;
+  std::set<uint64_t> to_be_migrated_, exported_, fed_;
   std::vector<BlockPool> pools_, host_pools_;
   std::vector<SlotPool> state_slots_, handoff_slots_, hisparse_slots_;
   std::unordered_map<uint64_t, int> affinity_;

@@ -35,6 +35,13 @@ class LLM:
     def step(self):
         return self.engine.step()
 
+    def feed(self, entries, want=()):
+        """Run given tokens instead of sampling, see LLMEngine.feed."""
+        return self.engine.feed(entries, want)
+
+    def end_feed(self, seq_ids) -> int:
+        return self.engine.end_feed(seq_ids)
+
     def is_finished(self) -> bool:
         return self.engine.is_finished()
 

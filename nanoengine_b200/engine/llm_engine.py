@@ -203,6 +203,24 @@ class LLMEngine:
             logger.info(self.scheduler.status_line(self.config.mode))
         return step_outs
 
+    def feed(self, entries, want=()):
+        """One step of given tokens: `entries` is a list of (seq_id, next tokens), run together as one batch from what earlier
+        steps left in the cache and the state slots; a sequence is admitted at its first entry and may skip steps.  `want` lists,
+        per entry, the places among its tokens whose logits are returned (fp32 [n, vocab], in entry order; None when there are
+        none).  Nothing is sampled.  `end_feed` gives back what finished sequences hold."""
+        self.scheduler.schedule_fed([(int(i), [int(t) for t in toks]) for i, toks in entries])
+        rows, base = [], 0
+        for k, (_, toks) in enumerate(entries):
+            for p in (want[k] if k < len(want) else ()):
+                if not 0 <= p < len(toks):
+                    raise ValueError(f"entry {k}: wanted place {p} outside its {len(toks)} tokens")
+                rows.append(base + p)
+            base += len(toks)
+        return self.executor.collective_rpc("run_logits", self.scheduler.serialize_run_batches()[0], rows)[0]
+
+    def end_feed(self, seq_ids) -> int:
+        return self.scheduler.release_fed([int(i) for i in seq_ids])
+
     def _run_static_pp_prefill_pipeline(self, res) -> List[bytes]:
         """Split each DP rank's prefill batch into `pp` micro-batches and keep them all in flight: every worker receives
         the micro-batches in order, so stage s works on micro-batch m while stage s+1 works on m-1."""

@@ -102,6 +102,10 @@ class ModelConfig:
     o_lora_rank: int = 0
     o_groups: int = 0
     num_hash_layers: int = 0                 # the first this-many MoE layers pick experts from a token-id table
+    # Tuvutar: every layer is listed with its own mixer ("latent_attention" | "delta"), the mixer's sizes and its feed-forward; the
+    # fields above describe one such layer only in the form `layer_config` derives for it
+    layer_specs: Optional[List[Dict[str, Any]]] = None
+    attn_scale: float = 0.0                  # > 0: softmax scale of the latent-attention layer (0: from the head dim)
     # MTP
     num_nextn_predict_layers: int = 0
     # quantisation of linear / expert weights: None (use dtype) or "fp8" (e4m3, 128x128 block scales)
@@ -118,7 +122,7 @@ class ModelConfig:
     def is_mla(self) -> bool:
         return self.architecture in ("DeepseekV2ForCausalLM", "DeepseekV3ForCausalLM", "DeepseekV32ForCausalLM",
                                      "GlmMoeDsaForCausalLM", "KimiK2ForCausalLM", "Glm5NextForConditionalGeneration",
-                                     "KimiK3ForConditionalGeneration")
+                                     "KimiK3ForConditionalGeneration", "Tuvutar")
 
     @property
     def is_dsv4(self) -> bool:
@@ -130,7 +134,24 @@ class ModelConfig:
 
     @property
     def is_hybrid_gdn(self) -> bool:
+        if self.layer_specs:
+            return any(s["type"] == "delta" for s in self.layer_specs)
         return self.linear_num_value_heads > 0
+
+    def layer_config(self, layer_idx: int) -> "ModelConfig":
+        """The sizes of one listed layer under the names the attention / delta-net / MLP modules read."""
+        import dataclasses
+        spec = self.layer_specs[layer_idx]
+        m, mlp = spec["mixer"], spec["mlp"]
+        over: Dict[str, Any] = {"layer_specs": None, "intermediate_size": int(mlp["ff"]) if mlp else 0}
+        if spec["type"] == "latent_attention":
+            over.update(num_attention_heads=int(m["heads"]), num_key_value_heads=int(m["heads"]), qk_nope_head_dim=int(m["dim"]),
+                        qk_rope_head_dim=int(m["rot_dim"]), v_head_dim=int(m["vdim"]), kv_lora_rank=int(m["kv_rank"]), q_lora_rank=None,
+                        attn_scale=float(m["scale"]), rope_theta=float(m["rot"]["base"]), rope_scaling=_yarn_of(m["rot"].get("scaling")))
+        else:
+            over.update(linear_num_key_heads=int(m["kv_heads"]), linear_num_value_heads=int(m["heads"]), linear_key_head_dim=int(m["dim"]),
+                        linear_value_head_dim=int(m["vdim"]), linear_conv_kernel_dim=int(m["conv"]))
+        return dataclasses.replace(self, **over)
 
     def attn_layer_type(self, layer_idx: int) -> str:
         """"sliding_attention" or "full_attention" for the families that mix window and global layers."""
@@ -147,7 +168,10 @@ class ModelConfig:
 
     def kv_source_layer(self, layer_idx: int) -> int:
         """The layer whose K / V cache layer `layer_idx` reads: itself, or for a KV-sharing layer the last earlier layer of the
-        same attention type that keeps its own."""
+        same attention type that keeps its own.  Listed layers name it themselves."""
+        if self.layer_specs:
+            src = self.layer_specs[layer_idx]["mixer"].get("kv_from")
+            return layer_idx if src is None else int(src)
         first = self.first_kv_shared_layer
         if layer_idx < first:
             return layer_idx
@@ -158,6 +182,8 @@ class ModelConfig:
         raise ValueError(f"no earlier {kind} layer to share keys and values with")
 
     def layer_type(self, layer_idx: int) -> str:
+        if self.layer_specs:
+            return "linear_attention" if self.layer_specs[layer_idx]["type"] == "delta" else "full_attention"
         if not self.is_hybrid_gdn:
             return "full_attention"
         if self.layer_types and layer_idx < len(self.layer_types):
@@ -238,6 +264,8 @@ class ModelConfig:
             if q.get("scale_fmt"):
                 d["scale_fmt"] = q["scale_fmt"]
         arch = d.get("architecture", "")
+        if arch == "Tuvutar" and "layers" in d:
+            d = _tuvutar_fields(d)
         la = d.pop("linear_attn_config", None)
         if isinstance(la, dict):                          # Kimi delta attention block of GLM5-next / Kimi-K3
             d["linear_kind"] = "kda"
@@ -342,6 +370,47 @@ class ModelConfig:
         d.pop("weight_block_size")
         d.pop("scale_fmt", None)
         return d
+
+
+def _yarn_of(sc: Optional[Dict[str, Any]]) -> Optional[Dict[str, Any]]:
+    """A {factor, original, fast, slow} block in the form `ops.reference.rope_inv_freq` reads; cos and sin carry 0.1 ln(factor) + 1."""
+    if not sc:
+        return None
+    import math
+    return {"type": "yarn", "factor": float(sc["factor"]), "original_max_position_embeddings": sc["original"], "beta_fast": float(sc["fast"]),
+            "beta_slow": float(sc["slow"]), "attention_factor": 0.1 * math.log(float(sc["factor"])) + 1.0}
+
+
+def _tuvutar_fields(d: Dict[str, Any]) -> Dict[str, Any]:
+    """config.json of a Tuvutar model ({architecture, layers, norm, vocab, width}) as ModelConfig fields.  The design has no
+    context limit of its own; the default only sizes the rotary table (Config raises it to max_model_len)."""
+    for i, s in enumerate(d["layers"]):
+        m = s["mixer"]
+        if s["type"] == "latent_attention":
+            if int(m["rot"]["dims"]) != int(m["rot_dim"]) or int(m["rot_dim"]) % 2:
+                raise ValueError(f"layer {i}: the rotated part is the whole (even) rot_dim")
+            src = m.get("kv_from")
+            if src is not None:
+                if not (0 <= int(src) < i) or d["layers"][int(src)]["type"] != "latent_attention" or d["layers"][int(src)]["mixer"].get("kv_from") is not None:
+                    raise ValueError(f"layer {i}: kv_from must name an earlier latent-attention layer that keeps its own rows")
+                o = d["layers"][int(src)]["mixer"]
+                if any(o[k] != m[k] for k in ("kv_rank", "rot_dim", "rot")):
+                    raise ValueError(f"layer {i}: kv_rank, rot_dim and rotation must equal those of layer {src}")
+        elif s["type"] == "delta":
+            if int(m["heads"]) % int(m["kv_heads"]):
+                raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {s['type']!r}")
+        if s.get("mlp") is not None and s["mlp"]["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {s['mlp']['kind']!r}")
+    out = {"architecture": d["architecture"], "vocab_size": int(d["vocab"]), "hidden_size": int(d["width"]), "num_hidden_layers": len(d["layers"]),
+           "rms_norm_eps": float(d["norm"]["eps"]), "norm_unit_offset": True, "hidden_activation": "gelu_pytorch_tanh", "q_lora_rank": None,
+           "n_routed_experts": 0, "n_shared_experts": 0, "max_position_embeddings": 131072, "tie_word_embeddings": False,
+           "layer_specs": [{"type": s["type"], "mixer": dict(s["mixer"]), "mlp": dict(s["mlp"]) if s.get("mlp") is not None else None} for s in d["layers"]]}
+    for k in ("eos_token_id", "bos_token_id", "max_position_embeddings"):
+        if d.get(k) is not None:
+            out[k] = d[k]
+    return out
 
 
 def tiny_deepseek_v3(**over) -> ModelConfig:
@@ -476,3 +545,47 @@ def tiny_gemma4(**over) -> ModelConfig:
                                          "full_attention": {"rope_theta": 1000000.0, "rope_type": "proportional", "partial_rotary_factor": 0.25}})
     base.update(over)
     return ModelConfig(**base)
+
+
+def _latent_spec(heads, dim, rot_dim, vdim, kv_rank, ff, kv_from=None, base=10000.0, scaling=None):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5,
+         "rot": {"base": base, "dims": rot_dim, "scaling": scaling}}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def _delta_spec(heads, kv_heads, dim, vdim, conv, ff=0):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def tiny_tuvutar(**over) -> ModelConfig:
+    """CPU-sized Tuvutar shape: latent attention, two delta layers (grouped key heads, one with a feed-forward), a latent layer that
+    reads the first one's rows."""
+    yarn = {"factor": 4.0, "original": 64, "fast": 32.0, "slow": 1.0}
+    c = ModelConfig.from_dict({"architecture": "Tuvutar", "vocab": 512, "width": 128, "norm": {"eps": 1e-6}, "layers": [
+        _latent_spec(4, 16, 8, 24, 48, 192, scaling=yarn), _delta_spec(4, 2, 32, 16, 4), _delta_spec(4, 4, 16, 32, 3, ff=96),
+        _latent_spec(2, 32, 8, 16, 48, 128, kv_from=0, scaling=yarn)]})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+def tuvutar_7b(**over) -> ModelConfig:
+    """A Tuvutar shape of a real model's layer sizes (7B class): width 4096, one latent-attention layer (32 heads, 128 + 64 / 128, rank
+    512) after every three delta layers (32 heads over 16 key heads, 128 x 128 states), every second latent layer reading its
+    predecessor's rows."""
+    layers = []
+    for i in range(8):
+        src = len(layers) - 4 if i % 2 else None
+        layers.append(_latent_spec(32, 128, 64, 128, 512, 12288, kv_from=src, base=1e6,
+                                   scaling={"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}))
+        layers += [_delta_spec(32, 16, 128, 128, 4, ff=12288 if j == 2 else 0) for j in range(3)]
+    c = ModelConfig.from_dict({"architecture": "Tuvutar", "vocab": 131072, "width": 4096, "norm": {"eps": 1e-6}, "layers": layers})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+PRESETS["tiny-tuvutar"], PRESETS["tuvutar-7b"] = tiny_tuvutar, tuvutar_7b

@@ -29,9 +29,14 @@ from .layers import QLinear, RMSNorm, RoutedExperts, SwiGLUMLP
 class MLAAttention(nn.Module):
     """`cache_idx`: which page family entry the layer uses (its rank among the full-attention layers in the hybrid families;
     the layer index otherwise).  With `cfg.mla_output_gate` the heads' output is multiplied by sigmoid(g_proj(x)) before
-    o_proj (reference models/kimi_k3/kimi_k3.py:73-100)."""
+    o_proj (reference models/kimi_k3/kimi_k3.py:73-100).
 
-    def __init__(self, cfg: ModelConfig, layer_idx: int, dtype, device, cache_idx: Optional[int] = None):
+    `merged_kv`: the form of the families that list their layers - no query bottleneck, [q | kv_a] is one GEMM (the query alone
+    when the layer reads another layer's rows, `reads_only`), and one kernel does the whole rotary / norm / cache-write step.
+    The softmax scale is `cfg.attn_scale` where the config gives one."""
+
+    def __init__(self, cfg: ModelConfig, layer_idx: int, dtype, device, cache_idx: Optional[int] = None, merged_kv: bool = False,
+                 reads_only: bool = False):
         super().__init__()
         self.cfg, self.layer_idx = cfg, layer_idx
         self.cache_idx = layer_idx if cache_idx is None else cache_idx
@@ -39,7 +44,10 @@ class MLAAttention(nn.Module):
         self.H, self.R, self.rope, self.nope, self.v = H, R, rope, nope, v
         self.q_lora = cfg.q_lora_rank
         q = cfg.quant
-        if self.q_lora:
+        self.merged, self.reads_only = merged_kv, reads_only
+        if merged_kv:
+            self.q_kv_proj = QLinear(cfg.hidden_size, H * (nope + rope) + (0 if reads_only else R + rope), dtype, device, q)
+        elif self.q_lora:
             # fused [q_a_proj ; kv_a_proj_with_mqa]
             self.qkv_a_proj = QLinear(cfg.hidden_size, self.q_lora + R + rope, dtype, device, q)
             self.q_a_layernorm = RMSNorm(self.q_lora, cfg.rms_norm_eps, dtype, device, quant_out=(q == "fp8"))
@@ -47,7 +55,7 @@ class MLAAttention(nn.Module):
         else:
             self.q_proj = QLinear(cfg.hidden_size, H * (nope + rope), dtype, device, q)
             self.kv_a_proj_with_mqa = QLinear(cfg.hidden_size, R + rope, dtype, device, q)
-        self.kv_a_layernorm = RMSNorm(R, cfg.rms_norm_eps, dtype, device)
+        self.kv_a_layernorm = None if reads_only else RMSNorm(R, cfg.rms_norm_eps, dtype, device)
         # absorbed halves of kv_b_proj
         self.kc = nn.Parameter(torch.empty(H, nope, R, dtype=dtype, device=device), requires_grad=False)   # W_UK
         self.vc = nn.Parameter(torch.empty(H, R, v, dtype=dtype, device=device), requires_grad=False)      # W_UV^T
@@ -55,9 +63,9 @@ class MLAAttention(nn.Module):
         self.kc_t: Optional[torch.Tensor] = None
         self.vc_t: Optional[torch.Tensor] = None
         self.o_proj = QLinear(H * v, cfg.hidden_size, dtype, device, q)
-        self.scale = (nope + rope) ** -0.5
+        self.scale = cfg.attn_scale if cfg.attn_scale > 0 else (nope + rope) ** -0.5
         sc = cfg.rope_scaling
-        if sc and sc.get("type", sc.get("rope_type")) == "yarn" and sc.get("mscale_all_dim"):
+        if cfg.attn_scale <= 0 and sc and sc.get("type", sc.get("rope_type")) == "yarn" and sc.get("mscale_all_dim"):
             m = ref.yarn_mscale(float(sc["factor"]), float(sc["mscale_all_dim"]))
             self.scale *= m * m
         self.indexer = None
@@ -73,6 +81,14 @@ class MLAAttention(nn.Module):
         w = w.view(self.H, self.nope + self.v, self.R)
         self.kc.copy_(w[:, : self.nope].to(self.kc.dtype))
         self.vc.copy_(w[:, self.nope:].transpose(1, 2).to(self.vc.dtype))
+        self.refresh_absorbed()
+
+    def set_uk_uv(self, uk: Optional[torch.Tensor] = None, uv: Optional[torch.Tensor] = None):
+        """The two halves stored apart: W_uk [H * nope, R], W_uv [H * v, R], both head by head."""
+        if uk is not None:
+            self.kc.copy_(uk.view(self.H, self.nope, self.R).to(self.kc.dtype))
+        if uv is not None:
+            self.vc.copy_(uv.view(self.H, self.v, self.R).transpose(1, 2).to(self.vc.dtype))
         self.refresh_absorbed()
 
     def refresh_absorbed(self):
@@ -91,6 +107,8 @@ class MLAAttention(nn.Module):
     def forward(self, x: torch.Tensor, positions: torch.Tensor, ctx: ForwardContext, rope_cache: torch.Tensor) -> torch.Tensor:
         T = x.shape[0]
         H, R, rope, nope = self.H, self.R, self.rope, self.nope
+        if self.merged:
+            return self._forward_merged(x, positions, ctx, rope_cache)
         if self.q_lora:
             a = self.qkv_a_proj(x)
             q_c = self.q_a_layernorm(a[:, : self.q_lora])
@@ -121,6 +139,22 @@ class MLAAttention(nn.Module):
         return self.o_proj(o)
 
 
+    def _forward_merged(self, x, positions, ctx: ForwardContext, rope_cache):
+        T, H, R, rope, nope = x.shape[0], self.H, self.R, self.rope, self.nope
+        qw = H * (nope + rope)
+        a = self.q_kv_proj(x)
+        q, kv_a = a[:, :qw].unflatten(-1, (H, nope + rope)), None if self.reads_only else a[:, qw:]
+        cache = ctx.kv_caches[self.cache_idx]
+        if (NONABSORBED_PREFILL and ctx.is_prefill and ctx.extras.get("no_prefix") and x.is_cuda and nope == 128 and rope == 64
+                and self.v == 128 and R % 8 == 0 and x.dtype == torch.bfloat16):
+            return self._prefill_nonabsorbed(x, q, kv_a, positions, ctx, rope_cache)
+        nw = None if self.reads_only else self.kv_a_layernorm
+        ops.latent_prepare(q, nope, kv_a, None if nw is None else nw.weight, 0.0 if nw is None else nw.eps, positions, rope_cache, cache,
+                           ctx.slot_mapping, R)
+        q_full = ops.latent_query(q, self.kc, nope, kc_t=self.kc_t)
+        o_lat = ops.mla_attention_paged(q_full, cache, ctx.block_tables, ctx.cu_seqlens_q, ctx.context_lens, self.scale, R)
+        return self.o_proj(ops.bmm_absorb(o_lat, self.vc, wt=self.vc_t).reshape(T, H * self.v))
+
     def _prefill_nonabsorbed(self, x, q, kv_a, positions, ctx: ForwardContext, rope_cache):
         """Prompts without a cached prefix: keys and values are expanded from the latent rows of the same tokens (two GEMMs against
         W_UK / W_UV) and attended in their own 192 / 128-wide geometry, 128 query tokens per tile - about a third of the
@@ -128,10 +162,21 @@ class MLAAttention(nn.Module):
         written just before (decode and later chunks read it).
         Parity: reference models/deepseek_v2/deepseek_v2.py:1792-1816 (non-absorbed ragged prefill)."""
         T, H, R, nope = x.shape[0], self.H, self.R, self.nope
-        ckv = ops.rmsnorm(kv_a[:, :R], self.kv_a_layernorm.weight, self.kv_a_layernorm.eps)
-        ckv = ops.dense(ckv)
-        k_pe = ops.apply_rope(kv_a[:, R:].contiguous().view(T, 1, self.rope), positions, rope_cache, True).view(T, self.rope)
-        ops.apply_rope(q[..., nope:], positions, rope_cache, True, q[..., nope:])           # in place on the strided view
+        if self.merged:
+            # the rows just written to the pages, gathered back: layers that read another layer's rows see the same values
+            cache = ctx.kv_caches[self.cache_idx]
+            norm = self.kv_a_layernorm
+            ops.latent_prepare(q, nope, kv_a, None if norm is None else norm.weight, 0.0 if norm is None else norm.eps, positions, rope_cache,
+                               cache, ctx.slot_mapping, R)
+            rows = ctx.extras.get(("latent_rows", self.cache_idx))
+            if rows is None:
+                rows = ctx.extras[("latent_rows", self.cache_idx)] = ops.latent_gather(cache, ctx.slot_mapping)
+            ckv, k_pe = rows[:, :R], rows[:, R:]
+        else:
+            ckv = ops.rmsnorm(kv_a[:, :R], self.kv_a_layernorm.weight, self.kv_a_layernorm.eps)
+            ckv = ops.dense(ckv)
+            k_pe = ops.apply_rope(kv_a[:, R:].contiguous().view(T, 1, self.rope), positions, rope_cache, True).view(T, self.rope)
+            ops.apply_rope(q[..., nope:], positions, rope_cache, True, q[..., nope:])           # in place on the strided view
         k_nope = ops.linear(ckv, self.kc.view(H * nope, R)).view(T, H, nope)
         v = ops.linear(ckv, self.vc_t.view(H * self.v, R)).view(T, H, self.v)
         o = ops.mla_prefill_ragged(q, k_nope, k_pe, v, ctx.cu_seqlens_q, self.scale).reshape(T, H * self.v)

@@ -34,9 +34,13 @@ from .layers import QLinear, RMSNorm, RoutedExperts, SwiGLUMLP
 
 
 class GatedDeltaNet(nn.Module):
-    def __init__(self, cfg: ModelConfig, state_idx: int, dtype, device):
+    """`exact`: everything between the projections is computed in 32-bit (`ops.gated_delta`: gates from fp32 logits, unit norms, the
+    recurrence and the gated output norm with one rounding at its end); any head sizes.  Otherwise the roundings of the Qwen3.5
+    release are kept."""
+
+    def __init__(self, cfg: ModelConfig, state_idx: int, dtype, device, exact: bool = False):
         super().__init__()
-        self.state_idx = state_idx
+        self.state_idx, self.exact = state_idx, exact
         self.hk, self.hv = cfg.linear_num_key_heads, cfg.linear_num_value_heads
         self.dk, self.dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
         self.key_dim, self.value_dim = self.hk * self.dk, self.hv * self.dv
@@ -55,6 +59,12 @@ class GatedDeltaNet(nn.Module):
     def forward(self, x, ctx: ForwardContext):
         T = x.shape[0]
         proj = self.in_proj(x)
+        if self.exact:
+            ab = ops.linear_fp32(x, self.in_proj_ab.weight)[:, : 2 * self.hv]
+            o = ops.gated_delta(proj, ab, self.conv_weight, self.A_log, self.dt_bias, self.norm_weight, ctx.conv_states[self.state_idx],
+                                ctx.rec_states[self.state_idx], ctx.state_slots, ctx.cu_seqlens_q, ctx.seq_fresh, self.hk, self.hv, self.dk, self.dv,
+                                self.eps, ctx.max_seqlen_q)
+            return self.out_proj(o)
         ab = self.in_proj_ab(x)
         qkv, z = proj[:, : self.conv_dim], proj[:, self.conv_dim:]
         uniform_one = (not ctx.is_prefill) and ctx.q_len_uniform == 1

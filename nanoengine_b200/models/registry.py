@@ -49,7 +49,21 @@ def _gemma4():
     return Gemma4ForCausalLM
 
 
+def _tuvutar():
+    from .tuvutar import TuvutarForCausalLM
+    return TuvutarForCausalLM
+
+
+# kernel sources (stems under csrc/) of the architectures that can be served from a partial build; None = all of them
+_KERNELS = {"Tuvutar": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_bf16", "mla_bf16", "delta")}
+
+
+def kernel_sources(architecture: str):
+    return _KERNELS.get(architecture)
+
+
 _LAZY = {
+    "Tuvutar": _tuvutar,
     "Gemma4ForCausalLM": _gemma4, "Gemma4ForConditionalGeneration": _gemma4,
     "Glm5NextForConditionalGeneration": _glm5_next, "KimiK3ForConditionalGeneration": _kimi_k3,
     "DeepseekV4ForCausalLM": _deepseek_v4,

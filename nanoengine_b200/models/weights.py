@@ -67,6 +67,9 @@ def hf_param_shapes(cfg: ModelConfig, include_mtp: bool = False) -> Dict[str, Tu
     out: Dict[str, Tuple[int, ...]] = {"model.embed_tokens.weight": (V, H), "model.norm.weight": (H,), "lm_head.weight": (V, H)}
     if cfg.architecture.startswith("Gemma4"):
         return _gemma4_param_shapes(cfg, out)
+    if cfg.layer_specs:
+        from .tuvutar import tuvutar_param_shapes
+        return tuvutar_param_shapes(cfg)
     if cfg.is_dsv4:
         from .deepseek_v4 import dsv4_param_shapes
         return dsv4_param_shapes(cfg, out)
@@ -234,6 +237,19 @@ def random_hf_weights(cfg: ModelConfig, seed: int = 0, device="cpu", keep: Optio
             continue
         g = torch.Generator(device=dev)
         g.manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
+        if cfg.layer_specs:                     # rows scaled by their fan-in, norm weights around zero or one
+            leaf = name.rsplit(".", 1)[-1]
+            if leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm":
+                t = 0.1 * torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
+            elif leaf == "norm":
+                t = 1.0 + 0.1 * torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
+            elif leaf in ("A_log", "dt_bias"):
+                t = 0.5 * torch.randn(shape, generator=g, device=dev, dtype=torch.float32) - (2.0 if leaf == "dt_bias" else 0.0)
+            else:
+                s = 1.0 if name == "embed" else 0.5 if leaf == "conv" else shape[-1] ** -0.5
+                t = s * torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
+            yield name, t
+            continue
         if name.endswith("tid2eid"):            # token id -> its experts: distinct ids per row
             t = torch.rand(shape[0], cfg.n_routed_experts, generator=g, device=dev).argsort(-1)[:, : shape[1]].to(torch.int32)
         elif name.endswith("attn_sink"):

@@ -70,6 +70,27 @@ def add_rmsnorm(x: torch.Tensor, residual: Optional[torch.Tensor], w: torch.Tens
     return rmsnorm(x, w, eps, quant, unit_offset), x
 
 
+def residual_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float, unit_offset: bool = True):
+    """Norms on both sides of a sublayer around a 32-bit residual stream: x <- x + rmsnorm(y, w_post), then the next sublayer's
+    input rmsnorm(x, w_next) in y's dtype.  y [T, W] (rows may be strided), x [T, W] fp32.  Returns (input, x); the CUDA body
+    updates x in place."""
+    off = 1.0 if unit_offset else 0.0
+
+    def norm(v, w):
+        return v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + off)
+
+    x = x + norm(y.float(), w_post)
+    return norm(x, w_next).to(y.dtype), x
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, w_next: torch.Tensor, eps: float, unit_offset: bool = True):
+    """The start of a 32-bit residual stream: x = table[ids] as fp32 and the first sublayer's input rmsnorm(x, w_next) in the
+    table's dtype.  Returns (input, x)."""
+    x = table[ids.long()].float()
+    w = w_next.float() + (1.0 if unit_offset else 0.0)
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(table.dtype), x
+
+
 def layernorm(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: float) -> torch.Tensor:
     return F.layer_norm(x.float(), (x.shape[-1],), w.float(), None if b is None else b.float(), eps).to(x.dtype)
 
@@ -164,6 +185,11 @@ def linear(x: torch.Tensor, w: torch.Tensor, w_scale: Optional[torch.Tensor] = N
     return y
 
 
+def linear_fp32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """y = x @ w^T with the accumulator handed on in fp32 (projections whose result enters a 32-bit computation)."""
+    return F.linear(dense(x).float(), w.float())
+
+
 # ---- rotary ------------------------------------------------------------------------------------
 def yarn_mscale(scale: float, mscale: float) -> float:
     return 1.0 if scale <= 1 else 0.1 * mscale * math.log(scale) + 1.0
@@ -186,6 +212,8 @@ def rope_inv_freq(dim: int, theta: float, scaling: Optional[dict]) -> Tuple[torc
     ramp = ((torch.arange(dim // 2, dtype=torch.float32) - low) / max(high - low, 1e-3)).clamp(0, 1)
     inv_mask = 1.0 - ramp
     inv = inv / factor * (1 - inv_mask) + inv * inv_mask
+    if scaling.get("attention_factor") is not None:            # the magnitude of cos and sin, given outright
+        return inv, float(scaling["attention_factor"])
     m = yarn_mscale(factor, float(scaling.get("mscale", 1.0))) / yarn_mscale(factor, float(scaling.get("mscale_all_dim", 0.0)))
     return inv, m
 
@@ -834,6 +862,26 @@ def mla_kv_prepare(kv_a: torch.Tensor, norm_w: torch.Tensor, eps: float, positio
     mla_kv_store(kv_cache, slot_mapping, ckv, k_pe)
 
 
+def latent_prepare(q: torch.Tensor, nope: int, kv_a: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
+                   rope_cache: torch.Tensor, kv_cache: torch.Tensor, slot_mapping: torch.Tensor, R: int) -> None:
+    """Everything of a latent-attention layer that turns by position, in one pass: the rotary part of every query head
+    (q [T, H, nope + rope]) is rotated in place, and - unless the layer reads another layer's rows (kv_a None) - the token's
+    cache row [RMSNorm(kv_a[:, :R]) | rope(kv_a[:, R:])] is written at `slot_mapping`."""
+    if kv_a is not None:
+        mla_kv_prepare(kv_a, norm_w, eps, positions, rope_cache, kv_cache, slot_mapping, R)
+    q[..., nope:] = apply_rope(q[..., nope:], positions, rope_cache, True)
+
+
+def latent_gather(kv_cache: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """Cache rows at `slots` as a [T, R + rope] tensor (slot -1: row 0, a padded token nobody reads)."""
+    return kv_cache.view(-1, kv_cache.shape[-1])[slots.clamp_min(0).long()]
+
+
+def latent_query(q: torch.Tensor, kc: torch.Tensor, nope: int, kc_t=None) -> torch.Tensor:
+    """Absorbed query [q_nope @ W_UK | q_rope] of an already rotated q [T, H, nope + rope] -> [T, H, R + rope]."""
+    return torch.cat([bmm_absorb(q[..., :nope], kc), q[..., nope:]], -1)
+
+
 def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """MoE router GEMM in fp32: x [T, H] (any dtype), w [E, H] fp32 -> [T, E] fp32."""
     return F.linear(x.float(), w.float())
@@ -874,7 +922,7 @@ def gdn_conv(x: torch.Tensor, weight: torch.Tensor, conv_state: torch.Tensor, sl
         for j in range(K):
             acc += full[j: j + (e - s)] * w[:, j]
         y[s:e] = torch.nn.functional.silu(acc).to(x.dtype)
-        conv_state[slot] = full[-(K - 1):].to(conv_state.dtype)
+        conv_state[slot] = full[full.shape[0] - (K - 1):].to(conv_state.dtype)
     return y
 
 
@@ -1104,6 +1152,36 @@ def gdn_recurrent(q, k, v, a, b, A_log, dt_bias, state, slots, cu_seqlens, fresh
             o[s:e], S = gdn_scan(qn[s:e], kn[s:e], vf[s:e], g[s:e], beta[s:e], S)
         state[slot] = S
     return rmsnorm_gated(o, z, norm_w, eps).reshape(T, Hv * Dv)
+
+
+def gated_delta(proj: torch.Tensor, ab: torch.Tensor, conv_w: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor,
+                window: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_seqlens: torch.Tensor, fresh: torch.Tensor, Hk: int,
+                Hv: int, Dk: int, Dv: int, eps: float, max_q_len: int = 1) -> torch.Tensor:
+    """Gated delta-rule mixer between its projections, 32-bit from the convolution on: proj [T, q | k | v | z] (Hk Dk, Hk Dk, Hv Dv,
+    Hv Dv columns), ab [T, 2 Hv] fp32 (decay and write-strength logits).  Short causal convolution + silu over q | k | v with the
+    carried `window` [S, K - 1, C], unit q and k, decay exp(-exp(A_log) softplus(a + dt_bias)), the recurrence on `state`
+    [S, Hv, Dv, Dk] fp32, then per head o / rms(o) * norm_w * silu(z).  Returns [T, Hv * Dv] in proj's dtype; any mix of sequence
+    lengths.  `max_q_len`: planning hint of the CUDA body."""
+    T = proj.shape[0]
+    C, kd = conv_w.shape[0], Hk * Dk
+    y = gdn_conv(proj[:, :C].float(), conv_w, window, slots, cu_seqlens, fresh)
+    g, beta = gdn_gates(ab[:, :Hv], ab[:, Hv:], A_log, dt_bias)
+    rep = Hv // Hk
+    qn = (_l2norm(y[:, :kd].view(T, Hk, Dk)) * Dk ** -0.5).repeat_interleave(rep, 1)
+    kn = _l2norm(y[:, kd: 2 * kd].view(T, Hk, Dk)).repeat_interleave(rep, 1)
+    v = y[:, 2 * kd:].view(T, Hv, Dv)
+    o = torch.empty(T, Hv, Dv, dtype=torch.float32, device=proj.device)
+    cu = cu_seqlens.tolist()
+    for i in range(len(cu) - 1):
+        s, e = cu[i], cu[i + 1]
+        if e <= s:
+            continue
+        slot = int(slots[i])
+        S = torch.zeros_like(state[slot]) if int(fresh[i]) else state[slot].clone()
+        o[s:e], state[slot] = gdn_scan(qn[s:e], kn[s:e], v[s:e], g[s:e], beta[s:e], S)
+    z = proj[:, C: C + Hv * Dv].float().view(T, Hv, Dv)
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float() * F.silu(z)
+    return o.to(proj.dtype).reshape(T, Hv * Dv)
 
 
 # ---- MTP draft verification -------------------------------------------------------------------------------

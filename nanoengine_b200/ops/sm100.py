@@ -20,6 +20,12 @@ _LIB = None
 _c = ctypes
 
 
+def use_library(path) -> None:
+    """Load the kernels from this file instead of the full library (a build of one architecture's kernels: build_native.build_for)."""
+    global _LIB
+    _LIB = ctypes.CDLL(str(path))
+
+
 def lib():
     global _LIB
     if _LIB is None:

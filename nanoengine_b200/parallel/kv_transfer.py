@@ -123,13 +123,17 @@ class LocalTransport:
              src_state: int = -1, dst_state: int = -1) -> int:
         s, d = self.src[src_dp], self.dst[dst_dp]
         sc, dc = s.cache, d.cache
-        si = torch.as_tensor(src_blocks, dtype=torch.long, device=sc.kv.device)
-        di = torch.as_tensor(dst_blocks, dtype=torch.long, device=dc.kv.device)
-        bdim = 1 if sc.plan.mla else 2
-        skv = sc.kv.view(torch.uint8) if sc.kv.dtype == torch.float8_e4m3fn else sc.kv
-        dkv = dc.kv.view(torch.uint8) if dc.kv.dtype == torch.float8_e4m3fn else dc.kv
-        dkv.index_copy_(bdim, di, skv.index_select(bdim, si).to(dkv.device))
-        n = skv.index_select(bdim, si).numel() * skv.element_size()
+        listed = sc.plan.latent_rows is not None             # one page tensor per layer, page id in front
+        bdim = 0 if listed else (1 if sc.plan.mla else 2)
+        si = torch.as_tensor(src_blocks, dtype=torch.long)
+        di = torch.as_tensor(dst_blocks, dtype=torch.long)
+        n = 0
+        for skv, dkv in zip(sc.layers if listed else [sc.kv], dc.layers if listed else [dc.kv]):
+            skv = skv.view(torch.uint8) if skv.dtype == torch.float8_e4m3fn else skv
+            dkv = dkv.view(torch.uint8) if dkv.dtype == torch.float8_e4m3fn else dkv
+            rows = skv.index_select(bdim, si.to(skv.device))
+            dkv.index_copy_(bdim, di.to(dkv.device), rows.to(dkv.device))
+            n += rows.numel() * rows.element_size()
         if sc.indexer is not None and dc.indexer is not None:
             # the indexer keys may sit on another device than the latent pages (hot / cold tier: pages in host memory)
             rows = sc.indexer.index_select(1, si.to(sc.indexer.device))
@@ -137,7 +141,7 @@ class LocalTransport:
             n += rows.numel()
         for t, u in zip(sc.comp or [], dc.comp or []):                    # pooled-row pages (DeepSeek-V4)
             if t is not None:
-                u.index_copy_(0, di, t.index_select(0, si).to(u.device))
+                u.index_copy_(0, di.to(u.device), t.index_select(0, si.to(t.device)).to(u.device))
                 n += len(src_blocks) * t[0].numel() * t.element_size()
         sfam, dfam = sc.slot_families(), dc.slot_families()
         if sfam:

@@ -14,6 +14,11 @@ DeepSeek-V4        one shared key / value row per token and layer in the latent-
                    compressor's carry [c * ratio, c * head_dim] fp32 twice (values and scores; c = 2 for ratio 4).  With an fp8 cache a row
                    is 584 packed bytes (448 e4m3 values, 64 bf16 rotated dims, 7 scale bytes + pad) instead of head_dim values.
 
+listed layers      families that list their layers one by one (Tuvutar) may give every latent layer its own row width and every
+                   delta layer its own state shape: one tensor per layer instead of the stacked ones ([blocks, block_size, D_l];
+                   [slots, Hv_l, Dv_l, Dk_l] fp32 and [slots, K_l - 1, conv_dim_l]), page families `latent_<n>`, slot families
+                   `delta_state_<n>` / `delta_conv_<n>`.  A layer that reads an earlier layer's rows owns none.
+
 One extra block past the scheduler-visible range is reserved as the scratch page that dummy batches of idle
 DP ranks write into.
 
@@ -64,6 +69,9 @@ class CachePlan:
     # the same number, or the bytes of a packed row when the cache keeps fp8 values)
     dsv4_ratios: Optional[List[int]] = None
     dsv4_head_dim: int = 0
+    # listed layers: row width of every latent layer that keeps rows, (heads, Dv, Dk, taps, conv channels) of every delta layer
+    latent_rows: Optional[List[int]] = None
+    delta_shapes: Optional[List[tuple]] = None
     hisparse: bool = False
     hot_rows: int = 0
     hs_slots: int = 0
@@ -88,6 +96,8 @@ class CachePlan:
         if not self.gdn:
             return 0
         e = 2 if self.kv_dtype in (torch.bfloat16, torch.float16, torch.float8_e4m3fn) else 4
+        if self.delta_shapes is not None:
+            return sum(h * dv * dk * 4 + (k - 1) * c * e for h, dv, dk, k, c in self.delta_shapes)
         return self.gdn_layers * (self.gdn_heads * self.gdn_dv * self.gdn_dk * 4 + (self.conv_k - 1) * self.conv_dim * e)
 
     @property
@@ -99,6 +109,8 @@ class CachePlan:
         e = torch.empty(0, dtype=self.kv_dtype).element_size()
         if self.dsv4:
             return (self.num_layers * self.block_size + sum(self.comp_entries_per_page(r) for r in self.dsv4_ratios if r)) * self.row_dim * e
+        if self.latent_rows is not None:
+            return self.block_size * sum(self.latent_rows) * e
         if self.mla:
             return self.num_layers * self.block_size * self.row_dim * e
         return 2 * self.num_layers * self.block_size * self.kv_heads_local * self.row_dim * e
@@ -157,6 +169,14 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
         return CachePlan(True, False, False, mc.num_hidden_layers, block_size, torch.uint8 if packed else dt,
                          dsv4_row_bytes(mc.head_dim, mc.qk_rope_head_dim) if packed else mc.head_dim, state_slots=state_slots,
                          dsv4_ratios=[mc.compress_ratio(i) for i in range(mc.num_hidden_layers)], dsv4_head_dim=mc.head_dim)
+    if mc.layer_specs:
+        n = mc.num_hidden_layers
+        own = [i for i in range(n) if mc.layer_type(i) == "full_attention" and mc.kv_source_layer(i) == i]
+        rows = [mc.layer_config(i).mla_cache_dim for i in own]
+        cfgs = [mc.layer_config(i) for i in range(n) if mc.layer_type(i) == "linear_attention"]
+        shapes = [(c.linear_num_value_heads, c.linear_value_head_dim, c.linear_key_head_dim, c.linear_conv_kernel_dim, c.gdn_conv_dim) for c in cfgs]
+        return CachePlan(True, False, False, len(rows), block_size, dt, max(rows, default=0), gdn=bool(shapes), gdn_layers=len(shapes),
+                         state_slots=state_slots, latent_rows=rows, delta_shapes=shapes)
     if mc.is_hybrid_gdn and mc.is_mla:
         # delta-attention layers between MLA layers (GLM5-next, Kimi-K3): latent pages for the full-attention layers (and the
         # MTP layers), one state slot per sequence for the linear ones
@@ -184,7 +204,7 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
 def kv_budget_blocks(plan: CachePlan, total: int, utilization: float, used: int, peak: int, current: int, reserved: int = 0) -> int:
     """blocks = (total*util - used - peak + current - reserved) // bytes_per_block."""
     budget = int(total * utilization) - used - peak + current - reserved
-    return max(0, budget // plan.block_bytes)
+    return max(0, budget // max(1, plan.block_bytes))
 
 
 class KVCache:
@@ -193,7 +213,11 @@ class KVCache:
         nb = num_blocks + 1   # + scratch page
         self.scratch_block = num_blocks
         self.hisparse = None
-        if plan.mla:
+        if plan.latent_rows is not None:
+            self.kv = None
+            sdt = torch.uint8 if plan.kv_dtype == torch.float8_e4m3fn else plan.kv_dtype
+            self.layers: List = [torch.zeros(nb, plan.block_size, d, dtype=sdt, device=device).view(plan.kv_dtype) for d in plan.latent_rows]
+        elif plan.mla:
             # under the hot / cold tier the logical pages are the cold tier: pinned host memory the staging kernel reads
             # through the unified address space
             kv_dev = "cpu" if plan.hisparse else device
@@ -202,7 +226,7 @@ class KVCache:
                 self.kv = self.kv.pin_memory()
             if plan.kv_dtype == torch.float8_e4m3fn:
                 self.kv = self.kv.view(torch.float8_e4m3fn)
-            self.layers: List = [self.kv[l] for l in range(plan.num_layers)]
+            self.layers = [self.kv[l] for l in range(plan.num_layers)]
         else:
             self.kv = torch.zeros(2, plan.num_layers, nb, plan.block_size, plan.kv_heads_local, plan.row_dim, dtype=plan.kv_dtype, device=device)
             self.layers = [(self.kv[0, l], self.kv[1, l]) for l in range(plan.num_layers)]
@@ -236,9 +260,13 @@ class KVCache:
                 self.comp_score_state.append(torch.full((ns, c * r, c * plan.dsv4_head_dim), float("-inf"), dtype=torch.float32, device=device))
         self.rec_states = self.conv_states = None
         self.scratch_slot = plan.state_slots
-        if plan.gdn:
-            ns = plan.state_slots + 1   # + scratch slot for padded graph rows and dummy batches
-            cdt = torch.bfloat16 if plan.kv_dtype == torch.float8_e4m3fn else plan.kv_dtype
+        ns = plan.state_slots + 1       # + scratch slot for padded graph rows and dummy batches
+        cdt = torch.bfloat16 if plan.kv_dtype == torch.float8_e4m3fn else plan.kv_dtype
+        if plan.delta_shapes is not None:
+            self.rec = self.conv = None
+            self.rec_states = [torch.zeros(ns, h, dv, dk, dtype=torch.float32, device=device) for h, dv, dk, _, _ in plan.delta_shapes]
+            self.conv_states = [torch.zeros(ns, k - 1, c, dtype=cdt, device=device) for _, _, _, k, c in plan.delta_shapes]
+        elif plan.gdn:
             self.rec = torch.zeros(plan.gdn_layers, ns, plan.gdn_heads, plan.gdn_dv, plan.gdn_dk, dtype=torch.float32, device=device)
             self.conv = torch.zeros(plan.gdn_layers, ns, plan.conv_k - 1, plan.conv_dim, dtype=cdt, device=device)
             self.rec_states = [self.rec[l] for l in range(plan.gdn_layers)]
@@ -255,6 +283,8 @@ class KVCache:
             per_plane = t.numel() * es // planes
             pages = self.num_blocks + 1
             return {"name": name, "tensor": t, "planes": planes, "plane_stride": per_plane, "page_bytes": per_plane // pages}
+        if self.plan.latent_rows is not None:
+            return [fam(f"latent_{l}", t, 1) for l, t in enumerate(self.layers)]
         out = [fam("mla_kv" if self.plan.mla else "gqa_kv", self.kv, self.kv.shape[0] if self.plan.mla else 2 * self.kv.shape[1])]
         if self.indexer is not None:
             out.append(fam("indexer", self.indexer, self.indexer.shape[0]))
@@ -268,7 +298,13 @@ class KVCache:
         window, compressor carries): same description, with `slot_bytes` in place of `page_bytes` and `slot_dim`, the tensor dimension
         the slot indexes."""
         out = []
-        if self.plan.gdn:
+        if self.plan.delta_shapes is not None:
+            for l, pair in enumerate(zip(self.rec_states, self.conv_states)):
+                for name, t in zip((f"delta_state_{l}", f"delta_conv_{l}"), pair):
+                    nbytes = t.numel() * t.element_size()
+                    if nbytes:
+                        out.append({"name": name, "tensor": t, "planes": 1, "plane_stride": nbytes, "slot_bytes": nbytes // t.shape[0], "slot_dim": 0})
+        elif self.plan.gdn:
             for name, t in (("gdn_state", self.rec), ("gdn_conv", self.conv)):
                 planes = t.shape[0]
                 per_plane = t.numel() * t.element_size() // planes
@@ -295,10 +331,12 @@ class KVCache:
         for f in self.page_families():
             self.host_families[f["name"]] = torch.zeros(f["planes"], num_host_blocks, f["page_bytes"], dtype=torch.uint8,
                                                         pin_memory=self.device.type == "cuda")
-        self.host_kv = self.host_families["mla_kv" if self.plan.mla else "gqa_kv"]
+        self.host_kv = self.host_families.get("mla_kv" if self.plan.mla else "gqa_kv")
 
     def block_views(self, bid: int) -> List[torch.Tensor]:
         """Byte views of everything block `bid` holds (all layers of every cache family), for the file-backed tier."""
+        if self.plan.latent_rows is not None:
+            return [(t.view(torch.uint8) if t.dtype == torch.float8_e4m3fn else t)[bid] for t in self.layers]
         kv = self.kv.view(torch.uint8) if self.kv.dtype == torch.float8_e4m3fn else self.kv
         out = [kv[:, bid] if self.plan.mla else kv[:, :, bid]]
         if self.indexer is not None:

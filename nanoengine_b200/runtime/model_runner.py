@@ -655,6 +655,22 @@ class ModelRunner:
         ids = [s for s, m in zip(b.seq_ids, mask) if m]
         return C.RunnerOut(ids, [[t] for t in toks], None if lps is None else [[x] for x in lps])
 
+    @torch.inference_mode()
+    def run_logits(self, blob: bytes, rows: List[int]) -> Optional[np.ndarray]:
+        """One step without sampling: the logits (fp32, [len(rows), vocab]) at the listed rows of the step's flat token list, or
+        None when none is asked for.  The forward pass is the one `run_batch` samples from (graph replay included)."""
+        b = C.RunnerIn.from_bytes(blob)
+        ctx = self.prepare(b)
+        hidden = self.forward(ctx)
+        out = None
+        if rows:
+            sel = self._to_dev(np.asarray(rows, dtype=np.int64))
+            out = self.model.compute_logits(hidden[sel]).float().cpu().numpy()
+        elif self.device.type == "cuda":
+            torch.cuda.current_stream().synchronize()
+        self._check_kernel_status()
+        return out
+
     # ---- benchmark helpers ----------------------------------------------------------------------
     @torch.inference_mode()
     def make_resident_decode_step(self):

@@ -89,6 +89,9 @@ def main(argv=None) -> int:
         from .ctrl import run_ctrl
         run_ctrl(a.host, a.port, a.ttl)
         return 0
+    if cmd == "replay":
+        from .replay import main as replay
+        return replay(rest)
     if cmd == "monitor":
         ap = argparse.ArgumentParser(prog="monitor")
         ap.add_argument("--targets", required=True)
@@ -121,7 +124,7 @@ def main(argv=None) -> int:
         serve(EncoderConfig(model=a.model, device=a.device, dtype=a.dtype, num_slots=a.num_slots, max_tokens_per_slot=a.max_tokens_per_slot,
                             endpoint=a.endpoint, engine_id=a.engine_id), a.host, a.port)
         return 0
-    raise SystemExit(f"unknown command {cmd}; expected serve | serve-encoder | monitor | router")
+    raise SystemExit(f"unknown command {cmd}; expected serve | serve-encoder | replay | monitor | ctrl | router")
 
 
 if __name__ == "__main__":
