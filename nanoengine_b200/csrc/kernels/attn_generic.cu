@@ -6,7 +6,8 @@
 //   MLA:  q [T, H, Dk], cache rows [Dk] (first Dv values double as V), out [T, H, Dv]
 //   GQA:  q [T, Hq, D], k/v caches [slots, Hkv, D], out [T, Hq, D]
 // Keys of a query: positions [0, limit] of its sequence through the block table (causal), or an explicit list of
-// physical slots (sparse, -1 = skip).  Cache dtype bf16 or e4m3 (query is then clamped and cast to e4m3 as well).
+// physical slots (sparse, -1 = skip).  Cache dtype bf16, e4m3 (query is then clamped and cast to e4m3 as well) or fp32 (query and
+// output fp32 too: runs in true 32-bit).
 //
 // Replaces in the reference: attention/base.py:451-525 (SDPA reference), flash_mla sparse decode call sites
 // (layers/backends/mla/flash_mla.py:22-121) for the sparse case, flashinfer / FA paged GQA wrappers.
@@ -18,14 +19,14 @@ constexpr int kKeysPerTile = 32;
 constexpr int kHeadsPerCta = 4;
 
 struct AttnArgs {
-  const __nv_bfloat16* q; long long q_tok_stride; int q_head_stride;
+  const void* q; long long q_tok_stride; int q_head_stride;
   const void* k_cache; const void* v_cache;      // v_cache == nullptr: V is the first Dv values of the K row (MLA)
   long long kv_slot_stride; int kv_head_stride;   // in elements
   int kv_group;                                   // query heads per kv head (1 for MLA where kv_head_stride = 0)
   const int* block_tables; int bt_stride; int block_size;
   const int* cu_seqlens_q; const int* context_lens; int num_seqs;
   const int* sparse; int topk;                    // [T, topk] physical slots or nullptr
-  __nv_bfloat16* out; long long o_tok_stride; int o_head_stride;
+  void* out; long long o_tok_stride; int o_head_stride;
   float* lse;                                     // optional [T, H] natural-log LSE
   int T, H, Dk, Dv; float scale; int fp8;
   int window;                                     // > 0: a query sees only the last `window` key positions up to its own (sliding-window layers)
@@ -33,8 +34,10 @@ struct AttnArgs {
   int heads_per_cta;                              // 4, or 1 when every query head has its own kv head (the CTA stages one kv head)
 };
 
-__device__ __forceinline__ float load_kv(const void* base, long long idx, int fp8) {
-  return fp8 ? e4m3_to_float(reinterpret_cast<const uint8_t*>(base)[idx]) : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(base)[idx]);
+// kind: 0 bf16, 1 e4m3, 2 fp32
+__device__ __forceinline__ float load_kv(const void* base, long long idx, int kind) {
+  if (kind == 2) return reinterpret_cast<const float*>(base)[idx];
+  return kind ? e4m3_to_float(reinterpret_cast<const uint8_t*>(base)[idx]) : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(base)[idx]);
 }
 
 __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
@@ -62,8 +65,8 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
 
   for (int i = threadIdx.x; i < kHeadsPerCta * Dk; i += blockDim.x) {
     int hh = h0 + i / Dk, d = i % Dk;
-    float v = (hh < a.H && i / Dk < a.heads_per_cta) ? __bfloat162float(a.q[(long long)t * a.q_tok_stride + (long long)hh * a.q_head_stride + d]) : 0.f;
-    if (a.fp8) v = e4m3_to_float(to_e4m3(fminf(fmaxf(v, -448.f), 448.f)));
+    float v = (hh < a.H && i / Dk < a.heads_per_cta) ? load_kv(a.q, (long long)t * a.q_tok_stride + (long long)hh * a.q_head_stride + d, a.fp8 == 2 ? 2 : 0) : 0.f;
+    if (a.fp8 == 1) v = e4m3_to_float(to_e4m3(fminf(fmaxf(v, -448.f), 448.f)));
     sq[i] = v;
   }
   // all 4 heads of a CTA must read the same kv head: heads per CTA divide the group size, or the group size is 1 with stride 0
@@ -129,7 +132,11 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
 #pragma unroll
   for (int j = 0; j < 20; j++) {
     int d = lane + 32 * j;
-    if (j < per_lane && d < Dv) a.out[(long long)t * a.o_tok_stride + (long long)h * a.o_head_stride + d] = __float2bfloat16(acc[j] * inv);
+    if (j < per_lane && d < Dv) {
+      const long long o = (long long)t * a.o_tok_stride + (long long)h * a.o_head_stride + d;
+      if (a.fp8 == 2) reinterpret_cast<float*>(a.out)[o] = acc[j] * inv;
+      else reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16(acc[j] * inv);
+    }
   }
   if (a.lse && lane == 0) a.lse[(long long)t * a.H + h] = l_run > 0.f ? (m_run * 0.6931471805599453f + logf(l_run)) : -INFINITY;
 }
@@ -223,10 +230,10 @@ extern "C" int ne_attn_generic(const void* q, long long q_tok_stride, int q_head
   if (T <= 0) return 0;
   if (Dv > 640 || (kv_group > 1 && kv_group % kHeadsPerCta != 0)) return 1001;
   AttnArgs a;
-  a.q = (const __nv_bfloat16*)q; a.q_tok_stride = q_tok_stride; a.q_head_stride = q_head_stride; a.k_cache = k_cache; a.v_cache = v_cache;
+  a.q = q; a.q_tok_stride = q_tok_stride; a.q_head_stride = q_head_stride; a.k_cache = k_cache; a.v_cache = v_cache;
   a.kv_slot_stride = kv_slot_stride; a.kv_head_stride = kv_head_stride; a.kv_group = kv_group; a.block_tables = block_tables;
   a.bt_stride = bt_stride; a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs;
-  a.sparse = sparse; a.topk = topk; a.out = (__nv_bfloat16*)out; a.o_tok_stride = o_tok_stride; a.o_head_stride = o_head_stride; a.lse = lse;
+  a.sparse = sparse; a.topk = topk; a.out = out; a.o_tok_stride = o_tok_stride; a.o_head_stride = o_head_stride; a.lse = lse;
   a.T = T; a.H = H; a.Dk = Dk; a.Dv = Dv; a.scale = scale; a.fp8 = fp8; a.window = window; a.noncausal = noncausal;
   // multi-head attention proper (one kv head per query head, separate V): the four query heads of a CTA would need four
   // different key tiles, so a CTA serves one head there

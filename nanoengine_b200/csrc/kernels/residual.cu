@@ -1,0 +1,255 @@
+// Row operators around a 32-bit residual stream, for bf16 and fp32 activations and any row width:
+//   * residual_norm: x += rmsnorm(y, w_post); out = rmsnorm(x, w_next)   (norm after a sublayer, residual add, norm before the next)
+//     or, as the start of the stream, x = table[id]; out = rmsnorm(x, w_next)
+//   * gated activation of [gate | up] rows
+//   * latent_prepare: rotary part of every query head in place, and the latent cache row [rmsnorm(kv[:R]) | rope(kv[R:])]
+//   * gather of cache rows
+#include "ptx.cuh"
+
+namespace ne {
+
+template <typename T> struct Vec4;
+template <> struct Vec4<float> {
+  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <> struct Vec4<__nv_bfloat16> {
+  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+  }
+};
+__device__ __forceinline__ float ldx(const float* p) { return *p; }
+__device__ __forceinline__ float ldx(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void stx(float* p, float v) { *p = v; }
+__device__ __forceinline__ void stx(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+// sum over the CTA; `red` holds two rows of partial sums used in turn, so one barrier per call is enough
+__device__ __forceinline__ float cta_sum(float v, float (*red)[32], int turn) {
+  v = warp_sum(v);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (l == 0) red[turn][w] = v;
+  __syncthreads();
+  return warp_sum(l < nw ? red[turn][l] : 0.f);
+}
+
+// One CTA per row.  V = 4: W, the row strides and the base addresses allow 4-element accesses; V = 1: anything.
+template <typename T, int V>
+__global__ void __launch_bounds__(512) residual_norm_kernel(const T* __restrict__ y, long long y_ld, float* __restrict__ x, const T* __restrict__ w_post,
+                                                           const T* __restrict__ w_next, T* __restrict__ out, int W, float eps, float w_off,
+                                                           const long long* __restrict__ ids, const T* __restrict__ table, int vocab) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  extern __shared__ float srow[];            // W floats
+  __shared__ float red[2][32];
+  const long long row = blockIdx.x;
+  float* xr = x + row * W;
+  float ss = 0.f;
+  if (ids) {
+    const long long id = ids[row];
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && threadIdx.x == 0) report(ST_BAD_INDEX, 40, (int)row, (int)id);
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+      if constexpr (V == 4) {
+        const float4 t = ok ? Vec4<T>::load(table + id * W + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        *reinterpret_cast<float4*>(srow + i) = t;
+        *reinterpret_cast<float4*>(xr + i) = t;
+        ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+      } else {
+        const float t = ok ? ldx(table + id * W + i) : 0.f;
+        srow[i] = t; xr[i] = t; ss += t * t;
+      }
+    }
+  } else {
+    const T* yr = y + row * y_ld;
+    float sy = 0.f;
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+      if constexpr (V == 4) {
+        const float4 t = Vec4<T>::load(yr + i);
+        *reinterpret_cast<float4*>(srow + i) = t;
+        sy += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+      } else {
+        const float t = ldx(yr + i);
+        srow[i] = t; sy += t * t;
+      }
+    }
+    const float r = rsqrtf(cta_sum(sy, red, 0) / (float)W + eps);
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {      // a thread rereads only what it stored itself
+      if constexpr (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(srow + i), w = Vec4<T>::load(w_post + i);
+        float4 v = *reinterpret_cast<const float4*>(xr + i);
+        v.x += t.x * r * (w.x + w_off); v.y += t.y * r * (w.y + w_off); v.z += t.z * r * (w.z + w_off); v.w += t.w * r * (w.w + w_off);
+        *reinterpret_cast<float4*>(srow + i) = v;
+        *reinterpret_cast<float4*>(xr + i) = v;
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      } else {
+        const float v = xr[i] + srow[i] * r * (ldx(w_post + i) + w_off);
+        srow[i] = v; xr[i] = v; ss += v * v;
+      }
+    }
+  }
+  const float r2 = rsqrtf(cta_sum(ss, red, 1) / (float)W + eps);
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(srow + i), w = Vec4<T>::load(w_next + i);
+      Vec4<T>::store(out + row * W + i, make_float4(v.x * r2 * (w.x + w_off), v.y * r2 * (w.y + w_off), v.z * r2 * (w.z + w_off), v.w * r2 * (w.w + w_off)));
+    } else {
+      stx(out + row * W + i, srow[i] * r2 * (ldx(w_next + i) + w_off));
+    }
+  }
+}
+
+// Gated activation (see elementwise.cu for the modes): x [T, >= 2I] rows with stride ld -> y [T, I]
+__device__ __forceinline__ float glu_exact(float g, float u, int act, float p0, float p1) {
+  if (act == 3) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  if (act == 1) { u = fminf(fmaxf(u, -p0), p0); g = fminf(g, p0); }
+  if (act == 2) {
+    if (p1 > 0.f) u = p1 * tanhf(u / p1);
+    return p0 * tanhf(g / p0) / (1.f + expf(-g)) * u;
+  }
+  return g / (1.f + expf(-g)) * u;
+}
+template <typename T, int V>
+__global__ void __launch_bounds__(256) glu_rows_kernel(const T* __restrict__ x, long long ld, T* __restrict__ y, long long n, int I, int act, float p0, float p1) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (i >= n) return;
+  const long long t = i / I;
+  const int c = (int)(i - t * I);
+  const T* g = x + t * ld + c;
+  if constexpr (V == 4) {
+    const float4 a = Vec4<T>::load(g), b = Vec4<T>::load(g + I);
+    Vec4<T>::store(y + i, make_float4(glu_exact(a.x, b.x, act, p0, p1), glu_exact(a.y, b.y, act, p0, p1), glu_exact(a.z, b.z, act, p0, p1),
+                                      glu_exact(a.w, b.w, act, p0, p1)));
+  } else {
+    stx(y + i, glu_exact(ldx(g), ldx(g + I), act, p0, p1));
+  }
+}
+
+// One warp per (token, unit): unit 0 .. H-1 rotates the rotary tail of that query head (q -> dst), unit H (when kv is given) writes the
+// token's cache row.  kv_kind: 0 bf16 rows, 1 e4m3 rows (clamped cast of the bf16 value), 2 fp32 rows.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q, long long q_ld, int q_hs, T* dst, long long d_ld, int d_hs, int H, const T* __restrict__ kv,
+                                                            long long kv_ld, const T* __restrict__ w, float eps, const long long* __restrict__ positions,
+                                                            const float* __restrict__ rope_cache, void* __restrict__ cache,
+                                                            const long long* __restrict__ slots, int T_, int R, int rope, int kv_kind) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const int units = H + (kv ? 1 : 0), lane = threadIdx.x & 31, half = rope / 2;
+  const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (wid >= (long long)T_ * units) return;
+  const int t = (int)(wid / units), u = (int)(wid % units);
+  const float* cs = rope_cache + positions[t] * rope;
+  if (u < H) {
+    const T* p = q + (long long)t * q_ld + (long long)u * q_hs;        // may be the destination itself
+    T* o = dst + (long long)t * d_ld + (long long)u * d_hs;
+    for (int i = lane; i < half; i += 32) {
+      const float a = ldx(p + 2 * i), b = ldx(p + 2 * i + 1), c = cs[i], s = cs[half + i];
+      stx(o + 2 * i, a * c - b * s);
+      stx(o + 2 * i + 1, b * c + a * s);
+    }
+    return;
+  }
+  const long long slot = slots[t];
+  if (slot < 0 || !NE_INDEX_OK(slot, BK_CACHE_ROWS, 41, __LINE__)) return;
+  const T* row = kv + (long long)t * kv_ld;
+  float ss = 0.f;
+  for (int c = lane; c < R; c += 32) { const float f = ldx(row + c); ss += f * f; }
+  const float r = rsqrtf(warp_sum(ss) / (float)R + eps);
+  auto put = [&](int c, float v) {
+    const long long o = slot * (R + rope) + c;
+    if (kv_kind == 2) reinterpret_cast<float*>(cache)[o] = v;
+    else if (kv_kind == 1) reinterpret_cast<uint8_t*>(cache)[o] = to_e4m3(__bfloat162float(__float2bfloat16(v)));
+    else reinterpret_cast<__nv_bfloat16*>(cache)[o] = __float2bfloat16(v);
+  };
+  for (int c = lane; c < R; c += 32) put(c, ldx(row + c) * r * ldx(w + c));
+  for (int i = lane; i < half; i += 32) {
+    const float a = ldx(row + R + 2 * i), b = ldx(row + R + 2 * i + 1), c = cs[i], s = cs[half + i];
+    put(R + 2 * i, a * c - b * s);
+    put(R + 2 * i + 1, b * c + a * s);
+  }
+}
+
+// rows[t] = cache[slots[t]] (slot -1: row 0); 16-byte pieces
+__global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ cache, const long long* __restrict__ slots, uint4* __restrict__ rows,
+                                                           int T, int pieces) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (long long)T * pieces) return;
+  const int t = (int)(i / pieces), c = (int)(i % pieces);
+  long long slot = slots[t];
+  if (slot < 0 || !NE_INDEX_OK(slot, BK_CACHE_ROWS, 42, __LINE__)) slot = 0;
+  rows[i] = cache[slot * pieces + c];
+}
+
+template <typename T>
+static int residual_norm_t(const void* y, long long y_ld, float* x, const void* w_post, const void* w_next, void* out, int T_, int W, float eps,
+                           float w_off, const long long* ids, const void* table, int vocab, cudaStream_t st) {
+  const size_t smem = (size_t)W * sizeof(float);
+  const uintptr_t al = (uintptr_t)y | (uintptr_t)x | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)out | (uintptr_t)table;
+  const bool vec = W % 4 == 0 && y_ld % 4 == 0 && al % 16 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((W + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+  auto k = vec ? residual_norm_kernel<T, 4> : residual_norm_kernel<T, 1>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl(k, dim3((unsigned)T_), dim3((unsigned)threads), smem, st, (const T*)y, y_ld, x, (const T*)w_post, (const T*)w_next, (T*)out, W, eps,
+                         w_off, ids, (const T*)table, vocab);
+}
+
+template <typename T>
+static int glu_rows_t(const void* x, long long ld, void* y, int T_, int I, int act, float p0, float p1, cudaStream_t st) {
+  const bool vec = I % 4 == 0 && ld % 4 == 0 && ((uintptr_t)x | (uintptr_t)y) % 16 == 0;
+  const long long n = (long long)T_ * I, items = vec ? n / 4 : n;
+  return (int)launch_pdl(vec ? glu_rows_kernel<T, 4> : glu_rows_kernel<T, 1>, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, st, (const T*)x, ld, (T*)y, n,
+                         I, act, p0, p1);
+}
+
+}  // namespace ne
+
+using namespace ne;
+
+// y [T, W] (row stride y_ld), x [T, W] fp32 updated in place, out [T, W].  With `ids` (and table [vocab, W]) y is not read: x = table[ids].
+extern "C" int ne_residual_norm(const void* y, long long y_ld, float* x, const void* w_post, const void* w_next, void* out, int T, int W, float eps,
+                                float w_off, const long long* ids, const void* table, int vocab, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (W <= 0 || W > 48 * 1024 || (!ids && (!y || !w_post)) || (ids && !table)) return 1001;
+  return fp32 ? residual_norm_t<float>(y, y_ld, x, w_post, w_next, out, T, W, eps, w_off, ids, table, vocab, st)
+              : residual_norm_t<__nv_bfloat16>(y, y_ld, x, w_post, w_next, out, T, W, eps, w_off, ids, table, vocab, st);
+}
+
+extern "C" int ne_glu_rows(const void* x, long long ld, void* y, int T, int I, int act, float p0, float p1, int fp32, cudaStream_t st) {
+  if (T <= 0 || I <= 0) return 0;
+  if (act < 0 || act > 3 || ld < 2 * I) return 1001;
+  return fp32 ? glu_rows_t<float>(x, ld, y, T, I, act, p0, p1, st) : glu_rows_t<__nv_bfloat16>(x, ld, y, T, I, act, p0, p1, st);
+}
+
+// q [T, H, rope], the rotary tails (row stride q_ld, head stride q_hs, elements), dst the same or another view; kv [T, R + rope] (row
+// stride kv_ld) or null
+extern "C" int ne_latent_prepare(const void* q, long long q_ld, int q_hs, void* dst, long long d_ld, int d_hs, int H, const void* kv, long long kv_ld, const void* w, float eps,
+                                 const long long* positions, const float* rope_cache, void* cache, const long long* slots, int T, int R, int rope,
+                                 int kv_kind, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (rope < 0 || rope % 2 || R <= 0 || kv_kind < 0 || kv_kind > 2 || (fp32 != 0) != (kv_kind == 2)) return 1001;
+  const long long warps = (long long)T * (H + (kv ? 1 : 0));
+  const dim3 grid((unsigned)((warps + 7) / 8));
+  if (fp32)
+    return (int)launch_pdl(latent_prepare_kernel<float>, grid, dim3(256), 0, st, (const float*)q, q_ld, q_hs, (float*)dst, d_ld, d_hs, H, (const float*)kv, kv_ld, (const float*)w, eps,
+                           positions, rope_cache, cache, slots, T, R, rope, kv_kind);
+  return (int)launch_pdl(latent_prepare_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)q, q_ld, q_hs, (__nv_bfloat16*)dst, d_ld, d_hs, H,
+                         (const __nv_bfloat16*)kv, kv_ld,
+                         (const __nv_bfloat16*)w, eps, positions, rope_cache, cache, slots, T, R, rope, kv_kind);
+}
+
+extern "C" int ne_latent_gather(const void* cache, const long long* slots, void* rows, int T, int row_bytes, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (row_bytes % 16) return 1001;
+  const int pieces = row_bytes / 16;
+  return (int)launch_pdl(latent_gather_kernel, dim3((unsigned)(((long long)T * pieces + 255) / 256)), dim3(256), 0, st, (const uint4*)cache, slots, (uint4*)rows, T,
+                         pieces);
+}

@@ -149,10 +149,12 @@ class MLAAttention(nn.Module):
                 and self.v == 128 and R % 8 == 0 and x.dtype == torch.bfloat16):
             return self._prefill_nonabsorbed(x, q, kv_a, positions, ctx, rope_cache)
         nw = None if self.reads_only else self.kv_a_layernorm
+        q_full = torch.empty(T, H, R + rope, dtype=q.dtype, device=q.device)
         ops.latent_prepare(q, nope, kv_a, None if nw is None else nw.weight, 0.0 if nw is None else nw.eps, positions, rope_cache, cache,
-                           ctx.slot_mapping, R)
-        q_full = ops.latent_query(q, self.kc, nope, kc_t=self.kc_t)
-        o_lat = ops.mla_attention_paged(q_full, cache, ctx.block_tables, ctx.cu_seqlens_q, ctx.context_lens, self.scale, R)
+                           ctx.slot_mapping, R, q_full)
+        ops.bmm_absorb(q[..., :nope], self.kc, out=q_full[..., :R], wt=self.kc_t)
+        o_lat = ops.mla_attention_paged(q_full, cache, ctx.block_tables, ctx.cu_seqlens_q, ctx.context_lens, self.scale, R,
+                                        max_q_len=ctx.max_seqlen_q)
         return self.o_proj(ops.bmm_absorb(o_lat, self.vc, wt=self.vc_t).reshape(T, H * self.v))
 
     def _prefill_nonabsorbed(self, x, q, kv_a, positions, ctx: ForwardContext, rope_cache):

@@ -293,7 +293,7 @@ def _gather_rows(cache: torch.Tensor, block_table: torch.Tensor, n: int) -> torc
 # ---- attention -----------------------------------------------------------------------------------
 def mla_attention_paged(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, cu_seqlens_q: torch.Tensor,
                         context_lens: torch.Tensor, scale: float, kv_lora_rank: int,
-                        sparse_indices: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        sparse_indices: Optional[torch.Tensor] = None, max_q_len: int = 0) -> torch.Tensor:
     """Absorbed MLA over the paged latent cache, causal within each sequence.
 
     q [T, H, R+rope] (already absorbed with W_UK and rotated); returns the latent output [T, H, R].
@@ -863,23 +863,18 @@ def mla_kv_prepare(kv_a: torch.Tensor, norm_w: torch.Tensor, eps: float, positio
 
 
 def latent_prepare(q: torch.Tensor, nope: int, kv_a: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
-                   rope_cache: torch.Tensor, kv_cache: torch.Tensor, slot_mapping: torch.Tensor, R: int) -> None:
+                   rope_cache: torch.Tensor, kv_cache: torch.Tensor, slot_mapping: torch.Tensor, R: int, q_full: Optional[torch.Tensor] = None) -> None:
     """Everything of a latent-attention layer that turns by position, in one pass: the rotary part of every query head
-    (q [T, H, nope + rope]) is rotated in place, and - unless the layer reads another layer's rows (kv_a None) - the token's
+    (q [T, H, nope + rope]) is rotated in place - or into q_full[..., R:], the tail of the absorbed query [T, H, R + rope] -, and - unless the layer reads another layer's rows (kv_a None) - the token's
     cache row [RMSNorm(kv_a[:, :R]) | rope(kv_a[:, R:])] is written at `slot_mapping`."""
     if kv_a is not None:
         mla_kv_prepare(kv_a, norm_w, eps, positions, rope_cache, kv_cache, slot_mapping, R)
-    q[..., nope:] = apply_rope(q[..., nope:], positions, rope_cache, True)
+    (q[..., nope:] if q_full is None else q_full[..., R:]).copy_(apply_rope(q[..., nope:], positions, rope_cache, True))
 
 
 def latent_gather(kv_cache: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
     """Cache rows at `slots` as a [T, R + rope] tensor (slot -1: row 0, a padded token nobody reads)."""
     return kv_cache.view(-1, kv_cache.shape[-1])[slots.clamp_min(0).long()]
-
-
-def latent_query(q: torch.Tensor, kc: torch.Tensor, nope: int, kc_t=None) -> torch.Tensor:
-    """Absorbed query [q_nope @ W_UK | q_rope] of an already rotated q [T, H, nope + rope] -> [T, H, R + rope]."""
-    return torch.cat([bmm_absorb(q[..., :nope], kc), q[..., nope:]], -1)
 
 
 def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:

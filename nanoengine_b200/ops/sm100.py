@@ -172,6 +172,33 @@ class PrequantizedActivation:
         self.q, self.scales, self.shape, self.device = q, scales, q.shape, q.device
 
 
+def _gemm_simt(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch):
+    """Tiled product on CUDA cores: true 32-bit operands, and bf16 shapes the tensor-core GEMM cannot address."""
+    f32 = A.dtype == torch.float32
+    assert A.dtype == B.dtype and D.dtype in (torch.float32, A.dtype)
+    _ck(lib().ne_gemm_simt(_p(A), _c.c_longlong(lda), _c.c_longlong(a_bs), _p(B), _c.c_longlong(ldb), _c.c_longlong(b_bs), _p(D), _c.c_longlong(ldd),
+                           _c.c_longlong(d_bs), _c.c_int(M), _c.c_int(N), _c.c_int(K), _c.c_int(batch), _c.c_int(int(f32)),
+                           _c.c_int(int(D.dtype == torch.float32)), _st()), "ne_gemm_simt")
+
+
+def _linear_simt(x, w, bias, out_fp32):
+    x2 = x.reshape(-1, x.shape[-1])
+    x2 = (x2 if x2.dtype == w.dtype else x2.to(w.dtype))
+    if x2.stride(-1) != 1:
+        x2 = x2.contiguous()
+    T, (N, K) = x2.shape[0], w.shape
+    out = torch.empty(T, N, dtype=torch.float32 if out_fp32 else w.dtype, device=x.device)
+    if T > 0:
+        _gemm_simt(x2, x2.stride(0), 0, w, w.stride(0), 0, out, N, 0, T, N, K, 1)
+    if bias is not None:
+        out = out + bias
+    return out.view(*x.shape[:-1], N)
+
+
+def linear_fp32(x, w: torch.Tensor) -> torch.Tensor:
+    return linear(x, w, out_fp32=True)
+
+
 def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None, out_fp32: bool = False) -> torch.Tensor:
     N, K = w.shape
     if isinstance(x, PrequantizedActivation):
@@ -185,6 +212,8 @@ def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None
     if isinstance(x, QAct):                   # (e4m3 [T, K], scales [K/128, T]) left by a fused norm + quant kernel
         pre = (x.q, x.scales) if x.q is not None else None
         x = x.x
+    if w.dtype == torch.float32 or (w.dtype == torch.bfloat16 and (K % 8 or N % 8)):
+        return _linear_simt(x, w, bias, out_fp32)
     x2 = _as_bf16_2d(x)
     T = x2.shape[0]
     out = torch.empty(T, N, dtype=torch.float32 if out_fp32 else torch.bfloat16, device=x.device)
@@ -206,9 +235,9 @@ def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None
 
 
 def kmajor(w: torch.Tensor) -> torch.Tensor:
-    """w [H, A, B] -> bf16 [H, B, A] contiguous: the K-major operand `bmm_absorb` multiplies with.  Owners of a weight build
-    this once when the weight is set (and again after an in-place update) and pass it as `wt`."""
-    return w.to(torch.bfloat16).transpose(1, 2).contiguous()
+    """w [H, A, B] -> bf16 (fp32 for fp32 weights) [H, B, A] contiguous: the K-major operand `bmm_absorb` multiplies with.  Owners of
+    a weight build this once when the weight is set (and again after an in-place update) and pass it as `wt`."""
+    return (w if w.dtype == torch.float32 else w.to(torch.bfloat16)).transpose(1, 2).contiguous()
 
 
 def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -238,12 +267,24 @@ def bmm_absorb(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = N
     Bd = w.shape[2]
     if wt is None:
         wt = kmajor(w)                                                                     # [H, B, A], K-major
+    if wt.dtype == torch.float32 or ((A % 8 or Bd % 8) and (out is None or out.dtype == torch.bfloat16)):
+        assert wt.shape == (H, Bd, A) and wt.is_contiguous()
+        x = x if (x.dtype == wt.dtype and x.stride(2) == 1) else x.to(wt.dtype).contiguous()
+        if out is None:
+            out = torch.empty(T, H, Bd, dtype=wt.dtype, device=x.device)
+        assert out.stride(2) == 1
+        if T > 0:
+            _gemm_simt(x, x.stride(0), x.stride(1), wt, A, Bd * A, out, out.stride(0), out.stride(1), T, Bd, A, H)
+        return out
     assert wt.shape == (H, Bd, A) and wt.dtype == torch.bfloat16 and wt.is_contiguous()
     if x.dtype != torch.bfloat16 or x.stride(2) != 1 or (x.stride(0) * 2) % 16 or (x.stride(1) * 2) % 16 or x.data_ptr() % 16:
         x = x.to(torch.bfloat16).contiguous()
     if out is None:
         out = torch.empty(T, H, Bd, dtype=torch.bfloat16, device=x.device)
     es = out.element_size()
+    if es == 2 and ((out.stride(0) * 2) % 16 or (out.stride(1) * 2) % 16 or out.data_ptr() % 16):
+        _gemm_simt(x, x.stride(0), x.stride(1), wt, A, Bd * A, out, out.stride(0), out.stride(1), T, Bd, A, H)      # rows TMA cannot address
+        return out
     assert es in (1, 2) and out.stride(2) == 1 and (out.stride(0) * es) % 16 == 0 and (out.stride(1) * es) % 16 == 0 and out.data_ptr() % 16 == 0
     if T > 0:
         _gemm(x, x.stride(0), x.stride(1), wt, out, out.stride(0), out.stride(1), T, Bd, A, H, None, None, False, None, 0, 0, None,
@@ -286,6 +327,30 @@ def add_rmsnorm(x: torch.Tensor, residual: Optional[torch.Tensor], w: torch.Tens
     return _rmsnorm(x, residual, w, eps, True, quant, unit_offset)
 
 
+def residual_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float, unit_offset: bool = True):
+    """Norm of a sublayer's output, 32-bit residual add (x is updated in place) and the norm before the next sublayer: one kernel,
+    one CTA per row."""
+    T, W = y.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.stride(1) == 1 and w_post.dtype == y.dtype and w_next.dtype == y.dtype
+    out = torch.empty(T, W, dtype=y.dtype, device=y.device)
+    _ck(lib().ne_residual_norm(_p(y), _c.c_longlong(y.stride(0)), _p(x), _p(w_post), _p(w_next), _p(out), _c.c_int(T), _c.c_int(W), _c.c_float(eps),
+                               _c.c_float(1.0 if unit_offset else 0.0), _p(None), _p(None), _c.c_int(0), _c.c_int(int(y.dtype == torch.float32)), _st()),
+        "ne_residual_norm")
+    return out, x
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, w_next: torch.Tensor, eps: float, unit_offset: bool = True):
+    """Embedding rows into a new 32-bit residual stream and the first norm, one kernel."""
+    T, (V, W) = ids.numel(), table.shape
+    assert table.is_contiguous() and w_next.dtype == table.dtype
+    x = torch.empty(T, W, dtype=torch.float32, device=table.device)
+    out = torch.empty(T, W, dtype=table.dtype, device=table.device)
+    _ck(lib().ne_residual_norm(_p(None), _c.c_longlong(0), _p(x), _p(None), _p(w_next), _p(out), _c.c_int(T), _c.c_int(W), _c.c_float(eps),
+                               _c.c_float(1.0 if unit_offset else 0.0), _p(_i64c(ids)), _p(table), _c.c_int(V), _c.c_int(int(table.dtype == torch.float32)), _st()),
+        "ne_residual_norm")
+    return out, x
+
+
 def layernorm(x, w, b, eps):
     """One warp per row of the last dimension."""
     shape = x.shape
@@ -319,6 +384,13 @@ def silu_and_mul(x: torch.Tensor, quant: bool = False, act=None):
     result (for an fp8 down projection)."""
     T, I2 = x.shape
     I = I2 // 2
+    if x.dtype == torch.float32 or I % 128:
+        if x.stride(1) != 1:
+            x = x.contiguous()
+        y = torch.empty(T, I, dtype=x.dtype, device=x.device)
+        _ck(lib().ne_glu_rows(_p(x), _c.c_longlong(x.stride(0)), _p(y), _c.c_int(T), _c.c_int(I), *_act_args(act),
+                              _c.c_int(int(x.dtype == torch.float32)), _st()), "ne_glu_rows")
+        return y
     x = x.contiguous()
     if quant and I % 128 == 0 and T > 0:
         q = torch.empty(T, I, dtype=FP8, device=x.device)
@@ -357,6 +429,32 @@ def mla_absorb_rope(q: torch.Tensor, kc: torch.Tensor, positions: torch.Tensor, 
     bmm_absorb(q[..., :nope], kc, out=out[..., :R], wt=kc_t)
     apply_rope(q[..., nope:], positions, cache, True, out=out[..., R:])
     return out
+
+
+def latent_prepare(q: torch.Tensor, nope: int, kv_a: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
+                   rope_cache: torch.Tensor, kv_cache: torch.Tensor, slot_mapping: torch.Tensor, R: int, q_full: Optional[torch.Tensor] = None) -> None:
+    """One kernel: rotary tails of the query heads in place or into q_full[..., R:], latent row normed / rotated / stored (kv_a None: no row)."""
+    T, H, D = q.shape
+    rope = D - nope
+    f32 = q.dtype == torch.float32
+    kind = 2 if kv_cache.dtype == torch.float32 else 1 if kv_cache.dtype == FP8 else 0
+    assert q.stride(2) == 1 and kv_cache.is_contiguous() and kv_cache.shape[-1] == R + rope and f32 == (kind == 2)
+    assert kv_a is None or (kv_a.dtype == q.dtype and kv_a.stride(1) == 1 and norm_w.dtype == q.dtype)
+    pe = q[..., nope:]
+    dst = pe if q_full is None else q_full[..., R:]
+    assert dst.dtype == q.dtype and dst.stride(2) == 1 and dst.shape == pe.shape
+    _ck(lib().ne_latent_prepare(_p(pe), _c.c_longlong(q.stride(0)), _c.c_int(q.stride(1)), _p(dst), _c.c_longlong(dst.stride(0)),
+                                _c.c_int(dst.stride(1)), _c.c_int(H), _p(kv_a),
+                                _c.c_longlong(0 if kv_a is None else kv_a.stride(0)), _p(norm_w), _c.c_float(eps), _p(_i64c(positions)), _p(rope_cache),
+                                _p(kv_cache), _p(_i64c(slot_mapping)), _c.c_int(T), _c.c_int(R), _c.c_int(rope), _c.c_int(kind), _c.c_int(int(f32)), _st()),
+        "ne_latent_prepare")
+
+
+def latent_gather(kv_cache: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    D, T = kv_cache.shape[-1], slots.numel()
+    rows = torch.empty(T, D, dtype=kv_cache.dtype, device=kv_cache.device)
+    _ck(lib().ne_latent_gather(_p(kv_cache), _p(_i64c(slots)), _p(rows), _c.c_int(T), _c.c_int(D * kv_cache.element_size()), _st()), "ne_latent_gather")
+    return rows
 
 
 def mla_query(q: torch.Tensor, kc: torch.Tensor, positions: torch.Tensor, rope_cache: torch.Tensor, nope: int, kv_cache: torch.Tensor,
@@ -597,9 +695,9 @@ def moe_experts_nvfp4(x, topk_idx, topk_w, w13_q, w13_sf, alpha1, a1_gscale, w2_
 
 
 # ---- attention / sampling: filled in by the dedicated kernel modules ---------------------------------
-def mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, sparse_indices=None):
+def mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, sparse_indices=None, max_q_len: int = 0):
     from . import sm100_attn
-    return sm100_attn.mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, sparse_indices)
+    return sm100_attn.mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, sparse_indices, max_q_len=max_q_len)
 
 
 def attention_varlen(q, k, v, cu_seqlens, scale, causal: bool = False):
@@ -852,6 +950,33 @@ def gdn_recurrent(q, k, v, a, b, A_log, dt_bias, state, slots, cu_seqlens, fresh
         else:
             rmsnorm_gated(dst, z, norm_w, eps, out)
     return out.view(T, Hv * Dv)
+
+
+def gated_delta(proj: torch.Tensor, ab: torch.Tensor, conv_w: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor,
+                window: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_seqlens: torch.Tensor, fresh: torch.Tensor, Hk: int,
+                Hv: int, Dk: int, Dv: int, eps: float, max_q_len: int = 1) -> torch.Tensor:
+    """Two kernels for single-token steps (prepare; recurrence with the output norm), three otherwise (the norm on its own)."""
+    T, K = proj.shape[0], conv_w.shape[1]
+    C = 2 * Hk * Dk + Hv * Dv
+    f32 = proj.dtype == torch.float32
+    assert proj.stride(1) == 1 and proj.shape[1] >= C + Hv * Dv and ab.dtype == torch.float32 and ab.stride(1) == 1 and ab.shape[1] >= 2 * Hv
+    assert conv_w.dtype == proj.dtype and conv_w.is_contiguous() and conv_w.shape[0] == C and norm_w.dtype == proj.dtype
+    assert window.dtype == proj.dtype and window.is_contiguous() and window.shape[1:] == (K - 1, C)
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (Hv, Dv, Dk) and A_log.dtype == dt_bias.dtype == torch.float32
+    out = torch.empty(T, Hv * Dv, dtype=proj.dtype, device=proj.device)
+    if T == 0:
+        return out
+    l = lib()
+    l.ne_delta_scratch_floats.restype = _c.c_longlong
+    scratch = torch.empty(l.ne_delta_scratch_floats(_c.c_int(T), _c.c_int(Hk), _c.c_int(Hv), _c.c_int(Dk), _c.c_int(Dv)), dtype=torch.float32, device=proj.device)
+    n = _c.c_int(1)
+    cu = _i32(cu_seqlens)
+    _ck(l.ne_gated_delta(_p(proj), _c.c_longlong(proj.stride(0)), _p(ab), _c.c_longlong(ab.stride(0)), _p(conv_w), _p(A_log), _p(dt_bias), _p(norm_w),
+                         _c.c_float(eps), _p(window), _p(state), _p(_i32(slots)), _p(cu), _p(_i32(fresh)), _p(scratch), _p(out), _c.c_int(T),
+                         _c.c_int(cu.numel() - 1), _c.c_int(Hk), _c.c_int(Hv), _c.c_int(Dk), _c.c_int(Dv), _c.c_int(K), _c.c_int(max_q_len), _c.c_int(int(f32)),
+                         _c.byref(n), _st()), "ne_gated_delta")
+    LAUNCHES[0] += n.value - 1
+    return out
 
 
 def kda_recurrent(q, k, v, raw_g, b, A_log, dt_bias, lower_bound, state, slots, cu_seqlens, fresh, gate, norm_w, eps: float) -> torch.Tensor:

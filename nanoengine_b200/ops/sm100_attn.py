@@ -1,8 +1,9 @@
 """CUDA bodies of attention and sampling.
 
 MLA over an fp8 latent cache with the DeepSeek-V3 geometry (576-value rows, 64-token pages, <= 128 heads) runs on the
-tcgen05 kernel, dense (paged) and DSA-sparse (listed rows gathered into the same pipeline) alike; every other shape and the
-bf16 cache run on the shape-generic CUDA-core kernel.
+tcgen05 kernel, dense (paged) and DSA-sparse (listed rows gathered into the same pipeline) alike; a bf16 latent cache with
+64-token pages on a tcgen05 kernel of its own (any rank up to 512); every other shape, and runs in 32-bit, on the shape-generic
+CUDA-core kernel.
 """
 from __future__ import annotations
 
@@ -15,6 +16,7 @@ from . import sm100 as _k
 FP8 = torch.float8_e4m3fn
 _NUM_SMS = None
 _sample_calls = 0
+LATENT_TC_CALLS = [0]        # launches of the bf16 latent tensor-core kernel
 SPARSE_TC_CALLS = [0]        # launches of the sparse tensor-core MLA kernel (tests check that the DSA path really takes it)
 
 
@@ -40,6 +42,13 @@ def mla_splits(T: int, max_pages: int) -> int:
     return max(1, min(want, max(1, max_pages // 4), 32))
 
 
+def latent_splits(ctas: int, max_pages: int) -> int:
+    """Key slices of the bf16 latent kernel: as many as still fit one wave, at least 4 pages each."""
+    if ctas * 5 >= _sms() * 3:
+        return 1
+    return max(1, min(_sms() // ctas, max(1, max_pages // 4), 32))
+
+
 def mla_partials(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, splits: int):
     """Un-merged split-KV results of the fp8 tcgen05 kernel: part [splits, T, H, R] fp32 (each slice normalised on its own) and
     lse2 [splits, T, H] fp32 (log2-sum-exp of the slice, -inf where a slice saw no key).  `ne_attn_merge` folds any stack of
@@ -63,19 +72,22 @@ def mla_partials(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_l
     return part, lse2
 
 
-def mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, sparse_indices=None, splits=None):
+def mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scale, kv_lora_rank, sparse_indices=None, splits=None, max_q_len=0):
+    """`max_q_len`: the longest run of new tokens of a sequence, where the caller knows it (0: derived from the batch size)."""
     T, H, Dk = q.shape
     R = kv_lora_rank
     lib = _k.lib()
     bt, cu, cl = _i32(block_tables), _i32(cu_seqlens_q), _i32(context_lens)
     B = cl.numel()
-    out = torch.empty(T, H, R, dtype=torch.bfloat16, device=q.device)
+    out = torch.empty(T, H, R, dtype=torch.float32 if cache.dtype == torch.float32 else torch.bfloat16, device=q.device)
     if T == 0:
         return out
     geom = cache.dtype == FP8 and Dk == 576 and R == 512 and cache.shape[1] == 64 and H <= 128
     fast = geom and sparse_indices is None
     if q.dtype == FP8:
         assert geom and q.is_contiguous(), "an e4m3 query is only produced for the fp8 tensor-core attention kernels"
+    elif cache.dtype == torch.float32:
+        q = q.float().contiguous()
     else:
         q = q if (q.dtype == torch.bfloat16 and q.is_contiguous()) else q.to(torch.bfloat16).contiguous()
     if geom and sparse_indices is not None:
@@ -118,14 +130,35 @@ def mla_attention_paged(q, cache, block_tables, cu_seqlens_q, context_lens, scal
             _k._ck(lib.ne_attn_merge(_k._p(part), _k._p(lse2), _k._p(out), _c.c_int(S), _c.c_longlong(T * H), _c.c_int(R), _c.c_int(R), _k._st()),
                    "ne_attn_merge")
         return out
+    if sparse_indices is None and cache.dtype == torch.bfloat16 and cache.shape[1] == 64:
+        # tiles of consecutive tokens only when every sequence could fill one: a decode batch keeps one token per tile
+        mq = max_q_len if max_q_len else (1 if T <= B else T)
+        tq = _c.c_int(0)
+        ctas = lib.ne_mla_bf16_plan(_c.c_int(H), _c.c_int(R), _c.c_int(Dk), _c.c_int(mq), _c.byref(tq))
+        if ctas:
+            tiles = min(T, T // tq.value + B)
+            S = splits if splits is not None else latent_splits(tiles * ctas, bt.shape[1])
+            part = lse2 = None
+            if S > 1:
+                part = torch.empty(S, T, H, R, dtype=torch.float32, device=q.device)
+                lse2 = torch.empty(S, T, H, dtype=torch.float32, device=q.device)
+            _k._ck(lib.ne_mla_bf16(_k._p(q), _k._p(cache), _c.c_int(cache.shape[0]), _k._p(bt), _c.c_int(bt.stride(0)), _k._p(cu), _k._p(cl), _c.c_int(B),
+                                   _c.c_int(T), _c.c_int(H), _c.c_int(R), _c.c_int(Dk), _c.c_int(mq), _c.c_int(tiles), _c.c_int(S), _c.c_float(scale),
+                                   _k._p(out), _k._p(part), _k._p(lse2), _k._st()), "ne_mla_bf16")
+            LATENT_TC_CALLS[0] += 1
+            if S > 1:
+                _k._ck(lib.ne_attn_merge(_k._p(part), _k._p(lse2), _k._p(out), _c.c_int(S), _c.c_longlong(T * H), _c.c_int(R), _c.c_int(R), _k._st()),
+                       "ne_attn_merge")
+            return out
     fp8 = cache.dtype == FP8
-    assert fp8 or cache.dtype == torch.bfloat16, "the CUDA attention kernels read bf16 or fp8 caches"
+    f32 = cache.dtype == torch.float32
+    assert fp8 or f32 or cache.dtype == torch.bfloat16, "the CUDA attention kernels read bf16, fp8 or fp32 caches"
     sp = None if sparse_indices is None else _i32(sparse_indices)
     _k._ck(lib.ne_attn_generic(_k._p(q), _c.c_longlong(q.stride(0)), _c.c_int(q.stride(1)), _k._p(cache), _k._p(None),
                                _c.c_longlong(cache.shape[-1]), _c.c_int(0), _c.c_int(0), _k._p(bt), _c.c_int(bt.stride(0)), _c.c_int(cache.shape[1]),
                                _k._p(cu), _k._p(cl), _c.c_int(B), _k._p(sp), _c.c_int(0 if sp is None else sp.shape[1]), _k._p(out),
                                _c.c_longlong(H * R), _c.c_int(R), _k._p(None), _c.c_int(T), _c.c_int(H), _c.c_int(Dk), _c.c_int(R),
-                               _c.c_float(scale), _c.c_int(1 if fp8 else 0), _c.c_int(0), _c.c_int(0), _k._st()), "ne_attn_generic")
+                               _c.c_float(scale), _c.c_int(2 if f32 else 1 if fp8 else 0), _c.c_int(0), _c.c_int(0), _k._st()), "ne_attn_generic")
     return out
 
 

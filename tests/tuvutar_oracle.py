@@ -60,8 +60,9 @@ def latent_rows(h, W, p, m, eps):
     return c, rotate(kv[:, R:], pos, m["rot"])
 
 
-def latent_attention(h, W, p, m, rows):
-    """Causal attention over the latent rows, keys and values expanded per head."""
+def latent_attention(h, W, p, m, rows, hide=None):
+    """Causal attention over the latent rows, keys and values expanded per head.  `hide`: plant a mistake - hide(i, n) returns the
+    keys query i leaves out."""
     n, H, d, r, vd = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
     c, kr = rows
     q = (h @ W[p + "q"].T).view(n, H, d + r)
@@ -71,6 +72,8 @@ def latent_attention(h, W, p, m, rows):
     out = torch.zeros(n, H, vd, dtype=h.dtype)
     for i in range(n):
         s = (torch.einsum("hd,jhd->hj", q[i, :, :d], k[: i + 1]) + qr[i] @ kr[: i + 1].T) * m["scale"]
+        if hide is not None:
+            s[:, [j for j in hide(i, n) if j <= i and i > 0]] = -1e30
         out[i] = torch.einsum("hj,jhv->hv", torch.softmax(s, -1), v[: i + 1])
     return out.reshape(n, H * vd) @ W[p + "o"].T
 
@@ -138,8 +141,9 @@ def dense_ff(h, W, p):
 
 
 # ---- the stack -------------------------------------------------------------------------------------------------------
-def forward(cfg, weights, tokens, dtype=torch.float64, trace=None):
-    """Logits [n, vocab] of one sequence.  `trace` (a list) receives the residual stream after every layer."""
+def forward(cfg, weights, tokens, dtype=torch.float64, trace=None, hide=None):
+    """Logits [n, vocab] of one sequence.  `trace` (a list) receives the residual stream after every layer; `hide`: see
+    latent_attention."""
     W = {k: v.to(dtype) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     x = W["embed"][torch.tensor(list(tokens))]
@@ -149,7 +153,7 @@ def forward(cfg, weights, tokens, dtype=torch.float64, trace=None):
         h = offset_norm(x, W[p + "norm1"], eps)
         if L["type"] == "latent_attention":
             rows[i] = rows[m["kv_from"]] if m.get("kv_from") is not None else latent_rows(h, W, p + "mix.", m, eps)
-            y = latent_attention(h, W, p + "mix.", m, rows[i])
+            y = latent_attention(h, W, p + "mix.", m, rows[i], hide)
         else:
             y = delta_mixer(h, W, p + "mix.", m, eps)
         x = x + offset_norm(y, W[p + "norm1b"], eps)
@@ -161,8 +165,9 @@ def forward(cfg, weights, tokens, dtype=torch.float64, trace=None):
 
 
 # ---- random models ---------------------------------------------------------------------------------------------------
-def random_weights(cfg, seed=0, std=1.0):
-    """Weights of every tensor of the design, bf16-representable, scaled so that no mechanism vanishes."""
+def random_weights(cfg, seed=0, sharp=1.5):
+    """Weights of every tensor of the design, bf16-representable, scaled so that no mechanism vanishes.  `sharp` scales the queries:
+    with a large value single keys stand out of hundreds."""
     g = torch.Generator().manual_seed(seed)
 
     def rnd(*shape, s=1.0):
@@ -177,7 +182,7 @@ def random_weights(cfg, seed=0, std=1.0):
         q = p + "mix."
         if L["type"] == "latent_attention":
             H, d, r, vd, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-            W[q + "q"] = rnd(H * (d + r), D, s=1.5 * D ** -0.5)
+            W[q + "q"] = rnd(H * (d + r), D, s=sharp * D ** -0.5)
             if m.get("kv_from") is None:
                 W[q + "dkv"] = rnd(R + r, D, s=D ** -0.5)
                 W[q + "dkv.norm"] = (1 + 0.2 * torch.randn(R, generator=g)).to(torch.bfloat16)
@@ -189,10 +194,18 @@ def random_weights(cfg, seed=0, std=1.0):
                 W[q + nm] = rnd(rows, D, s=D ** -0.5)
                 if nm in "qkv":
                     W[q + nm + ".conv"] = rnd(rows, K, s=0.6)
-            W[q + "A_log"], W[q + "dt_bias"] = rnd(H, s=0.5), rnd(H, s=0.5) - 2
+            W[q + "A_log"], W[q + "dt_bias"] = rnd(H, s=0.5), (rnd(H, s=0.5) - 3).to(torch.bfloat16)
             W[q + "norm"] = (1 + 0.2 * torch.randn(vd, generator=g)).to(torch.bfloat16)
             W[q + "o"] = rnd(D, H * vd, s=(H * vd) ** -0.5)
         if L["mlp"]:
             F = L["mlp"]["ff"]
             W[p + "mlp.gate"], W[p + "mlp.up"], W[p + "mlp.down"] = rnd(F, D, s=D ** -0.5), rnd(F, D, s=D ** -0.5), rnd(D, F, s=F ** -0.5)
     return W
+
+
+def greedy(cfg, weights, prompt, n):
+    """n greedily chosen tokens after `prompt`."""
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(cfg, weights, toks)[-1].argmax()))
+    return toks[len(prompt):]
