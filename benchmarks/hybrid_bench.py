@@ -1,0 +1,105 @@
+"""Prefill and decode throughput of a Tuvutar model beside the closest model of this package at equal sizes (`bench.py --model tuvutar`).
+
+The closest model is Kimi-K3's layer stack without experts and with a plain residual: latent attention between delta-rule layers and
+dense gated MLPs in bf16 (its delta layers decay per key channel, its latent layers carry an output gate).  Both get the same width,
+head counts and sizes, layer order, feed-forward in every layer, vocabulary, bf16 weights and caches, random weights, synthetic
+prompts, and run through the same engine: `prefill` is the device time of the scheduler's prompt steps (CUDA events around
+LLM.step), `decode` the replay of one decode step on resident inputs (graph + lm_head + sampling)."""
+from __future__ import annotations
+
+import json
+
+
+def sizes(name):
+    return {"small": dict(width=2048, heads=16, groups=4, ff=6144, vocab=32768), "medium": dict(width=4096, heads=32, groups=2, ff=12288, vocab=65536),
+            "large": dict(width=7168, heads=56, groups=1, ff=18432, vocab=65536)}[name]
+
+
+def tuvutar_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import ModelConfig, _delta_spec, _latent_spec
+    layers = []
+    for _ in range(groups):
+        layers.append(_latent_spec(heads, 128, 64, 128, 512, ff, base=1e6))
+        layers += [_delta_spec(heads, heads, 128, 128, 4, ff=ff) for _ in range(3)]
+    return ModelConfig.from_dict({"architecture": "Tuvutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers})
+
+
+def kimi_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import tiny_kimi_k3
+    return tiny_kimi_k3(vocab_size=vocab, hidden_size=width, num_hidden_layers=4 * groups, num_attention_heads=heads, num_key_value_heads=heads,
+                        q_lora_rank=None, kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128, intermediate_size=ff,
+                        n_routed_experts=0, n_shared_experts=0, layer_types=["full_attention", "linear_attention", "linear_attention", "linear_attention"] * groups,
+                        linear_num_key_heads=heads, linear_num_value_heads=heads, linear_key_head_dim=128, linear_value_head_dim=128, attn_res_block_size=0,
+                        routed_expert_hidden_size=0, max_position_embeddings=16384)
+
+
+def measure(mc, seqs, prompt, steps, warmup, seed=0):
+    import torch
+    from nanoengine_b200 import Config, LLM, SamplingParams
+    new = warmup + steps + 8
+    pages = (prompt + new + 63) // 64 + 1
+    llm = LLM(Config(model="bench", model_config=mc, dummy_weight=True, dtype="bfloat16", device="cuda", max_num_seqs=seqs, max_num_batched_tokens=8192,
+                     max_model_len=prompt + new + 64, num_kvcache_blocks=seqs * pages + 8, enable_prefix_caching=False, cuda_graph_max_bs=seqs, seed=seed,
+                     executor_backend="inproc", status_log_interval_s=0))
+    g = torch.Generator().manual_seed(1)
+    sp = SamplingParams(temperature=0.0, max_tokens=new, ignore_eos=True)
+    for _ in range(seqs):
+        llm.add_request(torch.randint(0, mc.vocab_size, (prompt,), generator=g).tolist(), sp)
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    sch, ms, toks, prev, n = llm.engine.scheduler, 0.0, 0, 0, 0
+    while sch.num_waiting() > 0 or sch.num_prefilling(0) > 0:
+        torch.cuda.synchronize()
+        e0.record()
+        llm.step()
+        e1.record()
+        e1.synchronize()
+        done = sch.metrics_summary()["prompt_tokens"]
+        if n >= 3:                                       # the first steps warm up
+            ms += e0.elapsed_time(e1)
+            toks += done - prev
+        prev, n = done, n + 1
+    for _ in range(max(3, warmup)):
+        llm.step()
+    runner = llm.engine.executor.runner
+    same, launches, step = runner.graph_step_equals_eager(), runner.count_step_launches(), runner.make_resident_decode_step()
+    for _ in range(3):
+        step()
+    torch.cuda.synchronize()
+    e0.record()
+    for _ in range(steps):
+        step()
+    e1.record()
+    e1.synchronize()
+    dev = e0.elapsed_time(e1) / steps
+    llm.shutdown()
+    del llm, runner, step
+    import gc
+    gc.collect()
+    torch.cuda.empty_cache()
+    return {"prefill_tok_s": round(toks / ms * 1e3, 1) if ms else None, "decode_tok_s": round(seqs / dev * 1e3, 1), "decode_ms": round(dev, 3),
+            "launches_per_step": launches, "graph_equals_eager": same}
+
+
+def main(args):
+    import threading
+    import torch
+    import bench
+    torch.cuda.set_device(0)
+    stop, samples = threading.Event(), []
+    th = threading.Thread(target=bench._clock_sampler, args=(stop, samples), daemon=True)
+    th.start()
+    rows = []
+    for name in args.sizes.split(","):
+        s = sizes(name)
+        for seqs, prompt in ((128, 2048), (16, 8192)):
+            rows.append({"size": name, **s, "seqs": seqs, "prompt": prompt, "tuvutar": measure(tuvutar_model(**s), seqs, prompt, args.steps, args.warmup),
+                         "kimi_k3_stack": measure(kimi_model(**s), seqs, prompt, args.steps, args.warmup) if not args.skip_closest else None})
+    stop.set()
+    th.join(timeout=2)
+    first = rows[0]["tuvutar"]
+    print(json.dumps({"metric": "Tuvutar decode out tok/s at the first size (prefill and the closest model in rows)", "value": first["decode_tok_s"],
+                      "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": first["decode_ms"], "higher_is_better": True,
+                      "vs_baseline": None, "dtype": "bf16", "data": "synthetic uniform-random token ids, random-init weights",
+                      "config": {"model": "tuvutar", "l2": "weights and states streamed every step exceed L2; no flush"}, "rows": rows,
+                      "clocks": bench._summarise_clocks(samples), "impl": "ours"}))
+    return 0

@@ -237,6 +237,58 @@ def case_absorb(T, which, H=128, nope=128, rope=64, R=512, v=128):
     return fn, w.numel() * 2 + T * H * (w.shape[1] + w.shape[2]) * 2, 2.0 * T * H * w.shape[1] * w.shape[2]
 
 
+def case_delta(B, q_len=1, Hk=16, Hv=32, Dk=128, Dv=128, K=4):
+    """The 32-bit gated delta mixer between its projections (prepare, scan, output norm).  Floor in a decode step: the fp32 state read
+    and written once; in a prompt: the projections in, the result out."""
+    T, C = B * q_len, 2 * Hk * Dk + Hv * Dv
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    kw = dict(proj=torch.randn(T, C + Hv * Dv, **bf), ab=torch.randn(T, 2 * Hv, device="cuda"), conv_w=(torch.randn(C, K, device="cuda") * 0.3).to(torch.bfloat16),
+              A_log=torch.rand(Hv, device="cuda"), dt_bias=torch.randn(Hv, device="cuda") - 2, norm_w=torch.ones(Dv, **bf),
+              window=torch.zeros(B + 1, K - 1, C, **bf), state=torch.randn(B + 1, Hv, Dv, Dk, device="cuda") * 0.1,
+              slots=torch.arange(B, device="cuda", dtype=torch.int32), cu_seqlens=(torch.arange(B + 1, device="cuda") * q_len).to(torch.int32),
+              fresh=torch.zeros(B, dtype=torch.int32, device="cuda"), Hk=Hk, Hv=Hv, Dk=Dk, Dv=Dv, eps=1e-6, max_q_len=q_len)
+    nbytes = B * Hv * Dv * Dk * 4 * 2 + T * (C + 2 * Hv * Dv) * 2 + T * 2 * Hv * 4 + B * (K - 1) * C * 2 * 2
+    return lambda: sm100.gated_delta(**kw), nbytes, 2.0 * T * Hv * Dv * Dk * 4
+
+
+def case_latent(B, ctx, H=32, R=512, rope=64, q_len=1, page=64):
+    """Absorbed latent attention over bf16 pages.  64-token pages take the tcgen05 kernel, other page sizes the generic one."""
+    nb, D, T = (ctx + page - 1) // page, R + rope, B * q_len
+    cache = torch.randn(B * nb + 1, page, D, device="cuda").to(torch.bfloat16)
+    bt = torch.arange(B * nb, device="cuda", dtype=torch.int32).view(B, nb)
+    q = torch.randn(T, H, D, device="cuda").to(torch.bfloat16)
+    cu = (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    cl = torch.full((B,), ctx, dtype=torch.int32, device="cuda")
+    fn = lambda: sm100_attn.mla_attention_paged(q, cache, bt, cu, cl, D ** -0.5, R, max_q_len=q_len)
+    causal = ctx - (q_len - 1) / 2.0
+    return fn, B * ctx * D * 2 + T * H * (D + R) * 2, 2.0 * T * H * causal * (D + R)
+
+
+def case_rows(kind, T, W=4096, H=32, nope=128, rope=64, R=512):
+    """Row kernels around the residual stream and the latent rows, and their 16-bit counterparts."""
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    y, w = torch.randn(T, W, **bf), torch.randn(W, **bf)
+    if kind == "residual_norm":
+        x = torch.randn(T, W, device="cuda")
+        return lambda: sm100.residual_norm(y, x, w, w, 1e-6), T * W * (2 + 4 + 4 + 2), 0.0
+    if kind == "add_rmsnorm":
+        x = torch.randn(T, W, **bf)
+        return lambda: sm100.add_rmsnorm(y, x, w, 1e-6), T * W * 2 * 4, 0.0
+    table = torch.randn(8192, rope, device="cuda")
+    pos = torch.arange(T, device="cuda") % 8192
+    a = torch.randn(T, H * (nope + rope) + R + rope, **bf)
+    q, kv = a[:, : H * (nope + rope)].unflatten(-1, (H, nope + rope)), a[:, H * (nope + rope):]
+    nw, cache = torch.ones(R, **bf), torch.zeros(T // 64 + 2, 64, R + rope, **bf)
+    full = torch.empty(T, H, R + rope, **bf)
+    nbytes = T * (R + rope) * 2 * 2 + T * H * rope * 2 * 2
+
+    def separate():
+        sm100.mla_kv_prepare(kv, nw, 1e-6, pos, table, cache, pos, R)
+        sm100.apply_rope(q[..., nope:], pos, table, True, full[..., R:])
+
+    return (separate if kind == "mla_kv_prepare_rope" else lambda: sm100.latent_prepare(q, nope, kv, nw, 1e-6, pos, table, cache, pos, R, full)), nbytes, 0.0
+
+
 def case_gdn(B, q_len=1, Hk=16, Hv=32, Dk=128, Dv=128, K=4):
     """Gated delta-net layer core at the Qwen3.5-MoE shape: conv over [q|k|v] with window shift, then the recurrent step with the gated
     norm.  The floor is one read and one write of every sequence's fp32 state."""
@@ -254,13 +306,14 @@ def case_gdn(B, q_len=1, Hk=16, Hv=32, Dk=128, Dv=128, K=4):
     fresh = torch.zeros(B, dtype=torch.int32, device="cuda")
     A_log, dtb = torch.rand(Hv, device="cuda"), torch.randn(Hv, device="cuda")
     nw = torch.ones(Dv, **bf)
+    cu_host = [i * q_len for i in range(B + 1)]
 
     def fn():
         y = sm100.gdn_conv(qkv, w, conv, slots, cu, fresh, q_len == 1)
         q = y[:, : Hk * Dk].view(T, Hk, Dk)
         k = y[:, Hk * Dk: 2 * Hk * Dk].view(T, Hk, Dk)
         v = y[:, 2 * Hk * Dk:].view(T, Hv, Dv)
-        return sm100.gdn_recurrent(q, k, v, ab[:, :Hv], ab[:, Hv:], A_log, dtb, state, slots, cu, fresh, z, nw, 1e-6, q_len, None)
+        return sm100.gdn_recurrent(q, k, v, ab[:, :Hv], ab[:, Hv:], A_log, dtb, state, slots, cu, fresh, z, nw, 1e-6, q_len, cu_host)
 
     nbytes = B * Hv * Dv * Dk * 4 * 2 + T * (C * 2 * 3 + Hv * Dv * 2 * 2) + B * (K - 1) * C * 2 * 2
     return fn, nbytes, 2.0 * T * Hv * Dv * Dk * 3
@@ -348,6 +401,28 @@ def build_cases(args):
         "absorb_v_decode": lambda: case_absorb(128, "v"),
         "gdn_decode": lambda: case_gdn(128),
         "gdn_verify2": lambda: case_gdn(128, q_len=2),
+        "gdn_prefill_4x2048": lambda: case_gdn(4, q_len=2048),
+        "gdn_prefill_1x8192": lambda: case_gdn(1, q_len=8192),
+        "delta_decode": lambda: case_delta(128),
+        "delta_decode_16": lambda: case_delta(16),
+        "delta_prefill_4x2048": lambda: case_delta(4, q_len=2048),
+        "delta_prefill_1x8192": lambda: case_delta(1, q_len=8192),
+        "latent_bf16_decode": lambda: case_latent(128, args.ctx),
+        "latent_bf16_decode_h128": lambda: case_latent(128, args.ctx, H=128),
+        "latent_bf16_decode_16x8192": lambda: case_latent(16, 8192),
+        "latent_bf16_decode_r128": lambda: case_latent(128, args.ctx, H=16, R=128, rope=16),
+        "latent_bf16_chunk_2048": lambda: case_latent(1, 8192, q_len=2048),
+        "latent_bf16_chunk_r256": lambda: case_latent(1, 8192, H=32, R=256, rope=64, q_len=2048),
+        "latent_generic_decode": lambda: case_latent(128, args.ctx, page=32),
+        "residual_norm_decode": lambda: case_rows("residual_norm", 128),
+        "residual_norm_prefill": lambda: case_rows("residual_norm", 8192),
+        "add_rmsnorm_decode": lambda: case_rows("add_rmsnorm", 128),
+        "add_rmsnorm_prefill": lambda: case_rows("add_rmsnorm", 8192),
+        "latent_prepare_decode": lambda: case_rows("latent_prepare", 128),
+        "latent_prepare_prefill": lambda: case_rows("latent_prepare", 8192),
+        "kv_prepare_rope_decode": lambda: case_rows("mla_kv_prepare_rope", 128),
+        "kv_prepare_rope_prefill": lambda: case_rows("mla_kv_prepare_rope", 8192),
+        "mla_fp8_decode_h32": lambda: case_mla(128, args.ctx, H=32),
         "kda_decode_256": lambda: case_kda(256),
         "kda_prefill_2048": lambda: case_kda(8, q_len=2048),
         "attn_res_decode": lambda: case_attn_res(128),
