@@ -40,8 +40,21 @@ __device__ __forceinline__ int seq_of(const int* cu, int B, int t) {
   return lo;
 }
 
+__device__ __forceinline__ float2 ldd2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 ldd2(const __nv_bfloat16* p) { return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p)); }
+__device__ __forceinline__ void ldd4(const float* p, float* o) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+}
+__device__ __forceinline__ void ldd4(const __nv_bfloat16* p, float* o) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 x = unpack_bf16x2(u.x), y = unpack_bf16x2(u.y);
+  o[0] = x.x; o[1] = x.y; o[2] = y.x; o[3] = y.y;
+}
+
 // One warp per (token, unit): units [0, Hk) are key heads (q and k), [Hk, Hk + Hv) value heads.  KT: taps (0 = any number).
-template <typename T, int KT>
+// V = 2 (four taps, even head sizes and strides): a lane takes two neighbouring channels at a time.
+template <typename T, int KT, int V>
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   const int units = a.Hk + a.Hv, lane = threadIdx.x & 31, K = KT ? KT : a.K, C = a.C;
@@ -68,24 +81,55 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a) {
     }
     return silu_exact(acc);
   };
+  auto conv2 = [&](int c) {                  // channels c and c + 1, four taps
+    float w0[4], w1[4];
+    ldd4(w + (long long)c * 4, w0); ldd4(w + (long long)c * 4 + 4, w1);
+    float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const int back = 3 - j;
+      float2 v = make_float2(0.f, 0.f);
+      if (back <= p) v = ldd2(x - back * a.proj_ld + c);
+      else if (carried) v = ldd2(win + (long long)(p + j) * C + c);
+      a0 += v.x * w0[j]; a1 += v.y * w1[j];
+    }
+    return make_float2(silu_exact(a0), silu_exact(a1));
+  };
   if (u < a.Hk) {
     const int Dk = a.Dk, q0 = u * Dk, k0 = a.Hk * Dk + u * Dk;
     float* qo = a.qn + ((long long)t * a.Hk + u) * Dk;
     float* ko = a.kn + ((long long)t * a.Hk + u) * Dk;
     float qq = 0.f, kk = 0.f, qk = 0.f;
-    for (int c = lane; c < Dk; c += 32) {
-      const float qv = conv(q0 + c), kv = conv(k0 + c);
-      qo[c] = qv; ko[c] = kv;
-      qq += qv * qv; kk += kv * kv; qk += qv * kv;
+    if constexpr (V == 2) {
+      for (int c = lane * 2; c < Dk; c += 64) {
+        const float2 qv = conv2(q0 + c), kv = conv2(k0 + c);
+        *reinterpret_cast<float2*>(qo + c) = qv; *reinterpret_cast<float2*>(ko + c) = kv;
+        qq += qv.x * qv.x + qv.y * qv.y; kk += kv.x * kv.x + kv.y * kv.y; qk += qv.x * kv.x + qv.y * kv.y;
+      }
+    } else {
+      for (int c = lane; c < Dk; c += 32) {
+        const float qv = conv(q0 + c), kv = conv(k0 + c);
+        qo[c] = qv; ko[c] = kv;
+        qq += qv * qv; kk += kv * kv; qk += qv * kv;
+      }
     }
     qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
     const float qr = rsqrtf(qq + 1e-6f) * rsqrtf((float)Dk), kr = rsqrtf(kk + 1e-6f);
-    for (int c = lane; c < Dk; c += 32) { qo[c] *= qr; ko[c] *= kr; }       // a lane rereads its own stores
+    if constexpr (V == 2) {                                                  // a lane rereads its own stores
+      for (int c = lane * 2; c < Dk; c += 64) {
+        float2 *q2 = reinterpret_cast<float2*>(qo + c), *k2 = reinterpret_cast<float2*>(ko + c);
+        const float2 qv = *q2, kv = *k2;
+        *q2 = make_float2(qv.x * qr, qv.y * qr); *k2 = make_float2(kv.x * kr, kv.y * kr);
+      }
+    } else {
+      for (int c = lane; c < Dk; c += 32) { qo[c] *= qr; ko[c] *= kr; }
+    }
     if (lane == 0) a.gates[(long long)t * (2 * a.Hv + a.Hk) + 2 * a.Hv + u] = qk * qr * kr;
   } else {
     const int h = u - a.Hk, Dv = a.Dv, v0 = 2 * a.Hk * a.Dk + h * Dv;
     float* vo = a.vn + ((long long)t * a.Hv + h) * Dv;
-    for (int c = lane; c < Dv; c += 32) vo[c] = conv(v0 + c);
+    if constexpr (V == 2) { for (int c = lane * 2; c < Dv; c += 64) *reinterpret_cast<float2*>(vo + c) = conv2(v0 + c); }
+    else { for (int c = lane; c < Dv; c += 32) vo[c] = conv(v0 + c); }
     if (lane == 0) {
       const float av = a.ab[(long long)t * a.ab_ld + h] + a.dt_bias[h], bv = a.ab[(long long)t * a.ab_ld + a.Hv + h];
       const float sp = av > 20.f ? av : log1pf(expf(av));
@@ -100,11 +144,11 @@ __device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
 }
 
-constexpr int kScanChunk = 8;      // tokens staged at a time (two chunks in flight)
+constexpr int kScanChunk = 16;     // tokens staged at a time (two chunks in flight)
 
 // grid = (Hv * splits, B), NW = blockDim.x / 32 warps of 4 R rows each; `splits` CTAs share a head's Dv rows.
 template <int CPL, int R, bool kFuse, typename T>
-__global__ void __launch_bounds__(kFuse ? 256 : 128, kFuse ? (CPL * R >= 40 ? 2 : 4) : (CPL * R >= 40 ? 4 : CPL * R >= 24 ? 6 : 8))
+__global__ void __launch_bounds__(kFuse ? 256 : 128, kFuse ? (CPL * R >= 40 ? 2 : CPL * R >= 32 ? 3 : 4) : (CPL * R >= 40 ? 4 : CPL * R >= 24 ? 6 : 8))
 delta_scan_kernel(const DeltaArgs a) {
   constexpr int DKP = CPL * 8;                 // columns a row is padded to
   extern __shared__ float sm[];
@@ -112,7 +156,7 @@ delta_scan_kernel(const DeltaArgs a) {
   const int splits = gridDim.x / a.Hv, h = blockIdx.x / splits, row0 = (blockIdx.x % splits) * rows, hk = h / (a.Hv / a.Hk);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cg = lane & 7, rg = lane >> 3;
   const int Dk = a.Dk, Dv = a.Dv, seq = blockIdx.y;
-  // per buffer: k [8][DKP] | q [8][DKP] | v [8][rows] | gates [8][4]
+  // per buffer (n = kScanChunk tokens): k [n][DKP] | q [n][DKP] | v [n][rows] | gates [n][4]
   const int buf_floats = kScanChunk * (2 * DKP + rows + 4);
   // columns past Dk stay zero: the copies below never touch them
   if (Dk < DKP)
@@ -120,11 +164,11 @@ delta_scan_kernel(const DeltaArgs a) {
       const int c = i % (DKP - Dk), r = i / (DKP - Dk);            // r: (buffer, k or q, token)
       sm[(r / (2 * kScanChunk)) * buf_floats + (r % (2 * kScanChunk)) * DKP + Dk + c] = 0.f;
     }
-  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  // The step's tables and the state were written before delta_prepare began (it triggers behind its own wait and writes none of
+  // them), so they are fetched while it still runs; only what it produces waits for it below.
   const int start = a.cu[seq], n = a.cu[seq + 1] - start;
-  if (n <= 0) return;
   const int slot = a.slots[seq];
-  if (!NE_INDEX_OK(slot, BK_STATE_SLOTS, 44, __LINE__)) return;
+  if (n <= 0 || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 44, __LINE__)) { pdl_wait(); return; }
   const bool is_fresh = a.fresh[seq] != 0;
 
   const bool vec = (Dk & 3) == 0;
@@ -157,7 +201,6 @@ delta_scan_kernel(const DeltaArgs a) {
     }
     cp_async_commit();
   };
-  stage(0, 0);
 
   // state rows of this thread: row0 + warp * 4R + r * 4 + rg; columns j * 32 + cg * 4 + {0..3}
   float* Sg = a.state + (((long long)slot * a.Hv + h) * Dv) * Dk;
@@ -177,6 +220,9 @@ delta_scan_kernel(const DeltaArgs a) {
       S[r][4 * j] = v.x; S[r][4 * j + 1] = v.y; S[r][4 * j + 2] = v.z; S[r][4 * j + 3] = v.w;
     }
   }
+  pdl_wait();
+  if (kFuse) pdl_trigger();       // a long scan triggers at its end
+  stage(0, 0);
   // the convolution window after this call: the last K - 1 inputs (older entries move up where the call is shorter)
   {
     const int K = a.K, C = a.C;
@@ -265,6 +311,7 @@ delta_scan_kernel(const DeltaArgs a) {
     }
     __syncthreads();          // everyone is done with this buffer before the next-but-one chunk is copied into it
   }
+  if (!kFuse) pdl_trigger();
 #pragma unroll
   for (int r = 0; r < R; r++) {
     const int row = row0 + warp * 4 * R + r * 4 + rg;
@@ -279,8 +326,8 @@ delta_scan_kernel(const DeltaArgs a) {
   }
 }
 
-// one warp per (token, head)
-template <typename T>
+// one warp per (token, head); V = 4: head size, strides and addresses allow groups of four
+template <typename T, int V>
 __global__ void __launch_bounds__(256) delta_out_norm_kernel(const DeltaArgs a) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   const long long row = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -290,6 +337,22 @@ __global__ void __launch_bounds__(256) delta_out_norm_kernel(const DeltaArgs a) 
   const float* o = a.raw + row * Dv;
   const T* z = reinterpret_cast<const T*>(a.proj) + t * a.proj_ld + a.C + h * Dv;
   float ss = 0.f;
+  if (V == 4 && Dv <= 128) {                 // one group of four per lane, held in registers
+    const bool on = lane * 4 < Dv;
+    const float4 f = on ? *reinterpret_cast<const float4*>(o + lane * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float r = rsqrtf(warp_sum(f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w) / (float)Dv + a.eps);
+    if (on) {
+      float zz[4], ww[4];
+      ldd4(z + lane * 4, zz); ldd4(reinterpret_cast<const T*>(a.norm_w) + lane * 4, ww);
+      T y[4];
+      std_(y, f.x * r * ww[0] * silu_exact(zz[0])); std_(y + 1, f.y * r * ww[1] * silu_exact(zz[1]));
+      std_(y + 2, f.z * r * ww[2] * silu_exact(zz[2])); std_(y + 3, f.w * r * ww[3] * silu_exact(zz[3]));
+      T* dst = reinterpret_cast<T*>(a.out) + row * Dv + lane * 4;
+      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<uint2*>(y);
+      else *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<uint4*>(y);
+    }
+    return;
+  }
   for (int d = lane; d < Dv; d += 32) { const float f = o[d]; ss += f * f; }
   const float r = rsqrtf(warp_sum(ss) / (float)Dv + a.eps);
   for (int d = lane; d < Dv; d += 32)
@@ -305,14 +368,22 @@ static int scan(const DeltaArgs& a, int warps, cudaStream_t st) {
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return (int)launch_pdl(k, dim3((unsigned)(a.Hv * splits), (unsigned)a.B), dim3((unsigned)(warps * 32)), smem, st, a);
+  const dim3 grid((unsigned)(a.Hv * splits), (unsigned)a.B), block((unsigned)(warps * 32));
+  if (kFuse) return (int)launch_pdl(k, grid, block, smem, st, a);
+  // A prompt's scan is a few long CTAs.  A dependent launch would place them while delta_prepare drains, several on the first SMs that
+  // have room, and leave the others empty for the whole scan (2.5 times as long for one 8192-token prompt); an ordinary launch
+  // spreads them over the machine.
+  k<<<grid, block, smem, st>>>(a);
+  return (int)cudaGetLastError();
 }
 
 template <typename T>
 static int delta_t(const DeltaArgs& a, int max_q, cudaStream_t st) {
   const long long warps = (long long)a.T * (a.Hk + a.Hv);
   const dim3 pgrid((unsigned)((warps + 7) / 8));
-  cudaError_t e = a.K == 4 ? launch_pdl(delta_prepare_kernel<T, 4>, pgrid, dim3(256), 0, st, a) : launch_pdl(delta_prepare_kernel<T, 0>, pgrid, dim3(256), 0, st, a);
+  const bool pairs = a.K == 4 && a.Dk % 2 == 0 && a.Dv % 2 == 0 && a.proj_ld % 2 == 0 && ((uintptr_t)a.proj | (uintptr_t)a.window | (uintptr_t)a.conv_w) % 16 == 0;
+  auto prep = pairs ? delta_prepare_kernel<T, 4, 2> : a.K == 4 ? delta_prepare_kernel<T, 4, 1> : delta_prepare_kernel<T, 0, 1>;
+  cudaError_t e = launch_pdl(prep, pgrid, dim3(256), 0, st, a);
   if (e != cudaSuccess) return (int)e;
   int rc;
   // whole heads per CTA (norm and gate in the same kernel) for single-token steps whose state fits the registers of 8 warps
@@ -337,7 +408,8 @@ static int delta_t(const DeltaArgs& a, int max_q, cudaStream_t st) {
 #undef NE_SCAN
   if (rc) return rc;
   const long long orows = (long long)a.T * a.Hv;
-  return (int)launch_pdl(delta_out_norm_kernel<T>, dim3((unsigned)((orows + 7) / 8)), dim3(256), 0, st, a);
+  const bool fours = a.Dv % 4 == 0 && a.C % 4 == 0 && a.proj_ld % 4 == 0 && ((uintptr_t)a.proj | (uintptr_t)a.norm_w | (uintptr_t)a.out) % 16 == 0;
+  return (int)launch_pdl(fours ? delta_out_norm_kernel<T, 4> : delta_out_norm_kernel<T, 1>, dim3((unsigned)((orows + 7) / 8)), dim3(256), 0, st, a);
 }
 
 }  // namespace ne

@@ -129,9 +129,15 @@ __global__ void __launch_bounds__(256) glu_rows_kernel(const T* __restrict__ x, 
   }
 }
 
+__device__ __forceinline__ float2 ldx2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 ldx2(const __nv_bfloat16* p) { return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p)); }
+__device__ __forceinline__ void stx2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void stx2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(a, b); }
+
 // One warp per (token, unit): unit 0 .. H-1 rotates the rotary tail of that query head (q -> dst), unit H (when kv is given) writes the
 // token's cache row.  kv_kind: 0 bf16 rows, 1 e4m3 rows (clamped cast of the bf16 value), 2 fp32 rows.
-template <typename T>
+// kPairs: R, the strides and the addresses allow two elements per access.
+template <typename T, bool kPairs>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q, long long q_ld, int q_hs, T* dst, long long d_ld, int d_hs, int H, const T* __restrict__ kv,
                                                             long long kv_ld, const T* __restrict__ w, float eps, const long long* __restrict__ positions,
                                                             const float* __restrict__ rope_cache, void* __restrict__ cache,
@@ -146,9 +152,15 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q, long lo
     const T* p = q + (long long)t * q_ld + (long long)u * q_hs;        // may be the destination itself
     T* o = dst + (long long)t * d_ld + (long long)u * d_hs;
     for (int i = lane; i < half; i += 32) {
-      const float a = ldx(p + 2 * i), b = ldx(p + 2 * i + 1), c = cs[i], s = cs[half + i];
-      stx(o + 2 * i, a * c - b * s);
-      stx(o + 2 * i + 1, b * c + a * s);
+      const float c = cs[i], s = cs[half + i];
+      if constexpr (kPairs) {
+        const float2 v = ldx2(p + 2 * i);
+        stx2(o + 2 * i, v.x * c - v.y * s, v.y * c + v.x * s);
+      } else {
+        const float a = ldx(p + 2 * i), b = ldx(p + 2 * i + 1);
+        stx(o + 2 * i, a * c - b * s);
+        stx(o + 2 * i + 1, b * c + a * s);
+      }
     }
     return;
   }
@@ -156,7 +168,8 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q, long lo
   if (slot < 0 || !NE_INDEX_OK(slot, BK_CACHE_ROWS, 41, __LINE__)) return;
   const T* row = kv + (long long)t * kv_ld;
   float ss = 0.f;
-  for (int c = lane; c < R; c += 32) { const float f = ldx(row + c); ss += f * f; }
+  if constexpr (kPairs) { for (int c = lane * 2; c < R; c += 64) { const float2 f = ldx2(row + c); ss += f.x * f.x + f.y * f.y; } }
+  else { for (int c = lane; c < R; c += 32) { const float f = ldx(row + c); ss += f * f; } }
   const float r = rsqrtf(warp_sum(ss) / (float)R + eps);
   auto put = [&](int c, float v) {
     const long long o = slot * (R + rope) + c;
@@ -164,6 +177,19 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q, long lo
     else if (kv_kind == 1) reinterpret_cast<uint8_t*>(cache)[o] = to_e4m3(__bfloat162float(__float2bfloat16(v)));
     else reinterpret_cast<__nv_bfloat16*>(cache)[o] = __float2bfloat16(v);
   };
+  if (kPairs && kv_kind != 1) {
+    T* dst = reinterpret_cast<T*>(cache) + slot * (R + rope);
+    for (int c = lane * 2; c < R; c += 64) {
+      const float2 f = ldx2(row + c), g = ldx2(w + c);
+      stx2(dst + c, f.x * r * g.x, f.y * r * g.y);
+    }
+    for (int i = lane; i < half; i += 32) {
+      const float2 v = ldx2(row + R + 2 * i);
+      const float c = cs[i], s = cs[half + i];
+      stx2(dst + R + 2 * i, v.x * c - v.y * s, v.y * c + v.x * s);
+    }
+    return;
+  }
   for (int c = lane; c < R; c += 32) put(c, ldx(row + c) * r * ldx(w + c));
   for (int i = lane; i < half; i += 32) {
     const float a = ldx(row + R + 2 * i), b = ldx(row + R + 2 * i + 1), c = cs[i], s = cs[half + i];
@@ -238,12 +264,14 @@ extern "C" int ne_latent_prepare(const void* q, long long q_ld, int q_hs, void* 
   if (rope < 0 || rope % 2 || R <= 0 || kv_kind < 0 || kv_kind > 2 || (fp32 != 0) != (kv_kind == 2)) return 1001;
   const long long warps = (long long)T * (H + (kv ? 1 : 0));
   const dim3 grid((unsigned)((warps + 7) / 8));
+  const bool pairs = R % 2 == 0 && q_ld % 2 == 0 && q_hs % 2 == 0 && d_ld % 2 == 0 && d_hs % 2 == 0 && kv_ld % 2 == 0 &&
+                     ((uintptr_t)q | (uintptr_t)dst | (uintptr_t)kv | (uintptr_t)w | (uintptr_t)cache) % (fp32 ? 8 : 4) == 0;
   if (fp32)
-    return (int)launch_pdl(latent_prepare_kernel<float>, grid, dim3(256), 0, st, (const float*)q, q_ld, q_hs, (float*)dst, d_ld, d_hs, H, (const float*)kv, kv_ld, (const float*)w, eps,
-                           positions, rope_cache, cache, slots, T, R, rope, kv_kind);
-  return (int)launch_pdl(latent_prepare_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)q, q_ld, q_hs, (__nv_bfloat16*)dst, d_ld, d_hs, H,
-                         (const __nv_bfloat16*)kv, kv_ld,
-                         (const __nv_bfloat16*)w, eps, positions, rope_cache, cache, slots, T, R, rope, kv_kind);
+    return (int)launch_pdl(pairs ? latent_prepare_kernel<float, true> : latent_prepare_kernel<float, false>, grid, dim3(256), 0, st, (const float*)q, q_ld, q_hs,
+                           (float*)dst, d_ld, d_hs, H, (const float*)kv, kv_ld, (const float*)w, eps, positions, rope_cache, cache, slots, T, R, rope, kv_kind);
+  return (int)launch_pdl(pairs ? latent_prepare_kernel<__nv_bfloat16, true> : latent_prepare_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, st,
+                         (const __nv_bfloat16*)q, q_ld, q_hs, (__nv_bfloat16*)dst, d_ld, d_hs, H, (const __nv_bfloat16*)kv, kv_ld, (const __nv_bfloat16*)w, eps,
+                         positions, rope_cache, cache, slots, T, R, rope, kv_kind);
 }
 
 extern "C" int ne_latent_gather(const void* cache, const long long* slots, void* rows, int T, int row_bytes, cudaStream_t st) {

@@ -698,8 +698,18 @@ class ModelRunner:
         ctx, temps = self._last_decode
         ids, pos = ctx.extras["input_ids"], ctx.extras["positions"]
         rows = ctx.last_token_indices.long()
+        # the step moves per-sequence state on: both runs start from the same one, and what was there before comes back afterwards
+        states = [t for t in (self.cache.rec_states or []) + (self.cache.conv_states or [])] if self.plan.gdn else []
+        saved = [t[ctx.state_slots.long()].clone() for t in states]
+
+        def restore():
+            for t, s in zip(states, saved):
+                t[ctx.state_slots.long()] = s
+
         a = self.sampler(self.model.compute_logits(self.forward(ctx)[rows]), torch.zeros_like(temps), False)[0]
+        restore()
         b = self.sampler(self.model.compute_logits(self.model(ids, pos, ctx)[rows]), torch.zeros_like(temps), False)[0]
+        restore()
         return bool(torch.equal(a, b))
 
     @torch.inference_mode()
