@@ -15,6 +15,7 @@ buffers, shared pool, capture per size, run).
 """
 from __future__ import annotations
 
+import gc
 from typing import Dict, List
 
 import torch
@@ -122,8 +123,16 @@ class DecodeGraphRunner:
         torch.cuda.current_stream().wait_stream(s)
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g, pool=self.pool):
-            out = self.r.model(ids, pos, sctx)
+        # no cycle collection inside a capture: an engine that died earlier in this process would free its graphs and caches there,
+        # which invalidates the capture
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(g, pool=self.pool):
+                out = self.r.model(ids, pos, sctx)
+        finally:
+            if collecting:
+                gc.enable()
         if self.pool is None:
             self.pool = g.pool()
         self.graphs[b], self.outputs[b] = g, out

@@ -237,6 +237,16 @@ def test_generation_in_32_bit_equals_the_oracle_and_graphs_equal_eager(tmp_path)
     assert runner.graphs is not None and runner.graphs.graphs and runner.graph_step_equals_eager()
 
 
+def test_fp8_latent_rows(tmp_path):
+    """Cache rows as e4m3 (an option of the engine): coarse, but the same in one prompt and token by token."""
+    cfg, W, path = build("latent_only", tmp_path)
+    toks = tokens(130, cfg["vocab"], 5)
+    want = oracle.forward(cfg, W, toks)
+    llm = make_llm(path, "bfloat16", DEV, pages=4, kv_cache_dtype="fp8")
+    a, b = feed_all(llm, None, toks, [130]), feed_all(llm, None, toks, [100, 1])
+    assert error(a, want) < 0.3 and error(b, a) < 0.1
+
+
 def test_long_decoding(tmp_path):
     """Several hundred single tokens through the decode graph: states and pages carried all the way."""
     cfg, W, path = build("delta_first", tmp_path, sharp=3.0)
