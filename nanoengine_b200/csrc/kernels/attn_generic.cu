@@ -7,11 +7,13 @@
 //   GQA:  q [T, Hq, D], k/v caches [slots, Hkv, D], out [T, Hq, D]
 // Keys of a query: positions [0, limit] of its sequence through the block table (causal), or an explicit list of
 // physical slots (sparse, -1 = skip).  Cache dtype bf16, e4m3 (query is then clamped and cast to e4m3 as well) or fp32 (query and
-// output fp32 too: runs in true 32-bit).
+// output fp32 too: runs in true 32-bit).  Options: a window of the last keys, scores capped as cap tanh(s / cap), a distance bias
+// -slope[head] (query position - key position) after the cap, the output of a head times sigmoid(gate[token, head]) and a constant.
 //
 // Replaces in the reference: attention/base.py:451-525 (SDPA reference), flash_mla sparse decode call sites
 // (layers/backends/mla/flash_mla.py:22-121) for the sparse case, flashinfer / FA paged GQA wrappers.
 #include "ptx.cuh"
+#include <cstring>
 
 namespace ne {
 
@@ -31,7 +33,10 @@ struct AttnArgs {
   int T, H, Dk, Dv; float scale; int fp8;
   int window;                                     // > 0: a query sees only the last `window` key positions up to its own (sliding-window layers)
   int noncausal;                                  // 1: every query sees all keys of its sequence (vision encoder)
-  int heads_per_cta;                              // 4, or 1 when every query head has its own kv head (the CTA stages one kv head)
+  int heads_per_cta;                              // 4 or the largest smaller divisor of the group: the heads of a CTA share one kv head
+  long long v_slot_stride; int v_head_stride;     // of the separate V rows
+  float softcap; const float* slopes;             // 0 / null: none
+  const void* gate; long long gate_ld; float out_scale;      // gate null: none
 };
 
 // kind: 0 bf16, 1 e4m3, 2 fp32
@@ -76,7 +81,8 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
 #pragma unroll
   for (int j = 0; j < 20; j++) acc[j] = 0.f;
   float m_run = -INFINITY, l_run = 0.f;
-  const float c = a.scale * 1.4426950408889634f;
+  constexpr float kLog2e = 1.4426950408889634f;
+  const float c = a.scale * kLog2e, slope = (a.slopes && head_ok) ? a.slopes[h] : 0.f;
   const int* bt = a.block_tables + (long long)seq * a.bt_stride;
 
   for (int k0 = first_key / kKeysPerTile * kKeysPerTile; k0 < n_keys; k0 += kKeysPerTile) {
@@ -95,7 +101,7 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
       for (int d = lane; d < Dk; d += 32)
         sk[r * (Dk + 1) + d] = slot >= 0 ? load_kv(a.k_cache, slot * a.kv_slot_stride + (long long)kvh * a.kv_head_stride + d, a.fp8) : 0.f;
       if (sv) for (int d = lane; d < Dv; d += 32)
-        sv[r * (Dv + 1) + d] = slot >= 0 ? load_kv(a.v_cache, slot * a.kv_slot_stride + (long long)kvh * a.kv_head_stride + d, a.fp8) : 0.f;
+        sv[r * (Dv + 1) + d] = slot >= 0 ? load_kv(a.v_cache, slot * a.v_slot_stride + (long long)kvh * a.v_head_stride + d, a.fp8) : 0.f;
       if (lane == 0) sk[r * (Dk + 1) + Dk] = slot >= 0 ? 1.f : 0.f;   // validity marker in the padding column
     }
     __syncthreads();
@@ -106,7 +112,10 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
     float s = 0.f;
     for (int d = 0; d < Dk; d++) s = fmaf(qr[d], kr[d], s);
     bool valid = (k0 + lane < n_keys) && (k0 + lane >= first_key) && kr[Dk] != 0.f;
-    float tl = valid ? s * c : -INFINITY;
+    float tl = s * c;
+    if (a.softcap > 0.f) tl = a.softcap * tanhf(s * a.scale / a.softcap) * kLog2e;
+    if (a.slopes) tl -= slope * (float)(limit - (k0 + lane)) * kLog2e;
+    if (!valid) tl = -INFINITY;
     float m_new = fmaxf(m_run, warp_max(tl));
     if (m_new == -INFINITY) continue;
     float alpha = exp2f(m_run - m_new);
@@ -128,7 +137,8 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
     }
   }
   if (!head_ok) return;
-  float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+  float inv = (l_run > 0.f ? 1.f / l_run : 0.f) * a.out_scale;
+  if (a.gate) inv /= 1.f + expf(-load_kv(a.gate, (long long)t * a.gate_ld + h, a.fp8 == 2 ? 2 : 0));
 #pragma unroll
   for (int j = 0; j < 20; j++) {
     int d = lane + 32 * j;
@@ -222,6 +232,37 @@ __global__ void __launch_bounds__(1024) sample_kernel(const float* __restrict__ 
 
 using namespace ne;
 
+static int attn_generic_launch(AttnArgs& a, cudaStream_t st) {
+  const size_t smem = sizeof(float) * ((size_t)kHeadsPerCta * a.Dk + (size_t)kKeysPerTile * (a.Dk + 1) + (a.v_cache ? (size_t)kKeysPerTile * (a.Dv + 1) : 0));
+  static size_t configured = 0;
+  if (smem > 48 * 1024 && smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(attn_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  return (int)launch_pdl(attn_generic_kernel, dim3(a.T, (a.H + a.heads_per_cta - 1) / a.heads_per_cta), dim3(128), smem, st, a);
+}
+
+// Paged grouped-query attention with the options of AttnArgs: q [T, H, D], k_cache [slots, Hkv, D], v_cache [slots, Hkv, Dv] (fp32 all of
+// them when fp32 = 1, else bf16), slopes [H] or null, gate [T, >= H] (row stride gate_ld) or null, out [T, ...] with row stride o_ld and head
+// stride Dv.  window 0: all earlier keys.
+extern "C" int ne_attn_biased(const void* q, long long q_ld, const void* k_cache, const void* v_cache, const int* block_tables, int bt_stride, int block_size,
+                              const int* cu_seqlens_q, const int* context_lens, int num_seqs, void* out, long long o_ld, int T, int H, int Hkv, int D, int Dv,
+                              float scale, float softcap, const float* slopes, int window, const void* gate, long long gate_ld, float out_scale, int fp32,
+                              cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (Hkv < 1 || H % Hkv || Dv < 1 || Dv > 640 || D < 1 || D > 640) return 1001;
+  AttnArgs a;
+  memset(&a, 0, sizeof(a));
+  a.q = q; a.q_tok_stride = q_ld; a.q_head_stride = D; a.k_cache = k_cache; a.v_cache = v_cache; a.kv_slot_stride = (long long)Hkv * D; a.kv_head_stride = D;
+  a.v_slot_stride = (long long)Hkv * Dv; a.v_head_stride = Dv; a.kv_group = H / Hkv; a.block_tables = block_tables; a.bt_stride = bt_stride;
+  a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs; a.out = out; a.o_tok_stride = o_ld;
+  a.o_head_stride = Dv; a.T = T; a.H = H; a.Dk = D; a.Dv = Dv; a.scale = scale; a.fp8 = fp32 ? 2 : 0; a.window = window; a.softcap = softcap; a.slopes = slopes;
+  a.gate = gate; a.gate_ld = gate_ld; a.out_scale = out_scale;
+  for (a.heads_per_cta = kHeadsPerCta; a.kv_group % a.heads_per_cta; a.heads_per_cta--) {}
+  return attn_generic_launch(a, st);
+}
+
 extern "C" int ne_attn_generic(const void* q, long long q_tok_stride, int q_head_stride, const void* k_cache, const void* v_cache,
                                long long kv_slot_stride, int kv_head_stride, int kv_group, const int* block_tables, int bt_stride,
                                int block_size, const int* cu_seqlens_q, const int* context_lens, int num_seqs, const int* sparse, int topk,
@@ -230,23 +271,17 @@ extern "C" int ne_attn_generic(const void* q, long long q_tok_stride, int q_head
   if (T <= 0) return 0;
   if (Dv > 640 || (kv_group > 1 && kv_group % kHeadsPerCta != 0)) return 1001;
   AttnArgs a;
+  memset(&a, 0, sizeof(a));
   a.q = q; a.q_tok_stride = q_tok_stride; a.q_head_stride = q_head_stride; a.k_cache = k_cache; a.v_cache = v_cache;
   a.kv_slot_stride = kv_slot_stride; a.kv_head_stride = kv_head_stride; a.kv_group = kv_group; a.block_tables = block_tables;
   a.bt_stride = bt_stride; a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs;
   a.sparse = sparse; a.topk = topk; a.out = out; a.o_tok_stride = o_tok_stride; a.o_head_stride = o_head_stride; a.lse = lse;
   a.T = T; a.H = H; a.Dk = Dk; a.Dv = Dv; a.scale = scale; a.fp8 = fp8; a.window = window; a.noncausal = noncausal;
+  a.v_slot_stride = kv_slot_stride; a.v_head_stride = kv_head_stride; a.out_scale = 1.f;
   // multi-head attention proper (one kv head per query head, separate V): the four query heads of a CTA would need four
   // different key tiles, so a CTA serves one head there
   a.heads_per_cta = (kv_group == 1 && kv_head_stride != 0 && v_cache != nullptr) ? 1 : kHeadsPerCta;
-  size_t smem = sizeof(float) * ((size_t)kHeadsPerCta * Dk + (size_t)kKeysPerTile * (Dk + 1) + (v_cache ? (size_t)kKeysPerTile * (Dv + 1) : 0));
-  static size_t configured = 0;
-  if (smem > 48 * 1024 && smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-    configured = smem;
-  }
-  dim3 grid(T, (H + a.heads_per_cta - 1) / a.heads_per_cta);
-  return (int)launch_pdl(attn_generic_kernel, dim3(grid), dim3(128), smem, st, a);
+  return attn_generic_launch(a, st);
 }
 
 extern "C" int ne_attn_merge(const float* part, const float* lse2, void* out, int splits, long long rows, int D, int out_row_stride, cudaStream_t st) {

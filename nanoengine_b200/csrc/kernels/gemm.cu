@@ -76,6 +76,7 @@ struct GemmArgs {
   int out_fp32;                         // 0: bf16 output, 1: fp32, 2: e4m3 (clamped cast, no scale; plain bf16 GEMMs only)
   const long long* row_dst;             // optional scatter epilogue: absolute address of every output row (bf16, may be peer memory),
   long long rd_group_stride;            // indexed [group * rd_group_stride + row]; used by the MoE combine
+  const float* bias;                    // optional [N]: added to the fp32 accumulator before the result is rounded (plain bf16 GEMMs)
   GemmComm comm;                        // hooks that fuse a collective into this GEMM (all null / zero for a plain GEMM)
 };
 
@@ -826,6 +827,17 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 32; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * al);
           }
+          if (!kFp4 && !kSplit && args.bias) {
+#pragma unroll
+            for (int q = 0; q < 4; q++) {
+              if (n0 + c * 32 + q * 8 >= args.N) continue;           // N is a multiple of 8
+              const float4 b0 = __ldg(reinterpret_cast<const float4*>(args.bias + n0 + c * 32 + q * 8));
+              const float4 b1 = __ldg(reinterpret_cast<const float4*>(args.bias + n0 + c * 32 + q * 8 + 4));
+              const float b[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+#pragma unroll
+              for (int j = 0; j < 8; j++) r[q * 8 + j] = __float_as_uint(__uint_as_float(r[q * 8 + j]) + b[j]);
+            }
+          }
           if (kSplit) {
             float4* P = reinterpret_cast<float4*>(smem);
 #pragma unroll
@@ -886,6 +898,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
         for (int pr = 0; pr < split; pr++) {
           const float4 v = ld_dsmem_f4(mapa_shared(local, (uint32_t)pr));
           s4.x += v.x; s4.y += v.y; s4.z += v.z; s4.w += v.w;
+        }
+        if (args.bias) {
+          const float4 b = __ldg(reinterpret_cast<const float4*>(args.bias + n));
+          s4.x += b.x; s4.y += b.y; s4.z += b.z; s4.w += b.w;
         }
         const long long off = (long long)grow * args.ldd + n;
         if (args.out_fp32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(args.D) + off) = s4;
@@ -1083,8 +1099,9 @@ using namespace ne;
 static int gemm_impl(const void* A, long long lda, long long a_gs, const void* B, void* D, long long ldd, long long d_gs,
                      int M, int N, int K, int groups, const int* masked_m, const int* row_start, int dtype, const float* sa, int sa_ld,
                      long long sa_gs, const float* sb, int out_fp32, int block_n_hint, const long long* row_dst, const GemmComm* comm,
-                     int a_rows_total, cudaStream_t stream) {
+                     int a_rows_total, cudaStream_t stream, const float* bias = nullptr) {
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
+  if (bias && (dtype != 0 || groups != 1 || ((uintptr_t)bias & 15))) return 1012;
   if (comm) {
     if (comm->wait_flags && (groups > kSchedCache || comm->wait_world > 16 || !masked_m)) return 1007;
     if (comm->gate_flags && (groups != 1 || row_start || masked_m || comm->gate_world > 16 || comm->gate_rpr < 1)) return 1008;
@@ -1163,7 +1180,7 @@ static int gemm_impl(const void* A, long long lda, long long a_gs, const void* B
   if (row_start) { a.d_group_stride = 0; sa_gs = 0; if (!masked_m) return 1004; }
   a.sa = sa; a.sa_ld = sa_ld; a.sa_group_stride = sa_gs; a.sb = sb;
   a.sb_group_stride = (long long)((N + 127) / 128) * (K / 128); a.out_fp32 = out_fp32; a.alpha = nullptr;
-  a.row_dst = row_dst; a.rd_group_stride = row_start ? 0 : M;
+  a.row_dst = row_dst; a.rd_group_stride = row_start ? 0 : M; a.bias = bias;
   if (row_dst && out_fp32) return 1005;
   if (comm) { a.comm = *comm; if (m_blocks <= 1 || groups != 1) a.comm.mb_rot = 0; else a.comm.mb_rot %= m_blocks; }
   else memset(&a.comm, 0, sizeof(a.comm));
@@ -1217,6 +1234,12 @@ extern "C" int ne_gemm(const void* A, long long lda, long long a_gs, const void*
                    nullptr, 0, stream);
 }
 
+// One dense bf16 GEMM with a bias row: D[m, n] = sum_k A[m, k] B[n, k] + bias[n], the sum rounded once.  bias fp32 [N].
+extern "C" int ne_gemm_bias(const void* A, long long lda, const void* B, const float* bias, void* D, long long ldd, int M, int N, int K, int out_fp32,
+                            cudaStream_t stream) {
+  return gemm_impl(A, lda, 0, B, D, ldd, 0, M, N, K, 1, nullptr, nullptr, 0, nullptr, 0, 0, nullptr, out_fp32, 0, nullptr, nullptr, 0, stream, bias);
+}
+
 // The same GEMM with a collective fused in (see GemmComm).  `a_rows_total` > 0 gives the number of rows the A tensor map must
 // cover when that is more than M (the double-buffered gather area of the gated form).
 extern "C" int ne_gemm_comm(const void* A, long long lda, long long a_gs, const void* B, void* D, long long ldd, long long d_gs,
@@ -1253,7 +1276,7 @@ extern "C" int ne_gemm_nvfp4(const void* A, const void* B, void* D, long long ld
   a.d_group_stride = row_start ? 0 : (long long)M * ldd;
   a.sa = reinterpret_cast<const float*>(sfa); a.sa_group_stride = row_start ? 0 : M;      // NVFP4: byte arrays; the stride counts rows
   a.sb = reinterpret_cast<const float*>(sfb);
-  a.alpha = alpha; a.out_fp32 = out_fp32 ? 1 : 0;
+  a.alpha = alpha; a.out_fp32 = out_fp32 ? 1 : 0; a.bias = nullptr;
   a.rd_group_stride = row_start ? 0 : M;
   const long long tiles = (row_start ? (long long)m_blocks + groups : (long long)groups * m_blocks) * ((N + bn - 1) / bn);
   const int grid = (int)(tiles < num_sms() ? tiles : num_sms());

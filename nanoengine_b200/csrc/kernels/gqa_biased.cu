@@ -1,0 +1,391 @@
+// Grouped-query paged attention on tcgen05 tensor cores with per-layer options: any head sizes up to 256 in multiples of 8 (query / key and
+// value sizes may differ), any group of query heads per key / value head up to 128, a window of the last keys, capped scores
+// cap tanh(s / cap), a distance bias -slope[head] (query position - key position) taken off after the cap, and an output gate: a head's
+// output times sigmoid(gate[token, head]) and a constant.  bf16, 64-token pages; decode and prompt portions alike.
+//
+// One CTA = one KV head x one tile of (token, head of the group) rows of ONE sequence x one slice of the pages its rows can see: pages in
+// front of the tile's window are never touched.  r = token_in_tile * g + head_in_group, at most 128 rows.
+//
+// Per 64-key page:  S = Q K^T   (nc chunks x 4 tcgen05.mma kind::f16, M=128 N=64 K=16; both K-major, 128B swizzle)
+//                   cap, bias, mask and online softmax in 32-bit by 128 threads reading S from TMEM; P -> bf16 -> shared memory
+//                   O += P V    (4 x tcgen05.mma, N = 64 nv; V read MN-major)
+// A head size that is not a multiple of 64 ends in a chunk whose missing columns TMA fills with zeros.  M = 128 rows are always multiplied;
+// rows past the tile's own read whatever shared memory follows and feed accumulator rows nobody reads.
+// Warp 0: TMA producer, warp 1: MMA issuer, warps 2-5: softmax / rescale / epilogue.  All waits are bounded.
+// With more than one slice the CTA writes a normalised partial result and its log2-sum-exp; gqa_biased_merge folds them and applies the gate.
+#include "ptx.cuh"
+#include "seq_tile.cuh"
+#include "tma_host.h"
+
+namespace ne {
+
+constexpr int kGbThreads = 192;
+constexpr int kKernelGb = 13;
+constexpr int kBPage = 64;                     // keys per page
+constexpr int kBChunk = kBPage * 128;          // one 64-column chunk of a page tile: 64 rows x 128 B
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct GbArgs {
+  const int* block_tables; int bt_stride;
+  const int* cu_seqlens_q; const int* context_lens; int num_seqs;
+  int T, H, Dv, g, tq, splits;
+  int nc, nv, rows8, stages, pbufs, window;
+  uint32_t tmem_cols;
+  float scale, softcap;
+  const float* slopes;                         // [H] or null
+  const __nv_bfloat16* gate; long long gate_ld; float out_scale;
+  __nv_bfloat16* out; long long o_ld;          // row t, head h: out + t o_ld + h Dv (splits == 1)
+  float* part; float* lse2;                    // [splits, T, H, Dv], [splits, T, H] (splits > 1)
+};
+
+__device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ld, long long t, int h, float scale) {
+  return gate ? scale / (1.f + __expf(-__bfloat162float(gate[t * ld + h]))) : scale;
+}
+
+template <bool kCap>
+__global__ void __launch_bounds__(kGbThreads, 1)
+gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const GbArgs a) {
+  pdl_wait();                     // dependent launch: nothing above this line touches global memory
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int q_chunk = a.rows8 * 128, p_bytes = a.rows8 * 128, stage_bytes = (a.nc + a.nv) * kBChunk;
+  uint8_t* sQ = smem;                                    // nc chunks of rows8 x 128 B
+  uint8_t* sP = sQ + a.nc * q_chunk;
+  uint8_t* sKV = sP + a.pbufs * p_bytes;                 // MMA reads of rows past rows8 end inside the page tiles
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sKV + a.stages * stage_bytes);
+  // q_full | kv_full[4] | kv_empty[4] | s_full[2] | s_empty[2] | p_full[2] | p_empty[2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  int* s_tile = reinterpret_cast<int*>(tmem_slot + 2);
+  const uint32_t b_qfull = smem_u32(bars), b_kvfull = smem_u32(bars + 1), b_kvempty = smem_u32(bars + 5);
+  const uint32_t b_sfull = smem_u32(bars + 9), b_sempty = smem_u32(bars + 11), b_pfull = smem_u32(bars + 13), b_pempty = smem_u32(bars + 15);
+
+  const int warp = threadIdx.x >> 5;
+  const int hkv = blockIdx.y, split = blockIdx.z;
+  if (warp == 0) {
+    int seq, tok;
+    find_seq_tile(a.cu_seqlens_q, a.num_seqs, a.tq, blockIdx.x, seq, tok);
+    if (lane_id() == 0) { s_tile[0] = seq; s_tile[1] = tok; }
+  }
+  if (threadIdx.x == 0) {
+    mbar_init(b_qfull, 1);
+    for (int i = 0; i < 4; i++) { mbar_init(b_kvfull + 8 * i, 1); mbar_init(b_kvempty + 8 * i, 1); }
+    for (int i = 0; i < 2; i++) {
+      mbar_init(b_sfull + 8 * i, 1); mbar_init(b_sempty + 8 * i, 4); mbar_init(b_pfull + 8 * i, 4); mbar_init(b_pempty + 8 * i, 1);
+    }
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) { tmem_alloc(smem_u32(tmem_slot), a.tmem_cols); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  pdl_trigger();                  // behind the TMEM allocation: a CTA of the next grid never holds columns this grid waits for
+  const uint32_t tmem_base = *tmem_slot, tmem_o = tmem_base + 128;
+  const int seq = s_tile[0], tok0 = s_tile[1];
+
+  int n_tiles = 0, pg_begin = 0, n_tok = 0, base_limit = -1;
+  const int* bt = a.block_tables;
+  if (seq >= 0) {
+    const int q_beg = a.cu_seqlens_q[seq], q_len = a.cu_seqlens_q[seq + 1] - q_beg;
+    n_tok = min(a.tq, q_beg + q_len - tok0);
+    base_limit = a.context_lens[seq] - q_len + (tok0 - q_beg);              // last key visible to the tile's first token
+    const int max_limit = base_limit + n_tok - 1;
+    const int first = a.window > 0 ? max(0, base_limit - a.window + 1) / kBPage : 0;
+    const int total = max_limit >= 0 ? max_limit / kBPage + 1 - first : 0;
+    const int per_split = (total + a.splits - 1) / a.splits;
+    pg_begin = first + split * per_split;
+    n_tiles = max(0, min(first + total, pg_begin + per_split) - pg_begin);
+    bt = a.block_tables + (long long)seq * a.bt_stride;
+  }
+
+  if (warp == 0) {
+    if (n_tiles > 0 && elect_one()) {
+      mbar_expect_tx(b_qfull, a.nc * a.g * a.tq * 128);
+      for (int c = 0; c < a.nc; c++) tma_load_3d(smem_u32(sQ + c * q_chunk), &q_map, b_qfull, c * 64, hkv * a.g, tok0);
+      for (int i = 0; i < n_tiles; i++) {
+        const int s = i % a.stages;
+        if (!mbar_wait(b_kvempty + 8 * s, ((i / a.stages) & 1) ^ 1, abort_flag, kKernelGb, 100 + s)) break;
+        uint8_t* dst = sKV + s * stage_bytes;
+        int block = bt[pg_begin + i];
+        if (!NE_INDEX_OK(block, BK_CACHE_PAGES, kKernelGb, __LINE__)) block = 0;      // a bad page id reads page 0
+        mbar_expect_tx(b_kvfull + 8 * s, stage_bytes);
+        for (int c = 0; c < a.nc; c++) tma_load_4d(smem_u32(dst + c * kBChunk), &k_map, b_kvfull + 8 * s, c * 64, hkv, 0, block);
+        for (int c = 0; c < a.nv; c++) tma_load_4d(smem_u32(dst + (a.nc + c) * kBChunk), &v_map, b_kvfull + 8 * s, c * 64, hkv, 0, block);
+      }
+    }
+  } else if (warp == 1) {
+    if (n_tiles > 0 && elect_one()) {
+      constexpr uint32_t kIdescQK = make_idesc(FMT_BF16, FMT_BF16, 128, kBPage);
+      const uint32_t idesc_pv = make_idesc(FMT_BF16, FMT_BF16, 128, (uint32_t)a.nv * 64, 0, 1);      // B (= V) is MN-major
+      bool ok = mbar_wait(b_qfull, 0, abort_flag, kKernelGb, 200);
+      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP), kv_addr = smem_u32(sKV);
+      auto pv = [&](int j) -> bool {
+        const int pb = j % a.pbufs;
+        if (!mbar_wait(b_pfull + 8 * pb, (j / a.pbufs) & 1, abort_flag, kKernelGb, 230)) return false;
+        tc_fence_after();
+        const int s = j % a.stages;
+        const uint32_t vt = kv_addr + s * stage_bytes + a.nc * kBChunk;
+#pragma unroll
+        for (int ks = 0; ks < 4; ks++) {                     // 16 keys per MMA
+          const uint64_t adesc = make_smem_desc(p_addr + pb * p_bytes + ks * 32, 16, 1024, SW_128B);
+          const uint64_t bdesc = make_smem_desc(vt + ks * 16 * 128, kBChunk, 1024, SW_128B);
+          umma_f16(tmem_o, adesc, bdesc, idesc_pv, (j | ks) != 0);
+        }
+        tc_commit(b_kvempty + 8 * s);
+        tc_commit(b_pempty + 8 * pb);
+        return true;
+      };
+      // barriers that gate S(i+1) are tested before the MMAs of S(i) are issued (see gqa_bf16.cu)
+      bool pre_se = true, pre_kv = mbar_test(b_kvfull, 0);
+      for (int i = 0; ok && i < n_tiles; i++) {
+        const int sb = i & 1, s = i % a.stages;
+        if (!pre_se && !mbar_wait(b_sempty + 8 * sb, ((i >> 1) & 1) ^ 1, abort_flag, kKernelGb, 210 + sb)) { ok = false; break; }
+        if (!pre_kv && !mbar_wait(b_kvfull + 8 * s, (i / a.stages) & 1, abort_flag, kKernelGb, 220 + s)) { ok = false; break; }
+        mbar_test2(b_sempty + 8 * ((i + 1) & 1), (((i + 1) >> 1) & 1) ^ 1, b_kvfull + 8 * ((i + 1) % a.stages), ((i + 1) / a.stages) & 1, pre_se, pre_kv);
+        tc_fence_after();
+        const uint32_t kt = kv_addr + s * stage_bytes, d = tmem_base + sb * kBPage;
+        for (int c = 0; c < a.nc; c++) {
+#pragma unroll
+          for (int ks = 0; ks < 4; ks++) {
+            const uint64_t adesc = make_smem_desc(q_addr + c * q_chunk + ks * 32, 16, 1024, SW_128B);
+            const uint64_t bdesc = make_smem_desc(kt + c * kBChunk + ks * 32, 16, 1024, SW_128B);
+            umma_f16(d, adesc, bdesc, kIdescQK, (c | ks) != 0);
+          }
+        }
+        tc_commit(b_sfull + 8 * sb);
+        if (i > 0 && !pv(i - 1)) { ok = false; break; }
+      }
+      if (ok) pv(n_tiles - 1);
+    }
+  } else {
+    const int wq = warp & 3;
+    const int row = wq * 32 + (int)lane_id();
+    const uint32_t lane_addr = (uint32_t)(wq * 32) << 16;
+    const int tl = row / a.g, head = hkv * a.g + row % a.g;
+    const bool row_ok = row < a.g * a.tq && tl < n_tok;
+    const int limit = row_ok ? base_limit + tl : -1;          // this row's last visible key
+    const int lowest = (row_ok && a.window > 0) ? limit - a.window + 1 : 0;
+    const float slope = (row_ok && a.slopes) ? __ldg(a.slopes + head) * kLog2e : 0.f;
+    const float c_in = kCap ? a.scale / a.softcap * (2.f * kLog2e) : a.scale * kLog2e, c_cap = a.softcap * kLog2e;
+    float m_run = -INFINITY, l_run = 0.f;
+    bool ok = true, s_ready = false;
+    for (int i = 0; ok && i < n_tiles; i++) {
+      const int sb = i & 1, pb = i % a.pbufs;
+      if (!s_ready && !mbar_wait(b_sfull + 8 * sb, (i >> 1) & 1, abort_flag, kKernelGb, 300 + sb)) { ok = false; break; }
+      tc_fence_after();
+      uint32_t r0[32], r1[32];
+      tmem_ld_32x32b_x32(tmem_base + lane_addr + sb * kBPage, r0);
+      tmem_ld_32x32b_x32(tmem_base + lane_addr + sb * kBPage + 32, r1);
+      tc_wait_ld();
+      tc_fence_before();
+      __syncwarp();
+      if (lane_id() == 0) mbar_arrive(b_sempty + 8 * sb);
+      const int key0 = (pg_begin + i) * kBPage;
+      const bool p_free = i < a.pbufs || mbar_test(b_pempty + 8 * pb, ((i - a.pbufs) / a.pbufs) & 1);     // needed only after the math
+      // score in the log2 domain: cap and bias
+      const float b0 = slope * (float)(key0 - limit);
+      auto score = [&](uint32_t r, int j) -> uint32_t {
+        float s = __uint_as_float(r) * c_in;
+        const float bias = fmaf(slope, (float)j, b0);
+        if (kCap) s = fmaf(c_cap, 1.f - __fdividef(2.f, 1.f + exp2f(fminf(s, 64.f))), bias);      // cap (1 - 2 / (e^(2x) + 1)) = cap tanh(x)
+        else s += bias;
+        return __float_as_uint(s);
+      };
+#pragma unroll
+      for (int j = 0; j < 32; j++) { r0[j] = score(r0[j], j); r1[j] = score(r1[j], 32 + j); }
+      if (key0 + kBPage - 1 > limit || key0 < lowest) {
+#pragma unroll
+        for (int j = 0; j < 32; j++) {
+          if (key0 + j > limit || key0 + j < lowest) r0[j] = 0xff800000u;
+          if (key0 + 32 + j > limit || key0 + 32 + j < lowest) r1[j] = 0xff800000u;
+        }
+      }
+      float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+      for (int j = 0; j < 32; j += 2) {
+        mx[0] = fmaxf(mx[0], __uint_as_float(r0[j])); mx[1] = fmaxf(mx[1], __uint_as_float(r0[j + 1]));
+        mx[2] = fmaxf(mx[2], __uint_as_float(r1[j])); mx[3] = fmaxf(mx[3], __uint_as_float(r1[j + 1]));
+      }
+      const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+      // lazy rescaling: the reference maximum only moves when the page's maximum exceeds it by more than 2^8
+      const bool first_valid = (m_run == -INFINITY);
+      const float m_new = (first_valid || m_tile > m_run + 8.f) ? fmaxf(m_run, m_tile) : m_run;
+      const float alpha = (m_new == -INFINITY || first_valid) ? 1.f : exp2f(m_run - m_new);
+      const float neg_m = (m_new == -INFINITY) ? 0.f : -m_new;
+      float psum = 0.f;
+      uint32_t pk[32];
+#pragma unroll
+      for (int j = 0; j < 16; j++) {
+        const float p0 = exp2f(__uint_as_float(r0[2 * j]) + neg_m), p1 = exp2f(__uint_as_float(r0[2 * j + 1]) + neg_m);
+        const float p2 = exp2f(__uint_as_float(r1[2 * j]) + neg_m), p3 = exp2f(__uint_as_float(r1[2 * j + 1]) + neg_m);
+        pk[j] = pack_bf16x2(p0, p1);
+        pk[16 + j] = pack_bf16x2(p2, p3);
+        // sum what the MMA will see (bf16-rounded probabilities), so numerator and denominator stay consistent
+        const float2 q0 = unpack_bf16x2(pk[j]), q1 = unpack_bf16x2(pk[16 + j]);
+        psum += (q0.x + q0.y) + (q1.x + q1.y);
+      }
+      l_run = l_run * alpha + psum;
+      m_run = m_new;
+      if (i > 0 && __any_sync(0xffffffffu, alpha < 1.f)) {
+        if (!mbar_wait(b_pempty + 8 * ((i - 1) % a.pbufs), ((i - 1) / a.pbufs) & 1, abort_flag, kKernelGb, 310)) { ok = false; break; }
+        tc_fence_after();
+#pragma unroll 1
+        for (int cblk = 0; cblk < a.nv * 4; cblk++) {
+          uint32_t o[16];
+          tmem_ld_32x32b_x16(tmem_o + lane_addr + cblk * 16, o);
+          tc_wait_ld();
+#pragma unroll
+          for (int j = 0; j < 16; j++) o[j] = __float_as_uint(__uint_as_float(o[j]) * alpha);
+          tmem_st_32x32b_x16(tmem_o + lane_addr + cblk * 16, o);
+        }
+        tc_wait_st();
+      }
+      if (!p_free && !mbar_wait(b_pempty + 8 * pb, ((i - a.pbufs) / a.pbufs) & 1, abort_flag, kKernelGb, 311)) { ok = false; break; }
+      s_ready = mbar_test(b_sfull + 8 * ((i + 1) & 1), ((i + 1) >> 1) & 1);
+      if (row < a.rows8) {       // P row (64 bf16 = 8 chunks of 16 bytes) into the 128B-swizzled K-major layout the MMA reads
+        uint8_t* prow = sP + pb * p_bytes + row * 128;
+        const int sw = row & 7;
+#pragma unroll
+        for (int cch = 0; cch < 8; cch++)
+          *reinterpret_cast<uint4*>(prow + ((cch ^ sw) << 4)) = make_uint4(pk[4 * cch], pk[4 * cch + 1], pk[4 * cch + 2], pk[4 * cch + 3]);
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      __syncwarp();
+      if (lane_id() == 0) mbar_arrive(b_pfull + 8 * pb);
+    }
+    if (ok && n_tiles > 0) ok = mbar_wait(b_pempty + 8 * ((n_tiles - 1) % a.pbufs), ((n_tiles - 1) / a.pbufs) & 1, abort_flag, kKernelGb, 320);
+    const long long tok = tok0 + tl, orow = row_ok ? tok * a.H + head : 0;
+    const bool have = ok && n_tiles > 0;
+    if (have) tc_fence_after();
+    float inv = (have && l_run > 0.f) ? 1.f / l_run : 0.f;
+    if (a.splits == 1 && row_ok) inv *= gate_of(a.gate, a.gate_ld, tok, head, a.out_scale);
+#pragma unroll 1
+    for (int cblk = 0; cblk < a.nv * 2; cblk++) {
+      uint32_t o[32];
+      if (have) {
+        tmem_ld_32x32b_x32(tmem_o + lane_addr + cblk * 32, o);
+        tc_wait_ld();
+      }
+      if (!row_ok) continue;
+#pragma unroll
+      for (int v = 0; v < 4; v++) {                            // Dv is a multiple of 8: whole groups of 8 columns
+        const int col = cblk * 32 + v * 8;
+        if (col >= a.Dv) continue;
+        float f[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) f[j] = have ? __uint_as_float(o[v * 8 + j]) * inv : 0.f;
+        if (a.splits == 1) {
+          *reinterpret_cast<uint4*>(a.out + tok * a.o_ld + (long long)head * a.Dv + col) =
+              make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+        } else {
+          float* dst = a.part + ((long long)split * a.T * a.H + orow) * a.Dv + col;
+          *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
+          *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
+        }
+      }
+    }
+    if (a.splits > 1 && row_ok)
+      a.lse2[(long long)split * a.T * a.H + orow] = (have && l_run > 0.f) ? m_run + log2f(l_run) : -INFINITY;
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_flag && threadIdx.x == 0) for (int i = 0; i < 2000; i++) __nanosleep(1000);      // copies in flight land before the CTA goes
+  __syncthreads();
+  if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem_base, a.tmem_cols); }
+}
+
+// out[t, h] = gate * sum_s softmax_s(lse2) part[s, t, h]; one CTA per (token, head)
+__global__ void __launch_bounds__(128) gqa_biased_merge_kernel(const GbArgs a) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const long long row = blockIdx.x, rows = (long long)a.T * a.H, t = row / a.H;
+  const int h = (int)(row - t * a.H);
+  float m = -INFINITY;
+  for (int s = 0; s < a.splits; s++) m = fmaxf(m, a.lse2[s * rows + row]);
+  float den = 0.f;
+  for (int s = 0; s < a.splits; s++) { const float l = a.lse2[s * rows + row]; den += l == -INFINITY ? 0.f : exp2f(l - m); }
+  const float inv = den > 0.f ? gate_of(a.gate, a.gate_ld, t, h, a.out_scale) / den : 0.f;
+  for (int d = threadIdx.x; d < a.Dv; d += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < a.splits; s++) {
+      const float l = a.lse2[s * rows + row];
+      if (l != -INFINITY) acc += exp2f(l - m) * a.part[(s * rows + row) * a.Dv + d];
+    }
+    a.out[t * a.o_ld + (long long)h * a.Dv + d] = __float2bfloat16(acc * inv);
+  }
+}
+
+struct GbPlan { int nc, nv, tq, rows8, stages, pbufs, smem; };
+
+// Tile geometry for groups of g heads, head sizes D / Dv and sequences of at most max_q new tokens; false: not covered.
+static bool gb_plan(int g, int D, int Dv, int max_q, GbPlan* p) {
+  if (g < 1 || g > 128 || D < 8 || D % 8 || D > 256 || Dv < 8 || Dv % 8 || Dv > 256 || max_q < 1) return false;
+  p->nc = (D + 63) / 64; p->nv = (Dv + 63) / 64;
+  p->tq = 128 / g < max_q ? 128 / g : max_q;
+  p->rows8 = (g * p->tq + 7) / 8 * 8;
+  const int limit = 232448 - 1024 - 256, kv = (p->nc + p->nv) * kBChunk, q = p->nc * p->rows8 * 128;
+  p->pbufs = q + 2 * p->rows8 * 128 + 2 * kv <= limit ? 2 : 1;
+  p->stages = (limit - q - p->pbufs * p->rows8 * 128) / kv;
+  if (p->stages > 4) p->stages = 4;
+  if (p->stages < 2) return false;
+  const int used = q + p->pbufs * p->rows8 * 128 + p->stages * kv;
+  p->smem = used + 1024 + 256;
+  // an MMA reads 128 rows from each chunk of Q and from each P buffer: those reads must end inside the allocation
+  const int last_q = (p->nc - 1) * p->rows8 * 128 + 16384, last_p = q + (p->pbufs - 1) * p->rows8 * 128 + 16384;
+  return (last_q > last_p ? last_q : last_p) <= used;
+}
+
+}  // namespace ne
+
+using namespace ne;
+
+// Tokens per tile (0: the shape is not covered)
+extern "C" int ne_gqa_biased_plan(int H, int Hkv, int D, int Dv, int max_q) {
+  GbPlan p;
+  return Hkv >= 1 && H % Hkv == 0 && gb_plan(H / Hkv, D, Dv, max_q, &p) ? p.tq : 0;
+}
+
+// q bf16 [T, H, D] (row stride q_ld elements), k_cache bf16 [num_blocks, 64, Hkv, D], v_cache bf16 [num_blocks, 64, Hkv, Dv];
+// max_tiles >= sum over sequences of ceil(q_len / tokens per tile).  softcap 0 / slopes null / window 0 / gate null: without.  out bf16, row
+// stride o_ld, heads Dv apart.  splits > 1: part fp32 [splits, T, H, Dv], lse2 [splits, T, H]; the merge kernel is launched too.
+extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache, const void* v_cache, int num_blocks, const int* block_tables, int bt_stride,
+                             const int* cu_seqlens_q, const int* context_lens, int num_seqs, int T, int H, int Hkv, int D, int Dv, int max_q, int max_tiles,
+                             int splits, float scale, float softcap, const float* slopes, int window, const void* gate, long long gate_ld, float out_scale,
+                             void* out, long long o_ld, float* part, float* lse2, cudaStream_t st) {
+  if (T <= 0) return 0;
+  GbPlan p;
+  if (Hkv < 1 || H % Hkv || splits < 1 || (splits > 1 && (!part || !lse2)) || max_tiles < 1 || !gb_plan(H / Hkv, D, Dv, max_q, &p)) return 1001;
+  if (q_ld % 8 || o_ld % 8 || q_ld < (long long)H * D || (((uintptr_t)q | (uintptr_t)out) & 15)) return 1002;
+  const int g = H / Hkv;
+  CUtensorMap mq, mk, mv;
+  int rc;
+  {
+    uint64_t dims[3] = {(uint64_t)D, (uint64_t)H, (uint64_t)T}; uint64_t strides[2] = {(uint64_t)D * 2, (uint64_t)q_ld * 2};
+    uint32_t box[3] = {64, (uint32_t)g, (uint32_t)p.tq};
+    rc = make_tmap(&mq, q, TMA_BF16, 3, dims, strides, box, TMA_SW_128); if (rc) return 2000 + rc;
+  }
+  for (int which = 0; which < 2; which++) {
+    const uint64_t w = which ? Dv : D;
+    uint64_t dims[4] = {w, (uint64_t)Hkv, (uint64_t)kBPage, (uint64_t)num_blocks};
+    uint64_t strides[3] = {w * 2, (uint64_t)Hkv * w * 2, (uint64_t)kBPage * Hkv * w * 2};
+    uint32_t box[4] = {64, 1, kBPage, 1};
+    rc = make_tmap(which ? &mv : &mk, which ? v_cache : k_cache, TMA_BF16, 4, dims, strides, box, TMA_SW_128); if (rc) return 2100 + rc;
+  }
+  auto kern = softcap > 0.f ? gqa_biased_kernel<true> : gqa_biased_kernel<false>;
+  static bool configured[2] = {false, false};
+  if (!configured[softcap > 0.f]) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
+    if (e != cudaSuccess) return (int)e;
+    configured[softcap > 0.f] = true;
+  }
+  GbArgs a;
+  a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs;
+  a.T = T; a.H = H; a.Dv = Dv; a.g = g; a.tq = p.tq; a.splits = splits; a.nc = p.nc; a.nv = p.nv; a.rows8 = p.rows8; a.stages = p.stages; a.pbufs = p.pbufs;
+  a.window = window; a.tmem_cols = p.nv <= 2 ? 256 : 512; a.scale = scale; a.softcap = softcap; a.slopes = slopes; a.gate = (const __nv_bfloat16*)gate;
+  a.gate_ld = gate_ld; a.out_scale = out_scale; a.out = (__nv_bfloat16*)out; a.o_ld = o_ld; a.part = part; a.lse2 = lse2;
+  cudaError_t e = launch_pdl(kern, dim3((unsigned)max_tiles, (unsigned)Hkv, (unsigned)splits), dim3(kGbThreads), (size_t)p.smem, st, mq, mk, mv, a);
+  if (e != cudaSuccess || splits == 1) return (int)e;
+  return (int)launch_pdl(gqa_biased_merge_kernel, dim3((unsigned)((long long)T * H)), dim3(128), 0, st, a);
+}

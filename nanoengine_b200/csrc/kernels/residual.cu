@@ -4,6 +4,8 @@
 //   * gated activation of [gate | up] rows
 //   * latent_prepare: rotary part of every query head in place, and the latent cache row [rmsnorm(kv[:R]) | rope(kv[R:])]
 //   * gather of cache rows
+//   * stream_mix: constant hyper-connections - the streams of a token mixed with a sublayer's output, the next sublayer's normed input
+//   * kv_rows: new key and value rows of any width into paged caches;  cap_rows: cap * tanh(x / cap) in place
 #include "ptx.cuh"
 
 namespace ne {
@@ -105,6 +107,7 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(const T* __restrict_
 // Gated activation (see elementwise.cu for the modes): x [T, >= 2I] rows with stride ld -> y [T, I]
 __device__ __forceinline__ float glu_exact(float g, float u, int act, float p0, float p1) {
   if (act == 3) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  if (act == 4) { g = fminf(g, p0); return g / (1.f + expf(-p1 * g)) * (fminf(fmaxf(u, -p0), p0) + 1.f); }
   if (act == 1) { u = fminf(fmaxf(u, -p0), p0); g = fminf(g, p0); }
   if (act == 2) {
     if (p1 > 0.f) u = p1 * tanhf(u / p1);
@@ -210,6 +213,149 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restr
   rows[i] = cache[slot * pieces + c];
 }
 
+// ---- constant hyper-connections -----------------------------------------------------------------------------------------
+// x [rows, S, W] fp32 streams.  y given: x_t <- sum_s mix[s, t] x_s + w_out[t] y (all streams from the old ones, written back unless
+// `last`).  ids given: every stream starts as table[id] + pos[position] instead.  Then u = sum_s w_in[s] x_s and out = rmsnorm(u) * w_next.
+// One CTA per row; S = 0: any number of streams up to kMaxStreams (then V = 1).
+constexpr int kMaxStreams = 16;
+struct StreamArgs {
+  const void* y; long long y_ld; float* x; const float* w_out; const float* mix; const float* w_in; const void* w_next; void* out;
+  const long long* ids; const long long* positions; const void* table; const void* pos;
+  int streams, W, vocab, n_pos, last; float eps;
+};
+template <typename T, int V, int S>
+__global__ void __launch_bounds__(512) stream_mix_kernel(const StreamArgs a) {
+  constexpr int SM = S ? S : kMaxStreams;
+  extern __shared__ float srow[];            // W floats: u
+  __shared__ float red[2][32];
+  __shared__ float s_in[SM], s_out[SM], s_mix[SM * SM];
+  const int ns = S ? S : a.streams, W = a.W;
+  // the coefficients are weights: they may be read before the kernel in front has finished
+  for (int i = threadIdx.x; i < ns; i += blockDim.x) { s_in[i] = a.w_in[i]; if (a.y) s_out[i] = a.w_out[i]; }
+  if (a.y) for (int i = threadIdx.x; i < ns * ns; i += blockDim.x) s_mix[i] = a.mix[i];
+  pdl_wait(); pdl_trigger();
+  __syncthreads();
+  const long long row = blockIdx.x;
+  float* xr = a.x + row * ns * W;
+  float ss = 0.f;
+  if (a.ids) {
+    const long long id = a.ids[row], p = a.positions[row];
+    const bool ok = id >= 0 && id < a.vocab && (!a.pos || (p >= 0 && p < a.n_pos));
+    if (!ok && threadIdx.x == 0) report(ST_BAD_INDEX, 45, (int)id, (int)p);
+    const T* tr = reinterpret_cast<const T*>(a.table) + (ok ? id : 0) * W;
+    const T* pr = a.pos ? reinterpret_cast<const T*>(a.pos) + (ok ? p : 0) * W : nullptr;
+    float wsum = 0.f;
+    for (int s = 0; s < ns; s++) wsum += s_in[s];
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+      if constexpr (V == 4) {
+        float4 t = Vec4<T>::load(tr + i);
+        if (pr) { const float4 q = Vec4<T>::load(pr + i); t.x += q.x; t.y += q.y; t.z += q.z; t.w += q.w; }
+        for (int s = 0; s < ns; s++) *reinterpret_cast<float4*>(xr + (long long)s * W + i) = t;
+        t.x *= wsum; t.y *= wsum; t.z *= wsum; t.w *= wsum;
+        *reinterpret_cast<float4*>(srow + i) = t;
+        ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+      } else {
+        float t = ldx(tr + i);
+        if (pr) t += ldx(pr + i);
+        for (int s = 0; s < ns; s++) xr[(long long)s * W + i] = t;
+        t *= wsum;
+        srow[i] = t; ss += t * t;
+      }
+    }
+  } else {
+    const T* yr = reinterpret_cast<const T*>(a.y) + row * a.y_ld;
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+      float xs[SM][V], yv[V], u[V];
+#pragma unroll
+      for (int s = 0; s < SM; s++) {
+        if (!S && s >= ns) break;
+        if constexpr (V == 4) {
+          const float4 t = *reinterpret_cast<const float4*>(xr + (long long)s * W + i);
+          xs[s][0] = t.x; xs[s][1] = t.y; xs[s][2] = t.z; xs[s][3] = t.w;
+        } else xs[s][0] = xr[(long long)s * W + i];
+      }
+      if constexpr (V == 4) { const float4 t = Vec4<T>::load(yr + i); yv[0] = t.x; yv[1] = t.y; yv[2] = t.z; yv[3] = t.w; }
+      else yv[0] = ldx(yr + i);
+#pragma unroll
+      for (int e = 0; e < V; e++) u[e] = 0.f;
+#pragma unroll (S ? SM : 1)
+      for (int t = 0; t < SM; t++) {
+        if (!S && t >= ns) break;
+        float n[V];
+#pragma unroll
+        for (int e = 0; e < V; e++) n[e] = s_out[t] * yv[e];
+#pragma unroll
+        for (int s = 0; s < SM; s++) {
+          if (!S && s >= ns) break;
+          const float m = s_mix[s * ns + t];
+#pragma unroll
+          for (int e = 0; e < V; e++) n[e] = fmaf(m, xs[s][e], n[e]);
+        }
+        const float wi = s_in[t];
+#pragma unroll
+        for (int e = 0; e < V; e++) u[e] = fmaf(wi, n[e], u[e]);
+        if (!a.last) {
+          if constexpr (V == 4) *reinterpret_cast<float4*>(xr + (long long)t * W + i) = make_float4(n[0], n[1], n[2], n[3]);
+          else xr[(long long)t * W + i] = n[0];
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; e++) { srow[i + e] = u[e]; ss += u[e] * u[e]; }
+    }
+  }
+  const float r = rsqrtf(cta_sum(ss, red, 0) / (float)W + a.eps);
+  const T* wn = reinterpret_cast<const T*>(a.w_next);
+  T* out = reinterpret_cast<T*>(a.out) + row * W;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {        // a thread rereads only what it stored itself
+    if constexpr (V == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(srow + i), w = Vec4<T>::load(wn + i);
+      Vec4<T>::store(out + i, make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w));
+    } else {
+      stx(out + i, srow[i] * r * ldx(wn + i));
+    }
+  }
+}
+
+template <typename T>
+static int stream_mix_t(const StreamArgs& a, int rows, cudaStream_t st) {
+  const size_t smem = (size_t)a.W * sizeof(float);
+  const uintptr_t al = (uintptr_t)a.y | (uintptr_t)a.x | (uintptr_t)a.w_next | (uintptr_t)a.out | (uintptr_t)a.table | (uintptr_t)a.pos;
+  const bool vec = a.W % 4 == 0 && a.y_ld % 4 == 0 && al % 16 == 0 && a.streams <= 4;
+  const int per = vec ? 4 : 1;
+  int threads = ((a.W + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+  void (*k)(const StreamArgs) = stream_mix_kernel<T, 1, 0>;
+  if (vec) k = a.streams == 1 ? stream_mix_kernel<T, 4, 1> : a.streams == 2 ? stream_mix_kernel<T, 4, 2> : a.streams == 3 ? stream_mix_kernel<T, 4, 3> : stream_mix_kernel<T, 4, 4>;
+  if (smem > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl(k, dim3((unsigned)rows), dim3((unsigned)threads), smem, st, a);
+}
+
+// ---- key / value rows into paged caches -------------------------------------------------------------------------------------
+// Row t of k (kw elements, row stride k_ld) goes to cache row slots[t], the same for v.  U: the access unit (uint4 where everything is
+// 16-byte aligned, else one element); widths and strides in units.
+template <typename U>
+__global__ void __launch_bounds__(256) kv_rows_kernel(const U* __restrict__ k, long long k_ld, const U* __restrict__ v, long long v_ld, U* __restrict__ kc, U* __restrict__ vc,
+                                                     const long long* __restrict__ slots, int T, int kw, int vw) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const int w = kw + vw;
+  if (i >= (long long)T * w) return;
+  const int t = (int)(i / w), c = (int)(i - (long long)t * w);
+  const long long slot = slots[t];
+  if (slot < 0 || !NE_INDEX_OK(slot, BK_CACHE_ROWS, 46, __LINE__)) return;
+  if (c < kw) kc[slot * kw + c] = k[(long long)t * k_ld + c];
+  else vc[slot * vw + c - kw] = v[(long long)t * v_ld + c - kw];
+}
+
+__global__ void __launch_bounds__(256) cap_rows_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
 template <typename T>
 static int residual_norm_t(const void* y, long long y_ld, float* x, const void* w_post, const void* w_next, void* out, int T_, int W, float eps,
                            float w_off, const long long* ids, const void* table, int vocab, cudaStream_t st) {
@@ -251,7 +397,7 @@ extern "C" int ne_residual_norm(const void* y, long long y_ld, float* x, const v
 
 extern "C" int ne_glu_rows(const void* x, long long ld, void* y, int T, int I, int act, float p0, float p1, int fp32, cudaStream_t st) {
   if (T <= 0 || I <= 0) return 0;
-  if (act < 0 || act > 3 || ld < 2 * I) return 1001;
+  if (act < 0 || act > 4 || ld < 2 * I) return 1001;
   return fp32 ? glu_rows_t<float>(x, ld, y, T, I, act, p0, p1, st) : glu_rows_t<__nv_bfloat16>(x, ld, y, T, I, act, p0, p1, st);
 }
 
@@ -280,4 +426,42 @@ extern "C" int ne_latent_gather(const void* cache, const long long* slots, void*
   const int pieces = row_bytes / 16;
   return (int)launch_pdl(latent_gather_kernel, dim3((unsigned)(((long long)T * pieces + 255) / 256)), dim3(256), 0, st, (const uint4*)cache, slots, (uint4*)rows, T,
                          pieces);
+}
+
+// See StreamArgs.  w_out [S], mix [S, S] (from, to), w_in [S] fp32; y / table / pos / w_next / out in the activation dtype.
+extern "C" int ne_stream_mix(const void* y, long long y_ld, float* x, const float* w_out, const float* mix, const float* w_in, const void* w_next, void* out,
+                             const long long* ids, const long long* positions, const void* table, int vocab, const void* pos, int n_pos, int T, int S, int W,
+                             float eps, int last, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (S < 1 || S > kMaxStreams || W < 1 || W > 48 * 1024 || (!ids && (!y || !w_out || !mix)) || (ids && (!table || !positions)) || !w_in) return 1001;
+  StreamArgs a;
+  a.y = ids ? nullptr : y; a.y_ld = ids ? 0 : y_ld; a.x = x; a.w_out = w_out; a.mix = mix; a.w_in = w_in; a.w_next = w_next; a.out = out; a.ids = ids;
+  a.positions = positions; a.table = ids ? table : nullptr; a.pos = ids ? pos : nullptr; a.streams = S; a.W = W; a.vocab = vocab; a.n_pos = n_pos; a.last = last; a.eps = eps;
+  return fp32 ? stream_mix_t<float>(a, T, st) : stream_mix_t<__nv_bfloat16>(a, T, st);
+}
+
+// k [T, kw], v [T, vw] (row strides k_ld, v_ld, elements of `es` bytes) -> rows slots[t] of caches [rows, kw] and [rows, vw]
+extern "C" int ne_kv_rows(const void* k, long long k_ld, const void* v, long long v_ld, void* kc, void* vc, const long long* slots, int T, int kw, int vw, int es,
+                          cudaStream_t st) {
+  if (T <= 0) return 0;
+  if ((es != 2 && es != 4) || kw < 1 || vw < 1) return 1001;
+  const int per = 16 / es;
+  const bool vec = kw % per == 0 && vw % per == 0 && k_ld % per == 0 && v_ld % per == 0 && ((uintptr_t)k | (uintptr_t)v | (uintptr_t)kc | (uintptr_t)vc) % 16 == 0;
+  const long long n = (long long)T * (kw + vw) / (vec ? per : 1);
+  const dim3 grid((unsigned)((n + 255) / 256));
+  if (vec)
+    return (int)launch_pdl(kv_rows_kernel<uint4>, grid, dim3(256), 0, st, (const uint4*)k, k_ld / per, (const uint4*)v, v_ld / per, (uint4*)kc, (uint4*)vc, slots, T,
+                           kw / per, vw / per);
+  if (es == 2)
+    return (int)launch_pdl(kv_rows_kernel<uint16_t>, grid, dim3(256), 0, st, (const uint16_t*)k, k_ld, (const uint16_t*)v, v_ld, (uint16_t*)kc, (uint16_t*)vc, slots, T,
+                           kw, vw);
+  return (int)launch_pdl(kv_rows_kernel<uint32_t>, grid, dim3(256), 0, st, (const uint32_t*)k, k_ld, (const uint32_t*)v, v_ld, (uint32_t*)kc, (uint32_t*)vc, slots, T, kw,
+                         vw);
+}
+
+// x [n] fp32 <- cap * tanh(x / cap)
+extern "C" int ne_cap_rows(float* x, long long n, float cap, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return 1001;
+  return (int)launch_pdl(cap_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, x, n, cap);
 }

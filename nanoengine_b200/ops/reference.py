@@ -83,6 +83,35 @@ def residual_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next
     return norm(x, w_next).to(y.dtype), x
 
 
+def stream_mix(y: torch.Tensor, x: torch.Tensor, w_out: torch.Tensor, mix: torch.Tensor, w_in: torch.Tensor, w_next: torch.Tensor, eps: float,
+               last: bool = False):
+    """Constant hyper-connections around a 32-bit residual of S streams: x_t <- sum_s mix[s, t] x_s + w_out[t] y, then the next sublayer's
+    input rmsnorm(sum_s w_in[s] x_s) * w_next in y's dtype.  y [T, W], x [T, S, W] fp32, w_out / w_in [S] and mix [S, S] (from, to) fp32.
+    Returns (input, x); the CUDA body updates x in place, unless `last` says that nothing reads the streams any more."""
+    x = torch.einsum("nsw,st->ntw", x, mix) + w_out[None, :, None] * y.float()[:, None]
+    return _stream_read(x, w_in, w_next, eps, y.dtype), x
+
+
+def stream_embed(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos: Optional[torch.Tensor], w_in: torch.Tensor, w_next: torch.Tensor,
+                 eps: float):
+    """The start of the streams of `stream_mix`: all of them table[id] (+ pos[position]) in fp32.  Returns (first sublayer's input, x)."""
+    e = table[ids.long()].float()
+    if pos is not None:
+        e = e + pos[positions.long()].float()
+    x = e[:, None].repeat(1, w_in.numel(), 1)
+    return _stream_read(x, w_in, w_next, eps, table.dtype), x
+
+
+def _stream_read(x, w_in, w_next, eps, dtype):
+    u = torch.einsum("nsw,s->nw", x, w_in)
+    return (u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * w_next.float()).to(dtype)
+
+
+def cap_logits(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap * tanh(logits / cap); the CUDA body works in place on fp32 logits."""
+    return cap * torch.tanh(logits / cap)
+
+
 def embed_norm(ids: torch.Tensor, table: torch.Tensor, w_next: torch.Tensor, eps: float, unit_offset: bool = True):
     """The start of a 32-bit residual stream: x = table[ids] as fp32 and the first sublayer's input rmsnorm(x, w_next) in the
     table's dtype.  Returns (input, x)."""
@@ -179,6 +208,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, w_scale: Optional[torch.Tensor] = N
         y = dequant_fp8_1x128(xq, xs) @ dequant_fp8_block(w, w_scale).t()
         y = y.view(*x.shape[:-1], w.shape[0]).to(x.dtype)
     else:
+        if bias is not None and bias.dtype == torch.float32:          # added to the accumulator: one rounding
+            return (F.linear(x.float(), w.float()) + bias).to(x.dtype)
         y = F.linear(x, w)
     if bias is not None:
         y = y + bias
@@ -262,6 +293,15 @@ def gqa_kv_store(k_cache, v_cache, slot_mapping, k, v) -> None:
     """k_cache/v_cache [blocks, block_size, kv_heads, head_dim]."""
     k_cache.view(-1, *k_cache.shape[2:])[slot_mapping.long()] = k.to(k_cache.dtype)
     v_cache.view(-1, *v_cache.shape[2:])[slot_mapping.long()] = v.to(v_cache.dtype)
+
+
+def kv_rows(k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> None:
+    """Rows of k [T, kv_heads * D] and v [T, kv_heads * Dv] (any widths, row strides free) into the paged caches [blocks, block_size,
+    kv_heads, D / Dv]; slot -1 writes nothing."""
+    keep = slot_mapping >= 0
+    slots = slot_mapping[keep].long()
+    for cache, t in ((k_cache, k), (v_cache, v)):
+        cache.view(-1, cache.shape[2] * cache.shape[3])[slots] = t[keep].to(cache.dtype)
 
 
 def gqa_qkv_prepare(qkv: torch.Tensor, hq: int, hkv: int, hd: int, q_norm_w, k_norm_w, eps: float, unit_offset: bool, positions,
@@ -355,6 +395,42 @@ def gqa_attention_paged(q, k_cache, v_cache, block_tables, cu_seqlens_q, context
             s = s.masked_fill(keys <= pos - window, float("-inf"))
         out[lo:hi] = torch.einsum("thn,nhd->thd", torch.softmax(s, -1), v)
     return out.to(q.dtype)
+
+
+def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0, softcap: float = 0.0, slopes=None,
+                         gate=None, out_scale: float = 1.0, out=None, max_q_len: int = 0) -> torch.Tensor:
+    """Causal grouped-query attention over paged caches with per-layer options.  q [T, Hq, D] (token stride free), k_cache [blocks, block_size,
+    Hkv, D], v_cache [..., Dv].  score = q.k scale, capped as softcap tanh(score / softcap) when softcap > 0, minus slopes[head] (query position
+    - key position) when slopes [Hq] are given; `window` > 0: a query sees its own and the window - 1 keys before it.  Head h's output is
+    multiplied by out_scale and, with gate [T, Hq], by sigmoid(gate[:, h]).  Writes into `out` [T, Hq * Dv] (rows may be strided) when given.
+    `max_q_len`: planning hint of the CUDA body."""
+    T, Hq, D = q.shape
+    Hkv, Dv = k_cache.shape[2], v_cache.shape[3]
+    o = torch.zeros(T, Hq, Dv, dtype=torch.float32, device=q.device)
+    for i in range(cu_seqlens_q.numel() - 1):
+        lo, hi = int(cu_seqlens_q[i]), int(cu_seqlens_q[i + 1])
+        if hi == lo:
+            continue
+        n, ql = int(context_lens[i]), hi - lo
+        k = _gather_rows(k_cache, block_tables[i], n).repeat_interleave(Hq // Hkv, 1)
+        v = _gather_rows(v_cache, block_tables[i], n).repeat_interleave(Hq // Hkv, 1)
+        s = torch.einsum("thd,nhd->thn", q[lo:hi].float(), k) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
+        dist = torch.arange(n - ql, n, device=q.device).view(ql, 1, 1) - torch.arange(n, device=q.device).view(1, 1, n)
+        if slopes is not None:
+            s = s - slopes.float().view(1, Hq, 1) * dist
+        s = s.masked_fill(dist < 0, float("-inf"))
+        if window > 0:
+            s = s.masked_fill(dist >= window, float("-inf"))
+        o[lo:hi] = torch.einsum("thn,nhd->thd", torch.softmax(s, -1), v)
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float())[:, :, None]
+    o = (o * out_scale).to(q.dtype).reshape(T, Hq * Dv)
+    if out is None:
+        return o
+    out.copy_(o)
+    return out
 
 
 def attention_varlen(q, k, v, cu_seqlens, scale, causal: bool = False) -> torch.Tensor:
@@ -481,13 +557,17 @@ def mxfp4_quant(w: torch.Tensor):
 
 def glu_act(a: torch.Tensor, b: torch.Tensor, act=None) -> torch.Tensor:
     """Gated activation of (gate a, up b) in fp32.  act None: silu(a) b.  ("gelu_tanh",): tanh-approximated GELU(a) b.  ("clamp", L): up in [-L, L], gate <= L, then
-    silu(a) b (reference layers/activation.py:86-92).  ("situ", beta, linear_beta): beta tanh(a / beta) sigmoid(a) times
+    silu(a) b (reference layers/activation.py:86-92).  ("clamp_linear", L, alpha): the same clamps, then a sigmoid(alpha a) (b + 1).  ("situ", beta, linear_beta): beta tanh(a / beta) sigmoid(a) times
     linear_beta tanh(b / linear_beta) (no clamp of b when linear_beta is None; reference kernel/triton/generic/situ.py:24-27)."""
     if act is None:
         return F.silu(a) * b
     if act[0] == "clamp":
         L = float(act[1])
         return F.silu(a.clamp(max=L)) * b.clamp(-L, L)
+    if act[0] == "clamp_linear":
+        L, alpha = float(act[1]), float(act[2])
+        a = a.clamp(max=L)
+        return a * torch.sigmoid(alpha * a) * (b.clamp(-L, L) + 1)
     if act[0] == "gelu_tanh":
         return F.gelu(a, approximate="tanh") * b
     if act[0] == "situ":
@@ -1177,6 +1257,81 @@ def gated_delta(proj: torch.Tensor, ab: torch.Tensor, conv_w: torch.Tensor, A_lo
     z = proj[:, C: C + Hv * Dv].float().view(T, Hv, Dv)
     o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float() * F.silu(z)
     return o.to(proj.dtype).reshape(T, Hv * Dv)
+
+
+# ---- linear attention with a scalar decay per head ---------------------------------------------------------
+def decay_scan(q, k, v, log_a, b, S, skip=None):
+    """S <- exp(log_a) S + b v k^T, o = S q (+ skip v), token by token for one sequence in fp32.  q, k [n, H, Dk], v [n, H, Dv], log_a and b
+    [n, H], S [H, Dv, Dk].  Returns (o [n, H, Dv], S)."""
+    o = torch.empty_like(v)
+    a = log_a.exp()
+    for t in range(q.shape[0]):
+        S = a[t, :, None, None] * S + (b[t, :, None] * v[t])[:, :, None] * k[t][:, None, :]
+        o[t] = torch.einsum("hvk,hk->hv", S, q[t])
+    if skip is not None:
+        o = o + skip.view(1, -1, 1) * v
+    return o, S
+
+
+def _decay_ragged(q, k, v, log_a, b, state, slots, cu_seqlens, fresh, skip=None):
+    o = torch.empty_like(v)
+    cu = cu_seqlens.tolist()
+    for i in range(len(cu) - 1):
+        s, e = cu[i], cu[i + 1]
+        if e <= s:
+            continue
+        slot = int(slots[i])
+        S = torch.zeros_like(state[slot]) if int(fresh[i]) else state[slot].clone()
+        o[s:e], state[slot] = decay_scan(q[s:e], k[s:e], v[s:e], log_a[s:e], b[s:e], S, skip)
+    return o
+
+
+def mamba2_mix(proj: torch.Tensor, dt_raw: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor,
+               D: torch.Tensor, norm_w: torch.Tensor, norm_groups: int, window: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+               cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, G: int, Dv: int, N: int, eps: float, max_q_len: int = 1) -> torch.Tensor:
+    """Mamba-2 mixer between its projections.  proj [T, z | x | B | C] (H Dv, H Dv, G N, G N columns), dt_raw [T, H] fp32.  Short causal
+    convolution + bias + silu over x | B | C (rounded to proj's dtype) with the carried `window` [S, K - 1, C]; dt = softplus(dt_raw + dt_bias);
+    per head S <- exp(-exp(A_log) dt) S + dt x B^T on `state` [S, H, Dv, N] fp32, y = S C + D x (head h reads group h // (H / G)); then
+    y silu(z), RMS-normed in `norm_groups` equal parts, times norm_w.  Returns [T, H Dv] in proj's dtype; any mix of sequence lengths.
+    `max_q_len`: planning hint of the CUDA body."""
+    T, inner = proj.shape[0], H * Dv
+    C, K = conv_w.shape
+    xbc = proj[:, inner: inner + C]
+    y = torch.empty(T, C, dtype=torch.float32, device=proj.device)
+    cu = cu_seqlens.tolist()
+    for i in range(len(cu) - 1):
+        s, e = cu[i], cu[i + 1]
+        if e <= s:
+            continue
+        slot = int(slots[i])
+        win = torch.zeros_like(window[slot]) if int(fresh[i]) else window[slot]
+        full = torch.cat([win, xbc[s:e].to(window.dtype)], 0)
+        y[s:e] = conv_b.float() + sum(full[j: j + e - s].float() * conv_w[:, j].float() for j in range(K))
+        window[slot] = full[full.shape[0] - (K - 1):]
+    y = F.silu(y).to(proj.dtype).float()
+    x, Bm, Cm = y[:, :inner].reshape(T, H, Dv), y[:, inner: inner + G * N].reshape(T, G, N), y[:, inner + G * N:].reshape(T, G, N)
+    dt = F.softplus(dt_raw.float() + dt_bias)
+    o = _decay_ragged(Cm.repeat_interleave(H // G, 1), Bm.repeat_interleave(H // G, 1), x, -A_log.exp() * dt, dt, state, slots, cu_seqlens, fresh, D)
+    o = (o.reshape(T, inner) * F.silu(proj[:, :inner].float())).reshape(T, norm_groups, inner // norm_groups)
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    return (o.reshape(T, inner) * norm_w.float()).to(proj.dtype)
+
+
+def lightning_mix(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor,
+                  slots: torch.Tensor, cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, Dk: int, Dv: int, eps: float, out_scale: float = 1.0,
+                  out: Optional[torch.Tensor] = None, max_q_len: int = 1) -> torch.Tensor:
+    """Linear attention with one constant decay per head: q, k [T, H Dk] and v [T, H Dv] projections (rows may be strided) pass silu, per head
+    S <- decay S + v k^T on `state` [S, H, Dv, Dk] fp32, o = S q; the concatenated heads are RMS-normed together, times norm_w, sigmoid(gate)
+    and out_scale.  Writes into `out` [T, H Dv] (rows may be strided) when given.  `max_q_len`: planning hint of the CUDA body."""
+    T = q.shape[0]
+    qf, kf, vf = F.silu(q.float()).reshape(T, H, Dk), F.silu(k.float()).reshape(T, H, Dk), F.silu(v.float()).reshape(T, H, Dv)
+    ones = torch.ones(T, H, dtype=torch.float32, device=q.device)
+    o = _decay_ragged(qf, kf, vf, decay.log().expand(T, H), ones, state, slots, cu_seqlens, fresh).reshape(T, H * Dv)
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float() * torch.sigmoid(gate.float()) * out_scale
+    if out is None:
+        return o.to(q.dtype)
+    out.copy_(o)
+    return out
 
 
 # ---- MTP draft verification -------------------------------------------------------------------------------

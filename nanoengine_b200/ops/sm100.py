@@ -172,13 +172,13 @@ class PrequantizedActivation:
         self.q, self.scales, self.shape, self.device = q, scales, q.shape, q.device
 
 
-def _gemm_simt(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch):
+def _gemm_simt(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias=None):
     """Tiled product on CUDA cores: true 32-bit operands, and bf16 shapes the tensor-core GEMM cannot address."""
     f32 = A.dtype == torch.float32
     assert A.dtype == B.dtype and D.dtype in (torch.float32, A.dtype)
     _ck(lib().ne_gemm_simt(_p(A), _c.c_longlong(lda), _c.c_longlong(a_bs), _p(B), _c.c_longlong(ldb), _c.c_longlong(b_bs), _p(D), _c.c_longlong(ldd),
                            _c.c_longlong(d_bs), _c.c_int(M), _c.c_int(N), _c.c_int(K), _c.c_int(batch), _c.c_int(int(f32)),
-                           _c.c_int(int(D.dtype == torch.float32)), _st()), "ne_gemm_simt")
+                           _c.c_int(int(D.dtype == torch.float32)), _p(bias), _st()), "ne_gemm_simt")
 
 
 def _linear_simt(x, w, bias, out_fp32):
@@ -188,9 +188,10 @@ def _linear_simt(x, w, bias, out_fp32):
         x2 = x2.contiguous()
     T, (N, K) = x2.shape[0], w.shape
     out = torch.empty(T, N, dtype=torch.float32 if out_fp32 else w.dtype, device=x.device)
+    fused = bias is not None and bias.dtype == torch.float32
     if T > 0:
-        _gemm_simt(x2, x2.stride(0), 0, w, w.stride(0), 0, out, N, 0, T, N, K, 1)
-    if bias is not None:
+        _gemm_simt(x2, x2.stride(0), 0, w, w.stride(0), 0, out, N, 0, T, N, K, 1, bias if fused else None)
+    if bias is not None and not fused:
         out = out + bias
     return out.view(*x.shape[:-1], N)
 
@@ -228,6 +229,11 @@ def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None
             _gemm(q, K, 0, w, out, N, 0, T, N, K, 1, None, None, True, s, T, 0, w_scale, out_fp32)
         else:
             assert w.dtype == torch.bfloat16, "CUDA linears take bf16 or fp8 weights"
+            if bias is not None and bias.dtype == torch.float32:              # added in the epilogue, before the one rounding
+                assert bias.numel() == N and bias.is_contiguous()
+                _ck(lib().ne_gemm_bias(_p(x2), _c.c_longlong(x2.stride(0)), _p(w), _p(bias), _p(out), _c.c_longlong(N), _c.c_int(T), _c.c_int(N), _c.c_int(K),
+                                       _c.c_int(int(out_fp32)), _st()), "ne_gemm_bias")
+                return out.view(*x.shape[:-1], N)
             _gemm(x2, x2.stride(0), 0, w, out, N, 0, T, N, K, 1, None, None, False, None, 0, 0, None, out_fp32)
     if bias is not None:
         out = out + bias
@@ -339,6 +345,40 @@ def residual_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next
     return out, x
 
 
+def _stream_mix(y, x, w_out, mix, w_in, w_next, eps, last, ids, positions, table, pos):
+    T, S, W = x.shape
+    dt = w_next.dtype
+    assert x.dtype == torch.float32 and x.is_contiguous() and w_in.dtype == torch.float32 and w_in.numel() == S and w_in.is_contiguous()
+    out = torch.empty(T, W, dtype=dt, device=x.device)
+    if y is not None:
+        assert y.dtype == dt and y.stride(1) == 1 and w_out.dtype == mix.dtype == torch.float32 and mix.shape == (S, S) and mix.is_contiguous()
+    else:
+        assert table.dtype == dt and table.is_contiguous() and (pos is None or (pos.dtype == dt and pos.is_contiguous()))
+    _ck(lib().ne_stream_mix(_p(y), _c.c_longlong(0 if y is None else y.stride(0)), _p(x), _p(w_out), _p(mix), _p(w_in), _p(w_next), _p(out), _p(ids), _p(positions),
+                            _p(table), _c.c_int(0 if table is None else table.shape[0]), _p(pos), _c.c_int(0 if pos is None else pos.shape[0]), _c.c_int(T), _c.c_int(S),
+                            _c.c_int(W), _c.c_float(eps), _c.c_int(int(last)), _c.c_int(int(dt == torch.float32)), _st()), "ne_stream_mix")
+    return out, x
+
+
+def stream_mix(y: torch.Tensor, x: torch.Tensor, w_out: torch.Tensor, mix: torch.Tensor, w_in: torch.Tensor, w_next: torch.Tensor, eps: float,
+               last: bool = False):
+    """Streams mixed with a sublayer's output (in place), contracted and normed for the next one: one kernel, one CTA per row."""
+    return _stream_mix(y, x, w_out, mix, w_in, w_next, eps, last, None, None, None, None)
+
+
+def stream_embed(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos: Optional[torch.Tensor], w_in: torch.Tensor, w_next: torch.Tensor,
+                 eps: float):
+    x = torch.empty(ids.numel(), w_in.numel(), table.shape[1], dtype=torch.float32, device=table.device)
+    return _stream_mix(None, x, None, None, w_in, w_next, eps, False, _i64c(ids), _i64c(positions), table, pos)
+
+
+def cap_logits(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    assert logits.dtype == torch.float32
+    logits = logits.contiguous()
+    _ck(lib().ne_cap_rows(_p(logits), _c.c_longlong(logits.numel()), _c.c_float(float(cap)), _st()), "ne_cap_rows")
+    return logits
+
+
 def embed_norm(ids: torch.Tensor, table: torch.Tensor, w_next: torch.Tensor, eps: float, unit_offset: bool = True):
     """Embedding rows into a new 32-bit residual stream and the first norm, one kernel."""
     T, (V, W) = ids.numel(), table.shape
@@ -374,6 +414,8 @@ def _act_args(act):
         return _c.c_int(1), _c.c_float(float(act[1])), _c.c_float(0.0)
     if act[0] == "situ":
         return _c.c_int(2), _c.c_float(float(act[1])), _c.c_float(float(act[2] or 0.0))
+    if act[0] == "clamp_linear":
+        return _c.c_int(4), _c.c_float(float(act[1])), _c.c_float(float(act[2]))
     if act[0] == "gelu_tanh":
         return _c.c_int(3), _c.c_float(1.0), _c.c_float(0.0)
     raise ValueError(f"unknown gated activation {act!r}")
@@ -514,6 +556,15 @@ def gqa_kv_store(k_cache, v_cache, slot_mapping, k, v):
         v2 = v2.contiguous()
     _ck(lib().ne_gqa_kv_store(_p(k2), _p(v2), _c.c_longlong(k2.stride(0)), _c.c_longlong(v2.stride(0)), _p(k_cache), _p(v_cache),
                               _p(_i64c(slot_mapping)), _c.c_int(T), _c.c_int(row), _st()), "ne_gqa_kv_store")
+
+
+def kv_rows(k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> None:
+    T = k.shape[0]
+    kw, vw = k_cache.shape[2] * k_cache.shape[3], v_cache.shape[2] * v_cache.shape[3]
+    assert k_cache.dtype == v_cache.dtype == k.dtype == v.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k.shape == (T, kw) and v.shape == (T, vw) and k.stride(1) == 1 and v.stride(1) == 1
+    _ck(lib().ne_kv_rows(_p(k), _c.c_longlong(k.stride(0)), _p(v), _c.c_longlong(v.stride(0)), _p(k_cache), _p(v_cache), _p(_i64c(slot_mapping)), _c.c_int(T),
+                         _c.c_int(kw), _c.c_int(vw), _c.c_int(k.element_size()), _st()), "ne_kv_rows")
 
 
 def _i64c(t):
@@ -731,6 +782,13 @@ def gelu(x: torch.Tensor, tanh: bool = True) -> torch.Tensor:
     y = torch.empty_like(x)
     _ck(lib().ne_gelu(_p(x), _p(y), _c.c_longlong(x.numel()), _c.c_int(1 if tanh else 0), _st()), "ne_gelu")
     return y
+
+
+def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0, softcap: float = 0.0, slopes=None,
+                         gate=None, out_scale: float = 1.0, out=None, max_q_len: int = 0) -> torch.Tensor:
+    from . import sm100_attn
+    return sm100_attn.gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window, softcap, slopes, gate, out_scale, out,
+                                           max_q_len)
 
 
 def gqa_attention_paged(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0):
@@ -977,6 +1035,64 @@ def gated_delta(proj: torch.Tensor, ab: torch.Tensor, conv_w: torch.Tensor, A_lo
                          _c.byref(n), _st()), "ne_gated_delta")
     LAUNCHES[0] += n.value - 1
     return out
+
+
+def _decay_scan(q, k, v, gates, decay, skip, state, slots, cu, fresh, raw, H, Hk, Dk, Dv, act, max_q_len):
+    T = q.shape[0]
+    for t in (q, k, v):
+        assert t.stride(1) == 1 and t.dtype == q.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, Dv, Dk)
+    _ck(lib().ne_decay_scan(_p(q), _c.c_longlong(q.stride(0)), _p(k), _c.c_longlong(k.stride(0)), _p(v), _c.c_longlong(v.stride(0)), _p(gates), _p(decay), _p(skip),
+                            _p(state), _p(slots), _p(cu), _p(fresh), _p(raw), _c.c_int(T), _c.c_int(cu.numel() - 1), _c.c_int(H), _c.c_int(Hk), _c.c_int(Dk),
+                            _c.c_int(Dv), _c.c_int(act), _c.c_int(max_q_len), _c.c_int(int(q.dtype == torch.float32)), _st()), "ne_decay_scan")
+
+
+def _gated_norm(raw, gate, w, out, parts, before, eps, scale):
+    T, W = out.shape
+    assert gate.stride(1) == 1 and out.stride(1) == 1 and gate.dtype == w.dtype == out.dtype and w.is_contiguous()
+    _ck(lib().ne_gated_norm(_p(raw), _p(gate), _c.c_longlong(gate.stride(0)), _p(w), _p(out), _c.c_longlong(out.stride(0)), _c.c_int(T), _c.c_int(W), _c.c_int(parts),
+                            _c.c_int(int(before)), _c.c_float(eps), _c.c_float(scale), _c.c_int(int(out.dtype == torch.float32)), _st()), "ne_gated_norm")
+    return out
+
+
+def mamba2_mix(proj: torch.Tensor, dt_raw: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor,
+               D: torch.Tensor, norm_w: torch.Tensor, norm_groups: int, window: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+               cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, G: int, Dv: int, N: int, eps: float, max_q_len: int = 1) -> torch.Tensor:
+    """Three kernels: convolution and step sizes, the recurrence, the gated norm."""
+    T, inner = proj.shape[0], H * Dv
+    C, K = conv_w.shape
+    f32 = proj.dtype == torch.float32
+    assert C == inner + 2 * G * N and proj.stride(1) == 1 and proj.shape[1] >= inner + C and dt_raw.dtype == torch.float32 and dt_raw.stride(1) == 1
+    assert conv_w.dtype == conv_b.dtype == window.dtype == proj.dtype and conv_w.is_contiguous() and window.is_contiguous() and window.shape[1:] == (K - 1, C)
+    assert A_log.dtype == dt_bias.dtype == D.dtype == torch.float32
+    out = torch.empty(T, inner, dtype=proj.dtype, device=proj.device)
+    if T == 0:
+        return out
+    slots, cu, fresh = _i32(slots), _i32(cu_seqlens), _i32(fresh)
+    xbc = torch.empty(T, C, dtype=proj.dtype, device=proj.device)
+    gates = torch.empty(T, H, 2, dtype=torch.float32, device=proj.device)
+    raw = torch.empty(T, inner, dtype=torch.float32, device=proj.device)
+    src = proj[:, inner: inner + C]
+    _ck(lib().ne_ssm_prepare(_p(src), _c.c_longlong(proj.stride(0)), _p(dt_raw), _c.c_longlong(dt_raw.stride(0)), _p(conv_w), _p(conv_b), _p(A_log), _p(dt_bias),
+                             _p(window), _p(slots), _p(cu), _p(fresh), _p(xbc), _p(gates), _c.c_int(T), _c.c_int(cu.numel() - 1), _c.c_int(H), _c.c_int(C), _c.c_int(K),
+                             _c.c_int(int(f32)), _st()), "ne_ssm_prepare")
+    _decay_scan(xbc[:, inner + G * N:], xbc[:, inner: inner + G * N], xbc[:, :inner], gates, None, D, state, slots, cu, fresh, raw, H, G, N, Dv, 0, max_q_len)
+    return _gated_norm(raw, proj[:, :inner], norm_w, out, norm_groups, True, eps, 1.0)
+
+
+def lightning_mix(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor,
+                  slots: torch.Tensor, cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, Dk: int, Dv: int, eps: float, out_scale: float = 1.0,
+                  out: Optional[torch.Tensor] = None, max_q_len: int = 1) -> torch.Tensor:
+    """Two kernels: the recurrence (silu of its inputs included) and the gated norm."""
+    T = q.shape[0]
+    if out is None:
+        out = torch.empty(T, H * Dv, dtype=q.dtype, device=q.device)
+    if T == 0:
+        return out
+    assert decay.dtype == torch.float32 and decay.numel() == H
+    raw = torch.empty(T, H * Dv, dtype=torch.float32, device=q.device)
+    _decay_scan(q, k, v, None, decay, None, state, _i32(slots), _i32(cu_seqlens), _i32(fresh), raw, H, H, Dk, Dv, 1, max_q_len)
+    return _gated_norm(raw, gate, norm_w, out, 1, False, eps, out_scale)
 
 
 def kda_recurrent(q, k, v, raw_g, b, A_log, dt_bias, lower_bound, state, slots, cu_seqlens, fresh, gate, norm_w, eps: float) -> torch.Tensor:

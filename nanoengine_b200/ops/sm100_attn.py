@@ -204,6 +204,59 @@ def gqa_attention_paged(q, k_cache, v_cache, block_tables, cu_seqlens_q, context
     return out
 
 
+BIASED_TC_CALLS = [0]        # launches of the tensor-core kernel of gqa_attention_biased
+
+
+def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window=0, softcap=0.0, slopes=None, gate=None, out_scale=1.0,
+                         out=None, max_q_len=0, splits=None):
+    """bf16 with head sizes in multiples of 8 up to 256 and 64-token pages: tensor cores; other shapes and 32-bit runs: the generic kernel."""
+    T, Hq, D = q.shape
+    Hkv, Dv = k_cache.shape[2], v_cache.shape[3]
+    lib = _k.lib()
+    bt, cu, cl = _i32(block_tables), _i32(cu_seqlens_q), _i32(context_lens)
+    B = cl.numel()
+    assert q.dtype == k_cache.dtype == v_cache.dtype and q.dtype in (torch.bfloat16, torch.float32) and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert q.stride(2) == 1 and q.stride(1) == D and k_cache.shape[3] == D and Hq % Hkv == 0
+    assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == Hq)
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
+    if out is None:
+        out = torch.empty(T, Hq * Dv, dtype=q.dtype, device=q.device)
+    assert out.dtype == q.dtype and out.shape == (T, Hq * Dv) and out.stride(1) == 1
+    if T == 0:
+        return out
+    gate_ld = 0 if gate is None else gate.stride(0)
+    mq = max_q_len if max_q_len else (1 if T <= B else T)
+    tq = 0
+    if (q.dtype == torch.bfloat16 and k_cache.shape[1] == 64 and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
+            and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
+        tq = lib.ne_gqa_biased_plan(_c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq))
+    if tq:
+        tiles = min(T, T // tq + B)
+        S = splits
+        if S is None:
+            pages = bt.shape[1] if window <= 0 else min(bt.shape[1], (window + tq + 62) // 64 + 1)
+            S = 1
+            if tiles * Hkv < 74:                       # few CTAs (small decode batches): slice the keys
+                S = max(1, min(148 // (tiles * Hkv), max(1, pages // 4), 16))
+        part = lse2 = None
+        if S > 1:
+            part = torch.empty(S, T, Hq, Dv, dtype=torch.float32, device=q.device)
+            lse2 = torch.empty(S, T, Hq, dtype=torch.float32, device=q.device)
+        _k._ck(lib.ne_gqa_biased(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _c.c_int(k_cache.shape[0]), _k._p(bt), _c.c_int(bt.stride(0)),
+                                 _k._p(cu), _k._p(cl), _c.c_int(B), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq),
+                                 _c.c_int(tiles), _c.c_int(S), _c.c_float(scale), _c.c_float(softcap), _k._p(slopes), _c.c_int(int(window)), _k._p(gate),
+                                 _c.c_longlong(gate_ld), _c.c_float(out_scale), _k._p(out), _c.c_longlong(out.stride(0)), _k._p(part), _k._p(lse2), _k._st()),
+               "ne_gqa_biased")
+        BIASED_TC_CALLS[0] += 1
+        _k.LAUNCHES[0] += int(S > 1)
+        return out
+    _k._ck(lib.ne_attn_biased(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _k._p(bt), _c.c_int(bt.stride(0)), _c.c_int(k_cache.shape[1]),
+                              _k._p(cu), _k._p(cl), _c.c_int(B), _k._p(out), _c.c_longlong(out.stride(0)), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D),
+                              _c.c_int(Dv), _c.c_float(scale), _c.c_float(softcap), _k._p(slopes), _c.c_int(int(window)), _k._p(gate), _c.c_longlong(gate_ld),
+                              _c.c_float(out_scale), _c.c_int(int(q.dtype == torch.float32)), _k._st()), "ne_attn_biased")
+    return out
+
+
 def attention_varlen(q, k, v, cu_seqlens, scale, causal: bool = False):
     """Attention over ragged sequences without a paged cache: q, k, v [T, H, D] of the same tokens, sequence i owns rows
     [cu[i], cu[i+1]).  Runs on the generic kernel, which addresses k / v as a one-row-per-page cache through a table of row
