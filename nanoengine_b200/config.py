@@ -203,8 +203,13 @@ class Config:
         if mc.layer_specs:
             if self.attention_tp != 1 or self.pp != 1:
                 raise ValueError("models with listed layers run with attention_tp = pp = 1")
-            # the design has no context limit: the rotary tables follow the engine's
-            mc.max_position_embeddings = max(mc.max_position_embeddings, self.max_model_len)
+            if mc.learned_positions:
+                if self.max_model_len > mc.max_position_embeddings:
+                    raise ValueError(f"max_model_len {self.max_model_len} is past the model's {mc.max_position_embeddings} learned positions")
+            else:                                       # no context limit of its own: the rotary tables follow the engine's
+                mc.max_position_embeddings = max(mc.max_position_embeddings, self.max_model_len)
+            if not mc.is_mla and self.resolved_kv_dtype() != self.dtype:
+                raise ValueError("key / value rows of listed layers are kept in the activation dtype: leave kv_cache_dtype at auto")
         if self.max_num_seqs < 1 or self.max_num_batched_tokens < 1:
             raise ValueError("max_num_seqs and max_num_batched_tokens must be positive")
         if not (0.0 < self.gpu_memory_utilization <= 1.0):

@@ -12,6 +12,10 @@ from dataclasses import dataclass, field, fields
 from typing import Any, Dict, List, Optional
 
 
+# mixers of listed layers that carry a recurrent state per sequence
+_STATE_MIXERS = ("delta", "mamba2", "parallel")
+
+
 @dataclass
 class ModelConfig:
     architecture: str = "DeepseekV3ForCausalLM"
@@ -102,10 +106,11 @@ class ModelConfig:
     o_lora_rank: int = 0
     o_groups: int = 0
     num_hash_layers: int = 0                 # the first this-many MoE layers pick experts from a token-id table
-    # Tuvutar: every layer is listed with its own mixer ("latent_attention" | "delta"), the mixer's sizes and its feed-forward; the
-    # fields above describe one such layer only in the form `layer_config` derives for it
+    # families that list every layer with its own mixer, the mixer's sizes and its feed-forward (Tuvutar: "latent_attention" | "delta",
+    # Filasun: "mamba2" | "parallel"); the fields above describe one such layer only in the form `layer_config` derives for it
     layer_specs: Optional[List[Dict[str, Any]]] = None
     attn_scale: float = 0.0                  # > 0: softmax scale of the latent-attention layer (0: from the head dim)
+    learned_positions: bool = False          # a learned vector per position, max_position_embeddings of them: a hard context limit
     # MTP
     num_nextn_predict_layers: int = 0
     # quantisation of linear / expert weights: None (use dtype) or "fp8" (e4m3, 128x128 block scales)
@@ -135,7 +140,7 @@ class ModelConfig:
     @property
     def is_hybrid_gdn(self) -> bool:
         if self.layer_specs:
-            return any(s["type"] == "delta" for s in self.layer_specs)
+            return any(s["type"] in _STATE_MIXERS for s in self.layer_specs)
         return self.linear_num_value_heads > 0
 
     def layer_config(self, layer_idx: int) -> "ModelConfig":
@@ -183,13 +188,28 @@ class ModelConfig:
 
     def layer_type(self, layer_idx: int) -> str:
         if self.layer_specs:
-            return "linear_attention" if self.layer_specs[layer_idx]["type"] == "delta" else "full_attention"
+            return "linear_attention" if self.layer_specs[layer_idx]["type"] in ("delta", "mamba2") else "full_attention"
         if not self.is_hybrid_gdn:
             return "full_attention"
         if self.layer_types and layer_idx < len(self.layer_types):
             return self.layer_types[layer_idx]
         n = self.full_attention_interval
         return "full_attention" if n > 0 and (layer_idx + 1) % n == 0 else "linear_attention"
+
+    def keeps_rows(self, layer_idx: int) -> bool:
+        """Does the listed layer own pages of the paged cache?"""
+        t = self.layer_specs[layer_idx]["type"]
+        return t in ("latent_attention", "parallel") and self.kv_source_layer(layer_idx) == layer_idx
+
+    def keeps_state(self, layer_idx: int) -> bool:
+        """Does the listed layer own a slot of recurrent state per sequence?  A "parallel" layer owns both."""
+        return self.layer_specs[layer_idx]["type"] in _STATE_MIXERS
+
+    def cache_rank(self, layer_idx: int) -> int:
+        return sum(1 for i in range(layer_idx) if self.keeps_rows(i))
+
+    def state_rank(self, layer_idx: int) -> int:
+        return sum(1 for i in range(layer_idx) if self.keeps_state(i))
 
     def num_layers_of(self, kind: str, upto: Optional[int] = None) -> int:
         return sum(1 for i in range(self.num_hidden_layers if upto is None else upto) if self.layer_type(i) == kind)
@@ -266,6 +286,8 @@ class ModelConfig:
         arch = d.get("architecture", "")
         if arch == "Tuvutar" and "layers" in d:
             d = _tuvutar_fields(d)
+        if arch == "Filasun" and "layers" in d:
+            d = _filasun_fields(d)
         la = d.pop("linear_attn_config", None)
         if isinstance(la, dict):                          # Kimi delta attention block of GLM5-next / Kimi-K3
             d["linear_kind"] = "kda"
@@ -408,6 +430,42 @@ def _tuvutar_fields(d: Dict[str, Any]) -> Dict[str, Any]:
            "n_routed_experts": 0, "n_shared_experts": 0, "max_position_embeddings": 131072, "tie_word_embeddings": False,
            "layer_specs": [{"type": s["type"], "mixer": dict(s["mixer"]), "mlp": dict(s["mlp"]) if s.get("mlp") is not None else None} for s in d["layers"]]}
     for k in ("eos_token_id", "bos_token_id", "max_position_embeddings"):
+        if d.get(k) is not None:
+            out[k] = d[k]
+    return out
+
+
+def _filasun_fields(d: Dict[str, Any]) -> Dict[str, Any]:
+    """config.json of a Filasun model ({architecture, layers, logit_softcap, max_positions, norm, streams, vocab, width}) as ModelConfig fields."""
+    def need(ok, i, what):
+        if not ok:
+            raise ValueError(f"layer {i}: {what}")
+
+    for i, s in enumerate(d["layers"]):
+        m = s["mixer"]
+        if s["type"] == "mamba2":
+            need(int(m["heads"]) % int(m["groups"]) == 0, i, "heads must be a multiple of groups")
+            need(int(m["heads"]) * int(m["vdim"]) % int(m["norm_groups"]) == 0, i, "norm_groups must divide heads * vdim")
+            need(1 <= int(m["conv"]) <= 16, i, "1 to 16 convolution taps")
+        elif s["type"] == "parallel":
+            l, r = m["left"], m["right"]
+            need(int(l["heads"]) % int(l["kv_heads"]) == 0, i, "heads must be a multiple of kv_heads")
+            need(int(l["mask"]["size"]) >= 1, i, "the window holds at least the token itself")
+            need(float(l["softcap"]) > 0, i, "softcap must be positive")
+            need(len(r["decay"]) == int(r["heads"]) and all(0 <= float(v) <= 1 for v in r["decay"]), i, "one decay in [0, 1] per head")
+        else:
+            need(False, i, f"unknown mixer type {s['type']!r}")
+        if s.get("mlp") is not None:
+            need(s["mlp"]["kind"] == "dense", i, f"unknown feed-forward kind {s['mlp']['kind']!r}")
+            need(float(s["mlp"]["limit"]) > 0, i, "limit must be positive")
+    if not 1 <= int(d["streams"]) <= 16 or not float(d["logit_softcap"]) > 0:
+        raise ValueError("1 to 16 streams and a positive logit_softcap")
+    out = {"architecture": d["architecture"], "vocab_size": int(d["vocab"]), "hidden_size": int(d["width"]), "num_hidden_layers": len(d["layers"]),
+           "rms_norm_eps": float(d["norm"]["eps"]), "q_lora_rank": None, "n_routed_experts": 0, "n_shared_experts": 0, "tie_word_embeddings": False,
+           "num_attention_heads": 1, "num_key_value_heads": 1, "max_position_embeddings": int(d["max_positions"]), "learned_positions": True,
+           "hc_mult": int(d["streams"]), "final_logit_softcapping": float(d["logit_softcap"]),
+           "layer_specs": [{"type": s["type"], "mixer": dict(s["mixer"]), "mlp": dict(s["mlp"]) if s.get("mlp") is not None else None} for s in d["layers"]]}
+    for k in ("eos_token_id", "bos_token_id"):
         if d.get(k) is not None:
             out[k] = d[k]
     return out
@@ -589,3 +647,42 @@ def tuvutar_7b(**over) -> ModelConfig:
 
 
 PRESETS["tiny-tuvutar"], PRESETS["tuvutar-7b"] = tiny_tuvutar, tuvutar_7b
+
+
+def _mamba2_spec(heads, vdim, state, groups, conv, norm_groups=1, ff=0, limit=7.0):
+    return {"type": "mamba2", "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups},
+            "mlp": {"kind": "dense", "ff": ff, "limit": limit} if ff else None}
+
+
+def _parallel_spec(heads, kv_heads, dim, vdim, window, l_heads, l_dim, l_vdim, ff=0, softcap=50.0, scales=(0.7, 0.7), limit=7.0):
+    decay = [1.0 - 2.0 ** (-(1.0 + 8.0 * i / l_heads)) for i in range(l_heads)]
+    return {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "softcap": softcap, "mask": {"size": window}},
+        "right": {"heads": l_heads, "dim": l_dim, "vdim": l_vdim, "decay": decay}, "left_scale": scales[0], "right_scale": scales[1]},
+        "mlp": {"kind": "dense", "ff": ff, "limit": limit} if ff else None}
+
+
+def tiny_filasun(**over) -> ModelConfig:
+    """CPU-sized Filasun shape: two parallel layers of unlike sizes around a Mamba-2 layer, three streams."""
+    c = ModelConfig.from_dict({"architecture": "Filasun", "vocab": 512, "width": 128, "norm": {"eps": 1e-6}, "streams": 3, "logit_softcap": 20.0,
+                               "max_positions": 1024, "layers": [_parallel_spec(4, 2, 16, 24, 40, 2, 32, 16, ff=192), _mamba2_spec(4, 16, 24, 2, 4, 2),
+                                                                 _parallel_spec(6, 1, 24, 16, 100, 3, 16, 24, ff=96)]})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+def filasun_7b(**over) -> ModelConfig:
+    """A Filasun shape of a real model's layer sizes (7B class): width 4096, one Mamba-2 layer (128 heads of 64, state 128, 8 groups) after every
+    three parallel layers (32 / 8 attention heads of 128 over a 4096-token window, 32 decayed heads of 128), two streams."""
+    layers = []
+    for _ in range(6):
+        layers += [_parallel_spec(32, 8, 128, 128, 4096, 32, 128, 128, ff=12288) for _ in range(3)] + [_mamba2_spec(128, 64, 128, 8, 4, 8)]
+    c = ModelConfig.from_dict({"architecture": "Filasun", "vocab": 131072, "width": 4096, "norm": {"eps": 1e-6}, "streams": 2, "logit_softcap": 30.0,
+                               "max_positions": 32768, "layers": layers})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+PRESETS["tiny-filasun"], PRESETS["filasun-7b"] = tiny_filasun, filasun_7b

@@ -162,7 +162,7 @@ class Gemma4ForCausalLM(nn.Module):
         w = self.model.embed_tokens.weight if self.lm_head is None else self.lm_head.weight
         logits = ops.lm_head(hidden, w)
         cap = self.cfg.final_logit_softcapping
-        return torch.tanh(logits / cap) * cap if cap else logits
+        return ops.cap_logits(logits, cap) if cap else logits
 
     # ---- weights ---------------------------------------------------------------------------
     def load_weights(self, weights: Iterable[Tuple[str, torch.Tensor]]) -> int:

@@ -22,9 +22,10 @@ def _ceil_div(a, b):
 
 
 class QLinear(nn.Module):
-    """y = x W^T with W [out, in] in the activation dtype or in fp8 e4m3 with 128x128 block scales."""
+    """y = x W^T with W [out, in] in the activation dtype or in fp8 e4m3 with 128x128 block scales.  `bias_fp32`: a bias kept in fp32
+    and added to the accumulator before the result is rounded (in the GEMM's epilogue on the GPU)."""
 
-    def __init__(self, in_features: int, out_features: int, dtype, device, quant: Optional[str] = None, bias: bool = False):
+    def __init__(self, in_features: int, out_features: int, dtype, device, quant: Optional[str] = None, bias: bool = False, bias_fp32: bool = False):
         super().__init__()
         self.in_features, self.out_features, self.quant = in_features, out_features, quant
         if quant == "fp8":
@@ -38,6 +39,8 @@ class QLinear(nn.Module):
                                        requires_grad=False)
             self.weight_scale_inv = None
         self.bias = nn.Parameter(torch.zeros(out_features, dtype=dtype, device=device), requires_grad=False) if bias else None
+        if bias_fp32:
+            self.bias = nn.Parameter(torch.zeros(self.weight.shape[0], dtype=torch.float32, device=device), requires_grad=False)
 
     def forward(self, x):
         y = ops.linear(x, self.weight, self.weight_scale_inv, self.bias)

@@ -1,0 +1,119 @@
+"""Sequence mixers with explicit sizes and constants, for families that list their layers one by one.
+
+Mamba2Mixer     z | x | B | C from one GEMM, the step sizes from a second one with an fp32 result; short convolution, state-space recurrence
+                and gated norm are `ops.mamba2_mix`.
+ParallelMixer   two mixers over the same input, summed with constant weights: windowed grouped-query attention with capped scores, a
+                distance bias and an output gate per head (`ops.gqa_attention_biased`), and linear attention with a constant decay per head
+                (`ops.lightning_mix`).  Both read one merged projection and write into one row, so the pair costs two GEMMs; the weights of
+                the sum are applied to the fp32 results before they are rounded.  The layer owns rows of the paged cache and a state."""
+from __future__ import annotations
+
+from typing import Dict, Sequence
+
+import torch
+import torch.nn as nn
+
+from .. import ops
+from ..runtime.context import ForwardContext
+from .layers import QLinear
+
+
+def _const(*shape, dtype=torch.float32, device=None, fill=0.0):
+    return nn.Parameter(torch.full(shape, fill, dtype=dtype, device=device), requires_grad=False)
+
+
+def distance_slopes(heads: int) -> torch.Tensor:
+    """Geometric slopes 2^(-8 (h + 1) / heads) of the distance bias."""
+    return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float32)
+
+
+class Mamba2Mixer(nn.Module):
+    def __init__(self, hidden: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_groups: int, eps: float, state_idx: int, dtype, device):
+        super().__init__()
+        self.heads, self.vdim, self.state, self.groups, self.norm_groups = heads, vdim, state, groups, norm_groups
+        self.eps, self.state_idx = eps, state_idx
+        self.inner = heads * vdim
+        self.conv_dim = self.inner + 2 * groups * state
+        self.in_proj = QLinear(hidden, self.inner + self.conv_dim, dtype, device, None)
+        self.dt_proj = QLinear(hidden, heads, dtype, device, None)
+        self.out_proj = QLinear(self.inner, hidden, dtype, device, None)
+        self.conv_weight, self.conv_bias = _const(self.conv_dim, conv, dtype=dtype, device=device), _const(self.conv_dim, dtype=dtype, device=device)
+        self.A_log, self.dt_bias, self.D = (_const(heads, device=device) for _ in range(3))
+        self.norm_weight = _const(self.inner, dtype=dtype, device=device, fill=1.0)
+
+    def forward(self, h, ctx: ForwardContext):
+        proj = self.in_proj(h)
+        dt = ops.linear_fp32(h, self.dt_proj.weight)[:, : self.heads]
+        y = ops.mamba2_mix(proj, dt, self.conv_weight, self.conv_bias, self.A_log, self.dt_bias, self.D, self.norm_weight, self.norm_groups,
+                           ctx.conv_states[self.state_idx], ctx.rec_states[self.state_idx], ctx.state_slots, ctx.cu_seqlens_q, ctx.seq_fresh,
+                           self.heads, self.groups, self.vdim, self.state, self.eps, ctx.max_seqlen_q)
+        return self.out_proj(y)
+
+    def parts(self):
+        """Tensor name below the mixer -> shape."""
+        D = self.in_proj.in_features
+        return {"in": (self.inner + self.conv_dim + self.heads, D), "conv": tuple(self.conv_weight.shape), "conv.b": (self.conv_dim,),
+                "dt_bias": (self.heads,), "A_log": (self.heads,), "D": (self.heads,), "norm": (self.inner,), "o": (D, self.inner)}
+
+    def load(self, w: Dict[str, torch.Tensor]) -> None:
+        rows = self.inner + self.conv_dim
+        self.in_proj.set_weight(w["in"][:rows])
+        self.dt_proj.set_weight(w["in"][rows:])
+        self.out_proj.set_weight(w["o"])
+        for p, n in ((self.conv_weight, "conv"), (self.conv_bias, "conv.b"), (self.A_log, "A_log"), (self.dt_bias, "dt_bias"), (self.D, "D"), (self.norm_weight, "norm")):
+            p.copy_(w[n])
+
+
+class ParallelMixer(nn.Module):
+    # rows of the merged projection; the gate of the attention heads, a few odd rows, comes last
+    ORDER = ("left.q", "left.k", "left.v", "right.q", "right.k", "right.v", "right.g", "left.g")
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, softcap: float, window: int, lin_heads: int, lin_dim: int,
+                 lin_vdim: int, decay: Sequence[float], left_scale: float, right_scale: float, eps: float, cache_idx: int, state_idx: int, dtype, device):
+        super().__init__()
+        self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = hidden, heads, kv_heads, dim, vdim
+        self.scale, self.softcap, self.window = scale, softcap, window
+        self.lin_heads, self.lin_dim, self.lin_vdim = lin_heads, lin_dim, lin_vdim
+        self.left_scale, self.right_scale, self.eps, self.cache_idx, self.state_idx = left_scale, right_scale, eps, cache_idx, state_idx
+        rows = {n: self.parts()[n][0] for n in self.ORDER}
+        self.rows = [rows[n] for n in self.ORDER]
+        self.left_width, self.right_width = heads * vdim, lin_heads * lin_vdim
+        self.in_proj = QLinear(hidden, sum(self.rows), dtype, device, None, bias_fp32=True)
+        self.out_proj = QLinear(self.left_width + self.right_width, hidden, dtype, device, None, bias_fp32=True)
+        self.norm_weight = _const(self.right_width, dtype=dtype, device=device, fill=1.0)
+        self.register_buffer("slopes", distance_slopes(heads).to(device), persistent=False)
+        self.register_buffer("decay", torch.tensor(list(decay), dtype=torch.float64).float().to(device), persistent=False)
+
+    def forward(self, h, ctx: ForwardContext):
+        T = h.shape[0]
+        q, k, v, lq, lk, lv, lg, gate = self.in_proj(h).split(self.rows, -1)
+        kc, vc = ctx.kv_caches[self.cache_idx]
+        ops.kv_rows(kc, vc, ctx.slot_mapping, k, v)
+        y = torch.empty(T, self.left_width + self.right_width, dtype=h.dtype, device=h.device)
+        ops.gqa_attention_biased(q.unflatten(-1, (self.heads, self.dim)), kc, vc, ctx.block_tables, ctx.cu_seqlens_q, ctx.context_lens, self.scale, self.window,
+                                 self.softcap, self.slopes, gate, self.left_scale, y[:, : self.left_width], ctx.max_seqlen_q)
+        ops.lightning_mix(lq, lk, lv, lg, self.decay, self.norm_weight, ctx.rec_states[self.state_idx], ctx.state_slots, ctx.cu_seqlens_q, ctx.seq_fresh,
+                          self.lin_heads, self.lin_dim, self.lin_vdim, self.eps, self.right_scale, y[:, self.left_width:], ctx.max_seqlen_q)
+        return self.out_proj(y)
+
+    def parts(self):
+        D, H, G = self.hidden, self.heads, self.kv_heads
+        out = {}
+        for n, r in (("q", H * self.dim), ("k", G * self.dim), ("v", G * self.vdim)):
+            out["left." + n], out[f"left.{n}.b"] = (r, D), (r,)
+        out["left.g"], out["left.o"], out["left.o.b"] = (H, D), (D, H * self.vdim), (D,)
+        lq, lv = self.lin_heads * self.lin_dim, self.lin_heads * self.lin_vdim
+        for n, r in (("q", lq), ("k", lq), ("v", lv), ("g", lv)):
+            out["right." + n] = (r, D)
+        out["right.norm"], out["right.o"] = (lv,), (D, lv)
+        return out
+
+    def load(self, w: Dict[str, torch.Tensor]) -> None:
+        self.in_proj.set_weight(torch.cat([w[n] for n in self.ORDER], 0))
+        b = torch.cat([w["left.q.b"], w["left.k.b"], w["left.v.b"]])
+        self.in_proj.bias.zero_()
+        self.in_proj.bias[: b.numel()].copy_(b)
+        self.out_proj.set_weight(torch.cat([w["left.o"], w["right.o"]], 1))
+        self.out_proj.bias.zero_()
+        self.out_proj.bias[: self.hidden].copy_(self.left_scale * w["left.o.b"])
+        self.norm_weight.copy_(w["right.norm"])

@@ -54,8 +54,14 @@ def _tuvutar():
     return TuvutarForCausalLM
 
 
+def _filasun():
+    from .filasun import FilasunForCausalLM
+    return FilasunForCausalLM
+
+
 # kernel sources (stems under csrc/) of the architectures that can be served from a partial build; None = all of them
-_KERNELS = {"Tuvutar": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_bf16", "mla_bf16", "delta")}
+_KERNELS = {"Tuvutar": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_bf16", "mla_bf16", "delta"),
+            "Filasun": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "linattn")}
 
 
 def kernel_sources(architecture: str):
@@ -63,7 +69,7 @@ def kernel_sources(architecture: str):
 
 
 _LAZY = {
-    "Tuvutar": _tuvutar,
+    "Tuvutar": _tuvutar, "Filasun": _filasun,
     "Gemma4ForCausalLM": _gemma4, "Gemma4ForConditionalGeneration": _gemma4,
     "Glm5NextForConditionalGeneration": _glm5_next, "KimiK3ForConditionalGeneration": _kimi_k3,
     "DeepseekV4ForCausalLM": _deepseek_v4,

@@ -68,6 +68,9 @@ def hf_param_shapes(cfg: ModelConfig, include_mtp: bool = False) -> Dict[str, Tu
     if cfg.architecture.startswith("Gemma4"):
         return _gemma4_param_shapes(cfg, out)
     if cfg.layer_specs:
+        if cfg.architecture == "Filasun":
+            from .filasun import filasun_param_shapes
+            return filasun_param_shapes(cfg)
         from .tuvutar import tuvutar_param_shapes
         return tuvutar_param_shapes(cfg)
     if cfg.is_dsv4:
@@ -239,6 +242,10 @@ def random_hf_weights(cfg: ModelConfig, seed: int = 0, device="cpu", keep: Optio
         g.manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
         if cfg.layer_specs:                     # rows scaled by their fan-in, norm weights around zero or one
             leaf = name.rsplit(".", 1)[-1]
+            if cfg.architecture == "Filasun":
+                from .filasun import filasun_random_tensor
+                yield name, filasun_random_tensor(name, shape, g, dev)
+                continue
             if leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm":
                 t = 0.1 * torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
             elif leaf == "norm":

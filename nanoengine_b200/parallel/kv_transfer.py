@@ -123,12 +123,12 @@ class LocalTransport:
              src_state: int = -1, dst_state: int = -1) -> int:
         s, d = self.src[src_dp], self.dst[dst_dp]
         sc, dc = s.cache, d.cache
-        listed = sc.plan.latent_rows is not None             # one page tensor per layer, page id in front
+        listed = sc.plan.listed                              # one page tensor per layer, page id in front
         bdim = 0 if listed else (1 if sc.plan.mla else 2)
         si = torch.as_tensor(src_blocks, dtype=torch.long)
         di = torch.as_tensor(dst_blocks, dtype=torch.long)
         n = 0
-        for skv, dkv in zip(sc.layers if listed else [sc.kv], dc.layers if listed else [dc.kv]):
+        for skv, dkv in zip(sc.row_tensors() if listed else [sc.kv], dc.row_tensors() if listed else [dc.kv]):
             skv = skv.view(torch.uint8) if skv.dtype == torch.float8_e4m3fn else skv
             dkv = dkv.view(torch.uint8) if dkv.dtype == torch.float8_e4m3fn else dkv
             rows = skv.index_select(bdim, si.to(skv.device))

@@ -14,10 +14,12 @@ DeepSeek-V4        one shared key / value row per token and layer in the latent-
                    compressor's carry [c * ratio, c * head_dim] fp32 twice (values and scores; c = 2 for ratio 4).  With an fp8 cache a row
                    is 584 packed bytes (448 e4m3 values, 64 bf16 rotated dims, 7 scale bytes + pad) instead of head_dim values.
 
-listed layers      families that list their layers one by one (Tuvutar) may give every latent layer its own row width and every
-                   delta layer its own state shape: one tensor per layer instead of the stacked ones ([blocks, block_size, D_l];
-                   [slots, Hv_l, Dv_l, Dk_l] fp32 and [slots, K_l - 1, conv_dim_l]), page families `latent_<n>`, slot families
-                   `delta_state_<n>` / `delta_conv_<n>`.  A layer that reads an earlier layer's rows owns none.
+listed layers      families that list their layers one by one (Tuvutar, Filasun) may give every layer its own row widths and state shape:
+                   one tensor per layer instead of the stacked ones - latent rows [blocks, block_size, D_l], or keys [blocks, block_size,
+                   G_l, D_l] and values [.., G_l, Dv_l]; states [slots, Hv_l, Dv_l, Dk_l] fp32 and convolution windows [slots, K_l - 1,
+                   conv_dim_l].  Page families `latent_<n>` or `key_<n>` / `value_<n>`, slot families `delta_state_<n>` / `delta_conv_<n>`.  A
+                   layer may own rows, a state, both (attention and linear attention side by side) or neither (it reads an earlier layer's
+                   rows); rows and states are numbered separately.
 
 One extra block past the scheduler-visible range is reserved as the scratch page that dummy batches of idle
 DP ranks write into.
@@ -69,8 +71,10 @@ class CachePlan:
     # the same number, or the bytes of a packed row when the cache keeps fp8 values)
     dsv4_ratios: Optional[List[int]] = None
     dsv4_head_dim: int = 0
-    # listed layers: row width of every latent layer that keeps rows, (heads, Dv, Dk, taps, conv channels) of every delta layer
+    # listed layers: row width of every latent layer that keeps rows, (kv heads, D, Dv) of every layer that keeps keys and values,
+    # (heads, Dv, Dk, taps, conv channels) of every layer with a recurrent state (taps 1, channels 0: no convolution)
     latent_rows: Optional[List[int]] = None
+    kv_shapes: Optional[List[tuple]] = None
     delta_shapes: Optional[List[tuple]] = None
     hisparse: bool = False
     hot_rows: int = 0
@@ -80,6 +84,11 @@ class CachePlan:
     @property
     def dsv4(self) -> bool:
         return self.dsv4_ratios is not None
+
+    @property
+    def listed(self) -> bool:
+        """One cache tensor per layer, page id in front."""
+        return self.latent_rows is not None or self.kv_shapes is not None
 
     @property
     def needs_state_slots(self) -> bool:
@@ -111,6 +120,8 @@ class CachePlan:
             return (self.num_layers * self.block_size + sum(self.comp_entries_per_page(r) for r in self.dsv4_ratios if r)) * self.row_dim * e
         if self.latent_rows is not None:
             return self.block_size * sum(self.latent_rows) * e
+        if self.kv_shapes is not None:
+            return self.block_size * sum(g * (d + dv) for g, d, dv in self.kv_shapes) * e
         if self.mla:
             return self.num_layers * self.block_size * self.row_dim * e
         return 2 * self.num_layers * self.block_size * self.kv_heads_local * self.row_dim * e
@@ -171,7 +182,20 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
                          dsv4_ratios=[mc.compress_ratio(i) for i in range(mc.num_hidden_layers)], dsv4_head_dim=mc.head_dim)
     if mc.layer_specs:
         n = mc.num_hidden_layers
-        own = [i for i in range(n) if mc.layer_type(i) == "full_attention" and mc.kv_source_layer(i) == i]
+        own = [i for i in range(n) if mc.keeps_rows(i)]
+        if not mc.is_mla:
+            mixers = [mc.layer_specs[i] for i in range(n)]
+            kv = [(int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])) for m in (mixers[i]["mixer"]["left"] for i in own)]
+            shapes = []
+            for s in mixers:
+                m = s["mixer"]
+                if s["type"] == "mamba2":
+                    shapes.append((int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["conv"]), int(m["heads"]) * int(m["vdim"]) + 2 * int(m["groups"]) * int(m["state"])))
+                elif s["type"] == "parallel":
+                    r = m["right"]
+                    shapes.append((int(r["heads"]), int(r["vdim"]), int(r["dim"]), 1, 0))
+            return CachePlan(False, True, False, len(kv), block_size, dt, max((d for _, d, _ in kv), default=0), gdn=bool(shapes), gdn_layers=len(shapes),
+                             state_slots=state_slots, kv_shapes=kv, delta_shapes=shapes)
         rows = [mc.layer_config(i).mla_cache_dim for i in own]
         cfgs = [mc.layer_config(i) for i in range(n) if mc.layer_type(i) == "linear_attention"]
         shapes = [(c.linear_num_value_heads, c.linear_value_head_dim, c.linear_key_head_dim, c.linear_conv_kernel_dim, c.gdn_conv_dim) for c in cfgs]
@@ -204,7 +228,9 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
 def kv_budget_blocks(plan: CachePlan, total: int, utilization: float, used: int, peak: int, current: int, reserved: int = 0) -> int:
     """blocks = (total*util - used - peak + current - reserved) // bytes_per_block."""
     budget = int(total * utilization) - used - peak + current - reserved
-    return max(0, budget // max(1, plan.block_bytes))
+    if plan.block_bytes == 0:              # no layer keeps rows: pages only count tokens
+        return 1 << 16
+    return max(0, budget // plan.block_bytes)
 
 
 class KVCache:
@@ -217,6 +243,9 @@ class KVCache:
             self.kv = None
             sdt = torch.uint8 if plan.kv_dtype == torch.float8_e4m3fn else plan.kv_dtype
             self.layers: List = [torch.zeros(nb, plan.block_size, d, dtype=sdt, device=device).view(plan.kv_dtype) for d in plan.latent_rows]
+        elif plan.kv_shapes is not None:
+            self.kv = None
+            self.layers = [tuple(torch.zeros(nb, plan.block_size, g, w, dtype=plan.kv_dtype, device=device) for w in (d, dv)) for g, d, dv in plan.kv_shapes]
         elif plan.mla:
             # under the hot / cold tier the logical pages are the cold tier: pinned host memory the staging kernel reads
             # through the unified address space
@@ -272,6 +301,10 @@ class KVCache:
             self.rec_states = [self.rec[l] for l in range(plan.gdn_layers)]
             self.conv_states = [self.conv[l] for l in range(plan.gdn_layers)]
 
+    def row_tensors(self) -> List[torch.Tensor]:
+        """Listed layers: every page tensor, page id in front."""
+        return [t for l in self.layers for t in (l if isinstance(l, tuple) else (l,))]
+
     # ---- byte layout of the per-page cache families (what a PD transfer or any other page mover needs to know) ----
     def page_families(self) -> List[dict]:
         """One entry per cache family that is indexed by page id: `tensor` (the whole family), `planes` (how many
@@ -285,6 +318,8 @@ class KVCache:
             return {"name": name, "tensor": t, "planes": planes, "plane_stride": per_plane, "page_bytes": per_plane // pages}
         if self.plan.latent_rows is not None:
             return [fam(f"latent_{l}", t, 1) for l, t in enumerate(self.layers)]
+        if self.plan.kv_shapes is not None:
+            return [fam(f"{name}_{l}", t, 1) for l, pair in enumerate(self.layers) for name, t in zip(("key", "value"), pair)]
         out = [fam("mla_kv" if self.plan.mla else "gqa_kv", self.kv, self.kv.shape[0] if self.plan.mla else 2 * self.kv.shape[1])]
         if self.indexer is not None:
             out.append(fam("indexer", self.indexer, self.indexer.shape[0]))
@@ -335,8 +370,8 @@ class KVCache:
 
     def block_views(self, bid: int) -> List[torch.Tensor]:
         """Byte views of everything block `bid` holds (all layers of every cache family), for the file-backed tier."""
-        if self.plan.latent_rows is not None:
-            return [(t.view(torch.uint8) if t.dtype == torch.float8_e4m3fn else t)[bid] for t in self.layers]
+        if self.plan.listed:
+            return [(t.view(torch.uint8) if t.dtype == torch.float8_e4m3fn else t)[bid] for t in self.row_tensors()]
         kv = self.kv.view(torch.uint8) if self.kv.dtype == torch.float8_e4m3fn else self.kv
         out = [kv[:, bid] if self.plan.mla else kv[:, :, bid]]
         if self.indexer is not None:

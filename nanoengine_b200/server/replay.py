@@ -51,8 +51,9 @@ def main(argv=None) -> int:
     torch.backends.cuda.matmul.allow_tf32 = torch.backends.cudnn.allow_tf32 = False
     from .. import LLM, Config
     pages = max(1, -(-a.max_tokens // PAGE))
+    longest = min(pages * PAGE, mc.max_position_embeddings) if mc.learned_positions else pages * PAGE
     llm = LLM(Config(model=a.model, model_config=mc, dtype=a.dtype, device=a.device, max_num_seqs=a.max_requests, kvcache_block_size=PAGE,
-                     num_kvcache_blocks=pages, max_model_len=pages * PAGE, max_num_batched_tokens=pages * PAGE, enable_prefix_caching=False,
+                     num_kvcache_blocks=pages, max_model_len=longest, max_num_batched_tokens=pages * PAGE, enable_prefix_caching=False,
                      executor_backend="inproc", enforce_eager=a.eager, status_log_interval_s=0))
     number = {}                     # request name -> sequence id of the engine
     next_id = 1
