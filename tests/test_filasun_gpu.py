@@ -9,7 +9,8 @@ from tuvutar_models import error, feed_all, make_llm, tokens
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda"
-TOL = {"float32": 5e-5, "bfloat16": 0.1}
+TOL = {"float32": 5e-5, "bfloat16": 0.08}
+ROUGH = {"mamba_only": 0.2}        # how far bf16 rounding alone takes a model, where that is more than the rest
 
 
 def _k():
@@ -221,7 +222,7 @@ def test_engine_agrees_with_the_oracle(name, dtype, tmp_path):
     want = oracle.forward(cfg, W, toks)
     llm = make_llm(path, dtype, DEV, pages=4)
     for cuts in ([200], [130, 1], [2], [64, 1, 63, 2, 20], [3, 7, 5, 49, 64]):
-        assert error(feed_all(llm, None, toks, cuts), want) < TOL[dtype], cuts
+        assert error(feed_all(llm, None, toks, cuts), want) < (ROUGH.get(name, TOL[dtype]) if dtype == "bfloat16" else TOL[dtype]), cuts
     assert llm.engine.scheduler.num_free_blocks(0) == 4
     assert _k().kernel_status()[0] == 0
 
