@@ -289,6 +289,61 @@ def case_rows(kind, T, W=4096, H=32, nope=128, rope=64, R=512):
     return (separate if kind == "mla_kv_prepare_rope" else lambda: sm100.latent_prepare(q, nope, kv, nw, 1e-6, pos, table, cache, pos, R, full)), nbytes, 0.0
 
 
+def case_mamba2(B, q_len=1, H=128, G=8, Dv=64, N=128, K=4, parts=8):
+    """Mamba-2 core between its projections (convolution, recurrence, gated norm).  The floor is one read and one write of every sequence's fp32
+    state and one pass over the projections and the result."""
+    T, inner = B * q_len, H * Dv
+    C = inner + 2 * G * N
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    proj, dt = torch.randn(T, inner + C, **bf), torch.randn(T, H, device="cuda")
+    cw, cb, nw = (torch.randn(C, K, device="cuda") * 0.3).to(torch.bfloat16), torch.zeros(C, **bf), torch.ones(inner, **bf)
+    A, db, D = torch.randn(H, device="cuda") * 0.5, torch.randn(H, device="cuda") - 2, torch.ones(H, device="cuda")
+    win, state = torch.zeros(B + 1, K - 1, C, **bf), torch.randn(B + 1, H, Dv, N, device="cuda") * 0.1
+    slots, cu = torch.arange(B, device="cuda", dtype=torch.int32), (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    fresh = torch.zeros(B, dtype=torch.int32, device="cuda")
+    fn = lambda: sm100.mamba2_mix(proj, dt, cw, cb, A, db, D, nw, parts, win, state, slots, cu, fresh, H, G, Dv, N, 1e-6, q_len)
+    return fn, B * H * Dv * N * 4 * 2 + T * (inner + C + inner) * 2, T * H * Dv * N * 4.0
+
+
+def case_lightning(B, q_len=1, H=32, Dk=128, Dv=128):
+    T = B * q_len
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    p = torch.randn(T, 2 * H * (Dk + Dv), **bf)
+    q, k, v, g = p.split([H * Dk, H * Dk, H * Dv, H * Dv], -1)
+    decay = 1 - torch.exp2(-torch.linspace(1, 9, H, device="cuda"))
+    nw, state = torch.ones(H * Dv, **bf), torch.randn(B + 1, H, Dv, Dk, device="cuda") * 0.1
+    slots, cu = torch.arange(B, device="cuda", dtype=torch.int32), (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    fresh = torch.zeros(B, dtype=torch.int32, device="cuda")
+    fn = lambda: sm100.lightning_mix(q, k, v, g, decay, nw, state, slots, cu, fresh, H, Dk, Dv, 1e-6, 0.5, None, q_len)
+    return fn, B * H * Dv * Dk * 4 * 2 + T * H * (2 * Dk + 3 * Dv) * 2, T * H * Dv * Dk * 4.0
+
+
+def case_biased(B, ctx, q_len, Hq, Hkv, window, cap=50.0, D=128, bs=64):
+    """Windowed attention with capped scores, distance bias and output gate; window 0, cap 0: none of it (the same kernel).  Bytes and FLOPs of the
+    keys inside the windows."""
+    nb = (ctx + bs - 1) // bs
+    k, v = (torch.randn(B * nb + 1, bs, Hkv, D, device="cuda", dtype=torch.bfloat16) for _ in range(2))
+    bt = torch.randperm(B * nb, device="cuda").view(B, nb).to(torch.int32)
+    T = B * q_len
+    q, gate = torch.randn(T, Hq, D, device="cuda", dtype=torch.bfloat16), torch.randn(T, Hq, device="cuda", dtype=torch.bfloat16)
+    cu = (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    cl = torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    slopes = torch.exp2(-8.0 * (torch.arange(Hq, device="cuda") + 1) / Hq) if window else None
+    out = torch.empty(T, Hq * D, device="cuda", dtype=torch.bfloat16)
+    fn = lambda: sm100_attn.gqa_attention_biased(q, k, v, bt, cu, cl, D ** -0.5, window, cap, slopes, gate if window else None, 1.0, out, q_len)
+    w = window or ctx
+    pairs = B * sum(min(w, ctx - q_len + i + 1) for i in range(q_len))
+    seen = min(ctx, w + q_len - 1)
+    return fn, B * seen * Hkv * D * 2 * 2 + T * Hq * D * 4, 4.0 * pairs * Hq * D
+
+
+def case_streams(T, S=2, W=4096):
+    y = torch.randn(T, W, device="cuda", dtype=torch.bfloat16)
+    x = torch.randn(T, S, W, device="cuda")
+    wo, wi, mix, wn = torch.ones(S, device="cuda"), torch.ones(S, device="cuda") / S, torch.eye(S, device="cuda"), torch.ones(W, device="cuda", dtype=torch.bfloat16)
+    return lambda: sm100.stream_mix(y, x, wo, mix, wi, wn, 1e-6), T * W * (S * 8 + 4), T * W * 2.0 * (S * S + 2 * S)
+
+
 def case_gdn(B, q_len=1, Hk=16, Hv=32, Dk=128, Dv=128, K=4):
     """Gated delta-net layer core at the Qwen3.5-MoE shape: conv over [q|k|v] with window shift, then the recurrent step with the gated
     norm.  The floor is one read and one write of every sequence's fp32 state."""
@@ -403,6 +458,25 @@ def build_cases(args):
         "gdn_verify2": lambda: case_gdn(128, q_len=2),
         "gdn_prefill_4x2048": lambda: case_gdn(4, q_len=2048),
         "gdn_prefill_1x8192": lambda: case_gdn(1, q_len=8192),
+        "mamba2_decode": lambda: case_mamba2(128),
+        "mamba2_decode_16": lambda: case_mamba2(16),
+        "mamba2_prefill_4x2048": lambda: case_mamba2(4, q_len=2048),
+        "mamba2_prefill_1x8192": lambda: case_mamba2(1, q_len=8192),
+        "lightning_decode": lambda: case_lightning(128),
+        "lightning_decode_16": lambda: case_lightning(16),
+        "lightning_prefill_4x2048": lambda: case_lightning(4, q_len=2048),
+        "lightning_prefill_1x8192": lambda: case_lightning(1, q_len=8192),
+        "biased_decode": lambda: case_biased(128, 8192, 1, 32, 8, 4096),
+        "biased_decode_nowindow": lambda: case_biased(128, 4096, 1, 32, 8, 0, 0.0),
+        "gqa_decode_same": lambda: case_gqa(128, 4096, 1, 32, 8),
+        "biased_decode_16": lambda: case_biased(16, 8192, 1, 32, 8, 4096),
+        "gqa_decode_same_16": lambda: case_gqa(16, 4096, 1, 32, 8),
+        "biased_prefill": lambda: case_biased(1, 8192, 8192, 32, 8, 4096),
+        "biased_prefill_nocap": lambda: case_biased(1, 8192, 8192, 32, 8, 4096, 0.0),
+        "biased_prefill_plain": lambda: case_biased(1, 8192, 8192, 32, 8, 0, 0.0),
+        "gqa_prefill_same": lambda: case_gqa(1, 8192, 8192, 32, 8),
+        "streams_decode": lambda: case_streams(128),
+        "streams_prefill": lambda: case_streams(8192),
         "delta_decode": lambda: case_delta(128),
         "delta_decode_16": lambda: case_delta(16),
         "delta_prefill_4x2048": lambda: case_delta(4, q_len=2048),

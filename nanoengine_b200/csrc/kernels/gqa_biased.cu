@@ -11,7 +11,8 @@
 //                   O += P V    (4 x tcgen05.mma, N = 64 nv; V read MN-major)
 // A head size that is not a multiple of 64 ends in a chunk whose missing columns TMA fills with zeros.  M = 128 rows are always multiplied;
 // rows past the tile's own read whatever shared memory follows and feed accumulator rows nobody reads.
-// Warp 0: TMA producer, warp 1: MMA issuer, warps 2-5: softmax / rescale / epilogue.  All waits are bounded.
+// Warp 0: TMA producer, warp 1: MMA issuer, warps 2-5: softmax / rescale / epilogue (those that own rows of the tile).  All waits are
+// bounded.  Two CTAs share an SM where the tiles are small enough: one's softmax runs beside the other's products and copies.
 // With more than one slice the CTA writes a normalised partial result and its log2-sum-exp; gqa_biased_merge folds them and applies the gate.
 #include "ptx.cuh"
 #include "seq_tile.cuh"
@@ -43,11 +44,12 @@ __device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ld
 }
 
 template <bool kCap>
-__global__ void __launch_bounds__(kGbThreads, 1)
+__global__ void __launch_bounds__(kGbThreads, 2)
 gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const GbArgs a) {
   pdl_wait();                     // dependent launch: nothing above this line touches global memory
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  uint8_t* smem = smem_raw;      // swizzled tiles need 1024-byte alignment: the dynamic allocation starts on such a boundary
+  if (smem_u32(smem) & 1023) { if (threadIdx.x == 0) report(ST_BAD_ARG, kKernelGb, 1, 0); return; }
   const int q_chunk = a.rows8 * 128, p_bytes = a.rows8 * 128, stage_bytes = (a.nc + a.nv) * kBChunk;
   uint8_t* sQ = smem;                                    // nc chunks of rows8 x 128 B
   uint8_t* sP = sQ + a.nc * q_chunk;
@@ -62,6 +64,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 
   const int warp = threadIdx.x >> 5;
   const int hkv = blockIdx.y, split = blockIdx.z;
+  const int live_warps = (a.g * a.tq + 31) / 32;         // softmax warps with rows of the tile
   if (warp == 0) {
     int seq, tok;
     find_seq_tile(a.cu_seqlens_q, a.num_seqs, a.tq, blockIdx.x, seq, tok);
@@ -71,7 +74,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     mbar_init(b_qfull, 1);
     for (int i = 0; i < 4; i++) { mbar_init(b_kvfull + 8 * i, 1); mbar_init(b_kvempty + 8 * i, 1); }
     for (int i = 0; i < 2; i++) {
-      mbar_init(b_sfull + 8 * i, 1); mbar_init(b_sempty + 8 * i, 4); mbar_init(b_pfull + 8 * i, 4); mbar_init(b_pempty + 8 * i, 1);
+      mbar_init(b_sfull + 8 * i, 1); mbar_init(b_sempty + 8 * i, live_warps); mbar_init(b_pfull + 8 * i, live_warps); mbar_init(b_pempty + 8 * i, 1);
     }
     *abort_flag = 0;
     mbar_fence_init();
@@ -158,7 +161,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       }
       if (ok) pv(n_tiles - 1);
     }
-  } else {
+  } else if ((warp & 3) < live_warps) {
     const int wq = warp & 3;
     const int row = wq * 32 + (int)lane_id();
     const uint32_t lane_addr = (uint32_t)(wq * 32) << 16;
@@ -185,15 +188,24 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       const bool p_free = i < a.pbufs || mbar_test(b_pempty + 8 * pb, ((i - a.pbufs) / a.pbufs) & 1);     // needed only after the math
       // score in the log2 domain: cap and bias
       const float b0 = slope * (float)(key0 - limit);
-      auto score = [&](uint32_t r, int j) -> uint32_t {
-        float s = __uint_as_float(r) * c_in;
-        const float bias = fmaf(slope, (float)j, b0);
-        if (kCap) s = fmaf(c_cap, 1.f - __fdividef(2.f, 1.f + exp2f(fminf(s, 64.f))), bias);      // cap (1 - 2 / (e^(2x) + 1)) = cap tanh(x)
-        else s += bias;
-        return __float_as_uint(s);
+      auto score4 = [&](uint32_t* r, int j0) {
+        float s[4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) s[e] = __uint_as_float(r[e]) * c_in;
+        if (kCap) {
+          // cap tanh(x) = cap - 2 cap / (e^(2x) + 1); one reciprocal for four: 1/a = bcd / abcd.  e^(2x) up to 2^30, where tanh has long been one.
+#pragma unroll
+          for (int e = 0; e < 4; e++) s[e] = 1.f + exp2f(fminf(s[e], 30.f));
+          const float ab = s[0] * s[1], cd = s[2] * s[3], rr = -2.f * c_cap * __fdividef(1.f, ab * cd);
+          const float rab = rr * cd, rcd = rr * ab;
+          const float t0 = fmaf(rab, s[1], c_cap), t1 = fmaf(rab, s[0], c_cap), t2 = fmaf(rcd, s[3], c_cap), t3 = fmaf(rcd, s[2], c_cap);
+          s[0] = t0; s[1] = t1; s[2] = t2; s[3] = t3;
+        }
+#pragma unroll
+        for (int e = 0; e < 4; e++) r[e] = __float_as_uint(s[e] + fmaf(slope, (float)(j0 + e), b0));
       };
 #pragma unroll
-      for (int j = 0; j < 32; j++) { r0[j] = score(r0[j], j); r1[j] = score(r1[j], 32 + j); }
+      for (int j = 0; j < 32; j += 4) { score4(r0 + j, j); score4(r1 + j, 32 + j); }
       if (key0 + kBPage - 1 > limit || key0 < lowest) {
 #pragma unroll
         for (int j = 0; j < 32; j++) {
@@ -325,13 +337,16 @@ static bool gb_plan(int g, int D, int Dv, int max_q, GbPlan* p) {
   p->nc = (D + 63) / 64; p->nv = (Dv + 63) / 64;
   p->tq = 128 / g < max_q ? 128 / g : max_q;
   p->rows8 = (g * p->tq + 7) / 8 * 8;
-  const int limit = 232448 - 1024 - 256, kv = (p->nc + p->nv) * kBChunk, q = p->nc * p->rows8 * 128;
-  p->pbufs = q + 2 * p->rows8 * 128 + 2 * kv <= limit ? 2 : 1;
-  p->stages = (limit - q - p->pbufs * p->rows8 * 128) / kv;
+  const int kv = (p->nc + p->nv) * kBChunk, pb = p->rows8 * 128, q = p->nc * pb;
+  // two CTAs per SM where half of its shared memory (and of its TMEM columns) holds a tile and two stages, else one with more stages
+  const int half = (233472 / 2 - 1024) - 256, whole = 232448 - 256;
+  const int limit = p->nv <= 2 && q + pb + 2 * kv <= half ? half : whole;
+  p->pbufs = q + 2 * pb + 2 * kv <= limit ? 2 : 1;
+  p->stages = (limit - q - p->pbufs * pb) / kv;
   if (p->stages > 4) p->stages = 4;
   if (p->stages < 2) return false;
-  const int used = q + p->pbufs * p->rows8 * 128 + p->stages * kv;
-  p->smem = used + 1024 + 256;
+  const int used = q + p->pbufs * pb + p->stages * kv;
+  p->smem = used + 256;
   // an MMA reads 128 rows from each chunk of Q and from each P buffer: those reads must end inside the allocation
   const int last_q = (p->nc - 1) * p->rows8 * 128 + 16384, last_p = q + (p->pbufs - 1) * p->rows8 * 128 + 16384;
   return (last_q > last_p ? last_q : last_p) <= used;

@@ -5,7 +5,8 @@
 //   1. ssm_prepare (Mamba-2): convolution + bias + silu over [x | B | C] with the carried window, dt = softplus(raw + bias) and the
 //      log-decay -exp(A_log) dt; moves the window on.  A thread walks a run of tokens of one channel.
 //   2. decay_scan: the recurrence token by token, any sizes, any mix of prompt portions and single tokens.  Rows of S are independent: a CTA
-//      owns some rows of one (sequence, head) in registers, 8 lanes share a row (each CPL of its columns).
+//      owns some rows of one (sequence, head) in registers, 8 lanes share a row (each CPL of its columns).  Long portions of bf16 models take
+//      the chunked tensor-core form instead (linattn_tc.cu).
 //   3. gated_norm: rows of heads, RMS-normed in equal parts, with the gate before (silu) or behind (sigmoid) the norm.
 // Whatever the portions are, the scan does the same arithmetic in the same order.
 #include "ptx.cuh"
@@ -31,6 +32,8 @@ __device__ __forceinline__ void sta4(__nv_bfloat16* p, const float* v) { *reinte
 template <int V, typename T> __device__ __forceinline__ void ldv(const T* p, float* o) { if constexpr (V == 4) lda4(p, o); else o[0] = lda(p); }
 template <int V, typename T> __device__ __forceinline__ void stv(T* p, const float* v) { if constexpr (V == 4) sta4(p, v); else sta(p, v[0]); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float round_as(float x, const float*) { return x; }
+__device__ __forceinline__ float round_as(float x, const __nv_bfloat16*) { return __bfloat162float(__float2bfloat16(x)); }
 
 // ---- Mamba-2: convolution, step sizes, log-decays ---------------------------------------------------------------------------
 constexpr int kRun = 16;              // tokens a thread walks
@@ -147,7 +150,8 @@ struct ScanArgs {
   const float* decay; const float* skip;      // [H]; skip null: no d v term
   float* state; const int* slots; const int* cu; const int* fresh;
   float* raw;                                 // [T, H, Dv] fp32
-  int T, B, H, Hk, Dk, Dv, act;               // act 1: silu on q, k and v
+  int T, B, H, Hk, Dk, Dv, act;               // act 1: silu on q, k and v, rounded to their type
+  int below;                                  // > 0: only sequences of fewer tokens (the others take the chunked form)
 };
 
 constexpr int kScanTok = 16;                  // tokens staged at a time
@@ -171,7 +175,7 @@ __global__ void __launch_bounds__(256, CPL * R >= 64 ? 2 : CPL * R >= 32 ? 3 : 4
   // wait, and that kernel writes none of these), so they are fetched while it still runs.
   const int start = a.cu[seq], n = a.cu[seq + 1] - start;
   const int slot = a.slots[seq];
-  if (n <= 0 || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 48, __LINE__)) { pdl_wait(); return; }
+  if (n <= 0 || (a.below > 0 && n >= a.below) || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 48, __LINE__)) { pdl_wait(); return; }
   const bool is_fresh = a.fresh[seq] != 0, vec = (Dk & 3) == 0;
   float* Sg = a.state + (((long long)slot * a.H + h) * Dv) * Dk;
   float S[R][CPL];                            // rows row0 + warp * 4R + r * 4 + rg, columns j * 32 + cg * 4 + {0..3}
@@ -206,7 +210,7 @@ __global__ void __launch_bounds__(256, CPL * R >= 64 ? 2 : CPL * R >= 32 ? 3 : 4
       float f[V];
       ldv<V>(which ? qg + (t0 + tok) * a.q_ld + c : kg + (t0 + tok) * a.k_ld + c, f);
 #pragma unroll
-      for (int e = 0; e < V; e++) (which ? sq : sk)[tok * DKP + c + e] = a.act ? silu_f(f[e]) : f[e];
+      for (int e = 0; e < V; e++) (which ? sq : sk)[tok * DKP + c + e] = a.act ? round_as(silu_f(f[e]), qg) : f[e];
     }
     for (int i = threadIdx.x; i < m * vper; i += blockDim.x) {
       const int r = (i % vper) * V, tok = i / vper;
@@ -214,7 +218,7 @@ __global__ void __launch_bounds__(256, CPL * R >= 64 ? 2 : CPL * R >= 32 ? 3 : 4
       float f[V];
       ldv<V>(vg + (t0 + tok) * a.v_ld + r, f);
 #pragma unroll
-      for (int e = 0; e < V; e++) sv[tok * rows + r + e] = a.act ? silu_f(f[e]) : f[e];
+      for (int e = 0; e < V; e++) sv[tok * rows + r + e] = a.act ? round_as(silu_f(f[e]), qg) : f[e];
     }
     for (int i = threadIdx.x; i < m; i += blockDim.x) {
       if (a.gates) {
@@ -403,15 +407,17 @@ extern "C" int ne_ssm_prepare(const void* xbc, long long ld, const float* dt_raw
 }
 
 // The recurrence token by token.  q, k [T, Hk, Dk], v [T, H, Dv] in the activation dtype (row strides in elements, heads packed), gates
-// [T, H, 2] or null (then decay [H]), skip [H] or null, state [S, H, Dv, Dk] fp32, raw [T, H, Dv] fp32.
+// [T, H, 2] or null (then decay [H]), skip [H] or null, state [S, H, Dv, Dk] fp32, raw [T, H, Dv] fp32.  below > 0: only the sequences with fewer
+// new tokens than that.
 extern "C" int ne_decay_scan(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld, const float* gates, const float* decay,
                              const float* skip, float* state, const int* slots, const int* cu, const int* fresh, float* raw, int T, int B, int H, int Hk, int Dk,
-                             int Dv, int act, int max_q, int fp32, cudaStream_t st) {
+                             int Dv, int act, int max_q, int below, int fp32, cudaStream_t st) {
   if (T <= 0 || B <= 0) return 0;
   if (Hk < 1 || H % Hk || Dk < 1 || Dk > 512 || Dv < 1 || B > 65535 || (!gates && !decay)) return 1001;
   ScanArgs a;
   a.q = q; a.k = k; a.v = v; a.q_ld = q_ld; a.k_ld = k_ld; a.v_ld = v_ld; a.gates = reinterpret_cast<const float2*>(gates); a.decay = decay; a.skip = skip;
-  a.state = state; a.slots = slots; a.cu = cu; a.fresh = fresh; a.raw = raw; a.T = T; a.B = B; a.H = H; a.Hk = Hk; a.Dk = Dk; a.Dv = Dv; a.act = act;
+  a.state = state; a.slots = slots; a.cu = cu; a.fresh = fresh; a.raw = raw; a.T = T; a.B = B; a.H = H; a.Hk = Hk; a.Dk = Dk; a.Dv = Dv; a.act = act; a.below = below;
+  if (below > 0 && max_q >= below) max_q = below - 1;
   return fp32 ? scan_t<float>(a, max_q, st) : scan_t<__nv_bfloat16>(a, max_q, st);
 }
 

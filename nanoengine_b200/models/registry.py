@@ -61,7 +61,7 @@ def _filasun():
 
 # kernel sources (stems under csrc/) of the architectures that can be served from a partial build; None = all of them
 _KERNELS = {"Tuvutar": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_bf16", "mla_bf16", "delta"),
-            "Filasun": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "linattn")}
+            "Filasun": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "linattn", "linattn_tc")}
 
 
 def kernel_sources(architecture: str):

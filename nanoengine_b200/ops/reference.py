@@ -1320,11 +1320,11 @@ def mamba2_mix(proj: torch.Tensor, dt_raw: torch.Tensor, conv_w: torch.Tensor, c
 def lightning_mix(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor,
                   slots: torch.Tensor, cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, Dk: int, Dv: int, eps: float, out_scale: float = 1.0,
                   out: Optional[torch.Tensor] = None, max_q_len: int = 1) -> torch.Tensor:
-    """Linear attention with one constant decay per head: q, k [T, H Dk] and v [T, H Dv] projections (rows may be strided) pass silu, per head
+    """Linear attention with one constant decay per head: q, k [T, H Dk] and v [T, H Dv] projections (rows may be strided) pass silu (rounded to their dtype), per head
     S <- decay S + v k^T on `state` [S, H, Dv, Dk] fp32, o = S q; the concatenated heads are RMS-normed together, times norm_w, sigmoid(gate)
     and out_scale.  Writes into `out` [T, H Dv] (rows may be strided) when given.  `max_q_len`: planning hint of the CUDA body."""
     T = q.shape[0]
-    qf, kf, vf = F.silu(q.float()).reshape(T, H, Dk), F.silu(k.float()).reshape(T, H, Dk), F.silu(v.float()).reshape(T, H, Dv)
+    qf, kf, vf = (F.silu(t.float()).to(t.dtype).float().reshape(T, H, w) for t, w in ((q, Dk), (k, Dk), (v, Dv)))
     ones = torch.ones(T, H, dtype=torch.float32, device=q.device)
     o = _decay_ragged(qf, kf, vf, decay.log().expand(T, H), ones, state, slots, cu_seqlens, fresh).reshape(T, H * Dv)
     o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float() * torch.sigmoid(gate.float()) * out_scale

@@ -1037,14 +1037,28 @@ def gated_delta(proj: torch.Tensor, ab: torch.Tensor, conv_w: torch.Tensor, A_lo
     return out
 
 
+CHUNKED_FROM = 64            # tokens of the longest portion from which bf16 calls use the chunked form (for portions of at least half as many)
+CHUNKED_CALLS = [0]          # launches of the chunked form
+
+
 def _decay_scan(q, k, v, gates, decay, skip, state, slots, cu, fresh, raw, H, Hk, Dk, Dv, act, max_q_len):
     T = q.shape[0]
     for t in (q, k, v):
         assert t.stride(1) == 1 and t.dtype == q.dtype
     assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, Dv, Dk)
+    B, below = cu.numel() - 1, 0
+    if (q.dtype == torch.bfloat16 and max_q_len >= CHUNKED_FROM and lib().ne_decay_chunk_covers(_c.c_int(Dk), _c.c_int(Dv))
+            and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v))):
+        below = CHUNKED_FROM // 2
+        _ck(lib().ne_decay_chunk(_p(q), _c.c_longlong(q.stride(0)), _p(k), _c.c_longlong(k.stride(0)), _p(v), _c.c_longlong(v.stride(0)), _p(gates), _p(decay),
+                                 _p(skip), _p(state), _p(slots), _p(cu), _p(fresh), _p(raw), _c.c_int(B), _c.c_int(H), _c.c_int(Hk), _c.c_int(Dk), _c.c_int(Dv),
+                                 _c.c_int(act), _c.c_int(below), _st()), "ne_decay_chunk")
+        CHUNKED_CALLS[0] += 1
+        if B == 1:
+            return
     _ck(lib().ne_decay_scan(_p(q), _c.c_longlong(q.stride(0)), _p(k), _c.c_longlong(k.stride(0)), _p(v), _c.c_longlong(v.stride(0)), _p(gates), _p(decay), _p(skip),
-                            _p(state), _p(slots), _p(cu), _p(fresh), _p(raw), _c.c_int(T), _c.c_int(cu.numel() - 1), _c.c_int(H), _c.c_int(Hk), _c.c_int(Dk),
-                            _c.c_int(Dv), _c.c_int(act), _c.c_int(max_q_len), _c.c_int(int(q.dtype == torch.float32)), _st()), "ne_decay_scan")
+                            _p(state), _p(slots), _p(cu), _p(fresh), _p(raw), _c.c_int(T), _c.c_int(B), _c.c_int(H), _c.c_int(Hk), _c.c_int(Dk),
+                            _c.c_int(Dv), _c.c_int(act), _c.c_int(max_q_len), _c.c_int(below), _c.c_int(int(q.dtype == torch.float32)), _st()), "ne_decay_scan")
 
 
 def _gated_norm(raw, gate, w, out, parts, before, eps, scale):

@@ -152,10 +152,6 @@ def _mamba_case(H, G, Dv, N, K, parts, lens, fresh, dtype, seed=0):
                 fresh=torch.tensor(fresh, dtype=torch.int32, device=DEV), H=H, G=G, Dv=Dv, N=N, eps=1e-4, max_q_len=max(lens))
 
 
-def _as32(c):
-    return {n: (v.float().clone() if isinstance(v, torch.Tensor) and v.is_floating_point() else v) for n, v in c.items()}
-
-
 @pytest.mark.parametrize("H,G,Dv,N,K,parts", [(6, 3, 10, 14, 3, 4), (6, 1, 48, 48, 3, 1), (8, 2, 32, 64, 4, 2), (3, 1, 24, 144, 5, 3), (4, 4, 88, 16, 1, 1), (8, 8, 16, 128, 9, 8),
                                               (16, 2, 64, 128, 4, 16), (2, 1, 160, 40, 2, 1), (1, 1, 33, 300, 4, 1), (4, 1, 64, 256, 16, 2)])
 @pytest.mark.parametrize("lens,fresh", LENS)
@@ -187,14 +183,46 @@ def _lightning_case(H, Dk, Dv, lens, fresh, dtype, seed=0, decay=None):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_lightning_mix(H, Dk, Dv, decay, lens, fresh, dtype):
     c = _lightning_case(H, Dk, Dv, lens, fresh, dtype, decay=decay)
-    want = _as32(c)
+    want = {n: (v.clone() if isinstance(v, torch.Tensor) else v) for n, v in c.items()}
     T = sum(lens)
     y = torch.zeros(T, 8 + H * Dv, device=DEV, dtype=dtype)
     _k().lightning_mix(**c, out=y[:, 8:])
     ref_out = _ref().lightning_mix(**want)
-    tol = 3e-5 if dtype == torch.float32 else 8e-3
+    tol = 3e-5 if dtype == torch.float32 else 1.2e-2
     assert rel(c["state"], want["state"]) < tol and rel(y[:, 8:], ref_out) < tol and float(y[:, :8].abs().max()) == 0.0
     assert _k().kernel_status()[0] == 0
+
+
+@pytest.mark.parametrize("H,Hk,Dk,Dv", [(4, 4, 64, 64), (2, 1, 128, 128), (3, 3, 48, 40), (2, 2, 8, 200), (8, 2, 120, 64)])
+@pytest.mark.parametrize("lens,fresh", [([128], [1]), ([64], [0]), ([129, 40, 31, 1], [0, 1, 0, 0]), ([1000, 2, 255], [1, 1, 0])])
+def test_chunked_recurrence_on_tensor_cores(H, Hk, Dk, Dv, lens, fresh):
+    """The chunked form against the token-by-token statement in 64-bit: head and remainder of every fp32 operand keep it near 32-bit accuracy,
+    for decays from none to complete."""
+    k, r = _k(), _ref()
+    g = torch.Generator(device=DEV).manual_seed(H * Dk)
+    T, B = sum(lens), len(lens)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=DEV)
+    qkv = rnd(T, 2 * Hk * Dk + H * Dv).to(torch.bfloat16)
+    q, kk, v = qkv.split([Hk * Dk, Hk * Dk, H * Dv], -1)
+    log_a = -torch.exp(3 * rnd(T, H)) * 0.05
+    log_a[:, 0] = 0.0
+    if T > 70:
+        log_a[33:70:9] = -300.0
+    b = rnd(T, H).abs()
+    gates, skip = torch.stack([log_a, b], -1).contiguous(), rnd(H)
+    state = 0.3 * rnd(B + 1, H, Dv, Dk)
+    want_s, slots, cu, fr = state.double(), torch.randperm(B + 1, generator=g, device=DEV)[:B].int(), _cu(lens), torch.tensor(fresh, dtype=torch.int32, device=DEV)
+    rep = H // Hk
+    dbl = lambda t, h, d: t.double().reshape(T, h, d)
+    want = r._decay_ragged(dbl(q, Hk, Dk).repeat_interleave(rep, 1), dbl(kk, Hk, Dk).repeat_interleave(rep, 1), dbl(v, H, Dv), log_a.double(), b.double(), want_s, slots, cu, fr,
+                           skip.double())
+    raw = torch.full((T, H * Dv), 9.0, device=DEV)
+    before = k.CHUNKED_CALLS[0]
+    k._decay_scan(q, kk, v, gates, None, skip, state, slots, cu, fr, raw, H, Hk, Dk, Dv, 0, max(lens))
+    assert k.CHUNKED_CALLS[0] == before + 1 and k.kernel_status()[0] == 0
+    scale = lambda t: t.abs().max()
+    assert float((raw.view(T, H, Dv).double() - want).abs().max() / scale(want)) < 4e-5
+    assert float((state.double() - want_s).abs().max() / scale(want_s)) < 4e-5
 
 
 @pytest.mark.parametrize("which", ["mamba2", "lightning"])
