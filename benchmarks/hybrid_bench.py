@@ -1,9 +1,17 @@
-"""Prefill and decode throughput of a Tuvutar model beside the closest model of this package at equal sizes (`bench.py --model tuvutar`).
+"""Prefill and decode throughput of a model with listed layers beside the closest model of this package at equal sizes (`bench.py --model
+tuvutar`, `bench.py --model filasun`).
 
-The closest model is Kimi-K3's layer stack without experts and with a plain residual: latent attention between delta-rule layers and
+Tuvutar: the closest model is Kimi-K3's layer stack without experts and with a plain residual: latent attention between delta-rule layers and
 dense gated MLPs in bf16 (its delta layers decay per key channel, its latent layers carry an output gate).  Both get the same width,
 head counts and sizes, layer order, feed-forward in every layer, vocabulary, bf16 weights and caches, random weights, synthetic
-prompts, and run through the same engine: `prefill` is the device time of the scheduler's prompt steps (CUDA events around
+prompts, and run through the same engine.
+
+Filasun: the closest model is the dense Qwen3.5 stack (grouped-query attention and gated delta-net layers, bf16, one residual).  A parallel layer
+(attention, decayed linear attention, a feed-forward of width ff) stands against an attention layer and a delta-net layer with a feed-forward of
+ff / 2 each, a Mamba-2 layer with a feed-forward of ff / 2 against a delta-net layer: the same head counts, head sizes, state sizes per layer,
+feed-forward weights, width and vocabulary; the attention window is the longest context, so that both read the same keys.
+
+`prefill` is the device time of the scheduler's prompt steps (CUDA events around
 LLM.step), `decode` the replay of one decode step on resident inputs (graph + lm_head + sampling)."""
 from __future__ import annotations
 
@@ -31,6 +39,27 @@ def kimi_model(width, heads, groups, ff, vocab):
                         n_routed_experts=0, n_shared_experts=0, layer_types=["full_attention", "linear_attention", "linear_attention", "linear_attention"] * groups,
                         linear_num_key_heads=heads, linear_num_value_heads=heads, linear_key_head_dim=128, linear_value_head_dim=128, attn_res_block_size=0,
                         routed_expert_hidden_size=0, max_position_embeddings=16384)
+
+
+def filasun_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import ModelConfig, _mamba2_spec, _parallel_spec
+    layers = []
+    for _ in range(groups):
+        layers += [_parallel_spec(heads, heads // 4, 128, 128, 16384, heads, 128, 128, ff=ff) for _ in range(2)]
+        layers.append(_mamba2_spec(2 * heads, 64, 128, max(1, heads // 8), 4, max(1, heads // 8), ff=ff // 2))
+    return ModelConfig.from_dict({"architecture": "Filasun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 2, "logit_softcap": 30.0,
+                                  "max_positions": 16384, "layers": layers})
+
+
+def qwen_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import tiny_qwen3_5
+    kinds = (["full_attention", "linear_attention"] * 2 + ["linear_attention"]) * groups
+    return tiny_qwen3_5(vocab_size=vocab, hidden_size=width, num_hidden_layers=len(kinds), layer_types=kinds, num_attention_heads=heads, num_key_value_heads=heads // 4,
+                        head_dim=128, intermediate_size=ff // 2, linear_num_key_heads=heads, linear_num_value_heads=heads, linear_key_head_dim=128,
+                        linear_value_head_dim=128, max_position_embeddings=16384)
+
+
+DESIGNS = {"tuvutar": ("Tuvutar", tuvutar_model, "kimi_k3_stack", kimi_model), "filasun": ("Filasun", filasun_model, "qwen3_5_stack", qwen_model)}
 
 
 def measure(mc, seqs, prompt, steps, warmup, seed=0):
@@ -85,6 +114,7 @@ def main(args):
     import torch
     import bench
     torch.cuda.set_device(0)
+    title, own, closest_name, closest = DESIGNS[args.model]
     stop, samples = threading.Event(), []
     th = threading.Thread(target=bench._clock_sampler, args=(stop, samples), daemon=True)
     th.start()
@@ -92,14 +122,14 @@ def main(args):
     for name in args.sizes.split(","):
         s = sizes(name)
         for seqs, prompt in ((128, 2048), (16, 8192)):
-            rows.append({"size": name, **s, "seqs": seqs, "prompt": prompt, "tuvutar": measure(tuvutar_model(**s), seqs, prompt, args.steps, args.warmup),
-                         "kimi_k3_stack": measure(kimi_model(**s), seqs, prompt, args.steps, args.warmup) if not args.skip_closest else None})
+            rows.append({"size": name, **s, "seqs": seqs, "prompt": prompt, args.model: measure(own(**s), seqs, prompt, args.steps, args.warmup),
+                         closest_name: measure(closest(**s), seqs, prompt, args.steps, args.warmup) if not args.skip_closest else None})
     stop.set()
     th.join(timeout=2)
-    first = rows[0]["tuvutar"]
-    print(json.dumps({"metric": "Tuvutar decode out tok/s at the first size (prefill and the closest model in rows)", "value": first["decode_tok_s"],
+    first = rows[0][args.model]
+    print(json.dumps({"metric": title + " decode out tok/s at the first size (prefill and the closest model in rows)", "value": first["decode_tok_s"],
                       "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": first["decode_ms"], "higher_is_better": True,
                       "vs_baseline": None, "dtype": "bf16", "data": "synthetic uniform-random token ids, random-init weights",
-                      "config": {"model": "tuvutar", "l2": "weights and states streamed every step exceed L2; no flush"}, "rows": rows,
+                      "config": {"model": args.model, "l2": "weights and states streamed every step exceed L2; no flush"}, "rows": rows,
                       "clocks": bench._summarise_clocks(samples), "impl": "ours"}))
     return 0

@@ -11,6 +11,9 @@
 //                   O += P V    (4 x tcgen05.mma, N = 64 nv; V read MN-major)
 // A head size that is not a multiple of 64 ends in a chunk whose missing columns TMA fills with zeros.  M = 128 rows are always multiplied;
 // rows past the tile's own read whatever shared memory follows and feed accumulator rows nobody reads.
+// Tiles of at most 32 rows (decode steps) with capped scores, where the softmax is the longer part, are laid out four times (kRep), rows 32 w .. of the products for softmax warp w, and warp w takes only
+// keys 16 w .. 16 w + 15 of every page: a quarter of the softmax work each, at no cost in products.  The four partial results of a row
+// (own maximum, sum and accumulator) are folded at the end.
 // Warp 0: TMA producer, warp 1: MMA issuer, warps 2-5: softmax / rescale / epilogue (those that own rows of the tile).  All waits are
 // bounded.  Two CTAs share an SM where the tiles are small enough: one's softmax runs beside the other's products and copies.
 // With more than one slice the CTA writes a normalised partial result and its log2-sum-exp; gqa_biased_merge folds them and applies the gate.
@@ -30,7 +33,7 @@ struct GbArgs {
   const int* block_tables; int bt_stride;
   const int* cu_seqlens_q; const int* context_lens; int num_seqs;
   int T, H, Dv, g, tq, splits;
-  int nc, nv, rows8, stages, pbufs, window;
+  int nc, nv, rows8, stages, pbufs, window;      // kRep: rows8 = 128
   uint32_t tmem_cols;
   float scale, softcap;
   const float* slopes;                         // [H] or null
@@ -43,7 +46,7 @@ __device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ld
   return gate ? scale / (1.f + __expf(-__bfloat162float(gate[t * ld + h]))) : scale;
 }
 
-template <bool kCap>
+template <bool kCap, bool kRep>
 __global__ void __launch_bounds__(kGbThreads, 2)
 gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const GbArgs a) {
   pdl_wait();                     // dependent launch: nothing above this line touches global memory
@@ -64,7 +67,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 
   const int warp = threadIdx.x >> 5;
   const int hkv = blockIdx.y, split = blockIdx.z;
-  const int live_warps = (a.g * a.tq + 31) / 32;         // softmax warps with rows of the tile
+  const int live_warps = kRep ? 4 : (a.g * a.tq + 31) / 32;         // softmax warps with rows of the tile
   if (warp == 0) {
     int seq, tok;
     find_seq_tile(a.cu_seqlens_q, a.num_seqs, a.tq, blockIdx.x, seq, tok);
@@ -104,8 +107,10 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 
   if (warp == 0) {
     if (n_tiles > 0 && elect_one()) {
-      mbar_expect_tx(b_qfull, a.nc * a.g * a.tq * 128);
-      for (int c = 0; c < a.nc; c++) tma_load_3d(smem_u32(sQ + c * q_chunk), &q_map, b_qfull, c * 64, hkv * a.g, tok0);
+      constexpr int kCopies = kRep ? 4 : 1;
+      mbar_expect_tx(b_qfull, kCopies * a.nc * a.g * a.tq * 128);
+      for (int r = 0; r < kCopies; r++)
+        for (int c = 0; c < a.nc; c++) tma_load_3d(smem_u32(sQ + c * q_chunk + r * 32 * 128), &q_map, b_qfull, c * 64, hkv * a.g, tok0);
       for (int i = 0; i < n_tiles; i++) {
         const int s = i % a.stages;
         if (!mbar_wait(b_kvempty + 8 * s, ((i / a.stages) & 1) ^ 1, abort_flag, kKernelGb, 100 + s)) break;
@@ -165,33 +170,42 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int wq = warp & 3;
     const int row = wq * 32 + (int)lane_id();
     const uint32_t lane_addr = (uint32_t)(wq * 32) << 16;
-    const int tl = row / a.g, head = hkv * a.g + row % a.g;
-    const bool row_ok = row < a.g * a.tq && tl < n_tok;
+    const int trow = kRep ? (int)lane_id() : row;             // row of the tile
+    const int tl = trow / a.g, head = hkv * a.g + trow % a.g;
+    const bool row_ok = trow < a.g * a.tq && tl < n_tok;
+    constexpr int kKeys = kRep ? 16 : 64;                     // keys of a page this thread scores, from kfirst on
+    const int kfirst = kRep ? wq * 16 : 0;
     const int limit = row_ok ? base_limit + tl : -1;          // this row's last visible key
     const int lowest = (row_ok && a.window > 0) ? limit - a.window + 1 : 0;
     const float slope = (row_ok && a.slopes) ? __ldg(a.slopes + head) * kLog2e : 0.f;
     const float c_in = kCap ? a.scale / a.softcap * (2.f * kLog2e) : a.scale * kLog2e, c_cap = a.softcap * kLog2e;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true, s_ready = false;
+    if constexpr (kRep)                                       // the columns of the other warps' keys stay zero
+      for (int i = 0; i < a.pbufs * 8; i++) *reinterpret_cast<uint4*>(sP + (i >> 3) * p_bytes + row * 128 + (i & 7) * 16) = make_uint4(0, 0, 0, 0);
     for (int i = 0; ok && i < n_tiles; i++) {
       const int sb = i & 1, pb = i % a.pbufs;
       if (!s_ready && !mbar_wait(b_sfull + 8 * sb, (i >> 1) & 1, abort_flag, kKernelGb, 300 + sb)) { ok = false; break; }
       tc_fence_after();
-      uint32_t r0[32], r1[32];
-      tmem_ld_32x32b_x32(tmem_base + lane_addr + sb * kBPage, r0);
-      tmem_ld_32x32b_x32(tmem_base + lane_addr + sb * kBPage + 32, r1);
+      uint32_t r[kKeys];
+      if constexpr (kRep) {
+        tmem_ld_32x32b_x16(tmem_base + lane_addr + sb * kBPage + kfirst, r);
+      } else {
+        tmem_ld_32x32b_x32(tmem_base + lane_addr + sb * kBPage, *reinterpret_cast<uint32_t(*)[32]>(r));
+        tmem_ld_32x32b_x32(tmem_base + lane_addr + sb * kBPage + 32, *reinterpret_cast<uint32_t(*)[32]>(r + 32));
+      }
       tc_wait_ld();
       tc_fence_before();
       __syncwarp();
       if (lane_id() == 0) mbar_arrive(b_sempty + 8 * sb);
-      const int key0 = (pg_begin + i) * kBPage;
+      const int key0 = (pg_begin + i) * kBPage + kfirst;
       const bool p_free = i < a.pbufs || mbar_test(b_pempty + 8 * pb, ((i - a.pbufs) / a.pbufs) & 1);     // needed only after the math
       // score in the log2 domain: cap and bias
       const float b0 = slope * (float)(key0 - limit);
-      auto score4 = [&](uint32_t* r, int j0) {
+      auto score4 = [&](uint32_t* rr4, int j0) {
         float s[4];
 #pragma unroll
-        for (int e = 0; e < 4; e++) s[e] = __uint_as_float(r[e]) * c_in;
+        for (int e = 0; e < 4; e++) s[e] = __uint_as_float(rr4[e]) * c_in;
         if (kCap) {
           // cap tanh(x) = cap - 2 cap / (e^(2x) + 1); one reciprocal for four: 1/a = bcd / abcd.  e^(2x) up to 2^30, where tanh has long been one.
 #pragma unroll
@@ -202,23 +216,18 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           s[0] = t0; s[1] = t1; s[2] = t2; s[3] = t3;
         }
 #pragma unroll
-        for (int e = 0; e < 4; e++) r[e] = __float_as_uint(s[e] + fmaf(slope, (float)(j0 + e), b0));
+        for (int e = 0; e < 4; e++) rr4[e] = __float_as_uint(s[e] + fmaf(slope, (float)(j0 + e), b0));
       };
 #pragma unroll
-      for (int j = 0; j < 32; j += 4) { score4(r0 + j, j); score4(r1 + j, 32 + j); }
-      if (key0 + kBPage - 1 > limit || key0 < lowest) {
+      for (int j = 0; j < kKeys; j += 4) score4(r + j, j);
+      if (key0 + kKeys - 1 > limit || key0 < lowest) {
 #pragma unroll
-        for (int j = 0; j < 32; j++) {
-          if (key0 + j > limit || key0 + j < lowest) r0[j] = 0xff800000u;
-          if (key0 + 32 + j > limit || key0 + 32 + j < lowest) r1[j] = 0xff800000u;
-        }
+        for (int j = 0; j < kKeys; j++)
+          if (key0 + j > limit || key0 + j < lowest) r[j] = 0xff800000u;
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-      for (int j = 0; j < 32; j += 2) {
-        mx[0] = fmaxf(mx[0], __uint_as_float(r0[j])); mx[1] = fmaxf(mx[1], __uint_as_float(r0[j + 1]));
-        mx[2] = fmaxf(mx[2], __uint_as_float(r1[j])); mx[3] = fmaxf(mx[3], __uint_as_float(r1[j + 1]));
-      }
+      for (int j = 0; j < kKeys; j++) mx[j & 3] = fmaxf(mx[j & 3], __uint_as_float(r[j]));
       const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
       // lazy rescaling: the reference maximum only moves when the page's maximum exceeds it by more than 2^8
       const bool first_valid = (m_run == -INFINITY);
@@ -226,16 +235,13 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       const float alpha = (m_new == -INFINITY || first_valid) ? 1.f : exp2f(m_run - m_new);
       const float neg_m = (m_new == -INFINITY) ? 0.f : -m_new;
       float psum = 0.f;
-      uint32_t pk[32];
+      uint32_t pk[kKeys / 2];
 #pragma unroll
-      for (int j = 0; j < 16; j++) {
-        const float p0 = exp2f(__uint_as_float(r0[2 * j]) + neg_m), p1 = exp2f(__uint_as_float(r0[2 * j + 1]) + neg_m);
-        const float p2 = exp2f(__uint_as_float(r1[2 * j]) + neg_m), p3 = exp2f(__uint_as_float(r1[2 * j + 1]) + neg_m);
-        pk[j] = pack_bf16x2(p0, p1);
-        pk[16 + j] = pack_bf16x2(p2, p3);
+      for (int j = 0; j < kKeys / 2; j++) {
+        pk[j] = pack_bf16x2(exp2f(__uint_as_float(r[2 * j]) + neg_m), exp2f(__uint_as_float(r[2 * j + 1]) + neg_m));
         // sum what the MMA will see (bf16-rounded probabilities), so numerator and denominator stay consistent
-        const float2 q0 = unpack_bf16x2(pk[j]), q1 = unpack_bf16x2(pk[16 + j]);
-        psum += (q0.x + q0.y) + (q1.x + q1.y);
+        const float2 q = unpack_bf16x2(pk[j]);
+        psum += q.x + q.y;
       }
       l_run = l_run * alpha + psum;
       m_run = m_new;
@@ -259,8 +265,8 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         uint8_t* prow = sP + pb * p_bytes + row * 128;
         const int sw = row & 7;
 #pragma unroll
-        for (int cch = 0; cch < 8; cch++)
-          *reinterpret_cast<uint4*>(prow + ((cch ^ sw) << 4)) = make_uint4(pk[4 * cch], pk[4 * cch + 1], pk[4 * cch + 2], pk[4 * cch + 3]);
+        for (int cch = 0; cch < kKeys / 8; cch++)
+          *reinterpret_cast<uint4*>(prow + (((kfirst / 8 + cch) ^ sw) << 4)) = make_uint4(pk[4 * cch], pk[4 * cch + 1], pk[4 * cch + 2], pk[4 * cch + 3]);
       }
       fence_proxy_async_smem();
       tc_fence_before();
@@ -271,35 +277,90 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const long long tok = tok0 + tl, orow = row_ok ? tok * a.H + head : 0;
     const bool have = ok && n_tiles > 0;
     if (have) tc_fence_after();
-    float inv = (have && l_run > 0.f) ? 1.f / l_run : 0.f;
-    if (a.splits == 1 && row_ok) inv *= gate_of(a.gate, a.gate_ld, tok, head, a.out_scale);
+    if constexpr (kRep) {
+      // fold the four partial results of every row: accumulators through shared memory (nothing else uses it any more)
+      float* fold = reinterpret_cast<float*>(smem);
+      const int ld = a.Dv + 4, rows = a.g * a.tq;
 #pragma unroll 1
-    for (int cblk = 0; cblk < a.nv * 2; cblk++) {
-      uint32_t o[32];
-      if (have) {
-        tmem_ld_32x32b_x32(tmem_o + lane_addr + cblk * 32, o);
-        tc_wait_ld();
-      }
-      if (!row_ok) continue;
+      for (int cblk = 0; cblk < a.nv * 2; cblk++) {
+        uint32_t o[32];
+        __syncwarp();                          // the lanes of rows outside the tile skip the stores below
+        if (have) {
+          tmem_ld_32x32b_x32(tmem_o + lane_addr + cblk * 32, o);
+          tc_wait_ld();
+        }
+        if (!row_ok) continue;
 #pragma unroll
-      for (int v = 0; v < 4; v++) {                            // Dv is a multiple of 8: whole groups of 8 columns
-        const int col = cblk * 32 + v * 8;
-        if (col >= a.Dv) continue;
-        float f[8];
-#pragma unroll
-        for (int j = 0; j < 8; j++) f[j] = have ? __uint_as_float(o[v * 8 + j]) * inv : 0.f;
-        if (a.splits == 1) {
-          *reinterpret_cast<uint4*>(a.out + tok * a.o_ld + (long long)head * a.Dv + col) =
-              make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
-        } else {
-          float* dst = a.part + ((long long)split * a.T * a.H + orow) * a.Dv + col;
-          *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
-          *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
+        for (int v = 0; v < 8; v++) {
+          const int col = cblk * 32 + v * 4;
+          if (col >= a.Dv) continue;
+          *reinterpret_cast<float4*>(fold + (wq * rows + trow) * ld + 4 + col) =
+              have ? make_float4(__uint_as_float(o[4 * v]), __uint_as_float(o[4 * v + 1]), __uint_as_float(o[4 * v + 2]), __uint_as_float(o[4 * v + 3]))
+                   : make_float4(0.f, 0.f, 0.f, 0.f);
         }
       }
+      if (row_ok) { fold[(wq * rows + trow) * ld] = have ? m_run : -INFINITY; fold[(wq * rows + trow) * ld + 1] = have ? l_run : 0.f; }
+      named_bar_sync(1, 128);
+      const int groups = a.Dv / 8;
+      for (int i = (int)threadIdx.x - 64; i < n_tok * a.g * groups; i += 128) {
+        const int rr = i / groups, col = (i - rr * groups) * 8, hd = hkv * a.g + rr % a.g;
+        const long long tk = tok0 + rr / a.g;
+        float m = -INFINITY, den = 0.f, f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int w = 0; w < 4; w++) m = fmaxf(m, fold[(w * rows + rr) * ld]);
+#pragma unroll
+        for (int w = 0; w < 4; w++) {
+          const float* src = fold + (w * rows + rr) * ld;
+          if (src[0] == -INFINITY) continue;
+          const float e = exp2f(src[0] - m);
+          den += e * src[1];
+#pragma unroll
+          for (int j = 0; j < 8; j++) f[j] = fmaf(e, src[4 + col + j], f[j]);
+        }
+        const float inv = (den > 0.f ? 1.f / den : 0.f) * (a.splits == 1 ? gate_of(a.gate, a.gate_ld, tk, hd, a.out_scale) : 1.f);
+        if (a.splits == 1) {
+          *reinterpret_cast<uint4*>(a.out + tk * a.o_ld + (long long)hd * a.Dv + col) =
+              make_uint4(pack_bf16x2(f[0] * inv, f[1] * inv), pack_bf16x2(f[2] * inv, f[3] * inv), pack_bf16x2(f[4] * inv, f[5] * inv), pack_bf16x2(f[6] * inv, f[7] * inv));
+        } else {
+          const long long o = (long long)split * a.T * a.H + tk * a.H + hd;
+          float* dst = a.part + o * a.Dv + col;
+          *reinterpret_cast<float4*>(dst) = make_float4(f[0] * inv, f[1] * inv, f[2] * inv, f[3] * inv);
+          *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4] * inv, f[5] * inv, f[6] * inv, f[7] * inv);
+          if (col == 0) a.lse2[o] = den > 0.f ? m + log2f(den) : -INFINITY;
+        }
+      }
+    } else {
+      float inv = (have && l_run > 0.f) ? 1.f / l_run : 0.f;
+      if (a.splits == 1 && row_ok) inv *= gate_of(a.gate, a.gate_ld, tok, head, a.out_scale);
+#pragma unroll 1
+      for (int cblk = 0; cblk < a.nv * 2; cblk++) {
+        uint32_t o[32];
+        __syncwarp();                          // the lanes of rows outside the tile skip the stores below
+        if (have) {
+          tmem_ld_32x32b_x32(tmem_o + lane_addr + cblk * 32, o);
+          tc_wait_ld();
+        }
+        if (!row_ok) continue;
+#pragma unroll
+        for (int v = 0; v < 4; v++) {                            // Dv is a multiple of 8: whole groups of 8 columns
+          const int col = cblk * 32 + v * 8;
+          if (col >= a.Dv) continue;
+          float f[8];
+#pragma unroll
+          for (int j = 0; j < 8; j++) f[j] = have ? __uint_as_float(o[v * 8 + j]) * inv : 0.f;
+          if (a.splits == 1) {
+            *reinterpret_cast<uint4*>(a.out + tok * a.o_ld + (long long)head * a.Dv + col) =
+                make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+          } else {
+            float* dst = a.part + ((long long)split * a.T * a.H + orow) * a.Dv + col;
+            *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
+            *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
+          }
+        }
+      }
+      if (a.splits > 1 && row_ok)
+        a.lse2[(long long)split * a.T * a.H + orow] = (have && l_run > 0.f) ? m_run + log2f(l_run) : -INFINITY;
     }
-    if (a.splits > 1 && row_ok)
-      a.lse2[(long long)split * a.T * a.H + orow] = (have && l_run > 0.f) ? m_run + log2f(l_run) : -INFINITY;
   }
 
   tc_fence_before();
@@ -329,14 +390,15 @@ __global__ void __launch_bounds__(128) gqa_biased_merge_kernel(const GbArgs a) {
   }
 }
 
-struct GbPlan { int nc, nv, tq, rows8, stages, pbufs, smem; };
+struct GbPlan { int nc, nv, tq, rep, rows8, stages, pbufs, smem; };
 
 // Tile geometry for groups of g heads, head sizes D / Dv and sequences of at most max_q new tokens; false: not covered.
-static bool gb_plan(int g, int D, int Dv, int max_q, GbPlan* p) {
+static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, GbPlan* p) {
   if (g < 1 || g > 128 || D < 8 || D % 8 || D > 256 || Dv < 8 || Dv % 8 || Dv > 256 || max_q < 1) return false;
   p->nc = (D + 63) / 64; p->nv = (Dv + 63) / 64;
   p->tq = 128 / g < max_q ? 128 / g : max_q;
-  p->rows8 = (g * p->tq + 7) / 8 * 8;
+  p->rep = rep && g * p->tq <= 32;
+  p->rows8 = p->rep ? 128 : (g * p->tq + 7) / 8 * 8;
   const int kv = (p->nc + p->nv) * kBChunk, pb = p->rows8 * 128, q = p->nc * pb;
   // two CTAs per SM where half of its shared memory (and of its TMEM columns) holds a tile and two stages, else one with more stages
   const int half = (233472 / 2 - 1024) - 256, whole = 232448 - 256;
@@ -347,6 +409,7 @@ static bool gb_plan(int g, int D, int Dv, int max_q, GbPlan* p) {
   if (p->stages < 2) return false;
   const int used = q + p->pbufs * pb + p->stages * kv;
   p->smem = used + 256;
+  if (p->rep && 4 * g * p->tq * (Dv + 4) * 4 > used) return false;      // the fold's buffer
   // an MMA reads 128 rows from each chunk of Q and from each P buffer: those reads must end inside the allocation
   const int last_q = (p->nc - 1) * p->rows8 * 128 + 16384, last_p = q + (p->pbufs - 1) * p->rows8 * 128 + 16384;
   return (last_q > last_p ? last_q : last_p) <= used;
@@ -359,7 +422,7 @@ using namespace ne;
 // Tokens per tile (0: the shape is not covered)
 extern "C" int ne_gqa_biased_plan(int H, int Hkv, int D, int Dv, int max_q) {
   GbPlan p;
-  return Hkv >= 1 && H % Hkv == 0 && gb_plan(H / Hkv, D, Dv, max_q, &p) ? p.tq : 0;
+  return Hkv >= 1 && H % Hkv == 0 && gb_plan(H / Hkv, D, Dv, max_q, false, &p) ? p.tq : 0;
 }
 
 // q bf16 [T, H, D] (row stride q_ld elements), k_cache bf16 [num_blocks, 64, Hkv, D], v_cache bf16 [num_blocks, 64, Hkv, Dv];
@@ -371,7 +434,8 @@ extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache,
                              void* out, long long o_ld, float* part, float* lse2, cudaStream_t st) {
   if (T <= 0) return 0;
   GbPlan p;
-  if (Hkv < 1 || H % Hkv || splits < 1 || (splits > 1 && (!part || !lse2)) || max_tiles < 1 || !gb_plan(H / Hkv, D, Dv, max_q, &p)) return 1001;
+  if (Hkv < 1 || H % Hkv || splits < 1 || (splits > 1 && (!part || !lse2)) || max_tiles < 1) return 1001;
+  if (!gb_plan(H / Hkv, D, Dv, max_q, softcap > 0.f, &p) && !gb_plan(H / Hkv, D, Dv, max_q, false, &p)) return 1001;
   if (q_ld % 8 || o_ld % 8 || q_ld < (long long)H * D || (((uintptr_t)q | (uintptr_t)out) & 15)) return 1002;
   const int g = H / Hkv;
   CUtensorMap mq, mk, mv;
@@ -388,12 +452,14 @@ extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache,
     uint32_t box[4] = {64, 1, kBPage, 1};
     rc = make_tmap(which ? &mv : &mk, which ? v_cache : k_cache, TMA_BF16, 4, dims, strides, box, TMA_SW_128); if (rc) return 2100 + rc;
   }
-  auto kern = softcap > 0.f ? gqa_biased_kernel<true> : gqa_biased_kernel<false>;
-  static bool configured[2] = {false, false};
-  if (!configured[softcap > 0.f]) {
+  const int variant = (softcap > 0.f ? 2 : 0) + p.rep;
+  auto kern = variant == 3 ? gqa_biased_kernel<true, true> : variant == 2 ? gqa_biased_kernel<true, false> : variant == 1 ? gqa_biased_kernel<false, true>
+                                                                                                                          : gqa_biased_kernel<false, false>;
+  static bool configured[4] = {false, false, false, false};
+  if (!configured[variant]) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
     if (e != cudaSuccess) return (int)e;
-    configured[softcap > 0.f] = true;
+    configured[variant] = true;
   }
   GbArgs a;
   a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs;

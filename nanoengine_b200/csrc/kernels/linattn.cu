@@ -121,25 +121,31 @@ __global__ void __launch_bounds__(128) ssm_prepare_kernel(const SsmArgs a) {
     }
   }
   T* out = reinterpret_cast<T*>(a.out) + c;
-  for (int t = t0; t < t1; t++) {
+  for (int tb = t0; tb < t1; tb += 4) {            // four tokens' loads in flight
+    float cur4[4][V];
 #pragma unroll
-    for (int j = 1; j < KM; j++)
+    for (int u = 0; u < 4; u++) if (tb + u < t1) ldv<V>(x + (long long)(tb + u) * a.ld, cur4[u]);
 #pragma unroll
-      for (int e = 0; e < V; e++) if (KT || j < K) h[j - 1][e] = h[j][e];
-    float cur[V], acc[V];
-    ldv<V>(x + (long long)t * a.ld, cur);
+    for (int u = 0; u < 4; u++) {
+      if (tb + u >= t1) break;
 #pragma unroll
-    for (int e = 0; e < V; e++) {
-      acc[e] = bias[e];
+      for (int j = 1; j < KM; j++)
 #pragma unroll
-      for (int j = 0; j < KM; j++) {
-        if (!KT && j >= K) break;
-        if (j == K - 1) h[j][e] = cur[e];
-        acc[e] = fmaf(h[j][e], w[j][e], acc[e]);
+        for (int e = 0; e < V; e++) if (KT || j < K) h[j - 1][e] = h[j][e];
+      float acc[V];
+#pragma unroll
+      for (int e = 0; e < V; e++) {
+        acc[e] = bias[e];
+#pragma unroll
+        for (int j = 0; j < KM; j++) {
+          if (!KT && j >= K) break;
+          if (j == K - 1) h[j][e] = cur4[u][e];
+          acc[e] = fmaf(h[j][e], w[j][e], acc[e]);
+        }
+        acc[e] = silu_f(acc[e]);
       }
-      acc[e] = silu_f(acc[e]);
+      stv<V>(out + (long long)(tb + u) * C, acc);
     }
-    stv<V>(out + (long long)t * C, acc);
   }
 }
 
@@ -355,11 +361,65 @@ __global__ void __launch_bounds__(512) gated_norm_kernel(const float* __restrict
   }
 }
 
+// The same for parts of up to IT * 8 elements per thread, held in registers: all of a thread's loads are in flight before the reduction.
+template <typename T, int IT>
+__global__ void __launch_bounds__(512) gated_norm_regs_kernel(const float* __restrict__ raw, const T* __restrict__ gate, long long g_ld, const T* __restrict__ w,
+                                                             T* __restrict__ out, long long o_ld, int W, int P, int before, float eps, float scale) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  __shared__ float red[16];
+  const long long t = blockIdx.x;
+  const int c0 = blockIdx.y * P;
+  const float* rr = raw + t * W + c0;
+  const T* gr = gate + t * g_ld + c0;
+  float f[IT][8], g[IT][8], ww[IT][8], ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < IT; it++) {
+    const int i = (it * blockDim.x + threadIdx.x) * 8;
+    if (i < P) { lda4(rr + i, f[it]); lda4(rr + i + 4, f[it] + 4); lda4(gr + i, g[it]); lda4(gr + i + 4, g[it] + 4); lda4(w + c0 + i, ww[it]); lda4(w + c0 + i + 4, ww[it] + 4); }
+    else {
+#pragma unroll
+      for (int e = 0; e < 8; e++) f[it][e] = g[it][e] = ww[it][e] = 0.f;
+    }
+  }
+#pragma unroll
+  for (int it = 0; it < IT; it++)
+#pragma unroll
+    for (int e = 0; e < 8; e++) {
+      if (before) f[it][e] *= silu_f(g[it][e]);
+      ss += f[it][e] * f[it][e];
+    }
+  ss = warp_sum(ss);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (nw > 1) {
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    ss = warp_sum(lane < nw ? red[lane] : 0.f);
+  }
+  const float r = rsqrtf(ss / (float)P + eps) * scale;
+#pragma unroll
+  for (int it = 0; it < IT; it++) {
+    const int i = (it * blockDim.x + threadIdx.x) * 8;
+    if (i >= P) continue;
+#pragma unroll
+    for (int e = 0; e < 8; e++) {
+      f[it][e] *= r * ww[it][e];
+      if (!before) f[it][e] /= 1.f + expf(-g[it][e]);
+    }
+    sta4(out + t * o_ld + c0 + i, f[it]); sta4(out + t * o_ld + c0 + i + 4, f[it] + 4);
+  }
+}
+
 template <typename T>
 static int gated_norm_t(const float* raw, const void* gate, long long g_ld, const void* w, void* out, long long o_ld, int T_, int W, int parts, int before,
                         float eps, float scale, cudaStream_t st) {
   const int P = W / parts;
   const bool vec = P % 4 == 0 && g_ld % 4 == 0 && o_ld % 4 == 0 && ((uintptr_t)raw | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) % 16 == 0;
+  if (vec && P % 8 == 0 && P <= 8 * 512 * 2) {
+    const int units = P / 8, two = units > 512;
+    const int th = ((two ? (units + 1) / 2 : units) + 31) / 32 * 32;
+    return (int)launch_pdl(two ? gated_norm_regs_kernel<T, 2> : gated_norm_regs_kernel<T, 1>, dim3((unsigned)T_, (unsigned)parts), dim3((unsigned)th), 0, st, raw,
+                           (const T*)gate, g_ld, (const T*)w, (T*)out, o_ld, W, P, before, eps, scale);
+  }
   const int per = vec ? 4 : 1;
   int threads = ((P + per - 1) / per + 31) / 32 * 32;
   threads = threads > 512 ? 512 : threads;

@@ -34,7 +34,9 @@ struct ChunkArgs {
 __device__ __forceinline__ int swz(int row, int piece) { return row * 128 + ((piece ^ (row & 7)) << 4); }      // byte offset of a 16-byte piece
 __device__ __forceinline__ uint32_t silu2(uint32_t u) {
   const float2 f = unpack_bf16x2(u);
-  return pack_bf16x2(f.x / (1.f + __expf(-f.x)), f.y / (1.f + __expf(-f.y)));
+  // one reciprocal for two; below -40 the result is zero in bf16 next to anything
+  const float a = 1.f + __expf(fminf(-f.x, 40.f)), b = 1.f + __expf(fminf(-f.y, 40.f)), r = __fdividef(1.f, a * b);
+  return pack_bf16x2(f.x * b * r, f.y * a * r);
 }
 // fp32 pair -> bf16 heads and bf16 remainders
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {

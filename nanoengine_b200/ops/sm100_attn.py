@@ -236,8 +236,9 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
         if S is None:
             pages = bt.shape[1] if window <= 0 else min(bt.shape[1], (window + tq + 62) // 64 + 1)
             S = 1
-            if tiles * Hkv < 74:                       # few CTAs (small decode batches): slice the keys
-                S = max(1, min(148 // (tiles * Hkv), max(1, pages // 4), 16))
+            slots = _sms() * (2 if Dv <= 128 else 1)   # resident CTAs
+            if tiles * Hkv * 2 <= slots:               # few CTAs (small decode batches): slice the keys
+                S = max(1, min(slots // (tiles * Hkv), max(1, pages // 4), 16))
         part = lse2 = None
         if S > 1:
             part = torch.empty(S, T, Hq, Dv, dtype=torch.float32, device=q.device)
