@@ -460,6 +460,7 @@ def build_cases(args):
         "gdn_prefill_1x8192": lambda: case_gdn(1, q_len=8192),
         "mamba2_decode": lambda: case_mamba2(128),
         "mamba2_decode_16": lambda: case_mamba2(16),
+        "mamba2_prefill_1x1024": lambda: case_mamba2(1, q_len=1024),
         "mamba2_prefill_4x2048": lambda: case_mamba2(4, q_len=2048),
         "mamba2_prefill_1x8192": lambda: case_mamba2(1, q_len=8192),
         "lightning_decode": lambda: case_lightning(128),

@@ -31,7 +31,11 @@ __device__ __forceinline__ void sta4(float* p, const float* v) { *reinterpret_ca
 __device__ __forceinline__ void sta4(__nv_bfloat16* p, const float* v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3])); }
 template <int V, typename T> __device__ __forceinline__ void ldv(const T* p, float* o) { if constexpr (V == 4) lda4(p, o); else o[0] = lda(p); }
 template <int V, typename T> __device__ __forceinline__ void stv(T* p, const float* v) { if constexpr (V == 4) sta4(p, v); else sta(p, v[0]); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// silu and sigmoid in the accuracy of the values they meet: exact functions for fp32, hardware exponentials (2^-21) where the result is rounded
+// to bf16
+__device__ __forceinline__ float sigm(float x, const float*) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigm(float x, const __nv_bfloat16*) { return __fdividef(1.f, 1.f + __expf(-x)); }
+template <typename T> __device__ __forceinline__ float silu_t(float x) { return x * sigm(x, (const T*)nullptr); }
 __device__ __forceinline__ float round_as(float x, const float*) { return x; }
 __device__ __forceinline__ float round_as(float x, const __nv_bfloat16*) { return __bfloat162float(__float2bfloat16(x)); }
 
@@ -142,7 +146,7 @@ __global__ void __launch_bounds__(128) ssm_prepare_kernel(const SsmArgs a) {
           if (j == K - 1) h[j][e] = cur4[u][e];
           acc[e] = fmaf(h[j][e], w[j][e], acc[e]);
         }
-        acc[e] = silu_f(acc[e]);
+        acc[e] = silu_t<T>(acc[e]);
       }
       stv<V>(out + (long long)(tb + u) * C, acc);
     }
@@ -216,7 +220,7 @@ __global__ void __launch_bounds__(256, CPL * R >= 64 ? 2 : CPL * R >= 32 ? 3 : 4
       float f[V];
       ldv<V>(which ? qg + (t0 + tok) * a.q_ld + c : kg + (t0 + tok) * a.k_ld + c, f);
 #pragma unroll
-      for (int e = 0; e < V; e++) (which ? sq : sk)[tok * DKP + c + e] = a.act ? round_as(silu_f(f[e]), qg) : f[e];
+      for (int e = 0; e < V; e++) (which ? sq : sk)[tok * DKP + c + e] = a.act ? round_as(silu_t<T>(f[e]), qg) : f[e];
     }
     for (int i = threadIdx.x; i < m * vper; i += blockDim.x) {
       const int r = (i % vper) * V, tok = i / vper;
@@ -224,7 +228,7 @@ __global__ void __launch_bounds__(256, CPL * R >= 64 ? 2 : CPL * R >= 32 ? 3 : 4
       float f[V];
       ldv<V>(vg + (t0 + tok) * a.v_ld + r, f);
 #pragma unroll
-      for (int e = 0; e < V; e++) sv[tok * rows + r + e] = a.act ? round_as(silu_f(f[e]), qg) : f[e];
+      for (int e = 0; e < V; e++) sv[tok * rows + r + e] = a.act ? round_as(silu_t<T>(f[e]), qg) : f[e];
     }
     for (int i = threadIdx.x; i < m; i += blockDim.x) {
       if (a.gates) {
@@ -334,7 +338,7 @@ __global__ void __launch_bounds__(512) gated_norm_kernel(const float* __restrict
     if (before) {
       ldv<V>(gr + i, g);
 #pragma unroll
-      for (int e = 0; e < V; e++) f[e] *= silu_f(g[e]);
+      for (int e = 0; e < V; e++) f[e] *= silu_t<T>(g[e]);
     }
 #pragma unroll
     for (int e = 0; e < V; e++) ss += f[e] * f[e];
@@ -355,7 +359,7 @@ __global__ void __launch_bounds__(512) gated_norm_kernel(const float* __restrict
 #pragma unroll
     for (int e = 0; e < V; e++) {
       f[e] *= r * ww[e];
-      if (!before) f[e] /= (1.f + expf(-g[e]));
+      if (!before) f[e] *= sigm(g[e], gr);
     }
     stv<V>(out + t * o_ld + c0 + i, f);
   }
@@ -385,7 +389,7 @@ __global__ void __launch_bounds__(512) gated_norm_regs_kernel(const float* __res
   for (int it = 0; it < IT; it++)
 #pragma unroll
     for (int e = 0; e < 8; e++) {
-      if (before) f[it][e] *= silu_f(g[it][e]);
+      if (before) f[it][e] *= silu_t<T>(g[it][e]);
       ss += f[it][e] * f[it][e];
     }
   ss = warp_sum(ss);
@@ -403,7 +407,7 @@ __global__ void __launch_bounds__(512) gated_norm_regs_kernel(const float* __res
 #pragma unroll
     for (int e = 0; e < 8; e++) {
       f[it][e] *= r * ww[it][e];
-      if (!before) f[it][e] /= 1.f + expf(-g[it][e]);
+      if (!before) f[it][e] *= sigm(g[it][e], gr);
     }
     sta4(out + t * o_ld + c0 + i, f[it]); sta4(out + t * o_ld + c0 + i + 4, f[it] + 4);
   }

@@ -12,12 +12,12 @@
 //     o  = e^(C_i) Yi + Y + d v
 // C: running sum of the log-decays, kept per block of 32 tokens so that no difference of large sums is taken: a factor between blocks is the
 // product of two exponentials of at most one, only the diagonal blocks take an exponential per element.
-// 256 threads: all of them load, convert and store; thread 0 issues the products.  All waits are bounded.
+// 512 threads: all of them load, convert and store; thread 0 issues the products.  All waits are bounded.
 #include "ptx.cuh"
 
 namespace ne {
 
-constexpr int kCtThreads = 256;
+constexpr int kCtThreads = 512;
 constexpr int kKernelCt = 14;
 constexpr int kCL = 128;                        // tokens per chunk
 constexpr int kCTile = kCL * 128;               // 128 rows x 64 bf16 columns, 128-byte swizzled
@@ -85,18 +85,15 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
   const bool s_row = wq * 32 < nk * 64;          // whole warps: rows of the state tile
 
   float* Sg = a.state + ((long long)slot * a.H + h) * Dv * Dk;
-  {                                              // the carried state: lane = column of Dk, 32 columns of Dv per thread
+  {                                              // the carried state: lane = column of Dk, 16 columns of Dv per thread
     const bool have = a.fresh[seq] == 0 && row < Dk;
+    uint32_t r[16];
 #pragma unroll
-    for (int c0 = 0; c0 < 32; c0 += 16) {
-      uint32_t r[16];
-#pragma unroll
-      for (int c = 0; c < 16; c++) {
-        const int d = hf * 32 + c0 + c;
-        r[c] = (have && d < vcols) ? __float_as_uint(Sg[(long long)(dv0 + d) * Dk + row]) : 0u;
-      }
-      tmem_st_32x32b_x16(t_s + lane_addr + hf * 32 + c0, r);
+    for (int c = 0; c < 16; c++) {
+      const int d = hf * 16 + c;
+      r[c] = (have && d < vcols) ? __float_as_uint(Sg[(long long)(dv0 + d) * Dk + row]) : 0u;
     }
+    tmem_st_32x32b_x16(t_s + lane_addr + hf * 16, r);
     tc_wait_st();
   }
   const float skip = a.skip ? a.skip[h] : 0.f;
@@ -109,20 +106,20 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
   constexpr uint32_t kIdY = make_idesc(FMT_BF16, FMT_BF16, 128, 64, 0, 1);       // B read MN-major: rows are tokens or columns of Dk
   constexpr uint32_t kIdS = make_idesc(FMT_BF16, FMT_BF16, 128, 64, 1, 1);
   // the next chunk's rows are fetched into registers while this one's products run
-  uint4 rq[4 * NK], rk[4 * NK], rv[4];
+  uint4 rq[2 * NK], rk[2 * NK], rv[2];
   float2 rg = make_float2(0.f, 0.f);
   auto fetch = [&](int i0) {
     const int m = min(kCL, n - i0);
     const long long t0 = start + i0;
 #pragma unroll
-    for (int e = 0; e < 4 * NK; e++) {
+    for (int e = 0; e < 2 * NK; e++) {
       const int j = tid + e * kCtThreads, r = j >> kShift, c = (j & (8 * NK - 1)) * 8;
       const bool in = r < m && c < Dk;
       rq[e] = in ? *reinterpret_cast<const uint4*>(qg + (t0 + r) * a.q_ld + c) : make_uint4(0, 0, 0, 0);
       rk[e] = in ? *reinterpret_cast<const uint4*>(kg + (t0 + r) * a.k_ld + c) : make_uint4(0, 0, 0, 0);
     }
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
+    for (int e = 0; e < 2; e++) {
       const int j = tid + e * kCtThreads, r = j >> 3, c = (j & 7) * 8;
       rv[e] = r < m && c < vcols ? *reinterpret_cast<const uint4*>(vg + (t0 + r) * a.v_ld + c) : make_uint4(0, 0, 0, 0);
     }
@@ -153,13 +150,13 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
     }
     // ---- q, k, v tiles
 #pragma unroll
-    for (int e = 0; e < 4 * NK; e++) {
+    for (int e = 0; e < 2 * NK; e++) {
       const int j = tid + e * kCtThreads, r = j >> kShift, p = j & (8 * NK - 1);
       put(sQ, r, p, rq[e]);
       put(sK, r, p, rk[e]);
     }
 #pragma unroll
-    for (int e = 0; e < 4; e++) { const int j = tid + e * kCtThreads; put(sV, j >> 3, j & 7, rv[e]); }
+    for (int e = 0; e < 2; e++) { const int j = tid + e * kCtThreads; put(sV, j >> 3, j & 7, rv[e]); }
     __syncthreads();
     const float bt0 = s_bt[0], bt1 = s_bt[1], bt2 = s_bt[2], bt3 = s_bt[3];
     const float after[4] = {bt1 + bt2 + bt3, bt2 + bt3, bt3, 0.f};
@@ -180,24 +177,21 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
     // ---- the state: head and remainder as it is, the accumulator scaled by the whole chunk's decay
     if (s_row) {
       const float dec = exp2f(bt0 + after[0]);
+      uint32_t r[16];
+      tmem_ld_32x32b_x16(t_s + lane_addr + hf * 16, r);
+      tc_wait_ld();
+      uint32_t hi[8], lo[8];
 #pragma unroll
-      for (int c0 = 0; c0 < 32; c0 += 16) {
-        uint32_t r[16];
-        tmem_ld_32x32b_x16(t_s + lane_addr + hf * 32 + c0, r);
-        tc_wait_ld();
-        uint32_t hi[8], lo[8];
+      for (int c = 0; c < 8; c++) split2(__uint_as_float(r[2 * c]), __uint_as_float(r[2 * c + 1]), hi[c], lo[c]);
 #pragma unroll
-        for (int c = 0; c < 8; c++) split2(__uint_as_float(r[2 * c]), __uint_as_float(r[2 * c + 1]), hi[c], lo[c]);
-#pragma unroll
-        for (int p = 0; p < 2; p++) {
-          const int o = swz(row, hf * 4 + (c0 >> 3) + p);
-          *reinterpret_cast<uint4*>(sSh + o) = make_uint4(hi[4 * p], hi[4 * p + 1], hi[4 * p + 2], hi[4 * p + 3]);
-          *reinterpret_cast<uint4*>(sSl + o) = make_uint4(lo[4 * p], lo[4 * p + 1], lo[4 * p + 2], lo[4 * p + 3]);
-        }
-#pragma unroll
-        for (int c = 0; c < 16; c++) r[c] = __float_as_uint(__uint_as_float(r[c]) * dec);
-        tmem_st_32x32b_x16(t_s + lane_addr + hf * 32 + c0, r);
+      for (int p = 0; p < 2; p++) {
+        const int o = swz(row, hf * 2 + p);
+        *reinterpret_cast<uint4*>(sSh + o) = make_uint4(hi[4 * p], hi[4 * p + 1], hi[4 * p + 2], hi[4 * p + 3]);
+        *reinterpret_cast<uint4*>(sSl + o) = make_uint4(lo[4 * p], lo[4 * p + 1], lo[4 * p + 2], lo[4 * p + 3]);
       }
+#pragma unroll
+      for (int c = 0; c < 16; c++) r[c] = __float_as_uint(__uint_as_float(r[c]) * dec);
+      tmem_st_32x32b_x16(t_s + lane_addr + hf * 16, r);
       tc_wait_st();
     }
     fence_proxy_async_smem();
@@ -222,12 +216,11 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
     }
     ok = mbar_wait(bar_g, phase, abort_flag, kKernelCt, 100);
     tc_fence_after();
-    // ---- decayed scores: this thread's row, blocks 2 hf and 2 hf + 1 of 32 columns
+    // ---- decayed scores: this thread's row, block hf of 32 columns
     if (ok) {
       const float li = s_lc[row];
-#pragma unroll
-      for (int x = 0; x < 2; x++) {
-        const int jb = 2 * hf + x;               // whole warps take the same branch: a warp's rows are one block
+      {
+        const int jb = hf;                       // whole warps take the same branch: a warp's rows are one block
         uint32_t hi[16], lo[16];
         if (jb > wq) {
 #pragma unroll
@@ -262,7 +255,7 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
         }
 #pragma unroll
         for (int p = 0; p < 4; p++) {
-          const int o = hf * kCTile + swz(row, x * 4 + p);
+          const int o = (hf >> 1) * kCTile + swz(row, (hf & 1) * 4 + p);
           *reinterpret_cast<uint4*>(sPh + o) = make_uint4(hi[4 * p], hi[4 * p + 1], hi[4 * p + 2], hi[4 * p + 3]);
           *reinterpret_cast<uint4*>(sPl + o) = make_uint4(lo[4 * p], lo[4 * p + 1], lo[4 * p + 2], lo[4 * p + 3]);
         }
@@ -284,25 +277,24 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
     if (i0 + kCL < n) fetch(i0 + kCL);
     ok = mbar_wait(bar_y, phase, abort_flag, kKernelCt, 200);
     tc_fence_after();
-    // ---- outputs: 32 columns of this thread's row
+    // ---- outputs: 16 columns of this thread's row
     if (ok) {
       const float before = (wq > 0 ? bt0 : 0.f) + (wq > 1 ? bt1 : 0.f) + (wq > 2 ? bt2 : 0.f);
       const float f = exp2f(s_lc[row] + before);
-#pragma unroll
-      for (int c0 = 0; c0 < 32; c0 += 16) {
+      {
         uint32_t yi[16], y[16];
-        tmem_ld_32x32b_x16(t_yi + lane_addr + hf * 32 + c0, yi);
-        tmem_ld_32x32b_x16(t_y + lane_addr + hf * 32 + c0, y);
+        tmem_ld_32x32b_x16(t_yi + lane_addr + hf * 16, yi);
+        tmem_ld_32x32b_x16(t_y + lane_addr + hf * 16, y);
         tc_wait_ld();
 #pragma unroll
         for (int p = 0; p < 2; p++) {
-          const uint4 u = *reinterpret_cast<const uint4*>(sV + swz(row, hf * 4 + (c0 >> 3) + p));
+          const uint4 u = *reinterpret_cast<const uint4*>(sV + swz(row, hf * 2 + p));
           const float2 v0 = unpack_bf16x2(u.x), v1 = unpack_bf16x2(u.y), v2 = unpack_bf16x2(u.z), v3 = unpack_bf16x2(u.w);
           const float vv[8] = {v0.x, v0.y, v1.x, v1.y, v2.x, v2.y, v3.x, v3.y};
           float o[8];
 #pragma unroll
           for (int e = 0; e < 8; e++) o[e] = fmaf(skip, vv[e], fmaf(f, __uint_as_float(yi[p * 8 + e]), __uint_as_float(y[p * 8 + e])));
-          float* dst = sY + row * kYld + hf * 32 + c0 + p * 8;
+          float* dst = sY + row * kYld + hf * 16 + p * 8;
           *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
           *reinterpret_cast<float4*>(dst + 4) = make_float4(o[4], o[5], o[6], o[7]);
         }
@@ -319,16 +311,13 @@ __global__ void __launch_bounds__(kCtThreads, 1) decay_chunk_kernel(const ChunkA
   }
   if (ok) {
     if (s_row) {
+      uint32_t r[16];
+      tmem_ld_32x32b_x16(t_s + lane_addr + hf * 16, r);
+      tc_wait_ld();
 #pragma unroll
-      for (int c0 = 0; c0 < 32; c0 += 16) {
-        uint32_t r[16];
-        tmem_ld_32x32b_x16(t_s + lane_addr + hf * 32 + c0, r);
-        tc_wait_ld();
-#pragma unroll
-        for (int c = 0; c < 16; c++) {
-          const int d = hf * 32 + c0 + c;
-          if (row < Dk && d < vcols) Sg[(long long)(dv0 + d) * Dk + row] = __uint_as_float(r[c]);
-        }
+      for (int c = 0; c < 16; c++) {
+        const int d = hf * 16 + c;
+        if (row < Dk && d < vcols) Sg[(long long)(dv0 + d) * Dk + row] = __uint_as_float(r[c]);
       }
     }
   }
