@@ -249,18 +249,22 @@ class ModelRunner:
 
     def _warmup_prefill(self, tokens: int) -> None:
         bs = self.plan.block_size
-        nb = (tokens + bs - 1) // bs
+        # one sequence, or several where the model's learned positions end before the token budget
+        longest = min(tokens, self.mc.max_position_embeddings) if self.mc.learned_positions else tokens
+        lens = [longest] * (tokens // longest) + ([tokens % longest] if tokens % longest else [])
+        nbs = [(n + bs - 1) // bs for n in lens]
+        nb, n_seq = sum(nbs), len(lens)
         import dataclasses
         tmp = KVCache(dataclasses.replace(self.plan, state_slots=0), nb, self.device)   # the scratch state slot is enough here
         b = C.RunnerIn()
         b.is_prefill = True
-        b.seq_ids = [0]
+        b.seq_ids = list(range(n_seq))
         b.input_ids = [1] * tokens
-        b.positions = list(range(tokens))
-        b.q_lens, b.seq_lens = [tokens], [tokens]
-        b.block_tables, b.block_offsets = list(range(nb)), [0, nb]
-        b.temperatures, b.sample_mask = [0.0], [1]
-        b.state_slots = b.handoff_slots = b.hisparse_slots = [-1]
+        b.positions = [p for n in lens for p in range(n)]
+        b.q_lens, b.seq_lens = lens, lens
+        b.block_tables, b.block_offsets = list(range(nb)), [sum(nbs[:i]) for i in range(n_seq + 1)]
+        b.temperatures, b.sample_mask = [0.0] * n_seq, [1] * n_seq
+        b.state_slots = b.handoff_slots = b.hisparse_slots = [-1] * n_seq
         saved, self.cache = self.cache, tmp
         try:
             self.run_batch(b)

@@ -27,7 +27,7 @@ CONFIGS = {
         mamba2(3, 18, 36, groups=1, conv=2, norm_groups=1, ff=44)]},
     # sizes the tensor-core paths take; windows of a page, less and more; grouped and single key / value heads
     "aligned": {"vocab": 192, "width": 128, "norm": {"eps": 1e-6}, "streams": 2, "logit_softcap": 30.0, "max_positions": 600, "layers": [
-        parallel(8, 2, 32, 48, 64, 4, 64, 32, ff=160, softcap=8.0), mamba2(8, 32, 64, groups=2, conv=4, norm_groups=2), parallel(6, 2, 80, 24, 21, 2, 128, 128),
+        parallel(8, 2, 32, 48, 64, 4, 64, 24, ff=160, softcap=8.0), mamba2(8, 32, 64, groups=2, conv=4, norm_groups=2), parallel(6, 2, 80, 24, 21, 2, 128, 128),
         parallel(4, 4, 64, 64, 130, 8, 16, 64, ff=96, softcap=50.0, scales=(1.0, 1.0))]},
     # Mamba-2 first and last, long convolution, one stream, eps that matters, a window of one token, decays of zero and one
     "mamba_first": {"vocab": 130, "width": 96, "norm": {"eps": 1e-2}, "streams": 1, "logit_softcap": 12.0, "max_positions": 520, "layers": [
