@@ -13,7 +13,9 @@ from typing import Any, Dict, List, Optional
 
 
 # mixers of listed layers that carry a recurrent state per sequence
-_STATE_MIXERS = ("delta", "mamba2", "parallel")
+_STATE_MIXERS = ("delta", "mamba2", "parallel", "general_delta")
+# ... and that keep rows in the paged cache
+_ROW_MIXERS = ("latent_attention", "parallel", "attention")
 
 
 @dataclass
@@ -107,9 +109,11 @@ class ModelConfig:
     o_groups: int = 0
     num_hash_layers: int = 0                 # the first this-many MoE layers pick experts from a token-id table
     # families that list every layer with its own mixer, the mixer's sizes and its feed-forward (Tuvutar: "latent_attention" | "delta",
-    # Filasun: "mamba2" | "parallel"); the fields above describe one such layer only in the form `layer_config` derives for it
+    # Filasun: "mamba2" | "parallel", Sapanex: "attention" | "general_delta"); the fields above describe one such layer only in the form `layer_config` derives for it
     layer_specs: Optional[List[Dict[str, Any]]] = None
     attn_scale: float = 0.0                  # > 0: softmax scale of the latent-attention layer (0: from the head dim)
+    embedding_scale: float = 1.0             # token embeddings enter the residual stream times this
+    postnorm_alpha: float = 0.0              # > 0: x <- norm(alpha x + sublayer(x)), the norm behind the sum
     learned_positions: bool = False          # a learned vector per position, max_position_embeddings of them: a hard context limit
     # MTP
     num_nextn_predict_layers: int = 0
@@ -188,7 +192,7 @@ class ModelConfig:
 
     def layer_type(self, layer_idx: int) -> str:
         if self.layer_specs:
-            return "linear_attention" if self.layer_specs[layer_idx]["type"] in ("delta", "mamba2") else "full_attention"
+            return "linear_attention" if self.layer_specs[layer_idx]["type"] not in _ROW_MIXERS else "full_attention"
         if not self.is_hybrid_gdn:
             return "full_attention"
         if self.layer_types and layer_idx < len(self.layer_types):
@@ -199,7 +203,7 @@ class ModelConfig:
     def keeps_rows(self, layer_idx: int) -> bool:
         """Does the listed layer own pages of the paged cache?"""
         t = self.layer_specs[layer_idx]["type"]
-        return t in ("latent_attention", "parallel") and self.kv_source_layer(layer_idx) == layer_idx
+        return t in _ROW_MIXERS and self.kv_source_layer(layer_idx) == layer_idx
 
     def keeps_state(self, layer_idx: int) -> bool:
         """Does the listed layer own a slot of recurrent state per sequence?  A "parallel" layer owns both."""
@@ -288,6 +292,8 @@ class ModelConfig:
             d = _tuvutar_fields(d)
         if arch == "Filasun" and "layers" in d:
             d = _filasun_fields(d)
+        if arch == "Sapanex" and "layers" in d:
+            d = _sapanex_fields(d)
         la = d.pop("linear_attn_config", None)
         if isinstance(la, dict):                          # Kimi delta attention block of GLM5-next / Kimi-K3
             d["linear_kind"] = "kda"
@@ -377,7 +383,12 @@ class ModelConfig:
                 q = json.load(f).get("quantization", {})
             if q.get("quant_algo"):
                 d["quantization_config"] = {"quant_method": "modelopt", **q}
-        return cls.from_dict(d)
+        mc = cls.from_dict(d)
+        for i, s in enumerate(mc.layer_specs or []):               # the rank of a low-rank projection is in the tensors only
+            if s["type"] == "general_delta" and "decay_rank" not in s["mixer"]:
+                from .weights import tensor_shape
+                s["mixer"]["decay_rank"] = tensor_shape(path, f"l{i}.mix.w1")[0]
+        return mc
 
     def to_dict(self) -> Dict[str, Any]:
         d = {f.name: getattr(self, f.name) for f in fields(self)}
@@ -464,6 +475,37 @@ def _filasun_fields(d: Dict[str, Any]) -> Dict[str, Any]:
            "rms_norm_eps": float(d["norm"]["eps"]), "q_lora_rank": None, "n_routed_experts": 0, "n_shared_experts": 0, "tie_word_embeddings": False,
            "num_attention_heads": 1, "num_key_value_heads": 1, "max_position_embeddings": int(d["max_positions"]), "learned_positions": True,
            "hc_mult": int(d["streams"]), "final_logit_softcapping": float(d["logit_softcap"]),
+           "layer_specs": [{"type": s["type"], "mixer": dict(s["mixer"]), "mlp": dict(s["mlp"]) if s.get("mlp") is not None else None} for s in d["layers"]]}
+    for k in ("eos_token_id", "bos_token_id"):
+        if d.get(k) is not None:
+            out[k] = d[k]
+    return out
+
+
+def _sapanex_fields(d: Dict[str, Any]) -> Dict[str, Any]:
+    """config.json of a Sapanex model ({architecture, embedding, layers, norm, postln_alpha, vocab, width}) as ModelConfig fields.  The design has
+    no context limit of its own; the default only sizes the rotary tables (Config raises it to max_model_len)."""
+    def need(ok, i, what):
+        if not ok:
+            raise ValueError(f"layer {i}: {what}")
+
+    for i, s in enumerate(d["layers"]):
+        m = s["mixer"]
+        if s["type"] == "attention":
+            need(int(m["heads"]) % int(m["kv_heads"]) == 0, i, "heads must be a multiple of kv_heads")
+            need(0 < int(m["rot"]["dims"]) <= int(m["dim"]) and int(m["rot"]["dims"]) % 2 == 0, i, "an even number of rotated dimensions, at most dim")
+            need(int(m["vdim"]) % 2 == 0, i, "rotated values need an even vdim")
+            need(int(m["mask"]["size"]) >= 1 and int(m["mask"]["pool"]) >= 1, i, "window and pooled blocks hold at least one token")
+        elif s["type"] == "general_delta":
+            need(1 <= int(m["dim"]) <= 512, i, "1 to 512 state rows per head")
+        else:
+            need(False, i, f"unknown mixer type {s['type']!r}")
+        if s.get("mlp") is not None:
+            need(s["mlp"]["kind"] == "dense", i, f"unknown feed-forward kind {s['mlp']['kind']!r}")
+    out = {"architecture": d["architecture"], "vocab_size": int(d["vocab"]), "hidden_size": int(d["width"]), "num_hidden_layers": len(d["layers"]),
+           "rms_norm_eps": float(d["norm"]["eps"]), "q_lora_rank": None, "n_routed_experts": 0, "n_shared_experts": 0, "tie_word_embeddings": True,
+           "num_attention_heads": 1, "num_key_value_heads": 1, "max_position_embeddings": int(d.get("max_position_embeddings") or 131072),
+           "embedding_scale": float(d["embedding"]["scale"]), "postnorm_alpha": float(d["postln_alpha"]),
            "layer_specs": [{"type": s["type"], "mixer": dict(s["mixer"]), "mlp": dict(s["mlp"]) if s.get("mlp") is not None else None} for s in d["layers"]]}
     for k in ("eos_token_id", "bos_token_id"):
         if d.get(k) is not None:
@@ -686,3 +728,41 @@ def filasun_7b(**over) -> ModelConfig:
 
 
 PRESETS["tiny-filasun"], PRESETS["filasun-7b"] = tiny_filasun, filasun_7b
+
+
+def _pooled_attention_spec(heads, kv_heads, dim, vdim, window, pool, rot_dims, ff=0, base=10000.0, scaling=None):
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": window, "pool": pool},
+                                           "rot": {"base": base, "dims": rot_dims, "scaling": scaling}},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def _general_delta_spec(heads, dim, rank, ff=0):
+    return {"type": "general_delta", "mixer": {"heads": heads, "dim": dim, "decay_rank": rank}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def tiny_sapanex(**over) -> ModelConfig:
+    """CPU-sized Sapanex shape: two attention layers of unlike windows and pools around two delta layers, one with a feed-forward."""
+    yarn = {"factor": 8.0, "original": 64, "fast": 16.0, "slow": 1.0}
+    c = ModelConfig.from_dict({"architecture": "Sapanex", "vocab": 512, "width": 128, "norm": {"eps": 1e-6}, "embedding": {"scale": 4.0}, "postln_alpha": 1.5, "layers": [
+        _pooled_attention_spec(4, 2, 32, 16, 24, 8, 16, ff=192, scaling=yarn), _general_delta_spec(4, 16, 8), _general_delta_spec(2, 32, 12, ff=96),
+        _pooled_attention_spec(6, 1, 16, 24, 70, 5, 16, ff=128)]})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+def sapanex_7b(**over) -> ModelConfig:
+    """A Sapanex shape of a real model's layer sizes (7B class): width 4096, one attention layer (32 / 8 heads of 128, a 4096-token window and
+    blocks of 16) after every three delta layers (32 heads of 128, rank 64)."""
+    yarn = {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+    layers = []
+    for _ in range(8):
+        layers += [_general_delta_spec(32, 128, 64, ff=16384) for _ in range(3)] + [_pooled_attention_spec(32, 8, 128, 128, 4096, 16, 64, ff=16384, base=5e5, scaling=yarn)]
+    c = ModelConfig.from_dict({"architecture": "Sapanex", "vocab": 131072, "width": 4096, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "postln_alpha": 2.0,
+                               "layers": layers})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+PRESETS["tiny-sapanex"], PRESETS["sapanex-7b"] = tiny_sapanex, sapanex_7b

@@ -42,8 +42,11 @@ class QLinear(nn.Module):
         if bias_fp32:
             self.bias = nn.Parameter(torch.zeros(self.weight.shape[0], dtype=torch.float32, device=device), requires_grad=False)
 
-    def forward(self, x):
-        y = ops.linear(x, self.weight, self.weight_scale_inv, self.bias)
+    def forward(self, x, act: Optional[str] = None, act_from: int = 0):
+        if act is not None:
+            y = ops.linear(x, self.weight, None, None, act=act, act_from=act_from)
+        else:
+            y = ops.linear(x, self.weight, self.weight_scale_inv, self.bias)
         return y if y.shape[-1] == self.out_features else y[..., : self.out_features]
 
     @torch.no_grad()
@@ -101,6 +104,17 @@ class SwiGLUMLP(nn.Module):
     def init_random(self, gen):
         self.gate_up_proj.init_random(gen)
         self.down_proj.init_random(gen)
+
+
+class DenseMLP(nn.Module):
+    """Two linears around an activation without a gate ("relu2": the square of relu), which is part of the first GEMM's epilogue."""
+
+    def __init__(self, hidden: int, inter: int, dtype, device, act: str):
+        super().__init__()
+        self.up_proj, self.down_proj, self.act = QLinear(hidden, inter, dtype, device), QLinear(inter, hidden, dtype, device), act
+
+    def forward(self, x):
+        return self.down_proj(self.up_proj(x, act=self.act))
 
 
 class TPSwiGLUMLP(nn.Module):

@@ -5,7 +5,12 @@ Mamba2Mixer     z | x | B | C from one GEMM, the step sizes from a second one wi
 ParallelMixer   two mixers over the same input, summed with constant weights: windowed grouped-query attention with capped scores, a
                 distance bias and an output gate per head (`ops.gqa_attention_biased`), and linear attention with a constant decay per head
                 (`ops.lightning_mix`).  Both read one merged projection and write into one row, so the pair costs two GEMMs; the weights of
-                the sum are applied to the fp32 results before they are rounded.  The layer owns rows of the paged cache and a state."""
+                the sum are applied to the fp32 results before they are rounded.  The layer owns rows of the paged cache and a state.
+PooledAttentionMixer   grouped-query attention over a window of tokens and the means of the blocks of tokens in front of it, with q and k
+                normed over all heads at once, partly rotated, and values that are cached rotated and whose sums are turned back
+                (`ops.pooled_attention_prepare`, `ops.gqa_attention_biased`).
+GeneralDeltaMixer   delta rule with a decay and a removal rate per key channel; everything from one GEMM, the decay's second, low-rank
+                factor from another one with an fp32 result; recurrence, norm and gate are `ops.general_delta`."""
 from __future__ import annotations
 
 from typing import Dict, Sequence
@@ -117,3 +122,67 @@ class ParallelMixer(nn.Module):
         self.out_proj.bias.zero_()
         self.out_proj.bias[: self.hidden].copy_(self.left_scale * w["left.o.b"])
         self.norm_weight.copy_(w["right.norm"])
+
+
+class PooledAttentionMixer(nn.Module):
+    ORDER = ("q", "k", "v")
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, pool: int, eps: float, cache_idx: int, dtype, device):
+        super().__init__()
+        self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = hidden, heads, kv_heads, dim, vdim
+        self.scale, self.window, self.pool, self.eps, self.cache_idx = scale, window, pool, eps, cache_idx
+        self.in_proj = QLinear(hidden, heads * dim + kv_heads * (dim + vdim), dtype, device)
+        self.out_proj = QLinear(heads * vdim, hidden, dtype, device)
+        self.q_norm, self.k_norm = _const(heads * dim, dtype=dtype, device=device, fill=1.0), _const(kv_heads * dim, dtype=dtype, device=device, fill=1.0)
+
+    def forward(self, h, positions, ctx: ForwardContext, key_table, value_table):
+        """The tables [positions, dims] (cos | sin): of the rotated part of queries and keys, and of whole values."""
+        kc, vc, kp, vp = ctx.kv_caches[self.cache_idx]
+        q = ops.pooled_attention_prepare(self.in_proj(h), self.heads, self.kv_heads, self.dim, self.vdim, self.q_norm, self.k_norm, self.eps, positions, key_table,
+                                         value_table, kc, vc, kp, vp, self.pool, ctx.slot_mapping, ctx.block_tables, ctx.cu_seqlens_q, ctx.max_seqlen_q)
+        return self.out_proj(ops.gqa_attention_biased(q, kc, vc, ctx.block_tables, ctx.cu_seqlens_q, ctx.context_lens, self.scale, self.window,
+                                                      max_q_len=ctx.max_seqlen_q, pooled=(kp, vp), pool=self.pool, turn_back=value_table))
+
+    def parts(self):
+        D, q, k, v = self.hidden, self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim
+        return {"q": (q, D), "k": (k, D), "v": (v, D), "q.norm": (q,), "k.norm": (k,), "o": (D, self.heads * self.vdim)}
+
+    def load(self, w: Dict[str, torch.Tensor]) -> None:
+        self.in_proj.set_weight(torch.cat([w[n] for n in self.ORDER], 0))
+        self.out_proj.set_weight(w["o"])
+        self.q_norm.copy_(w["q.norm"])
+        self.k_norm.copy_(w["k.norm"])
+
+
+class GeneralDeltaMixer(nn.Module):
+    # rows of the merged projection; the first factor of the decay's projection comes last: its tanh is part of the GEMM's epilogue
+    ORDER = ("r", "k", "a", "v", "g", "w1")
+
+    def __init__(self, hidden: int, heads: int, dim: int, rank: int, eps: float, state_idx: int, dtype, device):
+        super().__init__()
+        self.hidden, self.heads, self.dim, self.rank, self.eps, self.state_idx = hidden, heads, dim, rank, eps, state_idx
+        self.width = w = heads * dim
+        self.in_proj = QLinear(hidden, 5 * w + rank, dtype, device)
+        self.decay_proj = QLinear(rank, w, dtype, device)
+        self.out_proj = QLinear(w, hidden, dtype, device)
+        self.w0, self.a_bias = _const(w, device=device), _const(w, device=device)
+        self.norm_weight = _const(w, dtype=dtype, device=device, fill=1.0)
+
+    def forward(self, h, ctx: ForwardContext):
+        proj = self.in_proj(h, act="tanh", act_from=5 * self.width)
+        decay = ops.linear_fp32(proj[:, 5 * self.width: 5 * self.width + self.rank], self.decay_proj.weight)
+        return self.out_proj(ops.general_delta(proj, decay, self.w0, self.a_bias, self.norm_weight, ctx.rec_states[self.state_idx], ctx.state_slots, ctx.cu_seqlens_q,
+                                               ctx.seq_fresh, self.heads, self.dim, self.dim, self.eps, ctx.max_seqlen_q))
+
+    def parts(self):
+        D, w = self.hidden, self.width
+        out = {n: (w, D) for n in ("r", "k", "v", "g", "a")}
+        out.update({"a.b": (w,), "w1": (self.rank, D), "w2": (w, self.rank), "w0": (w,), "norm": (w,), "o": (D, w)})
+        return out
+
+    def load(self, w: Dict[str, torch.Tensor]) -> None:
+        self.in_proj.set_weight(torch.cat([w[n] for n in self.ORDER], 0))
+        self.decay_proj.set_weight(w["w2"])
+        self.out_proj.set_weight(w["o"])
+        for p, n in ((self.w0, "w0"), (self.a_bias, "a.b"), (self.norm_weight, "norm")):
+            p.copy_(w[n])

@@ -59,9 +59,15 @@ def _filasun():
     return FilasunForCausalLM
 
 
+def _sapanex():
+    from .sapanex import SapanexForCausalLM
+    return SapanexForCausalLM
+
+
 # kernel sources (stems under csrc/) of the architectures that can be served from a partial build; None = all of them
 _KERNELS = {"Tuvutar": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_bf16", "mla_bf16", "delta"),
-            "Filasun": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "linattn", "linattn_tc")}
+            "Filasun": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "linattn", "linattn_tc"),
+            "Sapanex": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "pooled", "general_delta")}
 
 
 def kernel_sources(architecture: str):
@@ -69,7 +75,7 @@ def kernel_sources(architecture: str):
 
 
 _LAZY = {
-    "Tuvutar": _tuvutar, "Filasun": _filasun,
+    "Tuvutar": _tuvutar, "Filasun": _filasun, "Sapanex": _sapanex,
     "Gemma4ForCausalLM": _gemma4, "Gemma4ForConditionalGeneration": _gemma4,
     "Glm5NextForConditionalGeneration": _glm5_next, "KimiK3ForConditionalGeneration": _kimi_k3,
     "DeepseekV4ForCausalLM": _deepseek_v4,

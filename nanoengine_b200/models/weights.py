@@ -61,6 +61,16 @@ def iterate_safetensors(path: str, keep: Optional[Callable[[str], bool]] = None,
                     yield name, sf.get_tensor(name)
 
 
+def tensor_shape(path: str, name: str) -> Tuple[int, ...]:
+    """Shape of one tensor of a checkpoint directory, from the shard headers."""
+    from safetensors import safe_open
+    for f in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(f, framework="pt") as sf:
+            if name in sf.keys():
+                return tuple(sf.get_slice(name).get_shape())
+    raise ValueError(f"{name}: not in the checkpoint under {path!r}")
+
+
 def hf_param_shapes(cfg: ModelConfig, include_mtp: bool = False) -> Dict[str, Tuple[int, ...]]:
     """Every tensor name of an HF-layout checkpoint of this architecture with its (high-precision) shape."""
     H, V = cfg.hidden_size, cfg.vocab_size
@@ -68,6 +78,9 @@ def hf_param_shapes(cfg: ModelConfig, include_mtp: bool = False) -> Dict[str, Tu
     if cfg.architecture.startswith("Gemma4"):
         return _gemma4_param_shapes(cfg, out)
     if cfg.layer_specs:
+        if cfg.architecture == "Sapanex":
+            from .sapanex import sapanex_param_shapes
+            return sapanex_param_shapes(cfg)
         if cfg.architecture == "Filasun":
             from .filasun import filasun_param_shapes
             return filasun_param_shapes(cfg)
@@ -242,6 +255,10 @@ def random_hf_weights(cfg: ModelConfig, seed: int = 0, device="cpu", keep: Optio
         g.manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
         if cfg.layer_specs:                     # rows scaled by their fan-in, norm weights around zero or one
             leaf = name.rsplit(".", 1)[-1]
+            if cfg.architecture == "Sapanex":
+                from .sapanex import sapanex_random_tensor
+                yield name, sapanex_random_tensor(name, shape, g, dev)
+                continue
             if cfg.architecture == "Filasun":
                 from .filasun import filasun_random_tensor
                 yield name, filasun_random_tensor(name, shape, g, dev)

@@ -120,6 +120,22 @@ def embed_norm(ids: torch.Tensor, table: torch.Tensor, w_next: torch.Tensor, eps
     return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(table.dtype), x
 
 
+def postnorm(y: torch.Tensor, x: torch.Tensor, alpha: float, w: torch.Tensor, eps: float, w_last: Optional[torch.Tensor] = None):
+    """Norm behind the sum around a 32-bit residual stream: x <- rmsnorm(alpha x + y, w); the next sublayer reads x itself in y's dtype, or
+    with `w_last` (the model's own norm) rmsnorm(x, w_last).  y [T, W] (rows may be strided), x [T, W] fp32.  Returns (input, x); the
+    CUDA body updates x in place."""
+    x = alpha * x + y.float()
+    x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    out = x if w_last is None else x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w_last.float()
+    return out.to(y.dtype), x
+
+
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float):
+    """The start of such a stream: x = scale * table[ids] in fp32, and its copy in the table's dtype.  Returns (input, x)."""
+    x = scale * table[ids.long()].float()
+    return x.to(table.dtype), x
+
+
 def layernorm(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: float) -> torch.Tensor:
     return F.layer_norm(x.float(), (x.shape[-1],), w.float(), None if b is None else b.float(), eps).to(x.dtype)
 
@@ -200,9 +216,15 @@ def dequant_fp8_block(q: torch.Tensor, s: torch.Tensor, block: int = 128) -> tor
     return q.float() * se
 
 
-def linear(x: torch.Tensor, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None) -> torch.Tensor:
-    """y = x @ w^T.  fp8 weights follow the DeepSeek recipe: activations quantised 1x128, fp32 accumulate."""
+def linear(x: torch.Tensor, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None, act: Optional[str] = None, act_from: int = 0) -> torch.Tensor:
+    """y = x @ w^T.  fp8 weights follow the DeepSeek recipe: activations quantised 1x128, fp32 accumulate.  `act` ("relu2": the square of relu,
+    "tanh"; not with fp8 weights or a bias): applied to the accumulators of the columns from `act_from` on, before the one rounding."""
     x = dense(x)
+    if act is not None:
+        assert w.dtype != FP8 and bias is None
+        y = F.linear(x.float(), w.float())
+        z = y[..., act_from:]
+        return torch.cat([y[..., :act_from], z.tanh() if act == "tanh" else F.relu(z).square()], -1).to(x.dtype)
     if w.dtype == FP8:
         xq, xs = quant_fp8_1x128(x.reshape(-1, x.shape[-1]))
         y = dequant_fp8_1x128(xq, xs) @ dequant_fp8_block(w, w_scale).t()
@@ -226,9 +248,9 @@ def yarn_mscale(scale: float, mscale: float) -> float:
     return 1.0 if scale <= 1 else 0.1 * mscale * math.log(scale) + 1.0
 
 
-def rope_inv_freq(dim: int, theta: float, scaling: Optional[dict]) -> Tuple[torch.Tensor, float]:
+def rope_inv_freq(dim: int, theta: float, scaling: Optional[dict], dtype=torch.float32) -> Tuple[torch.Tensor, float]:
     """Inverse frequencies (+ attention-magnitude factor) for plain RoPE and YaRN."""
-    inv = 1.0 / (theta ** (torch.arange(0, dim, 2, dtype=torch.float32) / dim))
+    inv = 1.0 / (theta ** (torch.arange(0, dim, 2, dtype=dtype) / dim))
     if not scaling or scaling.get("type", scaling.get("rope_type")) != "yarn":
         return inv, 1.0
     factor = float(scaling["factor"])
@@ -240,7 +262,7 @@ def rope_inv_freq(dim: int, theta: float, scaling: Optional[dict]) -> Tuple[torc
 
     low = max(math.floor(corr_dim(beta_fast)), 0)
     high = min(math.ceil(corr_dim(beta_slow)), dim - 1)
-    ramp = ((torch.arange(dim // 2, dtype=torch.float32) - low) / max(high - low, 1e-3)).clamp(0, 1)
+    ramp = ((torch.arange(dim // 2, dtype=dtype) - low) / max(high - low, 1e-3)).clamp(0, 1)
     inv_mask = 1.0 - ramp
     inv = inv / factor * (1 - inv_mask) + inv * inv_mask
     if scaling.get("attention_factor") is not None:            # the magnitude of cos and sin, given outright
@@ -249,11 +271,12 @@ def rope_inv_freq(dim: int, theta: float, scaling: Optional[dict]) -> Tuple[torc
     return inv, m
 
 
-def rope_cos_sin_cache(dim: int, max_pos: int, theta: float, scaling: Optional[dict] = None) -> torch.Tensor:
-    """[max_pos, dim] fp32: first half cos, second half sin (already multiplied by the YaRN magnitude)."""
-    inv, m = rope_inv_freq(dim, theta, scaling)
-    f = torch.outer(torch.arange(max_pos, dtype=torch.float32), inv)
-    return torch.cat([f.cos() * m, f.sin() * m], -1)
+def rope_cos_sin_cache(dim: int, max_pos: int, theta: float, scaling: Optional[dict] = None, exact: bool = False) -> torch.Tensor:
+    """[max_pos, dim] fp32: first half cos, second half sin (already multiplied by the YaRN magnitude).  `exact`: frequencies and angles in
+    64-bit, so that an entry is right to 32-bit however far its position."""
+    inv, m = rope_inv_freq(dim, theta, scaling, torch.float64 if exact else torch.float32)
+    f = torch.outer(torch.arange(max_pos, dtype=inv.dtype), inv)
+    return torch.cat([f.cos() * m, f.sin() * m], -1).float()
 
 
 def apply_rope(x: torch.Tensor, positions: torch.Tensor, cache: torch.Tensor, interleaved: bool) -> torch.Tensor:
@@ -320,6 +343,57 @@ def gqa_qkv_prepare(qkv: torch.Tensor, hq: int, hkv: int, hd: int, q_norm_w, k_n
     k = apply_rope(k.contiguous(), positions, rope_cache, False)
     keep = slot_mapping >= 0
     gqa_kv_store(k_cache, v_cache, slot_mapping[keep], k[keep], v[keep])
+    return q
+
+
+# ---- pooled rows --------------------------------------------------------------------------------------------
+def pooled_rows_per_page(pool: int, block_size: int) -> int:
+    """Pooled rows (means of `pool` tokens) a page has room for.  Eight neighbouring pooled rows are one group, kept together in the page of the
+    first token of its first block: a tile of pooled rows is whole groups, however `pool` and the page size divide."""
+    return -(-block_size // (8 * pool)) * 8
+
+
+def pooled_row_place(b: int, pool: int, block_size: int) -> Tuple[int, int]:
+    """(page of the sequence, row in that page's pooled rows) of pooled row b."""
+    g = b // 8
+    page = 8 * g * pool // block_size
+    return page, (g - -(-page * block_size // (8 * pool))) * 8 + b % 8
+
+
+def pooled_attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, q_norm: torch.Tensor, k_norm: torch.Tensor, eps: float, positions,
+                             key_table: torch.Tensor, value_table: torch.Tensor, k_cache, v_cache, k_pool, v_pool, pool: int, slots, block_tables,
+                             cu_seqlens, max_q_len: int = 0) -> torch.Tensor:
+    """What lies between the projection [T, q | k | v] and the attention over window and pooled blocks: RMS norm of q and of k over all heads
+    at once, rotation of the first key_table.shape[1] dims of every query and key head and of all dims of every value (pairs (i, i + half)),
+    key and value rows into the paged caches, and for every block of `pool` tokens that a token of this call completes the means of its
+    cached rows into the pooled rows of the page.  Returns q [T, H, D]; the CUDA body turns it in place.  `max_q_len`: planning hint."""
+    T = qkv.shape[0]
+    q, k, v = qkv.split([H * D, G * D, G * Dv], -1)
+    nd = key_table.shape[1]
+
+    def norm(x, w):
+        xf = x.float()
+        return xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+    def turn(x, table, n):
+        return torch.cat([apply_rope(x[..., :n], positions, table, False), x[..., n:]], -1)
+
+    q = turn(norm(q, q_norm).view(T, H, D), key_table, nd).to(qkv.dtype)
+    k = turn(norm(k, k_norm).view(T, G, D), key_table, nd).to(qkv.dtype)
+    v = turn(v.float().reshape(T, G, Dv), value_table, Dv).to(qkv.dtype)
+    kv_rows(k_cache, v_cache, slots, k.reshape(T, G * D), v.reshape(T, G * Dv))
+    bs, cu = k_cache.shape[1], cu_seqlens.tolist()
+    for s in range(len(cu) - 1):
+        for t in range(cu[s], cu[s + 1]):
+            p = int(positions[t])
+            if (p + 1) % pool or int(slots[t]) < 0:
+                continue
+            page, row = pooled_row_place(p // pool, pool, bs)
+            at = torch.arange(p - pool + 1, p + 1)
+            src = block_tables[s][(at // bs).to(block_tables.device)].long()
+            off = (at % bs).to(src.device)
+            for cache, dst in ((k_cache, k_pool), (v_cache, v_pool)):
+                dst[int(block_tables[s][page]), row] = cache[src, off].float().mean(0).to(cache.dtype)
     return q
 
 
@@ -398,14 +472,18 @@ def gqa_attention_paged(q, k_cache, v_cache, block_tables, cu_seqlens_q, context
 
 
 def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0, softcap: float = 0.0, slopes=None,
-                         gate=None, out_scale: float = 1.0, out=None, max_q_len: int = 0) -> torch.Tensor:
+                         gate=None, out_scale: float = 1.0, out=None, max_q_len: int = 0, pooled=None, pool: int = 0, turn_back=None) -> torch.Tensor:
     """Causal grouped-query attention over paged caches with per-layer options.  q [T, Hq, D] (token stride free), k_cache [blocks, block_size,
     Hkv, D], v_cache [..., Dv].  score = q.k scale, capped as softcap tanh(score / softcap) when softcap > 0, minus slopes[head] (query position
     - key position) when slopes [Hq] are given; `window` > 0: a query sees its own and the window - 1 keys before it.  Head h's output is
     multiplied by out_scale and, with gate [T, Hq], by sigmoid(gate[:, h]).  Writes into `out` [T, Hq * Dv] (rows may be strided) when given.
-    `max_q_len`: planning hint of the CUDA body."""
+    `max_q_len`: planning hint of the CUDA body.
+    `pooled` = (key rows, value rows) of blocks of `pool` tokens (`pooled_row_place`; with a window, without cap and slopes): a query at position
+    i also sees every block whose last token is at most i - window, in the same softmax.  `turn_back` [positions, Dv] (cos | sin): the output of
+    a query at position i is rotated by minus the angles of row i, pairs (m, m + Dv / 2), before the gate."""
     T, Hq, D = q.shape
     Hkv, Dv = k_cache.shape[2], v_cache.shape[3]
+    assert not pool or (window > 0 and softcap == 0 and slopes is None)
     o = torch.zeros(T, Hq, Dv, dtype=torch.float32, device=q.device)
     for i in range(cu_seqlens_q.numel() - 1):
         lo, hi = int(cu_seqlens_q[i]), int(cu_seqlens_q[i + 1])
@@ -423,7 +501,22 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
         s = s.masked_fill(dist < 0, float("-inf"))
         if window > 0:
             s = s.masked_fill(dist >= window, float("-inf"))
+        pos = torch.arange(n - ql, n, device=q.device)
+        nb = max(0, (n - window) // pool) if pool else 0
+        if nb:
+            at = [pooled_row_place(b, pool, k_cache.shape[1]) for b in range(nb)]
+            pages = block_tables[i][torch.tensor([p for p, _ in at], device=block_tables.device)].long()
+            rows = torch.tensor([r for _, r in at], device=pages.device)
+            kb, vb = (t[pages, rows].float().repeat_interleave(Hq // Hkv, 1) for t in pooled)
+            sb = torch.einsum("thd,nhd->thn", q[lo:hi].float(), kb) * scale
+            last = (torch.arange(nb, device=q.device) + 1) * pool - 1
+            sb = sb.masked_fill(last.view(1, 1, nb) > pos.view(ql, 1, 1) - window, float("-inf"))
+            s, v = torch.cat([s, sb], -1), torch.cat([v, vb], 0)
         o[lo:hi] = torch.einsum("thn,nhd->thd", torch.softmax(s, -1), v)
+        if turn_back is not None:
+            c, sn = (t.view(ql, 1, Dv // 2) for t in turn_back[pos].split(Dv // 2, -1))
+            a, b = o[lo:hi].split(Dv // 2, -1)
+            o[lo:hi] = torch.cat([a * c + b * sn, b * c - a * sn], -1)
     if gate is not None:
         o = o * torch.sigmoid(gate.float())[:, :, None]
     o = (o * out_scale).to(q.dtype).reshape(T, Hq * Dv)
@@ -1332,6 +1425,46 @@ def lightning_mix(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch
         return o.to(q.dtype)
     out.copy_(o)
     return out
+
+
+# ---- generalised delta rule ----------------------------------------------------------------------------------
+DECAY_RATE = math.exp(-0.5)      # largest decay rate per token of `general_delta`
+
+
+def general_delta_scan(r, k, v, w, a, S):
+    """S <- S diag(w) - (S u) (a u)^T + v k^T with u = k / sqrt(k.k + 1e-6), o = S r, token by token for one sequence in fp32.  r, k, w, a [n, H,
+    Dk], v [n, H, Dv], S [H, Dv, Dk].  Returns (o [n, H, Dv], S)."""
+    o = torch.empty_like(v)
+    u = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+    for t in range(r.shape[0]):
+        p = torch.einsum("hvk,hk->hv", S, u[t])
+        S = S * w[t][:, None, :] - p[:, :, None] * (a[t] * u[t])[:, None, :] + v[t][:, :, None] * k[t][:, None, :]
+        o[t] = torch.einsum("hvk,hk->hv", S, r[t])
+    return o, S
+
+
+def general_delta(proj: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor, a_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+                  cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, Dk: int, Dv: int, eps: float, max_q_len: int = 1) -> torch.Tensor:
+    """Generalised delta-rule mixer between its projections, 32-bit: proj [T, r | k | a | v | g (| anything)] (H Dk columns each for r, k, a, H Dv
+    for v, g), decay [T, >= H Dk] fp32.  Per key channel a decay exp(-DECAY_RATE sigmoid(decay + w0)) and a removal rate sigmoid(a + a_bias), then
+    `general_delta_scan` on `state` [S, H, Dv, Dk] fp32; per head o / rms(o), times norm_w [H Dv] and sigmoid(g).  Returns [T, H Dv] in proj's
+    dtype; any mix of sequence lengths.  `max_q_len`: planning hint of the CUDA body."""
+    T, nk, nv = proj.shape[0], H * Dk, H * Dv
+    r, k, a, v, g = (t.float() for t in proj[:, : 3 * nk + 2 * nv].split([nk, nk, nk, nv, nv], -1))
+    w = torch.exp(-DECAY_RATE * torch.sigmoid(decay[:, :nk].float() + w0)).view(T, H, Dk)
+    a = torch.sigmoid(a + a_bias).view(T, H, Dk)
+    r, k, v = r.reshape(T, H, Dk), k.reshape(T, H, Dk), v.reshape(T, H, Dv)
+    o = torch.empty(T, H, Dv, dtype=torch.float32, device=proj.device)
+    cu = cu_seqlens.tolist()
+    for i in range(len(cu) - 1):
+        s, e = cu[i], cu[i + 1]
+        if e <= s:
+            continue
+        slot = int(slots[i])
+        S = torch.zeros_like(state[slot]) if int(fresh[i]) else state[slot].clone()
+        o[s:e], state[slot] = general_delta_scan(r[s:e], k[s:e], v[s:e], w[s:e], a[s:e], S)
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    return (o.reshape(T, nv) * norm_w.float() * torch.sigmoid(g)).to(proj.dtype)
 
 
 # ---- MTP draft verification -------------------------------------------------------------------------------

@@ -14,12 +14,14 @@ DeepSeek-V4        one shared key / value row per token and layer in the latent-
                    compressor's carry [c * ratio, c * head_dim] fp32 twice (values and scores; c = 2 for ratio 4).  With an fp8 cache a row
                    is 584 packed bytes (448 e4m3 values, 64 bf16 rotated dims, 7 scale bytes + pad) instead of head_dim values.
 
-listed layers      families that list their layers one by one (Tuvutar, Filasun) may give every layer its own row widths and state shape:
+listed layers      families that list their layers one by one (Tuvutar, Filasun, Sapanex) may give every layer its own row widths and state shape:
                    one tensor per layer instead of the stacked ones - latent rows [blocks, block_size, D_l], or keys [blocks, block_size,
                    G_l, D_l] and values [.., G_l, Dv_l]; states [slots, Hv_l, Dv_l, Dk_l] fp32 and convolution windows [slots, K_l - 1,
-                   conv_dim_l].  Page families `latent_<n>` or `key_<n>` / `value_<n>`, slot families `delta_state_<n>` / `delta_conv_<n>`.  A
+                   conv_dim_l].  Page families `latent_<n>` or `key_<n>` / `value_<n>` (and `pooled_key_<n>` / `pooled_value_<n>`), slot families `delta_state_<n>` / `delta_conv_<n>`.  A
                    layer may own rows, a state, both (attention and linear attention side by side) or neither (it reads an earlier layer's
-                   rows); rows and states are numbered separately.
+                   rows); rows and states are numbered separately.  A layer that pools adds the means of blocks of P tokens, keys
+                   [blocks, R, G_l, D_l] and values [blocks, R, G_l, Dv_l]: eight neighbouring pooled rows sit together in the page of the
+                   first token of their first block (`ops.reference.pooled_rows_per_page`), so R = 8 for P >= 8.
 
 One extra block past the scheduler-visible range is reserved as the scratch page that dummy batches of idle
 DP ranks write into.
@@ -76,6 +78,7 @@ class CachePlan:
     latent_rows: Optional[List[int]] = None
     kv_shapes: Optional[List[tuple]] = None
     delta_shapes: Optional[List[tuple]] = None
+    pools: Optional[List[int]] = None          # tokens per pooled row of every layer in kv_shapes (0: the layer does not pool)
     hisparse: bool = False
     hot_rows: int = 0
     hs_slots: int = 0
@@ -89,6 +92,16 @@ class CachePlan:
     def listed(self) -> bool:
         """One cache tensor per layer, page id in front."""
         return self.latent_rows is not None or self.kv_shapes is not None
+
+    @property
+    def pooled(self) -> bool:
+        return any(self.pools or [])
+
+    def pooled_rows(self, layer: int) -> int:
+        """Pooled rows of a page of one kv_shapes layer."""
+        from ..ops.reference import pooled_rows_per_page
+        p = self.pools[layer] if self.pools else 0
+        return pooled_rows_per_page(p, self.block_size) if p else 0
 
     @property
     def needs_state_slots(self) -> bool:
@@ -121,7 +134,7 @@ class CachePlan:
         if self.latent_rows is not None:
             return self.block_size * sum(self.latent_rows) * e
         if self.kv_shapes is not None:
-            return self.block_size * sum(g * (d + dv) for g, d, dv in self.kv_shapes) * e
+            return sum((self.block_size + self.pooled_rows(l)) * g * (d + dv) for l, (g, d, dv) in enumerate(self.kv_shapes)) * e
         if self.mla:
             return self.num_layers * self.block_size * self.row_dim * e
         return 2 * self.num_layers * self.block_size * self.kv_heads_local * self.row_dim * e
@@ -149,6 +162,8 @@ class CachePlan:
         bits = C.PLAN_MLA if self.mla else C.PLAN_GQA
         if self.indexer:
             bits |= C.PLAN_INDEXER
+        if self.pooled:
+            bits |= C.PLAN_CSA          # pooled rows of one page cover tokens of later ones: no prefix reuse
         if self.gdn:
             bits |= C.PLAN_GDN          # one state slot per running sequence; no prefix reuse
         if self.hisparse:
@@ -185,7 +200,9 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
         own = [i for i in range(n) if mc.keeps_rows(i)]
         if not mc.is_mla:
             mixers = [mc.layer_specs[i] for i in range(n)]
-            kv = [(int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])) for m in (mixers[i]["mixer"]["left"] for i in own)]
+            rows = [mixers[i]["mixer"].get("left", mixers[i]["mixer"]) for i in own]
+            kv = [(int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])) for m in rows]
+            pools = [int(m["mask"].get("pool") or 0) for m in rows]
             shapes = []
             for s in mixers:
                 m = s["mixer"]
@@ -194,8 +211,10 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
                 elif s["type"] == "parallel":
                     r = m["right"]
                     shapes.append((int(r["heads"]), int(r["vdim"]), int(r["dim"]), 1, 0))
+                elif s["type"] == "general_delta":
+                    shapes.append((int(m["heads"]), int(m["dim"]), int(m["dim"]), 1, 0))
             return CachePlan(False, True, False, len(kv), block_size, dt, max((d for _, d, _ in kv), default=0), gdn=bool(shapes), gdn_layers=len(shapes),
-                             state_slots=state_slots, kv_shapes=kv, delta_shapes=shapes)
+                             state_slots=state_slots, kv_shapes=kv, delta_shapes=shapes, pools=pools)
         rows = [mc.layer_config(i).mla_cache_dim for i in own]
         cfgs = [mc.layer_config(i) for i in range(n) if mc.layer_type(i) == "linear_attention"]
         shapes = [(c.linear_num_value_heads, c.linear_value_head_dim, c.linear_key_head_dim, c.linear_conv_kernel_dim, c.gdn_conv_dim) for c in cfgs]
@@ -245,7 +264,9 @@ class KVCache:
             self.layers: List = [torch.zeros(nb, plan.block_size, d, dtype=sdt, device=device).view(plan.kv_dtype) for d in plan.latent_rows]
         elif plan.kv_shapes is not None:
             self.kv = None
-            self.layers = [tuple(torch.zeros(nb, plan.block_size, g, w, dtype=plan.kv_dtype, device=device) for w in (d, dv)) for g, d, dv in plan.kv_shapes]
+            # (keys, values) of every layer, with (pooled keys, pooled values) behind them where the layer pools
+            self.layers = [tuple(torch.zeros(nb, r, g, w, dtype=plan.kv_dtype, device=device) for r in (plan.block_size, plan.pooled_rows(l)) if r for w in (d, dv))
+                           for l, (g, d, dv) in enumerate(plan.kv_shapes)]
         elif plan.mla:
             # under the hot / cold tier the logical pages are the cold tier: pinned host memory the staging kernel reads
             # through the unified address space
@@ -319,7 +340,8 @@ class KVCache:
         if self.plan.latent_rows is not None:
             return [fam(f"latent_{l}", t, 1) for l, t in enumerate(self.layers)]
         if self.plan.kv_shapes is not None:
-            return [fam(f"{name}_{l}", t, 1) for l, pair in enumerate(self.layers) for name, t in zip(("key", "value"), pair)]
+            return [fam(f"{name}_{l}", t, 1) for l, parts in enumerate(self.layers)
+                    for name, t in zip(("key", "value", "pooled_key", "pooled_value"), parts)]
         out = [fam("mla_kv" if self.plan.mla else "gqa_kv", self.kv, self.kv.shape[0] if self.plan.mla else 2 * self.kv.shape[1])]
         if self.indexer is not None:
             out.append(fam("indexer", self.indexer, self.indexer.shape[0]))
