@@ -9,10 +9,13 @@
 // physical slots (sparse, -1 = skip).  Cache dtype bf16, e4m3 (query is then clamped and cast to e4m3 as well) or fp32 (query and
 // output fp32 too: runs in true 32-bit).  Options: a window of the last keys, scores capped as cap tanh(s / cap), a distance bias
 // -slope[head] (query position - key position) after the cap, the output of a head times sigmoid(gate[token, head]) and a constant.
+// With pooled rows (pooled.cuh) a query also sees the blocks wholly in front of its window, in the same softmax; an output may be rotated back by
+// its position (pairs of columns d, d + Dv / 2).
 //
 // Replaces in the reference: attention/base.py:451-525 (SDPA reference), flash_mla sparse decode call sites
 // (layers/backends/mla/flash_mla.py:22-121) for the sparse case, flashinfer / FA paged GQA wrappers.
 #include "ptx.cuh"
+#include "pooled.cuh"
 #include <cstring>
 
 namespace ne {
@@ -37,6 +40,8 @@ struct AttnArgs {
   long long v_slot_stride; int v_head_stride;     // of the separate V rows
   float softcap; const float* slopes;             // 0 / null: none
   const void* gate; long long gate_ld; float out_scale;      // gate null: none
+  const void* k_pool; const void* v_pool; int pool, pool_rows;      // pool 0: none
+  const float* turn; int n_pos;                              // [n_pos, Dv] cos | sin, or null
 };
 
 // kind: 0 bf16, 1 e4m3, 2 fp32
@@ -85,23 +90,33 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
   const float c = a.scale * kLog2e, slope = (a.slopes && head_ok) ? a.slopes[h] : 0.f;
   const int* bt = a.block_tables + (long long)seq * a.bt_stride;
 
-  for (int k0 = first_key / kKeysPerTile * kKeysPerTile; k0 < n_keys; k0 += kKeysPerTile) {
+  const int n_pool = a.pool ? pooled_visible(limit, a.window, a.pool) : 0, pool_tiles = (n_pool + kKeysPerTile - 1) / kKeysPerTile;
+  const int tile0 = first_key / kKeysPerTile, tiles = pool_tiles + max(0, (n_keys + kKeysPerTile - 1) / kKeysPerTile - tile0);
+  for (int it = 0; it < tiles; it++) {
+    const bool pooled = it < pool_tiles;
+    const int k0 = (pooled ? it : it - pool_tiles + tile0) * kKeysPerTile, k_end = pooled ? n_pool : n_keys, k_first = pooled ? 0 : first_key;
+    const void *kbase = pooled ? a.k_pool : a.k_cache, *vbase = pooled ? a.v_pool : a.v_cache;
     __syncthreads();
     // stage 32 key rows (and value rows) as fp32
     for (int r = warp; r < kKeysPerTile; r += 4) {
       int kidx = k0 + r;
       long long slot = -1;
-      if (kidx < n_keys) {
-        if (a.sparse) slot = a.sparse[(long long)t * a.topk + kidx];
+      if (kidx < k_end) {
+        if (pooled) {
+          int page, row;
+          pooled_place(kidx, a.pool, a.block_size, page, row);
+          page = bt[page];
+          slot = NE_INDEX_OK(page, BK_CACHE_PAGES, 24, __LINE__) ? (long long)page * a.pool_rows + row : -1;
+        } else if (a.sparse) slot = a.sparse[(long long)t * a.topk + kidx];
         else {
           const int page = bt[kidx / a.block_size];
           slot = (a.block_size == 1 || NE_INDEX_OK(page, BK_CACHE_PAGES, 23, __LINE__)) ? (long long)page * a.block_size + kidx % a.block_size : -1;
         }
       }
       for (int d = lane; d < Dk; d += 32)
-        sk[r * (Dk + 1) + d] = slot >= 0 ? load_kv(a.k_cache, slot * a.kv_slot_stride + (long long)kvh * a.kv_head_stride + d, a.fp8) : 0.f;
+        sk[r * (Dk + 1) + d] = slot >= 0 ? load_kv(kbase, slot * a.kv_slot_stride + (long long)kvh * a.kv_head_stride + d, a.fp8) : 0.f;
       if (sv) for (int d = lane; d < Dv; d += 32)
-        sv[r * (Dv + 1) + d] = slot >= 0 ? load_kv(a.v_cache, slot * a.v_slot_stride + (long long)kvh * a.v_head_stride + d, a.fp8) : 0.f;
+        sv[r * (Dv + 1) + d] = slot >= 0 ? load_kv(vbase, slot * a.v_slot_stride + (long long)kvh * a.v_head_stride + d, a.fp8) : 0.f;
       if (lane == 0) sk[r * (Dk + 1) + Dk] = slot >= 0 ? 1.f : 0.f;   // validity marker in the padding column
     }
     __syncthreads();
@@ -111,7 +126,7 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
     const float* qr = sq + warp * Dk;
     float s = 0.f;
     for (int d = 0; d < Dk; d++) s = fmaf(qr[d], kr[d], s);
-    bool valid = (k0 + lane < n_keys) && (k0 + lane >= first_key) && kr[Dk] != 0.f;
+    bool valid = (k0 + lane < k_end) && (k0 + lane >= k_first) && kr[Dk] != 0.f;
     float tl = s * c;
     if (a.softcap > 0.f) tl = a.softcap * tanhf(s * a.scale / a.softcap) * kLog2e;
     if (a.slopes) tl -= slope * (float)(limit - (k0 + lane)) * kLog2e;
@@ -136,9 +151,26 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
       }
     }
   }
+  if (a.turn) __syncthreads();                 // the tiles' memory is free
   if (!head_ok) return;
   float inv = (l_run > 0.f ? 1.f / l_run : 0.f) * a.out_scale;
   if (a.gate) inv /= 1.f + expf(-load_kv(a.gate, (long long)t * a.gate_ld + h, a.fp8 == 2 ? 2 : 0));
+  if (a.turn) {
+    float* so = sk + warp * Dv;                // a value of the pair sits in another lane
+#pragma unroll
+    for (int j = 0; j < 20; j++) { const int d = lane + 32 * j; if (j < per_lane && d < Dv) so[d] = acc[j]; }
+    __syncwarp();
+    const int half = Dv >> 1;
+    const float* tab = a.turn + (long long)min(max(limit, 0), a.n_pos - 1) * Dv;
+#pragma unroll
+    for (int j = 0; j < 20; j++) {
+      const int d = lane + 32 * j;
+      if (j < per_lane && d < Dv) {
+        const int m = d < half ? d : d - half;
+        acc[j] = d < half ? acc[j] * tab[m] + so[d + half] * tab[half + m] : acc[j] * tab[m] - so[m] * tab[half + m];
+      }
+    }
+  }
 #pragma unroll
   for (int j = 0; j < 20; j++) {
     int d = lane + 32 * j;
@@ -233,6 +265,7 @@ __global__ void __launch_bounds__(1024) sample_kernel(const float* __restrict__ 
 using namespace ne;
 
 static int attn_generic_launch(AttnArgs& a, cudaStream_t st) {
+  // (the way out of a rotated output, kHeadsPerCta rows of Dv, fits in the tiles of 32 keys and values)
   const size_t smem = sizeof(float) * ((size_t)kHeadsPerCta * a.Dk + (size_t)kKeysPerTile * (a.Dk + 1) + (a.v_cache ? (size_t)kKeysPerTile * (a.Dv + 1) : 0));
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
@@ -245,12 +278,14 @@ static int attn_generic_launch(AttnArgs& a, cudaStream_t st) {
 
 // Paged grouped-query attention with the options of AttnArgs: q [T, H, D], k_cache [slots, Hkv, D], v_cache [slots, Hkv, Dv] (fp32 all of
 // them when fp32 = 1, else bf16), slopes [H] or null, gate [T, >= H] (row stride gate_ld) or null, out [T, ...] with row stride o_ld and head
-// stride Dv.  window 0: all earlier keys.
+// stride Dv.  window 0: all earlier keys.  pool > 0: pooled rows k_pool [pages, pool_rows, Hkv, D], v_pool [.., Dv] in front of the window.
 extern "C" int ne_attn_biased(const void* q, long long q_ld, const void* k_cache, const void* v_cache, const int* block_tables, int bt_stride, int block_size,
                               const int* cu_seqlens_q, const int* context_lens, int num_seqs, void* out, long long o_ld, int T, int H, int Hkv, int D, int Dv,
                               float scale, float softcap, const float* slopes, int window, const void* gate, long long gate_ld, float out_scale, int fp32,
-                              cudaStream_t st) {
+                              const void* k_pool, const void* v_pool, int pool, int pool_rows, const float* turn, int n_pos, cudaStream_t st) {
   if (T <= 0) return 0;
+  if (pool > 0 && (window < 1 || softcap > 0.f || slopes || !k_pool || !v_pool || pool_rows < (block_size + 8 * pool - 1) / (8 * pool) * 8)) return 1004;
+  if (turn && (n_pos < 1 || Dv % 2)) return 1005;
   if (Hkv < 1 || H % Hkv || Dv < 1 || Dv > 640 || D < 1 || D > 640) return 1001;
   AttnArgs a;
   memset(&a, 0, sizeof(a));
@@ -258,7 +293,8 @@ extern "C" int ne_attn_biased(const void* q, long long q_ld, const void* k_cache
   a.v_slot_stride = (long long)Hkv * Dv; a.v_head_stride = Dv; a.kv_group = H / Hkv; a.block_tables = block_tables; a.bt_stride = bt_stride;
   a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs; a.out = out; a.o_tok_stride = o_ld;
   a.o_head_stride = Dv; a.T = T; a.H = H; a.Dk = D; a.Dv = Dv; a.scale = scale; a.fp8 = fp32 ? 2 : 0; a.window = window; a.softcap = softcap; a.slopes = slopes;
-  a.gate = gate; a.gate_ld = gate_ld; a.out_scale = out_scale;
+  a.gate = gate; a.gate_ld = gate_ld; a.out_scale = out_scale; a.k_pool = k_pool; a.v_pool = v_pool; a.pool = pool > 0 ? pool : 0; a.pool_rows = pool_rows;
+  a.turn = turn; a.n_pos = n_pos;
   for (a.heads_per_cta = kHeadsPerCta; a.kv_group % a.heads_per_cta; a.heads_per_cta--) {}
   return attn_generic_launch(a, st);
 }

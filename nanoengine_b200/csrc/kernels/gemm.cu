@@ -62,6 +62,12 @@ struct GemmComm {
   int* tail_advance;
 };
 
+// tanh as 1 - 2 / (e^2x + 1): the hardware's own is coarser than a bf16 result
+__device__ __forceinline__ float epi_act(float v, int act) {
+  if (act == 1) { v = fmaxf(v, 0.f); return v * v; }
+  return 1.f - __fdividef(2.f, 1.f + __expf(fminf(2.f * v, 60.f)));
+}
+
 struct GemmArgs {
   int M, N, K, groups;
   const int* masked_m;                  // [groups] valid rows per group, or nullptr (all M rows valid)
@@ -77,6 +83,7 @@ struct GemmArgs {
   const long long* row_dst;             // optional scatter epilogue: absolute address of every output row (bf16, may be peer memory),
   long long rd_group_stride;            // indexed [group * rd_group_stride + row]; used by the MoE combine
   const float* bias;                    // optional [N]: added to the fp32 accumulator before the result is rounded (plain bf16 GEMMs)
+  int act, act_from;                    // 1 square of relu, 2 tanh: applied to the fp32 accumulators of the columns from act_from on (plain bf16 GEMMs)
   GemmComm comm;                        // hooks that fuse a collective into this GEMM (all null / zero for a plain GEMM)
 };
 
@@ -838,6 +845,11 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               for (int j = 0; j < 8; j++) r[q * 8 + j] = __float_as_uint(__uint_as_float(r[q * 8 + j]) + b[j]);
             }
           }
+          if (!kFP8 && !kSplit && args.act && n0 + c * 32 + 32 > args.act_from) {
+#pragma unroll
+            for (int j = 0; j < 32; j++)
+              if (n0 + c * 32 + j >= args.act_from) r[j] = __float_as_uint(epi_act(__uint_as_float(r[j]), args.act));
+          }
           if (kSplit) {
             float4* P = reinterpret_cast<float4*>(smem);
 #pragma unroll
@@ -902,6 +914,12 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
         if (args.bias) {
           const float4 b = __ldg(reinterpret_cast<const float4*>(args.bias + n));
           s4.x += b.x; s4.y += b.y; s4.z += b.z; s4.w += b.w;
+        }
+        if (!kFP8 && args.act && n + 4 > args.act_from) {
+          if (n >= args.act_from) s4.x = epi_act(s4.x, args.act);
+          if (n + 1 >= args.act_from) s4.y = epi_act(s4.y, args.act);
+          if (n + 2 >= args.act_from) s4.z = epi_act(s4.z, args.act);
+          s4.w = epi_act(s4.w, args.act);
         }
         const long long off = (long long)grow * args.ldd + n;
         if (args.out_fp32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(args.D) + off) = s4;
@@ -1099,9 +1117,10 @@ using namespace ne;
 static int gemm_impl(const void* A, long long lda, long long a_gs, const void* B, void* D, long long ldd, long long d_gs,
                      int M, int N, int K, int groups, const int* masked_m, const int* row_start, int dtype, const float* sa, int sa_ld,
                      long long sa_gs, const float* sb, int out_fp32, int block_n_hint, const long long* row_dst, const GemmComm* comm,
-                     int a_rows_total, cudaStream_t stream, const float* bias = nullptr) {
+                     int a_rows_total, cudaStream_t stream, const float* bias = nullptr, int act = 0, int act_from = 0) {
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
   if (bias && (dtype != 0 || groups != 1 || ((uintptr_t)bias & 15))) return 1012;
+  if (act < 0 || act > 2 || (act && (dtype != 0 || groups != 1))) return 1013;
   if (comm) {
     if (comm->wait_flags && (groups > kSchedCache || comm->wait_world > 16 || !masked_m)) return 1007;
     if (comm->gate_flags && (groups != 1 || row_start || masked_m || comm->gate_world > 16 || comm->gate_rpr < 1)) return 1008;
@@ -1180,7 +1199,7 @@ static int gemm_impl(const void* A, long long lda, long long a_gs, const void* B
   if (row_start) { a.d_group_stride = 0; sa_gs = 0; if (!masked_m) return 1004; }
   a.sa = sa; a.sa_ld = sa_ld; a.sa_group_stride = sa_gs; a.sb = sb;
   a.sb_group_stride = (long long)((N + 127) / 128) * (K / 128); a.out_fp32 = out_fp32; a.alpha = nullptr;
-  a.row_dst = row_dst; a.rd_group_stride = row_start ? 0 : M; a.bias = bias;
+  a.row_dst = row_dst; a.rd_group_stride = row_start ? 0 : M; a.bias = bias; a.act = act; a.act_from = act_from;
   if (row_dst && out_fp32) return 1005;
   if (comm) { a.comm = *comm; if (m_blocks <= 1 || groups != 1) a.comm.mb_rot = 0; else a.comm.mb_rot %= m_blocks; }
   else memset(&a.comm, 0, sizeof(a.comm));
@@ -1238,6 +1257,13 @@ extern "C" int ne_gemm(const void* A, long long lda, long long a_gs, const void*
 extern "C" int ne_gemm_bias(const void* A, long long lda, const void* B, const float* bias, void* D, long long ldd, int M, int N, int K, int out_fp32,
                             cudaStream_t stream) {
   return gemm_impl(A, lda, 0, B, D, ldd, 0, M, N, K, 1, nullptr, nullptr, 0, nullptr, 0, 0, nullptr, out_fp32, 0, nullptr, nullptr, 0, stream, bias);
+}
+
+// One dense bf16 GEMM whose columns from act_from on pass an activation (1 square of relu, 2 tanh) before they are rounded.
+extern "C" int ne_gemm_act(const void* A, long long lda, const void* B, void* D, long long ldd, int M, int N, int K, int act, int act_from, int out_fp32,
+                           cudaStream_t stream) {
+  return gemm_impl(A, lda, 0, B, D, ldd, 0, M, N, K, 1, nullptr, nullptr, 0, nullptr, 0, 0, nullptr, out_fp32, 0, nullptr, nullptr, 0, stream, nullptr, act,
+                   act_from);
 }
 
 // The same GEMM with a collective fused in (see GemmComm).  `a_rows_total` > 0 gives the number of rows the A tensor map must

@@ -16,7 +16,7 @@ constexpr int kTile = 64, kTileK = 16;
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* __restrict__ A, long long lda, long long a_bs, const TI* __restrict__ B, long long ldb,
                                                        long long b_bs, TO* __restrict__ D, long long ldd, long long d_bs, int M, int N, int K,
-                                                       const float* __restrict__ bias) {
+                                                       const float* __restrict__ bias, int act, int act_from) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   __shared__ float sA[kTileK][kTile + 4], sB[kTileK][kTile + 4];
   A += blockIdx.z * a_bs; B += blockIdx.z * b_bs; D += blockIdx.z * d_bs;
@@ -46,15 +46,18 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* __restrict__ A
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (m < M && n < N) st_f(D + (long long)m * ldd + n, bias ? acc[i][j] + bias[n] : acc[i][j]);
+      if (m >= M || n >= N) continue;
+      float v = bias ? acc[i][j] + bias[n] : acc[i][j];
+      if (act && n >= act_from) { if (act == 1) { v = fmaxf(v, 0.f); v *= v; } else v = tanhf(v); }
+      st_f(D + (long long)m * ldd + n, v);
     }
 }
 
 template <typename TI, typename TO>
 static int simt(const void* A, long long lda, long long a_bs, const void* B, long long ldb, long long b_bs, void* D, long long ldd, long long d_bs,
-                int M, int N, int K, int batch, const float* bias, cudaStream_t st) {
+                int M, int N, int K, int batch, const float* bias, int act, int act_from, cudaStream_t st) {
   const dim3 grid((unsigned)((N + kTile - 1) / kTile), (unsigned)((M + kTile - 1) / kTile), (unsigned)batch);
-  return (int)launch_pdl(gemm_simt_kernel<TI, TO>, grid, dim3(256), 0, st, (const TI*)A, lda, a_bs, (const TI*)B, ldb, b_bs, (TO*)D, ldd, d_bs, M, N, K, bias);
+  return (int)launch_pdl(gemm_simt_kernel<TI, TO>, grid, dim3(256), 0, st, (const TI*)A, lda, a_bs, (const TI*)B, ldb, b_bs, (TO*)D, ldd, d_bs, M, N, K, bias, act, act_from);
 }
 
 }  // namespace ne
@@ -62,12 +65,13 @@ static int simt(const void* A, long long lda, long long a_bs, const void* B, lon
 using namespace ne;
 
 // A [batch, M, K] (row stride lda, batch stride a_bs, elements), B [batch, N, K], D [batch, M, N].  in_fp32 / out_fp32: element types
-// of the operands and of the result (bf16 otherwise).  bias (fp32 [N] or null) is added before the result is rounded.
+// of the operands and of the result (bf16 otherwise).  bias (fp32 [N] or null) is added before the result is rounded; then act (0 none,
+// 1 square of relu, 2 tanh) on the columns from act_from on.
 extern "C" int ne_gemm_simt(const void* A, long long lda, long long a_bs, const void* B, long long ldb, long long b_bs, void* D, long long ldd,
-                            long long d_bs, int M, int N, int K, int batch, int in_fp32, int out_fp32, const float* bias, cudaStream_t st) {
+                            long long d_bs, int M, int N, int K, int batch, int in_fp32, int out_fp32, const float* bias, int act, int act_from, cudaStream_t st) {
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
   if (K < 0 || batch > 65535 || (M + kTile - 1) / kTile > 65535) return 1001;
-  if (in_fp32) return out_fp32 ? simt<float, float>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, st) : 1002;
-  return out_fp32 ? simt<__nv_bfloat16, float>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, st)
-                  : simt<__nv_bfloat16, __nv_bfloat16>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, st);
+  if (in_fp32) return out_fp32 ? simt<float, float>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, act, act_from, st) : 1002;
+  return out_fp32 ? simt<__nv_bfloat16, float>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, act, act_from, st)
+                  : simt<__nv_bfloat16, __nv_bfloat16>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, act, act_from, st);
 }

@@ -16,8 +16,12 @@
 // (own maximum, sum and accumulator) are folded at the end.
 // Warp 0: TMA producer, warp 1: MMA issuer, warps 2-5: softmax / rescale / epilogue (those that own rows of the tile).  All waits are
 // bounded.  Two CTAs share an SM where the tiles are small enough: one's softmax runs beside the other's products and copies.
+// kExt: (1) beside the window a row sees the pooled rows (pooled.cuh) of blocks wholly in front of it: tiles of 64 pooled rows, fetched as eight
+// groups of eight, come before the window's pages, in one softmax; (2) a row's output is rotated back by its position (pairs of columns m, m + Dv / 2)
+// on its way out, through shared memory.
 // With more than one slice the CTA writes a normalised partial result and its log2-sum-exp; gqa_biased_merge folds them and applies the gate.
 #include "ptx.cuh"
+#include "pooled.cuh"
 #include "seq_tile.cuh"
 #include "tma_host.h"
 
@@ -40,15 +44,19 @@ struct GbArgs {
   const __nv_bfloat16* gate; long long gate_ld; float out_scale;
   __nv_bfloat16* out; long long o_ld;          // row t, head h: out + t o_ld + h Dv (splits == 1)
   float* part; float* lse2;                    // [splits, T, H, Dv], [splits, T, H] (splits > 1)
+  int pool;                                    // kExt: tokens per pooled row (0: none)
+  const float* turn; int n_pos;                // kExt: [n_pos, Dv] cos | sin, or null
+  int bar_off;                                 // where the barriers lie in shared memory
 };
 
 __device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ld, long long t, int h, float scale) {
   return gate ? scale / (1.f + __expf(-__bfloat162float(gate[t * ld + h]))) : scale;
 }
 
-template <bool kCap, bool kRep>
+template <bool kCap, bool kRep, bool kExt>
 __global__ void __launch_bounds__(kGbThreads, 2)
-gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const GbArgs a) {
+gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
+                  const __grid_constant__ CUtensorMap kp_map, const __grid_constant__ CUtensorMap vp_map, const GbArgs a) {
   pdl_wait();                     // dependent launch: nothing above this line touches global memory
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw;      // swizzled tiles need 1024-byte alignment: the dynamic allocation starts on such a boundary
@@ -57,7 +65,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   uint8_t* sQ = smem;                                    // nc chunks of rows8 x 128 B
   uint8_t* sP = sQ + a.nc * q_chunk;
   uint8_t* sKV = sP + a.pbufs * p_bytes;                 // MMA reads of rows past rows8 end inside the page tiles
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sKV + a.stages * stage_bytes);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + a.bar_off);
   // q_full | kv_full[4] | kv_empty[4] | s_full[2] | s_empty[2] | p_full[2] | p_empty[2]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -91,6 +99,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   const int seq = s_tile[0], tok0 = s_tile[1];
 
   int n_tiles = 0, pg_begin = 0, n_tok = 0, base_limit = -1;
+  int n_pt = 0, n_pool = 0, pt_first = 0;                // tiles of pooled rows in front of the pages, pooled rows visible to the tile's last token
   const int* bt = a.block_tables;
   if (seq >= 0) {
     const int q_beg = a.cu_seqlens_q[seq], q_len = a.cu_seqlens_q[seq + 1] - q_beg;
@@ -98,10 +107,13 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     base_limit = a.context_lens[seq] - q_len + (tok0 - q_beg);              // last key visible to the tile's first token
     const int max_limit = base_limit + n_tok - 1;
     const int first = a.window > 0 ? max(0, base_limit - a.window + 1) / kBPage : 0;
-    const int total = max_limit >= 0 ? max_limit / kBPage + 1 - first : 0;
+    if (kExt && a.pool) { n_pool = pooled_visible(max_limit, a.window, a.pool); n_pt = (n_pool + kBPage - 1) / kBPage; }
+    const int pages = max_limit >= 0 ? max_limit / kBPage + 1 - first : 0, total = pages + n_pt;
     const int per_split = (total + a.splits - 1) / a.splits;
-    pg_begin = first + split * per_split;
-    n_tiles = max(0, min(first + total, pg_begin + per_split) - pg_begin);
+    pg_begin = first - n_pt + split * per_split;                            // tiles of pooled rows count as the n_pt pages in front of the first one
+    n_tiles = max(0, min(first + pages, pg_begin + per_split) - pg_begin);
+    n_pt = max(0, first - pg_begin);                                        // those of this slice
+    pt_first = split * per_split;
     bt = a.block_tables + (long long)seq * a.bt_stride;
   }
 
@@ -115,6 +127,21 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         const int s = i % a.stages;
         if (!mbar_wait(b_kvempty + 8 * s, ((i / a.stages) & 1) ^ 1, abort_flag, kKernelGb, 100 + s)) break;
         uint8_t* dst = sKV + s * stage_bytes;
+        if (kExt && i < n_pt) {
+          int page[8], prow[8];
+#pragma unroll
+          for (int j = 0; j < 8; j++) pooled_group(min((pt_first + i) * 8 + j, (n_pool - 1) >> 3), a.pool, kBPage, page[j], prow[j]);      // past the last: masked
+#pragma unroll
+          for (int j = 0; j < 8; j++) { page[j] = bt[page[j]]; if (!NE_INDEX_OK(page[j], BK_CACHE_PAGES, kKernelGb, __LINE__)) page[j] = 0; }
+          mbar_expect_tx(b_kvfull + 8 * s, stage_bytes);
+          for (int c = 0; c < a.nc; c++)
+#pragma unroll
+            for (int j = 0; j < 8; j++) tma_load_4d(smem_u32(dst + c * kBChunk + j * 1024), &kp_map, b_kvfull + 8 * s, c * 64, hkv, prow[j], page[j]);
+          for (int c = 0; c < a.nv; c++)
+#pragma unroll
+            for (int j = 0; j < 8; j++) tma_load_4d(smem_u32(dst + (a.nc + c) * kBChunk + j * 1024), &vp_map, b_kvfull + 8 * s, c * 64, hkv, prow[j], page[j]);
+          continue;
+        }
         int block = bt[pg_begin + i];
         if (!NE_INDEX_OK(block, BK_CACHE_PAGES, kKernelGb, __LINE__)) block = 0;      // a bad page id reads page 0
         mbar_expect_tx(b_kvfull + 8 * s, stage_bytes);
@@ -177,6 +204,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int kfirst = kRep ? wq * 16 : 0;
     const int limit = row_ok ? base_limit + tl : -1;          // this row's last visible key
     const int lowest = (row_ok && a.window > 0) ? limit - a.window + 1 : 0;
+    const int pool_last = kExt && a.pool ? pooled_visible(limit, a.window, a.pool) - 1 : -1;      // last visible pooled row
     const float slope = (row_ok && a.slopes) ? __ldg(a.slopes + head) * kLog2e : 0.f;
     const float c_in = kCap ? a.scale / a.softcap * (2.f * kLog2e) : a.scale * kLog2e, c_cap = a.softcap * kLog2e;
     float m_run = -INFINITY, l_run = 0.f;
@@ -198,7 +226,9 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       tc_fence_before();
       __syncwarp();
       if (lane_id() == 0) mbar_arrive(b_sempty + 8 * sb);
-      const int key0 = (pg_begin + i) * kBPage + kfirst;
+      const bool pooled = kExt && i < n_pt;
+      const int key0 = (pooled ? pt_first + i : pg_begin + i) * kBPage + kfirst;
+      const int hi = pooled ? pool_last : limit, lo = pooled ? 0 : lowest;
       const bool p_free = i < a.pbufs || mbar_test(b_pempty + 8 * pb, ((i - a.pbufs) / a.pbufs) & 1);     // needed only after the math
       // score in the log2 domain: cap and bias
       const float b0 = slope * (float)(key0 - limit);
@@ -220,10 +250,10 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       };
 #pragma unroll
       for (int j = 0; j < kKeys; j += 4) score4(r + j, j);
-      if (key0 + kKeys - 1 > limit || key0 < lowest) {
+      if (key0 + kKeys - 1 > hi || key0 < lo) {
 #pragma unroll
         for (int j = 0; j < kKeys; j++)
-          if (key0 + j > limit || key0 + j < lowest) r[j] = 0xff800000u;
+          if (key0 + j > hi || key0 + j < lo) r[j] = 0xff800000u;
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -329,6 +359,42 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           if (col == 0) a.lse2[o] = den > 0.f ? m + log2f(den) : -INFINITY;
         }
       }
+    } else if (kExt && a.turn && a.splits == 1) {
+      // rows into shared memory (nothing else uses it any more), pairs of columns from there
+      float* fold = reinterpret_cast<float*>(smem);
+      const int ld = a.Dv + 4, half = a.Dv >> 1;
+      const float inv = ((have && l_run > 0.f) ? 1.f / l_run : 0.f) * (row_ok ? gate_of(a.gate, a.gate_ld, tok, head, a.out_scale) : 0.f);
+#pragma unroll 1
+      for (int cblk = 0; cblk < a.nv * 2; cblk++) {
+        uint32_t o[32];
+        __syncwarp();                          // the lanes of rows outside the tile skip the stores below
+        if (have) {
+          tmem_ld_32x32b_x32(tmem_o + lane_addr + cblk * 32, o);
+          tc_wait_ld();
+        }
+        if (!row_ok) continue;
+#pragma unroll
+        for (int v = 0; v < 8; v++) {
+          const int col = cblk * 32 + v * 4;
+          if (col >= a.Dv) continue;
+          *reinterpret_cast<float4*>(fold + trow * ld + col) =
+              have ? make_float4(__uint_as_float(o[4 * v]) * inv, __uint_as_float(o[4 * v + 1]) * inv, __uint_as_float(o[4 * v + 2]) * inv, __uint_as_float(o[4 * v + 3]) * inv)
+                   : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      }
+      named_bar_sync(1, live_warps * 32);
+      const int groups = half / 4, me = wq * 32 + (int)lane_id();      // Dv is a multiple of 8: groups of four pairs
+      for (int i = me; i < n_tok * a.g * groups; i += live_warps * 32) {
+        const int rr = i / groups, m = (i - rr * groups) * 4, tk = rr / a.g;
+        const float* src = fold + rr * ld + m;
+        const float* tab = a.turn + (long long)min(base_limit + tk, a.n_pos - 1) * a.Dv + m;
+        const float4 x = *reinterpret_cast<const float4*>(src), y = *reinterpret_cast<const float4*>(src + half);
+        const float4 c = __ldg(reinterpret_cast<const float4*>(tab)), s = __ldg(reinterpret_cast<const float4*>(tab + half));
+        __nv_bfloat16* dst = a.out + (long long)(tok0 + tk) * a.o_ld + (long long)(hkv * a.g + rr % a.g) * a.Dv + m;
+        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(x.x * c.x + y.x * s.x, x.y * c.y + y.y * s.y), pack_bf16x2(x.z * c.z + y.z * s.z, x.w * c.w + y.w * s.w));
+        *reinterpret_cast<uint2*>(dst + half) =
+            make_uint2(pack_bf16x2(y.x * c.x - x.x * s.x, y.y * c.y - x.y * s.y), pack_bf16x2(y.z * c.z - x.z * s.z, y.w * c.w - x.w * s.w));
+      }
     } else {
       float inv = (have && l_run > 0.f) ? 1.f / l_run : 0.f;
       if (a.splits == 1 && row_ok) inv *= gate_of(a.gate, a.gate_ld, tok, head, a.out_scale);
@@ -380,20 +446,34 @@ __global__ void __launch_bounds__(128) gqa_biased_merge_kernel(const GbArgs a) {
   float den = 0.f;
   for (int s = 0; s < a.splits; s++) { const float l = a.lse2[s * rows + row]; den += l == -INFINITY ? 0.f : exp2f(l - m); }
   const float inv = den > 0.f ? gate_of(a.gate, a.gate_ld, t, h, a.out_scale) / den : 0.f;
-  for (int d = threadIdx.x; d < a.Dv; d += blockDim.x) {
+  auto column = [&](int d) {
     float acc = 0.f;
     for (int s = 0; s < a.splits; s++) {
       const float l = a.lse2[s * rows + row];
       if (l != -INFINITY) acc += exp2f(l - m) * a.part[(s * rows + row) * a.Dv + d];
     }
-    a.out[t * a.o_ld + (long long)h * a.Dv + d] = __float2bfloat16(acc * inv);
+    return acc * inv;
+  };
+  __nv_bfloat16* out = a.out + t * a.o_ld + (long long)h * a.Dv;
+  if (a.turn) {
+    int lo = 0, hi = a.num_seqs - 1;          // last sequence whose first token is <= t
+    while (lo < hi) { const int mid = (lo + hi + 1) >> 1; if (a.cu_seqlens_q[mid] <= t) lo = mid; else hi = mid - 1; }
+    const int pos = min(max(a.context_lens[lo] - a.cu_seqlens_q[lo + 1] + (int)t, 0), a.n_pos - 1), half = a.Dv >> 1;
+    const float* tab = a.turn + (long long)pos * a.Dv;
+    for (int d = threadIdx.x; d < half; d += blockDim.x) {
+      const float x = column(d), y = column(d + half), c = tab[d], s = tab[half + d];
+      out[d] = __float2bfloat16(x * c + y * s);
+      out[d + half] = __float2bfloat16(y * c - x * s);
+    }
+    return;
   }
+  for (int d = threadIdx.x; d < a.Dv; d += blockDim.x) out[d] = __float2bfloat16(column(d));
 }
 
-struct GbPlan { int nc, nv, tq, rep, rows8, stages, pbufs, smem; };
+struct GbPlan { int nc, nv, tq, rep, rows8, stages, pbufs, bar_off, smem; };
 
 // Tile geometry for groups of g heads, head sizes D / Dv and sequences of at most max_q new tokens; false: not covered.
-static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, GbPlan* p) {
+static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, bool ext, GbPlan* p) {
   if (g < 1 || g > 128 || D < 8 || D % 8 || D > 256 || Dv < 8 || Dv % 8 || Dv > 256 || max_q < 1) return false;
   p->nc = (D + 63) / 64; p->nv = (Dv + 63) / 64;
   p->tq = 128 / g < max_q ? 128 / g : max_q;
@@ -408,7 +488,10 @@ static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, GbPlan* p) {
   if (p->stages > 4) p->stages = 4;
   if (p->stages < 2) return false;
   const int used = q + p->pbufs * pb + p->stages * kv;
-  p->smem = used + 256;
+  const int rows_out = ext ? g * p->tq * (Dv + 4) * 4 : 0;              // kExt's way out
+  p->bar_off = ((rows_out > used ? rows_out : used) + 15) / 16 * 16;
+  p->smem = p->bar_off + 256;
+  if (p->smem > 232448) return false;
   if (p->rep && 4 * g * p->tq * (Dv + 4) * 4 > used) return false;      // the fold's buffer
   // an MMA reads 128 rows from each chunk of Q and from each P buffer: those reads must end inside the allocation
   const int last_q = (p->nc - 1) * p->rows8 * 128 + 16384, last_p = q + (p->pbufs - 1) * p->rows8 * 128 + 16384;
@@ -420,22 +503,27 @@ static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, GbPlan* p) {
 using namespace ne;
 
 // Tokens per tile (0: the shape is not covered)
-extern "C" int ne_gqa_biased_plan(int H, int Hkv, int D, int Dv, int max_q) {
+extern "C" int ne_gqa_biased_plan(int H, int Hkv, int D, int Dv, int max_q, int ext) {
   GbPlan p;
-  return Hkv >= 1 && H % Hkv == 0 && gb_plan(H / Hkv, D, Dv, max_q, false, &p) ? p.tq : 0;
+  return Hkv >= 1 && H % Hkv == 0 && gb_plan(H / Hkv, D, Dv, max_q, false, ext != 0, &p) ? p.tq : 0;
 }
 
 // q bf16 [T, H, D] (row stride q_ld elements), k_cache bf16 [num_blocks, 64, Hkv, D], v_cache bf16 [num_blocks, 64, Hkv, Dv];
 // max_tiles >= sum over sequences of ceil(q_len / tokens per tile).  softcap 0 / slopes null / window 0 / gate null: without.  out bf16, row
-// stride o_ld, heads Dv apart.  splits > 1: part fp32 [splits, T, H, Dv], lse2 [splits, T, H]; the merge kernel is launched too.
+// stride o_ld, heads Dv apart.  pool > 0: pooled rows k_pool [num_blocks, pool_rows, Hkv, D], v_pool [.., Dv] (a window, no cap, no slopes); turn:
+// [n_pos, Dv] or null.  splits > 1: part fp32 [splits, T, H, Dv], lse2 [splits, T, H]; the merge kernel is launched too.
 extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache, const void* v_cache, int num_blocks, const int* block_tables, int bt_stride,
                              const int* cu_seqlens_q, const int* context_lens, int num_seqs, int T, int H, int Hkv, int D, int Dv, int max_q, int max_tiles,
                              int splits, float scale, float softcap, const float* slopes, int window, const void* gate, long long gate_ld, float out_scale,
-                             void* out, long long o_ld, float* part, float* lse2, cudaStream_t st) {
+                             void* out, long long o_ld, float* part, float* lse2, const void* k_pool, const void* v_pool, int pool, int pool_rows,
+                             const float* turn, int n_pos, cudaStream_t st) {
   if (T <= 0) return 0;
   GbPlan p;
+  const bool ext = pool > 0 || turn;
+  if (ext && (softcap > 0.f || slopes || (turn && n_pos < 1))) return 1003;
+  if (pool > 0 && (window < 1 || !k_pool || !v_pool || pool_rows < (kBPage + 8 * pool - 1) / (8 * pool) * 8)) return 1004;
   if (Hkv < 1 || H % Hkv || splits < 1 || (splits > 1 && (!part || !lse2)) || max_tiles < 1) return 1001;
-  if (!gb_plan(H / Hkv, D, Dv, max_q, softcap > 0.f, &p) && !gb_plan(H / Hkv, D, Dv, max_q, false, &p)) return 1001;
+  if (!gb_plan(H / Hkv, D, Dv, max_q, softcap > 0.f, ext, &p) && !gb_plan(H / Hkv, D, Dv, max_q, false, ext, &p)) return 1001;
   if (q_ld % 8 || o_ld % 8 || q_ld < (long long)H * D || (((uintptr_t)q | (uintptr_t)out) & 15)) return 1002;
   const int g = H / Hkv;
   CUtensorMap mq, mk, mv;
@@ -452,10 +540,18 @@ extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache,
     uint32_t box[4] = {64, 1, kBPage, 1};
     rc = make_tmap(which ? &mv : &mk, which ? v_cache : k_cache, TMA_BF16, 4, dims, strides, box, TMA_SW_128); if (rc) return 2100 + rc;
   }
-  const int variant = (softcap > 0.f ? 2 : 0) + p.rep;
-  auto kern = variant == 3 ? gqa_biased_kernel<true, true> : variant == 2 ? gqa_biased_kernel<true, false> : variant == 1 ? gqa_biased_kernel<false, true>
-                                                                                                                          : gqa_biased_kernel<false, false>;
-  static bool configured[4] = {false, false, false, false};
+  CUtensorMap mkp = mk, mvp = mv;
+  for (int which = 0; which < 2 && pool > 0; which++) {
+    const uint64_t w = which ? Dv : D;
+    uint64_t dims[4] = {w, (uint64_t)Hkv, (uint64_t)pool_rows, (uint64_t)num_blocks};
+    uint64_t strides[3] = {w * 2, (uint64_t)Hkv * w * 2, (uint64_t)pool_rows * Hkv * w * 2};
+    uint32_t box[4] = {64, 1, 8, 1};
+    rc = make_tmap(which ? &mvp : &mkp, which ? v_pool : k_pool, TMA_BF16, 4, dims, strides, box, TMA_SW_128); if (rc) return 2200 + rc;
+  }
+  const int variant = ext ? 4 : (softcap > 0.f ? 2 : 0) + p.rep;
+  auto kern = variant == 4 ? gqa_biased_kernel<false, false, true> : variant == 3 ? gqa_biased_kernel<true, true, false> : variant == 2 ? gqa_biased_kernel<true, false, false>
+              : variant == 1 ? gqa_biased_kernel<false, true, false> : gqa_biased_kernel<false, false, false>;
+  static bool configured[5] = {false, false, false, false, false};
   if (!configured[variant]) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
     if (e != cudaSuccess) return (int)e;
@@ -466,7 +562,8 @@ extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache,
   a.T = T; a.H = H; a.Dv = Dv; a.g = g; a.tq = p.tq; a.splits = splits; a.nc = p.nc; a.nv = p.nv; a.rows8 = p.rows8; a.stages = p.stages; a.pbufs = p.pbufs;
   a.window = window; a.tmem_cols = p.nv <= 2 ? 256 : 512; a.scale = scale; a.softcap = softcap; a.slopes = slopes; a.gate = (const __nv_bfloat16*)gate;
   a.gate_ld = gate_ld; a.out_scale = out_scale; a.out = (__nv_bfloat16*)out; a.o_ld = o_ld; a.part = part; a.lse2 = lse2;
-  cudaError_t e = launch_pdl(kern, dim3((unsigned)max_tiles, (unsigned)Hkv, (unsigned)splits), dim3(kGbThreads), (size_t)p.smem, st, mq, mk, mv, a);
+  a.pool = pool > 0 ? pool : 0; a.turn = turn; a.n_pos = n_pos; a.bar_off = p.bar_off;
+  cudaError_t e = launch_pdl(kern, dim3((unsigned)max_tiles, (unsigned)Hkv, (unsigned)splits), dim3(kGbThreads), (size_t)p.smem, st, mq, mk, mv, mkp, mvp, a);
   if (e != cudaSuccess || splits == 1) return (int)e;
   return (int)launch_pdl(gqa_biased_merge_kernel, dim3((unsigned)((long long)T * H)), dim3(128), 0, st, a);
 }

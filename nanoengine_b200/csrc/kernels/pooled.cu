@@ -1,0 +1,186 @@
+// Front end of attention over a window of tokens and pooled blocks of older ones, bf16 and fp32, any sizes:
+//   * pooled_prepare: RMS norm of q and of k over all heads at once, rotation of the first `dims` columns of every query and key head and of whole
+//     values (column i with column i + half), q back in place, key and value rows into the paged caches.  One CTA per token, its row in shared memory.
+//   * block means: a block of P tokens is pooled when its last token arrives - mean of the P rows as the caches hold them, in the order of
+//     positions.  Calls of single tokens do it in the same kernel, calls with portions in a second one, when all rows are stored.
+// Pooled rows are kept in groups of eight neighbours in the page of the first token of the group's first block.
+#include "ptx.cuh"
+#include "pooled.cuh"
+
+namespace ne {
+
+__device__ __forceinline__ float pl_ld(const float* p) { return *p; }
+__device__ __forceinline__ float pl_ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void pl_st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void pl_st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ float4 pl_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 pl_ld4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void pl_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void pl_st4(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
+
+struct PoolArgs {
+  void* qkv; long long ld;                   // [T, H D | G D | G Dv]
+  const void* q_norm; const void* k_norm; float eps;
+  const long long* positions; const float* k_table; const float* v_table; int n_pos;     // [n_pos, dims], [n_pos, Dv]: cos | sin
+  void* k_cache; void* v_cache; void* k_pool; void* v_pool; const long long* slots;
+  const int* block_tables; int bt_stride; const int* cu; int B;
+  int T, H, G, D, Dv, dims, pool, block_size, pool_rows;
+};
+
+// The block that token t completes (nothing to do when it completes none).  Whole CTA.
+template <typename T, int V>
+__device__ __forceinline__ void pool_block(const PoolArgs& a, int t) {
+  const long long p = a.positions[t];
+  if (p < 0 || (p + 1) % a.pool || a.slots[t] < 0) return;
+  int lo = 0, hi = a.B - 1;                   // last sequence whose first token is <= t
+  while (lo < hi) { const int mid = (lo + hi + 1) >> 1; if (a.cu[mid] <= t) lo = mid; else hi = mid - 1; }
+  const int* bt = a.block_tables + (long long)lo * a.bt_stride;
+  const int b = (int)(p / a.pool), bs = a.block_size;
+  int page, row;
+  pooled_place(b, a.pool, bs, page, row);
+  if (page >= a.bt_stride || p / bs >= a.bt_stride) { if (threadIdx.x == 0) report(ST_BAD_INDEX, 50, t, page); return; }
+  const long long dst = bt[page];
+  if (!NE_INDEX_OK(dst, BK_CACHE_PAGES, 50, __LINE__)) return;
+  const int kw = a.G * a.D, vw = a.G * a.Dv;
+  const float inv = 1.f / (float)a.pool;
+  for (int c = threadIdx.x * V; c < kw + vw; c += blockDim.x * V) {       // V divides kw: a group never straddles
+    const bool key = c < kw;
+    const int w = key ? kw : vw, cc = key ? c : c - kw;
+    const T* src = reinterpret_cast<const T*>(key ? a.k_cache : a.v_cache) + cc;
+    T* out = reinterpret_cast<T*>(key ? a.k_pool : a.v_pool) + (dst * a.pool_rows + row) * w + cc;
+    float s[V];
+#pragma unroll
+    for (int e = 0; e < V; e++) s[e] = 0.f;
+#pragma unroll 4
+    for (int j = 0; j < a.pool; j++) {
+      const int q = (int)p - a.pool + 1 + j, pg = bt[q / bs];
+      if (!NE_INDEX_OK(pg, BK_CACHE_PAGES, 51, __LINE__)) continue;
+      const T* r = src + ((long long)pg * bs + q % bs) * w;
+      if constexpr (V == 4) { const float4 v = pl_ld4(r); s[0] += v.x; s[1] += v.y; s[2] += v.z; s[3] += v.w; }
+      else s[0] += pl_ld(r);
+    }
+    if constexpr (V == 4) pl_st4(out, make_float4(s[0] * inv, s[1] * inv, s[2] * inv, s[3] * inv));
+    else pl_st(out, s[0] * inv);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, const int pool_here) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  extern __shared__ __align__(16) float sm[];       // the row (fp32) | key table | value table
+  __shared__ float red[2][16];
+  const int t = blockIdx.x, nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.Dv, W = nq + nk + nv, D = a.D, Dv = a.Dv, dims = a.dims;
+  float* s_kt = sm + (W + 3) / 4 * 4;
+  float* s_vt = s_kt + (dims + 3) / 4 * 4;
+  T* row = reinterpret_cast<T*>(a.qkv) + (long long)t * a.ld;
+  long long p = a.positions[t];
+  const long long slot = a.slots[t];
+  if (p < 0 || p >= a.n_pos) { if (threadIdx.x == 0) report(ST_BAD_INDEX, 52, t, (int)p); p = 0; }
+  for (int i = threadIdx.x; i < dims; i += blockDim.x) s_kt[i] = a.k_table[p * dims + i];
+  for (int i = threadIdx.x; i < Dv; i += blockDim.x) s_vt[i] = a.v_table[p * Dv + i];
+  float qq = 0.f, kk = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {             // V divides nq and nk
+    float s;
+    if constexpr (V == 4) {
+      const float4 v = pl_ld4(row + i);
+      *reinterpret_cast<float4*>(sm + i) = v;
+      s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    } else { const float v = pl_ld(row + i); sm[i] = v; s = v * v; }
+    if (i < nq) qq += s; else if (i < nq + nk) kk += s;
+  }
+  qq = warp_sum(qq); kk = warp_sum(kk);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (lane == 0) { red[0][warp] = qq; red[1][warp] = kk; }
+  __syncthreads();
+  const float rq = rsqrtf(warp_sum(lane < nw ? red[0][lane] : 0.f) / (float)nq + a.eps), rk = rsqrtf(warp_sum(lane < nw ? red[1][lane] : 0.f) / (float)nk + a.eps);
+  const bool store = slot >= 0 && NE_INDEX_OK(slot, BK_CACHE_ROWS, 53, __LINE__);
+  const T *qw = reinterpret_cast<const T*>(a.q_norm), *kw = reinterpret_cast<const T*>(a.k_norm);
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    const int part = i < nq ? 0 : i < nq + nk ? 1 : 2;
+    const int j = part == 0 ? i : part == 1 ? i - nq : i - nq - nk;        // column within q, k or v
+    if (part && !store) continue;
+    const int width = part == 2 ? Dv : D, turned = part == 2 ? Dv : dims, half = turned >> 1, d = j % width;
+    const float* tab = part == 2 ? s_vt : s_kt;
+    const T* w = part == 0 ? qw : kw;
+    const float r = part == 0 ? rq : rk;
+    // columns d .. d + V - 1 lie on one side of the rotation: V divides half and width
+    const int other = d < half ? half : -half, ti = d < half ? d : d - half;
+    const float sign = d < half ? -1.f : 1.f;
+    T* dst = part == 0 ? row + i : part == 1 ? reinterpret_cast<T*>(a.k_cache) + slot * nk + j : reinterpret_cast<T*>(a.v_cache) + slot * nv + j;
+    if constexpr (V == 4) {
+      float4 x = *reinterpret_cast<const float4*>(sm + i);
+      if (part < 2) { const float4 g = pl_ld4(w + j); x.x *= r * g.x; x.y *= r * g.y; x.z *= r * g.z; x.w *= r * g.w; }
+      if (d < turned) {
+        float4 y = *reinterpret_cast<const float4*>(sm + i + other);
+        if (part < 2) { const float4 g = pl_ld4(w + j + other); y.x *= r * g.x; y.y *= r * g.y; y.z *= r * g.z; y.w *= r * g.w; }
+        const float4 c = *reinterpret_cast<const float4*>(tab + ti), s = *reinterpret_cast<const float4*>(tab + half + ti);
+        x.x = x.x * c.x + sign * y.x * s.x; x.y = x.y * c.y + sign * y.y * s.y; x.z = x.z * c.z + sign * y.z * s.z; x.w = x.w * c.w + sign * y.w * s.w;
+      }
+      pl_st4(dst, x);
+    } else {
+      float x = sm[i];
+      if (part < 2) x *= r * pl_ld(w + j);
+      if (d < turned) {
+        float y = sm[i + other];
+        if (part < 2) y *= r * pl_ld(w + j + other);
+        x = x * tab[ti] + sign * y * tab[half + ti];
+      }
+      pl_st(dst, x);
+    }
+  }
+  if (!pool_here) return;
+  __syncthreads();                                   // this token's rows are stored
+  pool_block<T, V>(a, t);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) pooled_means_kernel(const PoolArgs a) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  pool_block<T, V>(a, blockIdx.x);
+}
+
+template <typename T>
+static int pooled_t(const PoolArgs& a, int max_q, cudaStream_t st) {
+  const int W = a.H * a.D + a.G * (a.D + a.Dv);
+  const uintptr_t al = (uintptr_t)a.qkv | (uintptr_t)a.q_norm | (uintptr_t)a.k_norm | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache | (uintptr_t)a.k_pool | (uintptr_t)a.v_pool;
+  const bool vec = a.D % 4 == 0 && a.Dv % 8 == 0 && a.dims % 8 == 0 && a.ld % 4 == 0 && al % 16 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((W + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+  const size_t smem = sizeof(float) * ((size_t)(W + 3) / 4 * 4 + (a.dims + 3) / 4 * 4 + a.Dv);
+  auto k = vec ? pooled_prepare_kernel<T, 4> : pooled_prepare_kernel<T, 1>;
+  if (smem > 40 * 1024) {
+    if (smem > 227 * 1024) return 1001;
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  cudaError_t e = launch_pdl(k, dim3((unsigned)a.T), dim3((unsigned)threads), smem, st, a, max_q == 1 ? 1 : 0);
+  if (e != cudaSuccess || max_q == 1) return (int)e;
+  int mt = (a.G * (a.D + a.Dv) / per + 31) / 32 * 32;
+  mt = mt > 256 ? 256 : mt < 32 ? 32 : mt;
+  return (int)launch_pdl(vec ? pooled_means_kernel<T, 4> : pooled_means_kernel<T, 1>, dim3((unsigned)a.T), dim3((unsigned)mt), 0, st, a);
+}
+
+}  // namespace ne
+
+using namespace ne;
+
+// See PoolArgs.  Caches [pages, block_size, G, D / Dv], pooled rows [pages, pool_rows, G, D / Dv], all in the activation dtype (fp32 = 1: float).
+// max_q: most tokens a sequence brings; 1 pools in the same kernel (a call then has no two tokens of one sequence).
+extern "C" int ne_pooled_prepare(void* qkv, long long ld, const void* q_norm, const void* k_norm, float eps, const long long* positions, const float* k_table,
+                                 const float* v_table, int n_pos, void* k_cache, void* v_cache, void* k_pool, void* v_pool, const long long* slots,
+                                 const int* block_tables, int bt_stride, const int* cu, int B, int T, int H, int G, int D, int Dv, int dims, int pool, int block_size,
+                                 int pool_rows, int max_q, int fp32, cudaStream_t st) {
+  if (T <= 0 || B <= 0) return 0;
+  if (H < 1 || G < 1 || D < 1 || Dv < 2 || Dv % 2 || dims < 0 || dims % 2 || dims > D || pool < 1 || block_size < 1 || n_pos < 1 ||
+      pool_rows < (block_size + 8 * pool - 1) / (8 * pool) * 8 || ld < (long long)H * D + (long long)G * (D + Dv)) return 1001;
+  PoolArgs a;
+  a.qkv = qkv; a.ld = ld; a.q_norm = q_norm; a.k_norm = k_norm; a.eps = eps; a.positions = positions; a.k_table = k_table; a.v_table = v_table; a.n_pos = n_pos;
+  a.k_cache = k_cache; a.v_cache = v_cache; a.k_pool = k_pool; a.v_pool = v_pool; a.slots = slots; a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu = cu;
+  a.B = B; a.T = T; a.H = H; a.G = G; a.D = D; a.Dv = Dv; a.dims = dims; a.pool = pool; a.block_size = block_size; a.pool_rows = pool_rows;
+  return fp32 ? pooled_t<float>(a, max_q, st) : pooled_t<__nv_bfloat16>(a, max_q, st);
+}

@@ -1,6 +1,7 @@
 // Row operators around a 32-bit residual stream, for bf16 and fp32 activations and any row width:
 //   * residual_norm: x += rmsnorm(y, w_post); out = rmsnorm(x, w_next)   (norm after a sublayer, residual add, norm before the next)
 //     or, as the start of the stream, x = table[id]; out = rmsnorm(x, w_next)
+//   * postnorm: x <- rmsnorm(alpha x + y, w); out = x, or rmsnorm(x, w_last) in front of the head; or, as the start, x = scale * table[id]
 //   * gated activation of [gate | up] rows
 //   * latent_prepare: rotary part of every query head in place, and the latent cache row [rmsnorm(kv[:R]) | rope(kv[R:])]
 //   * gather of cache rows
@@ -102,6 +103,97 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(const T* __restrict_
       stx(out + row * W + i, srow[i] * r2 * (ldx(w_next + i) + w_off));
     }
   }
+}
+
+// One CTA per row, the row in shared memory between the passes.  ids given: x = alpha table[id], out = x.
+struct PostnormArgs {
+  const void* y; long long y_ld; float* x; const void* w; const void* w_last; void* out; const long long* ids; const void* table; int W, vocab; float alpha, eps;
+};
+template <typename T, int V>
+__global__ void __launch_bounds__(512) postnorm_kernel(const PostnormArgs a) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  extern __shared__ float srow[];            // W floats
+  __shared__ float red[2][32];
+  const long long row = blockIdx.x;
+  const int W = a.W;
+  float* xr = a.x + row * W;
+  T* out = reinterpret_cast<T*>(a.out) + row * W;
+  if (a.ids) {
+    const long long id = a.ids[row];
+    const bool ok = id >= 0 && id < a.vocab;
+    if (!ok && threadIdx.x == 0) report(ST_BAD_INDEX, 47, (int)row, (int)id);
+    const T* tr = reinterpret_cast<const T*>(a.table) + (ok ? id : 0) * W;
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+      if constexpr (V == 4) {
+        float4 t = Vec4<T>::load(tr + i);
+        t.x *= a.alpha; t.y *= a.alpha; t.z *= a.alpha; t.w *= a.alpha;
+        *reinterpret_cast<float4*>(xr + i) = t;
+        Vec4<T>::store(out + i, t);
+      } else {
+        const float t = ldx(tr + i) * a.alpha;
+        xr[i] = t; stx(out + i, t);
+      }
+    }
+    return;
+  }
+  const T* yr = reinterpret_cast<const T*>(a.y) + row * a.y_ld;
+  const T* w = reinterpret_cast<const T*>(a.w);
+  const T* wl = reinterpret_cast<const T*>(a.w_last);
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 t = Vec4<T>::load(yr + i);
+      float4 v = *reinterpret_cast<const float4*>(xr + i);
+      v.x = fmaf(a.alpha, v.x, t.x); v.y = fmaf(a.alpha, v.y, t.y); v.z = fmaf(a.alpha, v.z, t.z); v.w = fmaf(a.alpha, v.w, t.w);
+      *reinterpret_cast<float4*>(srow + i) = v;
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    } else {
+      const float v = fmaf(a.alpha, xr[i], ldx(yr + i));
+      srow[i] = v; ss += v * v;
+    }
+  }
+  const float r = rsqrtf(cta_sum(ss, red, 0) / (float)W + a.eps);
+  float s2 = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {        // a thread rereads only what it stored itself
+    if constexpr (V == 4) {
+      float4 v = *reinterpret_cast<const float4*>(srow + i);
+      const float4 g = Vec4<T>::load(w + i);
+      v.x *= r * g.x; v.y *= r * g.y; v.z *= r * g.z; v.w *= r * g.w;
+      *reinterpret_cast<float4*>(xr + i) = v;
+      if (wl) { *reinterpret_cast<float4*>(srow + i) = v; s2 += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+      else Vec4<T>::store(out + i, v);
+    } else {
+      const float v = srow[i] * r * ldx(w + i);
+      xr[i] = v;
+      if (wl) { srow[i] = v; s2 += v * v; } else stx(out + i, v);
+    }
+  }
+  if (!wl) return;
+  const float r2 = rsqrtf(cta_sum(s2, red, 1) / (float)W + a.eps);
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(srow + i), g = Vec4<T>::load(wl + i);
+      Vec4<T>::store(out + i, make_float4(v.x * r2 * g.x, v.y * r2 * g.y, v.z * r2 * g.z, v.w * r2 * g.w));
+    } else {
+      stx(out + i, srow[i] * r2 * ldx(wl + i));
+    }
+  }
+}
+
+template <typename T>
+static int postnorm_t(const PostnormArgs& a, int rows, cudaStream_t st) {
+  const size_t smem = (size_t)a.W * sizeof(float);
+  const uintptr_t al = (uintptr_t)a.y | (uintptr_t)a.x | (uintptr_t)a.w | (uintptr_t)a.w_last | (uintptr_t)a.out | (uintptr_t)a.table;
+  const bool vec = a.W % 4 == 0 && a.y_ld % 4 == 0 && al % 16 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((a.W + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+  auto k = vec ? postnorm_kernel<T, 4> : postnorm_kernel<T, 1>;
+  if (smem > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl(k, dim3((unsigned)rows), dim3((unsigned)threads), smem, st, a);
 }
 
 // Gated activation (see elementwise.cu for the modes): x [T, >= 2I] rows with stride ld -> y [T, I]
@@ -393,6 +485,18 @@ extern "C" int ne_residual_norm(const void* y, long long y_ld, float* x, const v
   if (W <= 0 || W > 48 * 1024 || (!ids && (!y || !w_post)) || (ids && !table)) return 1001;
   return fp32 ? residual_norm_t<float>(y, y_ld, x, w_post, w_next, out, T, W, eps, w_off, ids, table, vocab, st)
               : residual_norm_t<__nv_bfloat16>(y, y_ld, x, w_post, w_next, out, T, W, eps, w_off, ids, table, vocab, st);
+}
+
+// y [T, W] (row stride y_ld), x [T, W] fp32 updated in place, out [T, W]; w_last null: out is x itself.  With `ids` (and table [vocab, W]) y and
+// the norms are not read: x = out = alpha * table[ids].
+extern "C" int ne_postnorm(const void* y, long long y_ld, float* x, float alpha, const void* w, const void* w_last, void* out, int T, int W, float eps,
+                           const long long* ids, const void* table, int vocab, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (W <= 0 || W > 48 * 1024 || (!ids && (!y || !w)) || (ids && !table)) return 1001;
+  PostnormArgs a;
+  a.y = ids ? nullptr : y; a.y_ld = ids ? 0 : y_ld; a.x = x; a.w = ids ? nullptr : w; a.w_last = ids ? nullptr : w_last; a.out = out; a.ids = ids;
+  a.table = ids ? table : nullptr; a.W = W; a.vocab = vocab; a.alpha = alpha; a.eps = eps;
+  return fp32 ? postnorm_t<float>(a, T, st) : postnorm_t<__nv_bfloat16>(a, T, st);
 }
 
 extern "C" int ne_glu_rows(const void* x, long long ld, void* y, int T, int I, int act, float p0, float p1, int fp32, cudaStream_t st) {

@@ -172,16 +172,19 @@ class PrequantizedActivation:
         self.q, self.scales, self.shape, self.device = q, scales, q.shape, q.device
 
 
-def _gemm_simt(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias=None):
+_ACTS = {None: 0, "relu2": 1, "tanh": 2}        # of linear(act=...)
+
+
+def _gemm_simt(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias=None, act=None, act_from=0):
     """Tiled product on CUDA cores: true 32-bit operands, and bf16 shapes the tensor-core GEMM cannot address."""
     f32 = A.dtype == torch.float32
     assert A.dtype == B.dtype and D.dtype in (torch.float32, A.dtype)
     _ck(lib().ne_gemm_simt(_p(A), _c.c_longlong(lda), _c.c_longlong(a_bs), _p(B), _c.c_longlong(ldb), _c.c_longlong(b_bs), _p(D), _c.c_longlong(ldd),
                            _c.c_longlong(d_bs), _c.c_int(M), _c.c_int(N), _c.c_int(K), _c.c_int(batch), _c.c_int(int(f32)),
-                           _c.c_int(int(D.dtype == torch.float32)), _p(bias), _st()), "ne_gemm_simt")
+                           _c.c_int(int(D.dtype == torch.float32)), _p(bias), _c.c_int(_ACTS[act]), _c.c_int(act_from), _st()), "ne_gemm_simt")
 
 
-def _linear_simt(x, w, bias, out_fp32):
+def _linear_simt(x, w, bias, out_fp32, act=None, act_from=0):
     x2 = x.reshape(-1, x.shape[-1])
     x2 = (x2 if x2.dtype == w.dtype else x2.to(w.dtype))
     if x2.stride(-1) != 1:
@@ -190,7 +193,7 @@ def _linear_simt(x, w, bias, out_fp32):
     out = torch.empty(T, N, dtype=torch.float32 if out_fp32 else w.dtype, device=x.device)
     fused = bias is not None and bias.dtype == torch.float32
     if T > 0:
-        _gemm_simt(x2, x2.stride(0), 0, w, w.stride(0), 0, out, N, 0, T, N, K, 1, bias if fused else None)
+        _gemm_simt(x2, x2.stride(0), 0, w, w.stride(0), 0, out, N, 0, T, N, K, 1, bias if fused else None, act, act_from)
     if bias is not None and not fused:
         out = out + bias
     return out.view(*x.shape[:-1], N)
@@ -200,8 +203,10 @@ def linear_fp32(x, w: torch.Tensor) -> torch.Tensor:
     return linear(x, w, out_fp32=True)
 
 
-def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None, out_fp32: bool = False) -> torch.Tensor:
+def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None, out_fp32: bool = False, act: Optional[str] = None,
+           act_from: int = 0) -> torch.Tensor:
     N, K = w.shape
+    assert act is None or (w.dtype != FP8 and bias is None and isinstance(x, torch.Tensor))
     if isinstance(x, PrequantizedActivation):
         assert w.dtype == FP8 and x.shape[-1] == K, "a pre-quantised activation feeds fp8 linears only"
         T = x.shape[0]
@@ -214,7 +219,7 @@ def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None
         pre = (x.q, x.scales) if x.q is not None else None
         x = x.x
     if w.dtype == torch.float32 or (w.dtype == torch.bfloat16 and (K % 8 or N % 8)):
-        return _linear_simt(x, w, bias, out_fp32)
+        return _linear_simt(x, w, bias, out_fp32, act, act_from)
     x2 = _as_bf16_2d(x)
     T = x2.shape[0]
     out = torch.empty(T, N, dtype=torch.float32 if out_fp32 else torch.bfloat16, device=x.device)
@@ -233,6 +238,10 @@ def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None
                 assert bias.numel() == N and bias.is_contiguous()
                 _ck(lib().ne_gemm_bias(_p(x2), _c.c_longlong(x2.stride(0)), _p(w), _p(bias), _p(out), _c.c_longlong(N), _c.c_int(T), _c.c_int(N), _c.c_int(K),
                                        _c.c_int(int(out_fp32)), _st()), "ne_gemm_bias")
+                return out.view(*x.shape[:-1], N)
+            if act is not None:
+                _ck(lib().ne_gemm_act(_p(x2), _c.c_longlong(x2.stride(0)), _p(w), _p(out), _c.c_longlong(N), _c.c_int(T), _c.c_int(N), _c.c_int(K),
+                                      _c.c_int(_ACTS[act]), _c.c_int(act_from), _c.c_int(int(out_fp32)), _st()), "ne_gemm_act")
                 return out.view(*x.shape[:-1], N)
             _gemm(x2, x2.stride(0), 0, w, out, N, 0, T, N, K, 1, None, None, False, None, 0, 0, None, out_fp32)
     if bias is not None:
@@ -389,6 +398,27 @@ def embed_norm(ids: torch.Tensor, table: torch.Tensor, w_next: torch.Tensor, eps
                                _c.c_float(1.0 if unit_offset else 0.0), _p(_i64c(ids)), _p(table), _c.c_int(V), _c.c_int(int(table.dtype == torch.float32)), _st()),
         "ne_residual_norm")
     return out, x
+
+
+def _postnorm(y, x, alpha, w, eps, w_last, ids, table, dt):
+    T, W = x.shape
+    out = torch.empty(T, W, dtype=dt, device=x.device)
+    _ck(lib().ne_postnorm(_p(y), _c.c_longlong(0 if y is None else y.stride(0)), _p(x), _c.c_float(alpha), _p(w), _p(w_last), _p(out), _c.c_int(T), _c.c_int(W),
+                          _c.c_float(eps), _p(ids), _p(table), _c.c_int(0 if table is None else table.shape[0]), _c.c_int(int(dt == torch.float32)), _st()),
+        "ne_postnorm")
+    return out, x
+
+
+def postnorm(y: torch.Tensor, x: torch.Tensor, alpha: float, w: torch.Tensor, eps: float, w_last: Optional[torch.Tensor] = None):
+    """Sum, norm behind it, and the next reader's copy (or the model's own norm): one kernel, one CTA per row; x is updated in place."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.stride(1) == 1 and y.dtype == w.dtype and (w_last is None or w_last.dtype == w.dtype)
+    return _postnorm(y, x, alpha, w, eps, w_last, None, None, y.dtype)
+
+
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float):
+    assert table.is_contiguous()
+    x = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
+    return _postnorm(None, x, scale, None, 0.0, None, _i64c(ids), table, table.dtype)
 
 
 def layernorm(x, w, b, eps):
@@ -565,6 +595,29 @@ def kv_rows(k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Te
     assert k.shape == (T, kw) and v.shape == (T, vw) and k.stride(1) == 1 and v.stride(1) == 1
     _ck(lib().ne_kv_rows(_p(k), _c.c_longlong(k.stride(0)), _p(v), _c.c_longlong(v.stride(0)), _p(k_cache), _p(v_cache), _p(_i64c(slot_mapping)), _c.c_int(T),
                          _c.c_int(kw), _c.c_int(vw), _c.c_int(k.element_size()), _st()), "ne_kv_rows")
+
+
+def pooled_attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, q_norm: torch.Tensor, k_norm: torch.Tensor, eps: float, positions,
+                             key_table: torch.Tensor, value_table: torch.Tensor, k_cache, v_cache, k_pool, v_pool, pool: int, slots, block_tables,
+                             cu_seqlens, max_q_len: int = 0) -> torch.Tensor:
+    """One kernel for single-token steps, two otherwise (the block means read rows that other CTAs store); q is turned in place."""
+    T = qkv.shape[0]
+    dt = qkv.dtype
+    mq = max_q_len if max_q_len else (T if T > cu_seqlens.numel() - 1 else 1)
+    assert all(t.dtype == dt for t in (q_norm, k_norm, k_cache, v_cache, k_pool, v_pool)) and qkv.stride(1) == 1
+    assert all(t.is_contiguous() for t in (k_cache, v_cache, k_pool, v_pool, key_table, value_table))
+    assert k_cache.shape[2:] == k_pool.shape[2:] == (G, D) and v_cache.shape[2:] == v_pool.shape[2:] == (G, Dv) and value_table.shape[1] == Dv
+    assert key_table.dtype == value_table.dtype == torch.float32 and key_table.shape[0] == value_table.shape[0]
+    q = qkv[:, : H * D].unflatten(-1, (H, D))
+    if T == 0:
+        return q
+    bt, cu = _i32(block_tables), _i32(cu_seqlens)
+    _ck(lib().ne_pooled_prepare(_p(qkv), _c.c_longlong(qkv.stride(0)), _p(q_norm), _p(k_norm), _c.c_float(eps), _p(_i64c(positions)), _p(key_table), _p(value_table),
+                                _c.c_int(key_table.shape[0]), _p(k_cache), _p(v_cache), _p(k_pool), _p(v_pool), _p(_i64c(slots)), _p(bt), _c.c_int(bt.stride(0)), _p(cu),
+                                _c.c_int(cu.numel() - 1), _c.c_int(T), _c.c_int(H), _c.c_int(G), _c.c_int(D), _c.c_int(Dv), _c.c_int(key_table.shape[1]), _c.c_int(pool),
+                                _c.c_int(k_cache.shape[1]), _c.c_int(k_pool.shape[1]), _c.c_int(mq), _c.c_int(int(dt == torch.float32)), _st()), "ne_pooled_prepare")
+    LAUNCHES[0] += int(mq != 1)
+    return q
 
 
 def _i64c(t):
@@ -785,10 +838,10 @@ def gelu(x: torch.Tensor, tanh: bool = True) -> torch.Tensor:
 
 
 def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0, softcap: float = 0.0, slopes=None,
-                         gate=None, out_scale: float = 1.0, out=None, max_q_len: int = 0) -> torch.Tensor:
+                         gate=None, out_scale: float = 1.0, out=None, max_q_len: int = 0, pooled=None, pool: int = 0, turn_back=None) -> torch.Tensor:
     from . import sm100_attn
     return sm100_attn.gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window, softcap, slopes, gate, out_scale, out,
-                                           max_q_len)
+                                           max_q_len, pooled, pool, turn_back)
 
 
 def gqa_attention_paged(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0):
@@ -1107,6 +1160,28 @@ def lightning_mix(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch
     raw = torch.empty(T, H * Dv, dtype=torch.float32, device=q.device)
     _decay_scan(q, k, v, None, decay, None, state, _i32(slots), _i32(cu_seqlens), _i32(fresh), raw, H, H, Dk, Dv, 1, max_q_len)
     return _gated_norm(raw, gate, norm_w, out, 1, False, eps, out_scale)
+
+
+def general_delta(proj: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor, a_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+                  cu_seqlens: torch.Tensor, fresh: torch.Tensor, H: int, Dk: int, Dv: int, eps: float, max_q_len: int = 1) -> torch.Tensor:
+    """One kernel for single-token steps (heads up to 128 x 128), three otherwise (vectors of every token; recurrence; norm and gate)."""
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and proj.shape[1] >= H * (3 * Dk + 2 * Dv) and decay.dtype == torch.float32 and decay.stride(1) == 1 and decay.shape[1] >= H * Dk
+    assert w0.dtype == a_bias.dtype == torch.float32 and w0.numel() == a_bias.numel() == H * Dk and norm_w.dtype == proj.dtype and norm_w.numel() == H * Dv
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, Dv, Dk)
+    out = torch.empty(T, H * Dv, dtype=proj.dtype, device=proj.device)
+    if T == 0:
+        return out
+    l, mq = lib(), max(1, max_q_len)
+    l.ne_general_delta_scratch.restype = _c.c_longlong
+    n_scratch = l.ne_general_delta_scratch(_c.c_int(T), _c.c_int(H), _c.c_int(Dk), _c.c_int(Dv), _c.c_int(mq))
+    scratch = torch.empty(n_scratch, dtype=torch.float32, device=proj.device) if n_scratch else None
+    cu, n = _i32(cu_seqlens), _c.c_int(1)
+    _ck(l.ne_general_delta(_p(proj), _c.c_longlong(proj.stride(0)), _p(decay), _c.c_longlong(decay.stride(0)), _p(w0), _p(a_bias), _p(norm_w), _c.c_float(eps),
+                           _p(state), _p(_i32(slots)), _p(cu), _p(_i32(fresh)), _p(scratch), _p(out), _c.c_int(T), _c.c_int(cu.numel() - 1), _c.c_int(H), _c.c_int(Dk),
+                           _c.c_int(Dv), _c.c_int(mq), _c.c_int(int(proj.dtype == torch.float32)), _c.byref(n), _st()), "ne_general_delta")
+    LAUNCHES[0] += n.value - 1
+    return out
 
 
 def kda_recurrent(q, k, v, raw_g, b, A_log, dt_bias, lower_bound, state, slots, cu_seqlens, fresh, gate, norm_w, eps: float) -> torch.Tensor:

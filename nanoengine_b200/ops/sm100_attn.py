@@ -208,7 +208,7 @@ BIASED_TC_CALLS = [0]        # launches of the tensor-core kernel of gqa_attenti
 
 
 def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window=0, softcap=0.0, slopes=None, gate=None, out_scale=1.0,
-                         out=None, max_q_len=0, splits=None):
+                         out=None, max_q_len=0, pooled=None, pool=0, turn_back=None, splits=None):
     """bf16 with head sizes in multiples of 8 up to 256 and 64-token pages: tensor cores; other shapes and 32-bit runs: the generic kernel."""
     T, Hq, D = q.shape
     Hkv, Dv = k_cache.shape[2], v_cache.shape[3]
@@ -225,16 +225,23 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
     if T == 0:
         return out
     gate_ld = 0 if gate is None else gate.stride(0)
+    kp, vp = pooled if pool else (None, None)
+    assert not pool or (kp.dtype == vp.dtype == q.dtype and kp.is_contiguous() and vp.is_contiguous() and kp.shape[2:] == k_cache.shape[2:] and vp.shape[2:] == v_cache.shape[2:])
+    assert turn_back is None or (turn_back.dtype == torch.float32 and turn_back.is_contiguous() and turn_back.shape[1] == Dv)
+    extra = (_k._p(kp), _k._p(vp), _c.c_int(pool), _c.c_int(kp.shape[1] if pool else 0), _k._p(turn_back), _c.c_int(0 if turn_back is None else turn_back.shape[0]))
     mq = max_q_len if max_q_len else (1 if T <= B else T)
     tq = 0
     if (q.dtype == torch.bfloat16 and k_cache.shape[1] == 64 and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
             and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
-        tq = lib.ne_gqa_biased_plan(_c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq))
+        tq = lib.ne_gqa_biased_plan(_c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq),
+                                    _c.c_int(int(bool(pool) or turn_back is not None)))
     if tq:
         tiles = min(T, T // tq + B)
         S = splits
         if S is None:
             pages = bt.shape[1] if window <= 0 else min(bt.shape[1], (window + tq + 62) // 64 + 1)
+            if pool:
+                pages += bt.shape[1] // pool
             S = 1
             slots = _sms() * (2 if Dv <= 128 else 1)   # resident CTAs
             if tiles * Hkv * 2 <= slots:               # few CTAs (small decode batches): slice the keys
@@ -246,7 +253,7 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
         _k._ck(lib.ne_gqa_biased(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _c.c_int(k_cache.shape[0]), _k._p(bt), _c.c_int(bt.stride(0)),
                                  _k._p(cu), _k._p(cl), _c.c_int(B), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq),
                                  _c.c_int(tiles), _c.c_int(S), _c.c_float(scale), _c.c_float(softcap), _k._p(slopes), _c.c_int(int(window)), _k._p(gate),
-                                 _c.c_longlong(gate_ld), _c.c_float(out_scale), _k._p(out), _c.c_longlong(out.stride(0)), _k._p(part), _k._p(lse2), _k._st()),
+                                 _c.c_longlong(gate_ld), _c.c_float(out_scale), _k._p(out), _c.c_longlong(out.stride(0)), _k._p(part), _k._p(lse2), *extra, _k._st()),
                "ne_gqa_biased")
         BIASED_TC_CALLS[0] += 1
         _k.LAUNCHES[0] += int(S > 1)
@@ -254,7 +261,7 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
     _k._ck(lib.ne_attn_biased(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _k._p(bt), _c.c_int(bt.stride(0)), _c.c_int(k_cache.shape[1]),
                               _k._p(cu), _k._p(cl), _c.c_int(B), _k._p(out), _c.c_longlong(out.stride(0)), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D),
                               _c.c_int(Dv), _c.c_float(scale), _c.c_float(softcap), _k._p(slopes), _c.c_int(int(window)), _k._p(gate), _c.c_longlong(gate_ld),
-                              _c.c_float(out_scale), _c.c_int(int(q.dtype == torch.float32)), _k._st()), "ne_attn_biased")
+                              _c.c_float(out_scale), _c.c_int(int(q.dtype == torch.float32)), *extra, _k._st()), "ne_attn_biased")
     return out
 
 
