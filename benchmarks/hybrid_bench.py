@@ -1,5 +1,5 @@
 """Prefill and decode throughput of a model with listed layers beside the closest model of this package at equal sizes (`bench.py --model
-tuvutar`, `bench.py --model filasun`).
+tuvutar`, `--model filasun`, `--model sapanex`).
 
 Tuvutar: the closest model is Kimi-K3's layer stack without experts and with a plain residual: latent attention between delta-rule layers and
 dense gated MLPs in bf16 (its delta layers decay per key channel, its latent layers carry an output gate).  Both get the same width,
@@ -10,6 +10,10 @@ Filasun: the closest model is the dense Qwen3.5 stack (grouped-query attention a
 (attention, decayed linear attention, a feed-forward of width ff) stands against an attention layer and a delta-net layer with a feed-forward of
 ff / 2 each, a Mamba-2 layer with a feed-forward of ff / 2 against a delta-net layer: the same head counts, head sizes, state sizes per layer,
 feed-forward weights, width and vocabulary; the attention window is the longest context, so that both read the same keys.
+
+Sapanex: the closest model is the dense Qwen3.5 stack again, an attention layer after every three delta layers in both, the same head counts, head
+sizes, state sizes, width and vocabulary; a feed-forward of two matrices of 3 ff / 2 stands against a gated one of three of ff.  Sapanex's attention
+layers see a window of 1024 tokens and blocks of 16, Qwen3.5's the whole context.
 
 `prefill` is the device time of the scheduler's prompt steps (CUDA events around
 LLM.step), `decode` the replay of one decode step on resident inputs (graph + lm_head + sampling)."""
@@ -59,7 +63,28 @@ def qwen_model(width, heads, groups, ff, vocab):
                         linear_value_head_dim=128, max_position_embeddings=16384)
 
 
-DESIGNS = {"tuvutar": ("Tuvutar", tuvutar_model, "kimi_k3_stack", kimi_model), "filasun": ("Filasun", filasun_model, "qwen3_5_stack", qwen_model)}
+def sapanex_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import ModelConfig, _general_delta_spec, _pooled_attention_spec
+    yarn = {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+    layers = []
+    for _ in range(groups):
+        layers += [_general_delta_spec(heads, 128, 64, ff=3 * ff // 2) for _ in range(3)]
+        layers.append(_pooled_attention_spec(heads, heads // 4, 128, 128, 1024, 16, 64, ff=3 * ff // 2, base=5e5, scaling=yarn))
+    return ModelConfig.from_dict({"architecture": "Sapanex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "postln_alpha": 2.0,
+                                  "max_position_embeddings": 16384, "layers": layers})
+
+
+def qwen_3to1_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import tiny_qwen3_5
+    kinds = (["linear_attention"] * 3 + ["full_attention"]) * groups
+    return tiny_qwen3_5(vocab_size=vocab, hidden_size=width, num_hidden_layers=len(kinds), layer_types=kinds, num_attention_heads=heads, num_key_value_heads=heads // 4,
+                        head_dim=128, intermediate_size=ff, linear_num_key_heads=heads, linear_num_value_heads=heads, linear_key_head_dim=128,
+                        linear_value_head_dim=128, max_position_embeddings=16384)
+
+
+DESIGNS = {"sapanex": ("Sapanex", sapanex_model, "qwen3_5_stack", qwen_3to1_model),
+           "tuvutar": ("Tuvutar", tuvutar_model, "kimi_k3_stack", kimi_model),
+           "filasun": ("Filasun", filasun_model, "qwen3_5_stack", qwen_model)}
 
 
 def measure(mc, seqs, prompt, steps, warmup, seed=0):

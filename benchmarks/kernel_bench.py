@@ -337,6 +337,62 @@ def case_biased(B, ctx, q_len, Hq, Hkv, window, cap=50.0, D=128, bs=64):
     return fn, B * seen * Hkv * D * 2 * 2 + T * Hq * D * 4, 4.0 * pairs * Hq * D
 
 
+def case_general_delta(B, q_len=1, H=32, D=128):
+    """The generalised delta-rule mixer between its projections (gates, unit keys, recurrence, norm, gate); floor as for the delta mixer."""
+    T, W = B * q_len, H * D
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    kw = dict(proj=torch.randn(T, 5 * W + 64, **bf), decay=torch.randn(T, W, device="cuda"), w0=torch.randn(W, device="cuda") - 2, a_bias=torch.randn(W, device="cuda"),
+              norm_w=torch.ones(W, **bf), state=torch.randn(B + 1, H, D, D, device="cuda") * 0.1, slots=torch.arange(B, device="cuda", dtype=torch.int32),
+              cu_seqlens=(torch.arange(B + 1, device="cuda") * q_len).to(torch.int32), fresh=torch.zeros(B, dtype=torch.int32, device="cuda"), H=H, Dk=D, Dv=D,
+              eps=1e-6, max_q_len=q_len)
+    return lambda: sm100.general_delta(**kw), B * H * D * D * 4 * 2 + T * W * (6 * 2 + 4), 2.0 * T * H * D * D * 4
+
+
+def case_pooled(B, ctx, q_len, Hq, Hkv, window, pool, D=128, bs=64):
+    """Attention over a window and pooled blocks, outputs turned back; pool 0: the window alone.  Bytes and FLOPs of the tokens and blocks a query
+    sees."""
+    from nanoengine_b200.ops.reference import pooled_rows_per_page
+    nb, T = (ctx + bs - 1) // bs, B * q_len
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    k, v = (torch.randn(B * nb + 1, bs, Hkv, D, **bf) for _ in range(2))
+    pooled = tuple(torch.randn(B * nb + 1, pooled_rows_per_page(pool, bs), Hkv, D, **bf) for _ in range(2)) if pool else None
+    bt = torch.randperm(B * nb, device="cuda").view(B, nb).to(torch.int32)
+    q, out = torch.randn(T, Hq, D, **bf), torch.empty(T, Hq * D, **bf)
+    cu = (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    cl = torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    turn = torch.rand(ctx, D, device="cuda")
+    fn = lambda: sm100_attn.gqa_attention_biased(q, k, v, bt, cu, cl, D ** -0.5, window, out=out, max_q_len=q_len, pooled=pooled, pool=pool, turn_back=turn)
+    blocks = lambda i: max(0, (i - window + 1) // pool) if pool else 0
+    pairs = B * sum(min(window, i + 1) + blocks(i) for i in range(ctx - q_len, ctx))
+    seen = min(ctx, window + q_len - 1) + blocks(ctx - 1)
+    return fn, B * seen * Hkv * D * 2 * 2 + T * Hq * D * 4, 4.0 * pairs * Hq * D
+
+
+def case_pooled_prepare(B, q_len, H=32, G=8, D=128, dims=64, pool=16, at=4096, bs=64):
+    """q / k norm over all heads, rotations, key and value rows, block means; at: position of the first token."""
+    T, W, nb = B * q_len, H * D + 2 * G * D, (at + q_len + bs - 1) // bs
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    qkv, qn, kn = torch.randn(T, W, **bf), torch.ones(H * D, **bf), torch.ones(G * D, **bf)
+    kc, vc = (torch.zeros(B * nb + 1, bs, G, D, **bf) for _ in range(2))
+    kp, vp = (torch.zeros(B * nb + 1, -(-bs // (8 * pool)) * 8, G, D, **bf) for _ in range(2))
+    bt = torch.randperm(B * nb, device="cuda").view(B, nb).to(torch.int32)
+    # single tokens: the sequences stand at different places of their blocks
+    pos = at - at % pool + (torch.arange(B, device="cuda") % pool if q_len == 1 else torch.arange(T, device="cuda") % q_len)
+    seq = torch.arange(T, device="cuda") // q_len
+    pos = pos.clamp_max(nb * bs - 1)
+    slots = bt[seq, pos // bs].long() * bs + pos % bs
+    kt, vt = torch.rand(nb * bs, dims, device="cuda"), torch.rand(nb * bs, D, device="cuda")
+    cu = (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    fn = lambda: sm100.pooled_attention_prepare(qkv, H, G, D, D, qn, kn, 1e-6, pos, kt, vt, kc, vc, kp, vp, pool, slots, bt, cu, q_len)
+    means = T / pool * G * 2 * D * 2 * (pool + 1)
+    return fn, T * W * 2 * 2 + means, 0.0
+
+
+def case_postnorm(T, W=4096):
+    y, w, x = torch.randn(T, W, device="cuda", dtype=torch.bfloat16), torch.ones(W, device="cuda", dtype=torch.bfloat16), torch.randn(T, W, device="cuda")
+    return lambda: sm100.postnorm(y, x, 2.0, w, 1e-6), T * W * (2 + 4 + 4 + 2), 0.0
+
+
 def case_streams(T, S=2, W=4096):
     y = torch.randn(T, W, device="cuda", dtype=torch.bfloat16)
     x = torch.randn(T, S, W, device="cuda")
@@ -476,6 +532,20 @@ def build_cases(args):
         "biased_prefill_nocap": lambda: case_biased(1, 8192, 8192, 32, 8, 4096, 0.0),
         "biased_prefill_plain": lambda: case_biased(1, 8192, 8192, 32, 8, 0, 0.0),
         "gqa_prefill_same": lambda: case_gqa(1, 8192, 8192, 32, 8),
+        "general_delta_decode": lambda: case_general_delta(128),
+        "general_delta_decode_16": lambda: case_general_delta(16),
+        "general_delta_prefill_4x2048": lambda: case_general_delta(4, q_len=2048),
+        "general_delta_prefill_1x8192": lambda: case_general_delta(1, q_len=8192),
+        "pooled_decode": lambda: case_pooled(128, 8192, 1, 32, 8, 4096, 16),
+        "pooled_decode_16": lambda: case_pooled(16, 8192, 1, 32, 8, 4096, 16),
+        "pooled_decode_small_window": lambda: case_pooled(128, 8192, 1, 32, 8, 512, 16),
+        "pooled_prefill": lambda: case_pooled(1, 8192, 8192, 32, 8, 1024, 16),
+        "pooled_prefill_nopool": lambda: case_pooled(1, 8192, 8192, 32, 8, 8192, 0),
+        "pooled_prefill_w1024": lambda: case_pooled(1, 8192, 8192, 32, 8, 1024, 0),
+        "pooled_prepare_decode": lambda: case_pooled_prepare(128, 1),
+        "pooled_prepare_prefill": lambda: case_pooled_prepare(4, 2048),
+        "postnorm_decode": lambda: case_postnorm(128),
+        "postnorm_prefill": lambda: case_postnorm(8192),
         "streams_decode": lambda: case_streams(128),
         "streams_prefill": lambda: case_streams(8192),
         "delta_decode": lambda: case_delta(128),

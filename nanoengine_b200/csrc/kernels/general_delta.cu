@@ -9,7 +9,7 @@
 //   single tokens: one kernel.  A CTA holds a whole head; its state is fetched while the kernel in front still runs; gates and unit keys are
 //   made in it, and norm and gate are applied before the row leaves.
 //   otherwise: general_delta_prepare (one warp per (token, head)) writes u | w | a u | r w, general_delta_scan runs the recurrence with the
-//   next tokens' vectors on their way (cp.async), general_delta_norm finishes.
+//   next tokens' vectors on their way (bulk copies), general_delta_norm finishes.
 // The same arithmetic in the same order runs whatever the portions are, so a sequence cut differently gives the same state.
 #include "ptx.cuh"
 
@@ -44,9 +44,9 @@ struct GdArgs {
   const void* norm_w; float eps;             // [H Dv]
   float* state;                              // [S, H, Dv, Dk]
   const int* slots; const int* cu; const int* fresh;
-  float* vec; float* val; float* scal;       // [T, H, 4, DkP]: u, w, a u, r w (zeros past Dk); [T, H, Dv]: |k| v, then o; [T, H, 2]: r.u, r.(a u)
+  float* vec; float* val; float* scal;       // [T, H, 4, DkP]: u, w, a u, r w (zeros past Dk); [T, H, DvP]: |k| v, then o; [T, H, 4]: r.u, r.(a u)
   void* out;                                 // [T, H, Dv]
-  int T, B, H, Dk, Dv, DkP;
+  int T, B, H, Dk, Dv, DkP, DvP;
 };
 
 // Whole warp: the vectors of one (token, head), `ld` floats apart, zeros from Dk to `pad`.  Returns |k|; r.u and r.(a u) in ru, rau.
@@ -107,7 +107,7 @@ __global__ void __launch_bounds__(256) general_delta_prepare_kernel(const GdArgs
   float ru, rau;
   const float kn = head_vectors<T, V>(a, t, h, a.vec + i * 4 * a.DkP, a.DkP, a.DkP, ru, rau);
   const T* v = reinterpret_cast<const T*>(a.proj) + t * a.proj_ld + 3 * a.H * a.Dk + h * a.Dv;
-  float* vo = a.val + i * a.Dv;
+  float* vo = a.val + i * a.DvP;
   if (V == 4 && a.Dv % 4 == 0) {
     for (int c = lane * 4; c < a.Dv; c += 128) {
       float x[4];
@@ -117,19 +117,23 @@ __global__ void __launch_bounds__(256) general_delta_prepare_kernel(const GdArgs
   } else {
     for (int c = lane; c < a.Dv; c += 32) vo[c] = kn * ldg_(v + c);
   }
-  if (lane == 0) { a.scal[i * 2] = ru; a.scal[i * 2 + 1] = rau; }
+  if (lane == 0) { a.scal[i * 4] = ru; a.scal[i * 4 + 1] = rau; }
 }
 
 // One token for the rows of a row group.  S: packed columns j * 32 + cg * 4 + {0, 1}, {2, 3}; vec: u | w | a u | r w, `ld` floats apart; kv: |k| v of
-// the thread's rows, kv_o that of the row whose output this lane returns (see out_row).
-template <int CPL, int R>
+// the thread's rows, kv_o that of the row whose output this lane returns (see out_row).  kHold: u stays in
+// registers for the update.
+template <int CPL, int R, bool kHold>
 __device__ __forceinline__ float delta_token(f2 (&S)[R][CPL / 2], const float* vec, int ld, int cg, const float (&kv)[R], float kv_o, float ru, float rau) {
   f2 p2[R], q2[R];
 #pragma unroll
   for (int r = 0; r < R; r++) p2[r] = q2[r] = 0ull;
+  ulonglong2 uh[kHold ? CPL / 4 : 1];
 #pragma unroll
   for (int j = 0; j < CPL / 4; j++) {
-    const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(vec + j * 32 + cg * 4), q = *reinterpret_cast<const ulonglong2*>(vec + 3 * ld + j * 32 + cg * 4);
+    const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(vec + j * 32 + cg * 4);
+    if (kHold) uh[j] = u;
+    const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(vec + 3 * ld + j * 32 + cg * 4);
 #pragma unroll
     for (int r = 0; r < R; r++) {
       p2[r] = fma2(S[r][2 * j], u.x, p2[r]); q2[r] = fma2(S[r][2 * j], q.x, q2[r]);
@@ -166,7 +170,8 @@ __device__ __forceinline__ float delta_token(f2 (&S)[R][CPL / 2], const float* v
   for (int r = 0; r < R; r++) { kv2[r] = pack2(kv[r], kv[r]); np2[r] = pack2(-p[r], -p[r]); }
 #pragma unroll
   for (int j = 0; j < CPL / 4; j++) {
-    const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(vec + j * 32 + cg * 4), w = *reinterpret_cast<const ulonglong2*>(vec + ld + j * 32 + cg * 4),
+    const ulonglong2 u = kHold ? uh[kHold ? j : 0] : *reinterpret_cast<const ulonglong2*>(vec + j * 32 + cg * 4);
+    const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(vec + ld + j * 32 + cg * 4),
                      au = *reinterpret_cast<const ulonglong2*>(vec + 2 * ld + j * 32 + cg * 4);
 #pragma unroll
     for (int r = 0; r < R; r++) {
@@ -216,113 +221,153 @@ __device__ __forceinline__ void store_state(const f2 (&S)[R][CPL / 2], float* Sg
   }
 }
 
-// Single tokens (a sequence may bring a few): grid (H, B), one CTA holds a head, warps of 16 rows.
-template <int CPL, typename T, int V>
-__global__ void __launch_bounds__(256, CPL >= 8 ? 2 : 3) general_delta_step_kernel(const GdArgs a) {
+// up to four elements from column c of n; vec: one access
+template <typename T>
+__device__ __forceinline__ void ld_up4(const T* p, int c, int n, bool vec, float* o) {
+  if (vec) { if (c < n) ldv4(p + c, o); else o[0] = o[1] = o[2] = o[3] = 0.f; return; }
+#pragma unroll
+  for (int e = 0; e < 4; e++) o[e] = c + e < n ? ldg_(p + c + e) : 0.f;
+}
+
+// Single tokens (a sequence may bring a few): grid (H, B), one CTA holds a head in warps of 16 rows; warp 0 makes the token's vectors while the
+// state is on its way.
+template <int CPL, typename T, bool VEC>
+__global__ void __launch_bounds__(256, 2) general_delta_step_kernel(const GdArgs a) {
   constexpr int DKP = CPL * 8, R = 4;
+  constexpr float kRate = 0.60653065971263342f;      // exp(-1/2)
   __shared__ float4 s_vec4[DKP];             // u | w | a u | r w
-  __shared__ float s_scal[4], s_red[8];
-  float* s_vec = reinterpret_cast<float*>(s_vec4);
+  __shared__ float4 s_kv4[32], s_out4[32];   // v; norm weight * sigmoid(g)
+  __shared__ float s_scal[3], s_red[8];      // r.u, r.(a u), |k|
+  float *s_vec = reinterpret_cast<float*>(s_vec4), *s_kv = reinterpret_cast<float*>(s_kv4), *s_out = reinterpret_cast<float*>(s_out4);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cg = lane & 7, rg = lane >> 3, nw = blockDim.x >> 5;
-  const int h = blockIdx.x, seq = blockIdx.y, Dk = a.Dk, Dv = a.Dv;
+  const int h = blockIdx.x, seq = blockIdx.y, Dk = a.Dk, Dv = a.Dv, hk = a.H * Dk, c = lane * 4;
   // The step's tables and the state are older than the kernel in front (every kernel triggers behind its own wait): fetched while it runs.
   const int start = a.cu[seq], n = a.cu[seq + 1] - start, slot = a.slots[seq];
   if (n <= 0 || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 48, __LINE__)) { pdl_wait(); return; }
   float* Sg = a.state + (((long long)slot * a.H + h) * Dv) * Dk;
+  const bool fresh = a.fresh[seq] != 0;
   f2 S[R][CPL / 2];
-  load_state<CPL, R>(S, Sg, warp * 16, rg, cg, Dv, Dk, a.fresh[seq] != 0);
+  if (warp != 0) load_state<CPL, R>(S, Sg, warp * 16, rg, cg, Dv, Dk, fresh);
   pdl_wait(); pdl_trigger();
   const int orow = out_row<R>(cg), lrow = warp * 16 + max(orow, 0) * 4 + rg;
   for (int i = 0; i < n; i++) {
     const long long t = start + i;
-    const T* v = reinterpret_cast<const T*>(a.proj) + t * a.proj_ld + 3 * a.H * Dk + h * Dv;
-    float kv[R];
+    if (warp == 0) {                         // the vectors' loads in front of the state's
+      const T* p = reinterpret_cast<const T*>(a.proj) + t * a.proj_ld + h * Dk;
+      float r[4], k[4], s[4], z[4], w0[4], ab[4];
+      ld_up4(p + hk, c, Dk, VEC, k); ld_up4(a.decay + t * a.decay_ld + h * Dk, c, Dk, VEC, z); ld_up4(p + 2 * hk, c, Dk, VEC, s); ld_up4(p, c, Dk, VEC, r);
+      ld_up4(a.w0 + h * Dk, c, Dk, VEC, w0); ld_up4(a.a_bias + h * Dk, c, Dk, VEC, ab);
+      if (i == 0) load_state<CPL, R>(S, Sg, 0, rg, cg, Dv, Dk, fresh);
+      const float kk = warp_sum(k[0] * k[0] + k[1] * k[1] + k[2] * k[2] + k[3] * k[3]) + 1e-6f;
+      const float inv = rsqrtf(kk);
+      float ru = 0.f, rau = 0.f, o[4][4];
 #pragma unroll
-    for (int r = 0; r < R; r++) { const int row = warp * 16 + r * 4 + rg; kv[r] = row < Dv ? ldg_(v + row) : 0.f; }
-    if (warp == 0) {
-      float ru, rau;
-      const float kn = head_vectors<T, V>(a, t, h, s_vec, DKP, DKP, ru, rau);
-      if (lane == 0) { s_scal[0] = ru; s_scal[1] = rau; s_scal[2] = kn; }
+      for (int e = 0; e < 4; e++) {
+        const float w = expf(-kRate * sigmoid_(z[e] + w0[e])), u = k[e] * inv, au = sigmoid_(s[e] + ab[e]) * u;
+        o[0][e] = u; o[1][e] = w; o[2][e] = au; o[3][e] = r[e] * w;
+        ru = fmaf(r[e], u, ru); rau = fmaf(r[e], au, rau);
+      }
+      if (c < DKP)
+#pragma unroll
+        for (int x = 0; x < 4; x++) *reinterpret_cast<float4*>(s_vec + x * DKP + c) = make_float4(o[x][0], o[x][1], o[x][2], o[x][3]);
+      ru = warp_sum(ru); rau = warp_sum(rau);
+      if (lane == 0) { s_scal[0] = ru; s_scal[1] = rau; s_scal[2] = kk * inv; }
+    }
+    if (warp == nw / 2) {                    // and another warp those of its rows
+      const T* pv = reinterpret_cast<const T*>(a.proj) + t * a.proj_ld + 3 * hk + h * Dv;
+      float v[4], g[4], nw4[4];
+      ld_up4(pv, c, Dv, VEC, v); ld_up4(pv + a.H * Dv, c, Dv, VEC, g); ld_up4(reinterpret_cast<const T*>(a.norm_w) + h * Dv, c, Dv, VEC, nw4);
+      s_kv4[lane] = make_float4(v[0], v[1], v[2], v[3]);
+      s_out4[lane] = make_float4(nw4[0] * sigmoid_(g[0]), nw4[1] * sigmoid_(g[1]), nw4[2] * sigmoid_(g[2]), nw4[3] * sigmoid_(g[3]));
     }
     __syncthreads();
     const float kn = s_scal[2];
+    float kv[R];
 #pragma unroll
-    for (int r = 0; r < R; r++) kv[r] *= kn;
-    const float kv_o = orow <= 0 ? kv[0] : orow == 1 ? kv[1] : orow == 2 ? kv[2] : kv[3];
-    const float o = delta_token<CPL, R>(S, s_vec, DKP, cg, kv, kv_o, s_scal[0], s_scal[1]);
+    for (int r = 0; r < R; r++) kv[r] = kn * s_kv[warp * 16 + r * 4 + rg];
+    const float o = delta_token<CPL, R, false>(S, s_vec, DKP, cg, kv, kn * s_kv[lrow], s_scal[0], s_scal[1]);
     const bool mine = orow >= 0 && lrow < Dv;
     const float ss = warp_sum(mine ? o * o : 0.f);
     if (lane == 0) s_red[warp] = ss;
+    if (i + 1 == n) store_state<CPL, R>(S, Sg, warp * 16, rg, cg, Dv, Dk);
     __syncthreads();
     float tot = 0.f;
     for (int w = 0; w < nw; w++) tot += s_red[w];
-    if (mine) {
-      const float g = ldg_(v + a.H * Dv + lrow);
-      stg_(reinterpret_cast<T*>(a.out) + (t * a.H + h) * Dv + lrow,
-           o * rsqrtf(tot / (float)Dv + a.eps) * ldg_(reinterpret_cast<const T*>(a.norm_w) + h * Dv + lrow) * sigmoid_(g));
-    }
+    if (mine) stg_(reinterpret_cast<T*>(a.out) + (t * a.H + h) * Dv + lrow, o * rsqrtf(tot / (float)Dv + a.eps) * s_out[lrow]);
     if (i + 1 < n) __syncthreads();          // the vectors and sums are read by now
   }
-  store_state<CPL, R>(S, Sg, warp * 16, rg, cg, Dv, Dk);
 }
 
-__device__ __forceinline__ void cp_async4_(uint32_t dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
+// untiled bulk copy: addresses and size in multiples of 16 bytes
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
+constexpr int kKernelGd = 15;
 
-// grid = (H * splits, B), 4 warps of 4 R rows; `splits` CTAs share a head's Dv rows.  CH tokens are staged at a time, two buffers.
+// grid = (H * splits, B), 4 warps of 4 R rows; `splits` CTAs share a head's Dv rows.  CH tokens are staged at a time, two buffers; warp 0 issues the
+// copies of a token's vectors, one bulk copy each.
 template <int CPL, int R, int CH>
 __global__ void __launch_bounds__(128, CPL * R >= 64 ? 3 : CPL * R >= 32 ? 4 : 6) general_delta_scan_kernel(const GdArgs a) {
   constexpr int DKP = CPL * 8, rows = 16 * R, kBuf = CH * (4 * DKP + rows + 4);
-  extern __shared__ __align__(16) float sm[];                     // per buffer: vectors [CH][4][DKP] | |k| v [CH][rows] | r.u, r.(a u) [CH][4]
+  extern __shared__ __align__(128) float sm[];                    // per buffer: vectors [CH][4][DKP] | |k| v [CH][rows] | r.u, r.(a u) [CH][4]
+  __shared__ uint64_t bars[2];
+  __shared__ int abort_word;
+  volatile int* abort_flag = &abort_word;
   const int splits = gridDim.x / a.H, h = blockIdx.x / splits, row0 = (blockIdx.x % splits) * rows;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cg = lane & 7, rg = lane >> 3;
-  const int Dk = a.Dk, Dv = a.Dv, DkP = a.DkP, seq = blockIdx.y;
+  const int Dk = a.Dk, Dv = a.Dv, seq = blockIdx.y;
   const int start = a.cu[seq], n = a.cu[seq + 1] - start, slot = a.slots[seq];
   if (n <= 0 || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 49, __LINE__)) return;
-  for (int i = threadIdx.x; i < 2 * kBuf; i += blockDim.x) sm[i] = 0.f;      // columns past DkP and rows past Dv stay zero
+  if (threadIdx.x == 0) { mbar_init(smem_u32(bars), 1); mbar_init(smem_u32(bars + 1), 1); abort_word = 0; mbar_fence_init(); }
   __syncthreads();
-  const int pieces = DkP;                                           // 16-byte pieces of a token's four vectors
-  auto stage = [&](int buf, int i0) {
+  const int vrows = min(rows, a.DvP - row0);                       // a multiple of 4; rows past Dv read whatever their scratch holds and are not kept
+  auto stage = [&](int buf, int i0) {                              // warp 0
     const int m = min(CH, n - i0);
     float* base = sm + buf * kBuf;
-    const long long t0 = start + i0;
-    for (int i = threadIdx.x; i < m * pieces; i += blockDim.x) {
-      const int tok = i / pieces, c = (i - tok * pieces) * 4, which = c / DkP;
-      cp_async16(smem_u32(base + (tok * 4 + which) * DKP + c - which * DkP), a.vec + ((t0 + tok) * a.H + h) * 4 * DkP + c, 16);
+    const uint32_t bar = smem_u32(bars + buf);
+    if (lane == 0) mbar_expect_tx(bar, m * (4 * DKP + vrows + 4) * 4);
+    __syncwarp();
+    for (int i = lane; i < 3 * m; i += 32) {
+      const int tok = i / 3, which = i - 3 * tok;
+      const long long th = (long long)(start + i0 + tok) * a.H + h;
+      if (which == 0) bulk_load(smem_u32(base + tok * 4 * DKP), a.vec + th * 4 * DKP, 16 * DKP, bar);
+      else if (which == 1) bulk_load(smem_u32(base + CH * 4 * DKP + tok * rows), a.val + th * a.DvP + row0, vrows * 4, bar);
+      else bulk_load(smem_u32(base + CH * (4 * DKP + rows) + tok * 4), a.scal + th * 4, 16, bar);
     }
-    float* sv = base + CH * 4 * DKP;
-    for (int i = threadIdx.x; i < m * rows; i += blockDim.x) {
-      const int r = i % rows, tok = i / rows;
-      if (row0 + r < Dv) cp_async4_(smem_u32(sv + i), a.val + ((t0 + tok) * a.H + h) * Dv + row0 + r);
-    }
-    float* sg = sv + CH * rows;
-    if ((int)threadIdx.x < m * 2) cp_async4_(smem_u32(sg + (threadIdx.x >> 1) * 4 + (threadIdx.x & 1)), a.scal + ((t0 + (threadIdx.x >> 1)) * a.H + h) * 2 + (threadIdx.x & 1));
-    cp_async_commit();
   };
-  stage(0, 0);
+  if (warp == 0) stage(0, 0);
   float* Sg = a.state + (((long long)slot * a.H + h) * Dv) * Dk;
   f2 S[R][CPL / 2];
   const int wrow = warp * 4 * R;
   load_state<CPL, R>(S, Sg, row0 + wrow, rg, cg, Dv, Dk, a.fresh[seq] != 0);
   const int orow = out_row<R>(cg), lrow = wrow + max(orow, 0) * 4 + rg;
-  for (int i0 = 0, buf = 0; i0 < n; i0 += CH, buf ^= 1) {
-    const int m = min(CH, n - i0);
-    if (i0 + CH < n) { stage(buf ^ 1, i0 + CH); cp_async_wait<1>(); } else cp_async_wait<0>();
-    __syncthreads();
-    const float* sv = sm + buf * kBuf + CH * 4 * DKP;
-    const float* sg = sv + CH * rows;
+  const bool keep = orow >= 0 && row0 + lrow < Dv;
+  bool ok = true;
+  for (int i0 = 0, it = 0; i0 < n; i0 += CH, it++) {
+    const int m = min(CH, n - i0), buf = it & 1;
+    if (warp == 0 && i0 + CH < n) stage(buf ^ 1, i0 + CH);
+    if (!mbar_wait(smem_u32(bars + buf), (it >> 1) & 1, abort_flag, kKernelGd, 400 + buf)) { ok = false; *abort_flag = 1; }
+    const float* vec = sm + buf * kBuf;
+    const float *sv = vec + CH * 4 * DKP, *sg = sv + CH * rows;
+    float* ov = a.val + ((long long)(start + i0) * a.H + h) * a.DvP + row0 + lrow;       // |k| v of these places has been read
+#pragma unroll 2
     for (int i = 0; i < m; i++) {
       float kv[R];
 #pragma unroll
       for (int r = 0; r < R; r++) kv[r] = sv[i * rows + wrow + r * 4 + rg];
       const float2 gt = *reinterpret_cast<const float2*>(sg + i * 4);
-      const float o = delta_token<CPL, R>(S, sm + buf * kBuf + i * 4 * DKP, DKP, cg, kv, sv[i * rows + lrow], gt.x, gt.y);
-      if (orow >= 0 && row0 + lrow < Dv) a.val[((start + i0 + i) * (long long)a.H + h) * Dv + row0 + lrow] = o;      // |k| v of this place has been read
+      const float o = delta_token<CPL, R, (CPL <= 16)>(S, vec + i * 4 * DKP, DKP, cg, kv, sv[i * rows + lrow], gt.x, gt.y);
+      if (keep) ov[(long long)i * a.H * a.DvP] = o;
     }
     __syncthreads();          // everyone is done with this buffer before the next-but-one chunk is copied into it
+    if (*abort_flag) break;
   }
-  store_state<CPL, R>(S, Sg, row0 + wrow, rg, cg, Dv, Dk);
+  if (*abort_flag) {          // a wait gave up (reported): copies in flight land before the CTA goes; the state is left as it was
+    if (threadIdx.x == 0) for (int i = 0; i < 2000; i++) __nanosleep(1000);
+    __syncthreads();
+    return;
+  }
+  if (ok) store_state<CPL, R>(S, Sg, row0 + wrow, rg, cg, Dv, Dk);
 }
 
 // One warp per (token, head): out = o / rms(o) * norm_w * sigmoid(g).  V = 4: sizes, strides and addresses allow groups of four.
@@ -332,7 +377,7 @@ __global__ void __launch_bounds__(256) general_delta_norm_kernel(const GdArgs a)
   const long long i = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (i >= (long long)a.T * a.H) return;
   const int lane = threadIdx.x & 31, h = (int)(i % a.H), Dv = a.Dv;
-  const float* o = a.val + i * Dv;
+  const float* o = a.val + i * a.DvP;
   const T* g = reinterpret_cast<const T*>(a.proj) + (i / a.H) * a.proj_ld + a.H * (3 * a.Dk + Dv) + h * Dv;
   const T* w = reinterpret_cast<const T*>(a.norm_w) + h * Dv;
   T* out = reinterpret_cast<T*>(a.out) + i * Dv;
@@ -361,7 +406,7 @@ __global__ void __launch_bounds__(256) general_delta_norm_kernel(const GdArgs a)
 
 template <int CPL, int R>
 static int gd_scan(const GdArgs& a, cudaStream_t st) {
-  constexpr int CH = CPL <= 16 ? 16 : CPL <= 32 ? 8 : 4, rows = 16 * R;
+  constexpr int CH = CPL <= 32 ? 8 : 4, rows = 16 * R;
   const size_t smem = sizeof(float) * 2 * CH * (4 * CPL * 8 + rows + 4);
   auto k = general_delta_scan_kernel<CPL, R, CH>;
   cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -371,6 +416,8 @@ static int gd_scan(const GdArgs& a, cudaStream_t st) {
   return (int)cudaGetLastError();
 }
 
+// columns a row is held in: 8 lanes times the columns of the kernel that takes the size
+static int gd_padded(int Dk) { return Dk <= 32 ? 32 : Dk <= 64 ? 64 : Dk <= 96 ? 96 : Dk <= 128 ? 128 : Dk <= 192 ? 192 : Dk <= 256 ? 256 : 512; }
 static bool gd_whole(int Dk, int Dv, int max_q) { return max_q <= 2 && Dk <= 128 && Dv <= 128; }
 
 template <typename T>
@@ -379,15 +426,15 @@ static int general_delta_t(const GdArgs& a, int max_q, cudaStream_t st) {
                      ((uintptr_t)a.proj | (uintptr_t)a.decay | (uintptr_t)a.w0 | (uintptr_t)a.a_bias | (uintptr_t)a.norm_w | (uintptr_t)a.out) % 16 == 0;
   if (gd_whole(a.Dk, a.Dv, max_q)) {
     const dim3 grid((unsigned)a.H, (unsigned)a.B), block((unsigned)((a.Dv + 15) / 16 * 32));
-#define NE_STEP(CPL_) (int)launch_pdl(fours ? general_delta_step_kernel<CPL_, T, 4> : general_delta_step_kernel<CPL_, T, 1>, grid, block, 0, st, a)
+#define NE_STEP(CPL_) (int)launch_pdl(fours ? general_delta_step_kernel<CPL_, T, true> : general_delta_step_kernel<CPL_, T, false>, grid, block, 0, st, a)
     return a.Dk <= 32 ? NE_STEP(4) : a.Dk <= 64 ? NE_STEP(8) : a.Dk <= 96 ? NE_STEP(12) : NE_STEP(16);
 #undef NE_STEP
   }
   const dim3 wgrid((unsigned)(((long long)a.T * a.H + 7) / 8));
   cudaError_t e = launch_pdl(fours ? general_delta_prepare_kernel<T, 4> : general_delta_prepare_kernel<T, 1>, wgrid, dim3(256), 0, st, a);
   if (e != cudaSuccess) return (int)e;
-  // rows spread over the machine: two rows per thread while that leaves warp schedulers idle, four otherwise
-  const bool wide = (long long)a.H * a.Dv * a.B >= 148ll * 4 * 16 * 2;
+  // the vectors of a token are read from shared memory by every warp, whatever its rows: four rows per thread, unless that leaves SMs idle
+  const bool wide = (long long)a.H * a.Dv * a.B > 148ll * 64;
 #define NE_SCAN(CPL_) (wide ? gd_scan<CPL_, 4>(a, st) : gd_scan<CPL_, 2>(a, st))
   int rc;
   if (a.Dk <= 32) rc = NE_SCAN(4);
@@ -409,8 +456,7 @@ using namespace ne;
 // fp32 elements of scratch a call needs (none for single-token steps whose heads fit a CTA)
 extern "C" long long ne_general_delta_scratch(int T, int H, int Dk, int Dv, int max_q) {
   if (gd_whole(Dk, Dv, max_q)) return 0;
-  const long long th = (long long)T * H, DkP = (Dk + 3) / 4 * 4;
-  return th * 4 * DkP + (th * Dv + 3) / 4 * 4 + th * 2;
+  return (long long)T * H * (4 * gd_padded(Dk) + (Dv + 3) / 4 * 4 + 4);
 }
 
 extern "C" int ne_general_delta(const void* proj, long long proj_ld, const float* decay, long long decay_ld, const float* w0, const float* a_bias, const void* norm_w,
@@ -422,9 +468,9 @@ extern "C" int ne_general_delta(const void* proj, long long proj_ld, const float
   if (!whole && (!scratch || ((uintptr_t)scratch & 15))) return 1002;
   GdArgs a;
   a.proj = proj; a.proj_ld = proj_ld; a.decay = decay; a.decay_ld = decay_ld; a.w0 = w0; a.a_bias = a_bias; a.norm_w = norm_w; a.eps = eps; a.state = state;
-  a.slots = slots; a.cu = cu; a.fresh = fresh; a.out = out; a.T = T; a.B = B; a.H = H; a.Dk = Dk; a.Dv = Dv; a.DkP = (Dk + 3) / 4 * 4;
+  a.slots = slots; a.cu = cu; a.fresh = fresh; a.out = out; a.T = T; a.B = B; a.H = H; a.Dk = Dk; a.Dv = Dv; a.DkP = gd_padded(Dk); a.DvP = (Dv + 3) / 4 * 4;
   const long long th = (long long)T * H;
-  a.vec = scratch; a.val = whole ? nullptr : a.vec + th * 4 * a.DkP; a.scal = whole ? nullptr : a.val + (th * Dv + 3) / 4 * 4;
+  a.vec = scratch; a.val = whole ? nullptr : a.vec + th * 4 * a.DkP; a.scal = whole ? nullptr : a.val + th * a.DvP;
   *launches = whole ? 1 : 3;
   return fp32 ? general_delta_t<float>(a, max_q, st) : general_delta_t<__nv_bfloat16>(a, max_q, st);
 }

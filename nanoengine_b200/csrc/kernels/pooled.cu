@@ -31,38 +31,69 @@ struct PoolArgs {
   int T, H, G, D, Dv, dims, pool, block_size, pool_rows;
 };
 
-// The block that token t completes (nothing to do when it completes none).  Whole CTA.
-template <typename T, int V>
-__device__ __forceinline__ void pool_block(const PoolArgs& a, int t) {
-  const long long p = a.positions[t];
-  if (p < 0 || (p + 1) % a.pool || a.slots[t] < 0) return;
+constexpr int kOffs = 64;                    // rows whose places are looked up at a time
+
+// Where the pooled row goes that token t completes: row of the pooled caches, -1 when it completes none.  bt: the sequence's block table.
+__device__ __forceinline__ long long block_place(const PoolArgs& a, int t, long long p, const int*& bt) {
+  if (p < 0 || (p + 1) % a.pool || a.slots[t] < 0) return -1;
   int lo = 0, hi = a.B - 1;                   // last sequence whose first token is <= t
+  if (t < a.B && a.cu[t] == t && a.cu[t + 1] == t + 1) lo = hi = t;      // single tokens
   while (lo < hi) { const int mid = (lo + hi + 1) >> 1; if (a.cu[mid] <= t) lo = mid; else hi = mid - 1; }
-  const int* bt = a.block_tables + (long long)lo * a.bt_stride;
-  const int b = (int)(p / a.pool), bs = a.block_size;
+  bt = a.block_tables + (long long)lo * a.bt_stride;
   int page, row;
-  pooled_place(b, a.pool, bs, page, row);
-  if (page >= a.bt_stride || p / bs >= a.bt_stride) { if (threadIdx.x == 0) report(ST_BAD_INDEX, 50, t, page); return; }
-  const long long dst = bt[page];
-  if (!NE_INDEX_OK(dst, BK_CACHE_PAGES, 50, __LINE__)) return;
-  const int kw = a.G * a.D, vw = a.G * a.Dv;
+  pooled_place((int)(p / a.pool), a.pool, a.block_size, page, row);
+  if (page >= a.bt_stride || p / a.block_size >= a.bt_stride) { if (threadIdx.x == 0) report(ST_BAD_INDEX, 50, t, page); return -1; }
+  const int dst = bt[page];
+  return NE_INDEX_OK(dst, BK_CACHE_PAGES, 50, __LINE__) ? (long long)dst * a.pool_rows + row : -1;
+}
+
+// Mean of rows p - pool + 1 .. p into pooled row `dst`, summed in the order of positions.  Whole CTA; the rows are stored by now.
+template <typename T, int V>
+__device__ __forceinline__ void pool_block(const PoolArgs& a, long long p, long long dst, const int* bt, long long* offs) {
+  const int kw = a.G * a.D, vw = a.G * a.Dv, bs = a.block_size;
   const float inv = 1.f / (float)a.pool;
-  for (int c = threadIdx.x * V; c < kw + vw; c += blockDim.x * V) {       // V divides kw: a group never straddles
-    const bool key = c < kw;
+  for (int c0 = 0; c0 < kw + vw; c0 += blockDim.x * V) {
+    const int c = c0 + threadIdx.x * V;                                   // V divides kw: a group never straddles
+    const bool key = c < kw, on = c < kw + vw;
     const int w = key ? kw : vw, cc = key ? c : c - kw;
     const T* src = reinterpret_cast<const T*>(key ? a.k_cache : a.v_cache) + cc;
-    T* out = reinterpret_cast<T*>(key ? a.k_pool : a.v_pool) + (dst * a.pool_rows + row) * w + cc;
     float s[V];
 #pragma unroll
     for (int e = 0; e < V; e++) s[e] = 0.f;
-#pragma unroll 4
-    for (int j = 0; j < a.pool; j++) {
-      const int q = (int)p - a.pool + 1 + j, pg = bt[q / bs];
-      if (!NE_INDEX_OK(pg, BK_CACHE_PAGES, 51, __LINE__)) continue;
-      const T* r = src + ((long long)pg * bs + q % bs) * w;
-      if constexpr (V == 4) { const float4 v = pl_ld4(r); s[0] += v.x; s[1] += v.y; s[2] += v.z; s[3] += v.w; }
-      else s[0] += pl_ld(r);
+    for (int j0 = 0; j0 < a.pool; j0 += kOffs) {
+      const int m = min(kOffs, a.pool - j0);
+      if (a.pool > kOffs || c0 == 0) {
+        __syncthreads();
+        if ((int)threadIdx.x < m) {
+          const int q = (int)p - a.pool + 1 + j0 + threadIdx.x, pg = bt[q / bs];
+          offs[threadIdx.x] = NE_INDEX_OK(pg, BK_CACHE_PAGES, 51, __LINE__) ? (long long)pg * bs + q % bs : 0;
+        }
+        __syncthreads();
+      }
+      if (!on) continue;
+      int j = 0;
+      for (; j + 8 <= m; j += 8) {
+        if constexpr (V == 4) {
+          float4 v[8];
+#pragma unroll
+          for (int e = 0; e < 8; e++) v[e] = pl_ld4(src + offs[j + e] * w);
+#pragma unroll
+          for (int e = 0; e < 8; e++) { s[0] += v[e].x; s[1] += v[e].y; s[2] += v[e].z; s[3] += v[e].w; }
+        } else {
+          float v[8];
+#pragma unroll
+          for (int e = 0; e < 8; e++) v[e] = pl_ld(src + offs[j + e] * w);
+#pragma unroll
+          for (int e = 0; e < 8; e++) s[0] += v[e];
+        }
+      }
+      for (; j < m; j++) {
+        if constexpr (V == 4) { const float4 v = pl_ld4(src + offs[j] * w); s[0] += v.x; s[1] += v.y; s[2] += v.z; s[3] += v.w; }
+        else s[0] += pl_ld(src + offs[j] * w);
+      }
     }
+    if (!on) continue;
+    T* out = reinterpret_cast<T*>(key ? a.k_pool : a.v_pool) + dst * w + cc;
     if constexpr (V == 4) pl_st4(out, make_float4(s[0] * inv, s[1] * inv, s[2] * inv, s[3] * inv));
     else pl_st(out, s[0] * inv);
   }
@@ -73,6 +104,7 @@ __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, c
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   extern __shared__ __align__(16) float sm[];       // the row (fp32) | key table | value table
   __shared__ float red[2][16];
+  __shared__ long long offs[kOffs];
   const int t = blockIdx.x, nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.Dv, W = nq + nk + nv, D = a.D, Dv = a.Dv, dims = a.dims;
   float* s_kt = sm + (W + 3) / 4 * 4;
   float* s_vt = s_kt + (dims + 3) / 4 * 4;
@@ -80,6 +112,8 @@ __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, c
   long long p = a.positions[t];
   const long long slot = a.slots[t];
   if (p < 0 || p >= a.n_pos) { if (threadIdx.x == 0) report(ST_BAD_INDEX, 52, t, (int)p); p = 0; }
+  const int* bt = nullptr;
+  const long long place = pool_here ? block_place(a, t, p, bt) : -1;
   for (int i = threadIdx.x; i < dims; i += blockDim.x) s_kt[i] = a.k_table[p * dims + i];
   for (int i = threadIdx.x; i < Dv; i += blockDim.x) s_vt[i] = a.v_table[p * Dv + i];
   float qq = 0.f, kk = 0.f;
@@ -98,49 +132,54 @@ __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, c
   __syncthreads();
   const float rq = rsqrtf(warp_sum(lane < nw ? red[0][lane] : 0.f) / (float)nq + a.eps), rk = rsqrtf(warp_sum(lane < nw ? red[1][lane] : 0.f) / (float)nk + a.eps);
   const bool store = slot >= 0 && NE_INDEX_OK(slot, BK_CACHE_ROWS, 53, __LINE__);
-  const T *qw = reinterpret_cast<const T*>(a.q_norm), *kw = reinterpret_cast<const T*>(a.k_norm);
-  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
-    const int part = i < nq ? 0 : i < nq + nk ? 1 : 2;
-    const int j = part == 0 ? i : part == 1 ? i - nq : i - nq - nk;        // column within q, k or v
-    if (part && !store) continue;
-    const int width = part == 2 ? Dv : D, turned = part == 2 ? Dv : dims, half = turned >> 1, d = j % width;
+  const float* x0 = sm;                              // one warp per head; V divides the head sizes and the halves of the rotations
+  for (int u = warp; u < a.H + 2 * a.G; u += nw) {
+    const int part = u < a.H ? 0 : u < a.H + a.G ? 1 : 2;
+    if (part && !store) break;
+    const int j0 = part == 0 ? u * D : part == 1 ? (u - a.H) * D : (u - a.H - a.G) * Dv, i0 = part == 0 ? j0 : part == 1 ? nq + j0 : nq + nk + j0;
+    const int width = part == 2 ? Dv : D, turned = part == 2 ? Dv : dims, half = turned >> 1;
     const float* tab = part == 2 ? s_vt : s_kt;
-    const T* w = part == 0 ? qw : kw;
+    const T* w = reinterpret_cast<const T*>(part == 0 ? a.q_norm : a.k_norm) + j0;
     const float r = part == 0 ? rq : rk;
-    // columns d .. d + V - 1 lie on one side of the rotation: V divides half and width
-    const int other = d < half ? half : -half, ti = d < half ? d : d - half;
-    const float sign = d < half ? -1.f : 1.f;
-    T* dst = part == 0 ? row + i : part == 1 ? reinterpret_cast<T*>(a.k_cache) + slot * nk + j : reinterpret_cast<T*>(a.v_cache) + slot * nv + j;
-    if constexpr (V == 4) {
-      float4 x = *reinterpret_cast<const float4*>(sm + i);
-      if (part < 2) { const float4 g = pl_ld4(w + j); x.x *= r * g.x; x.y *= r * g.y; x.z *= r * g.z; x.w *= r * g.w; }
-      if (d < turned) {
-        float4 y = *reinterpret_cast<const float4*>(sm + i + other);
-        if (part < 2) { const float4 g = pl_ld4(w + j + other); y.x *= r * g.x; y.y *= r * g.y; y.z *= r * g.z; y.w *= r * g.w; }
-        const float4 c = *reinterpret_cast<const float4*>(tab + ti), s = *reinterpret_cast<const float4*>(tab + half + ti);
-        x.x = x.x * c.x + sign * y.x * s.x; x.y = x.y * c.y + sign * y.y * s.y; x.z = x.z * c.z + sign * y.z * s.z; x.w = x.w * c.w + sign * y.w * s.w;
+    T* dst = part == 0 ? row + j0 : part == 1 ? reinterpret_cast<T*>(a.k_cache) + slot * nk + j0 : reinterpret_cast<T*>(a.v_cache) + slot * nv + j0;
+    for (int d = lane * V; d < width; d += 32 * V) {
+      const int other = d < half ? d + half : d - half, ti = d < half ? d : d - half;
+      const float sign = d < half ? -1.f : 1.f;
+      if constexpr (V == 4) {
+        float4 x = *reinterpret_cast<const float4*>(x0 + i0 + d);
+        if (part < 2) { const float4 g = pl_ld4(w + d); x.x *= r * g.x; x.y *= r * g.y; x.z *= r * g.z; x.w *= r * g.w; }
+        if (d < turned) {
+          float4 y = *reinterpret_cast<const float4*>(x0 + i0 + other);
+          if (part < 2) { const float4 g = pl_ld4(w + other); y.x *= r * g.x; y.y *= r * g.y; y.z *= r * g.z; y.w *= r * g.w; }
+          const float4 c = *reinterpret_cast<const float4*>(tab + ti), s = *reinterpret_cast<const float4*>(tab + half + ti);
+          x.x = x.x * c.x + sign * y.x * s.x; x.y = x.y * c.y + sign * y.y * s.y; x.z = x.z * c.z + sign * y.z * s.z; x.w = x.w * c.w + sign * y.w * s.w;
+        }
+        pl_st4(dst + d, x);
+      } else {
+        float x = x0[i0 + d];
+        if (part < 2) x *= r * pl_ld(w + d);
+        if (d < turned) {
+          float y = x0[i0 + other];
+          if (part < 2) y *= r * pl_ld(w + other);
+          x = x * tab[ti] + sign * y * tab[half + ti];
+        }
+        pl_st(dst + d, x);
       }
-      pl_st4(dst, x);
-    } else {
-      float x = sm[i];
-      if (part < 2) x *= r * pl_ld(w + j);
-      if (d < turned) {
-        float y = sm[i + other];
-        if (part < 2) y *= r * pl_ld(w + j + other);
-        x = x * tab[ti] + sign * y * tab[half + ti];
-      }
-      pl_st(dst, x);
     }
   }
-  if (!pool_here) return;
+  if (place < 0) return;
   __syncthreads();                                   // this token's rows are stored
-  pool_block<T, V>(a, t);
+  pool_block<T, V>(a, p, place, bt, offs);
 }
 
 template <typename T, int V>
 __global__ void __launch_bounds__(256) pooled_means_kernel(const PoolArgs a) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
-  pool_block<T, V>(a, blockIdx.x);
+  __shared__ long long offs[kOffs];
+  const long long p = a.positions[blockIdx.x];
+  const int* bt = nullptr;
+  const long long place = block_place(a, blockIdx.x, p, bt);
+  if (place >= 0) pool_block<T, V>(a, p, place, bt, offs);
 }
 
 template <typename T>
@@ -150,7 +189,8 @@ static int pooled_t(const PoolArgs& a, int max_q, cudaStream_t st) {
   const bool vec = a.D % 4 == 0 && a.Dv % 8 == 0 && a.dims % 8 == 0 && a.ld % 4 == 0 && al % 16 == 0;
   const int per = vec ? 4 : 1;
   int threads = ((W + per - 1) / per + 31) / 32 * 32;
-  threads = threads > 512 ? 512 : threads;
+  const int most = max_q == 1 ? 512 : 256;           // few CTAs: wide ones
+  threads = threads > most ? most : threads < 64 ? 64 : threads;
   const size_t smem = sizeof(float) * ((size_t)(W + 3) / 4 * 4 + (a.dims + 3) / 4 * 4 + a.Dv);
   auto k = vec ? pooled_prepare_kernel<T, 4> : pooled_prepare_kernel<T, 1>;
   if (smem > 40 * 1024) {
@@ -161,7 +201,7 @@ static int pooled_t(const PoolArgs& a, int max_q, cudaStream_t st) {
   cudaError_t e = launch_pdl(k, dim3((unsigned)a.T), dim3((unsigned)threads), smem, st, a, max_q == 1 ? 1 : 0);
   if (e != cudaSuccess || max_q == 1) return (int)e;
   int mt = (a.G * (a.D + a.Dv) / per + 31) / 32 * 32;
-  mt = mt > 256 ? 256 : mt < 32 ? 32 : mt;
+  mt = mt > 256 ? 256 : mt < 64 ? 64 : mt;           // at least kOffs threads
   return (int)launch_pdl(vec ? pooled_means_kernel<T, 4> : pooled_means_kernel<T, 1>, dim3((unsigned)a.T), dim3((unsigned)mt), 0, st, a);
 }
 
