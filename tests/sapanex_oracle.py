@@ -50,14 +50,13 @@ def yarn_frequencies(dims, base, scaling):
 
 def rotate(x, freq, factor=1.0, back=False):
     """x [n, heads, width], row = position: the first 2 len(freq) columns turn (column i with column i + len(freq)), the rest pass."""
-    n, half = x.shape[0], len(freq)
+    half = len(freq)
     out = x.clone()
-    for p in range(n):
-        for i, f in enumerate(freq):
-            a = (-p if back else p) * f
-            c, s = math.cos(a) * factor, math.sin(a) * factor
-            u, v = x[p, :, i], x[p, :, i + half]
-            out[p, :, i], out[p, :, i + half] = u * c - v * s, v * c + u * s
+    for p in range(x.shape[0]):
+        a = torch.tensor([(-p if back else p) * f for f in freq], dtype=torch.float64)
+        c, s = (a.cos() * factor).to(x.dtype), (a.sin() * factor).to(x.dtype)
+        u, v = x[p, :, :half], x[p, :, half: 2 * half]
+        out[p, :, :half], out[p, :, half: 2 * half] = u * c - v * s, v * c + u * s
     return out
 
 
@@ -75,16 +74,19 @@ def visible(i, size, pool):
     return tokens, blocks
 
 
-def window_attention(q, k, v, scale, size, pool):
-    """q [n, H, d], k [n, G, d], v [n, G, dv] -> [n, H, dv]."""
+def window_attention(q, k, v, scale, size, pool, hide=None):
+    """q [n, H, d], k [n, G, d], v [n, G, dv] -> [n, H, dv].  `hide` plants a mistake: hide(i) gives the tokens and the blocks query i leaves out."""
     n, H, _ = q.shape
     rep = H // k.shape[1]
     kb, vb = pool_blocks(k, pool), pool_blocks(v, pool)
     out = torch.zeros(n, H, v.shape[2], dtype=q.dtype)
     for i in range(n):
         tokens, blocks = visible(i, size, pool)
-        keys = torch.stack([k[j] for j in tokens] + [kb[b] for b in blocks])
-        values = torch.stack([v[j] for j in tokens] + [vb[b] for b in blocks])
+        if hide is not None:
+            no_tokens, no_blocks = hide(i)
+            tokens, blocks = [j for j in tokens if j not in no_tokens or j == i], [b for b in blocks if b not in no_blocks]
+        keys = torch.cat([k[tokens]] + [kb[b][None] for b in blocks])
+        values = torch.cat([v[tokens]] + [vb[b][None] for b in blocks])
         for h in range(H):
             s = keys[:, h // rep] @ q[i, h] * scale
             e = torch.exp(s - s.max())
@@ -92,7 +94,7 @@ def window_attention(q, k, v, scale, size, pool):
     return out
 
 
-def attention(h, W, m, eps):
+def attention(h, W, m, eps, hide=None):
     n, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q = rms_norm(h @ W["q"].T, W["q.norm"], eps).view(n, H, d)
     k = rms_norm(h @ W["k"].T, W["k.norm"], eps).view(n, G, d)
@@ -100,16 +102,26 @@ def attention(h, W, m, eps):
     freq, factor = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
     vfreq = plain_frequencies(dv, m["rot"]["base"])
     q, k, v = rotate(q, freq, factor), rotate(k, freq, factor), rotate(v, vfreq)
-    o = window_attention(q, k, v, m["scale"], m["mask"]["size"], m["mask"]["pool"])
+    o = window_attention(q, k, v, m["scale"], m["mask"]["size"], m["mask"]["pool"], hide)
     return rotate(o, vfreq, back=True).reshape(n, H * dv) @ W["o"].T
 
 
 # ---- generalised delta rule --------------------------------------------------------------------------------------------
 def delta_step(S, r, k, v, w, a):
-    """One head, one token: S [dim of keys, dim of values]."""
-    u = k / torch.sqrt((k * k).sum() + 1e-6)
-    new = w[:, None] * S - (a * u)[:, None] * (u @ S)[None, :] + k[:, None] * v[None, :]
-    return new, new.T @ r
+    """One token: S [heads, dim of keys, dim of values], the rest [heads, dim]."""
+    u = k / torch.sqrt((k * k).sum(-1, keepdim=True) + 1e-6)
+    seen = (u[:, :, None] * S).sum(1)                                        # u^T S
+    new = w[:, :, None] * S - (a * u)[:, :, None] * seen[:, None, :] + k[:, :, None] * v[:, None, :]
+    return new, (new * r[:, :, None]).sum(1)
+
+
+def recurrence(r, k, v, w, a):
+    """[n, heads, dim] each -> o [n, heads, dim of values] and the state after the last token."""
+    S = torch.zeros(r.shape[1], r.shape[2], v.shape[2], dtype=r.dtype)
+    o = torch.zeros(r.shape[0], r.shape[1], v.shape[2], dtype=r.dtype)
+    for t in range(r.shape[0]):
+        S, o[t] = delta_step(S, r[t], k[t], v[t], w[t], a[t])
+    return o, S
 
 
 def general_delta(h, W, m, eps):
@@ -117,11 +129,7 @@ def general_delta(h, W, m, eps):
     r, k, v = ((h @ W[x].T).view(n, H, d) for x in ("r", "k", "v"))
     w = torch.exp(-math.exp(-0.5) * sigmoid(torch.tanh(h @ W["w1"].T) @ W["w2"].T + W["w0"])).view(n, H, d)
     a = sigmoid(h @ W["a"].T + W["a.b"]).view(n, H, d)
-    o = torch.zeros(n, H, d, dtype=h.dtype)
-    for head in range(H):
-        S = torch.zeros(d, d, dtype=h.dtype)
-        for t in range(n):
-            S, o[t, head] = delta_step(S, r[t, head], k[t, head], v[t, head], w[t, head], a[t, head])
+    o, _ = recurrence(r, k, v, w, a)
     o = unit_rms(o, eps).reshape(n, H * d) * W["norm"] * sigmoid(h @ W["g"].T)
     return o @ W["o"].T
 
@@ -131,14 +139,15 @@ def part(weights, prefix):
     return {k[len(prefix):]: v for k, v in weights.items() if k.startswith(prefix)}
 
 
-def forward(cfg, weights, tokens, layers_out=None):
-    """Logits [n, vocab] of one sequence; `layers_out` (a list) receives the residual stream after every layer."""
+def forward(cfg, weights, tokens, layers_out=None, hide=None):
+    """Logits [n, vocab] of one sequence; `layers_out` (a list) receives the residual stream after every layer; hide: see window_attention."""
     eps, alpha = cfg["norm"]["eps"], cfg["postln_alpha"]
     x = weights["embed"][torch.tensor(tokens)] * cfg["embedding"]["scale"]
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
-        mixer = {"attention": attention, "general_delta": general_delta}[layer["type"]]
-        x = rms_norm(alpha * x + mixer(x, part(weights, p + "mix."), layer["mixer"], eps), weights[p + "norm1"], eps)
+        args = (x, part(weights, p + "mix."), layer["mixer"], eps)
+        y = attention(*args, hide) if layer["type"] == "attention" else general_delta(*args)
+        x = rms_norm(alpha * x + y, weights[p + "norm1"], eps)
         if layer["mlp"] is not None:
             y = squared_relu(x @ weights[p + "mlp.up"].T) @ weights[p + "mlp.down"].T
             x = rms_norm(alpha * x + y, weights[p + "norm2"], eps)
@@ -147,8 +156,15 @@ def forward(cfg, weights, tokens, layers_out=None):
     return rms_norm(x, weights["final.norm"], eps) @ weights["embed"].T
 
 
+def greedy(cfg, weights, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(cfg, weights, toks)[-1].argmax()))
+    return toks[len(prompt):]
+
+
 def shapes(cfg):
-    """Every tensor name with its shape; the rank of the decay's projection is not in the config: `rank` of a layer here."""
+    """Every tensor name with its shape; cfg["ranks"]: the rank of every layer's decay projection (None for attention)."""
     D = cfg["width"]
     out = {"embed": (cfg["vocab"], D), "final.norm": (D,)}
     for i, s in enumerate(cfg["layers"]):
