@@ -155,7 +155,7 @@ def _as_bf16_2d(x):
     if x2.dtype != torch.bfloat16:
         x2 = x2.to(torch.bfloat16)
     if x2.stride(-1) != 1 or (x2.stride(0) * 2) % 16 != 0 or x2.data_ptr() % 16 != 0:
-        x2 = x2.contiguous()
+        x2 = x2.clone(memory_format=torch.contiguous_format)      # (contiguous() would hand a single unaligned row back as it is)
     return x2
 
 

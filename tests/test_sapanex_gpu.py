@@ -65,6 +65,15 @@ def test_norm_behind_the_sum(T, W, dtype):
     assert torch.equal(x0, 6.5 * table[ids].float()) and torch.equal(h, x0.to(dtype))
 
 
+@pytest.mark.parametrize("T", [1, 3])
+def test_products_of_rows_that_start_anywhere(T):
+    """The second factor of the decay's projection reads a slice of the merged projection, wherever that lies."""
+    k = _k()
+    y, w = torch.randn(T, 80, device=DEV).to(torch.bfloat16), torch.randn(16, 8, device=DEV).to(torch.bfloat16)
+    for at in (60, 61, 64):
+        assert rel(k.linear_fp32(y[:, at: at + 8], w), y[:, at: at + 8].double() @ w.double().T) < 1e-5
+
+
 def _paged(q_lens, ctx, G, D, Dv, pool, dtype, g, page=64):
     pages = [(c + page - 1) // page for c in ctx]
     perm = torch.randperm(sum(pages) + 3, generator=g, device=DEV)
