@@ -6,7 +6,7 @@
 // a row (each CPL of its columns), a warp holds 4 R rows.  A token costs two dot products with the old state, p = S.u and q = S.(r w), and one
 // update, all in packed pairs of fp32; o = q + (|k| v) (r.u) - p (r.(a u)), so nothing waits for the new state.  The 2 R sums of a row group are
 // reduced over its lanes by halving (every exchange leaves each lane half of the sums) and the p handed back.
-//   single tokens: one kernel.  A CTA holds a whole head; its state is fetched while the kernel in front still runs; gates and unit keys are
+//   single tokens: one kernel.  A CTA or a pair of them holds a whole head; its state is fetched while the kernel in front still runs; gates and unit keys are
 //   made in it, and norm and gate are applied before the row leaves.
 //   otherwise: general_delta_prepare (one warp per (token, head)) writes u | w | a u | r w, general_delta_scan runs the recurrence with the
 //   next tokens' vectors on their way (bulk copies), general_delta_norm finishes.
@@ -186,6 +186,24 @@ template <int R> __device__ __forceinline__ int out_row(int cg) { return cg < 4 
 
 template <int CPL, int R>
 __device__ __forceinline__ void load_state(f2 (&S)[R][CPL / 2], const float* Sg, int row0, int rg, int cg, int Dv, int Dk, bool zero) {
+  if (Dk == CPL * 8 && row0 + 4 * R <= Dv) {          // whole rows: nothing between one load and the next
+    if (zero) {
+#pragma unroll
+      for (int r = 0; r < R; r++)
+#pragma unroll
+        for (int j = 0; j < CPL / 2; j++) S[r][j] = 0ull;
+      return;
+    }
+    const float* src = Sg + (long long)(row0 + rg) * Dk + cg * 4;
+#pragma unroll
+    for (int r = 0; r < R; r++)
+#pragma unroll
+      for (int j = 0; j < CPL / 4; j++) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(src + r * 4 * CPL * 8 + j * 32);
+        S[r][2 * j] = v.x; S[r][2 * j + 1] = v.y;
+      }
+    return;
+  }
   const bool vec = (Dk & 3) == 0;
 #pragma unroll
   for (int r = 0; r < R; r++) {
@@ -205,6 +223,14 @@ __device__ __forceinline__ void load_state(f2 (&S)[R][CPL / 2], const float* Sg,
 }
 template <int CPL, int R>
 __device__ __forceinline__ void store_state(const f2 (&S)[R][CPL / 2], float* Sg, int row0, int rg, int cg, int Dv, int Dk) {
+  if (Dk == CPL * 8 && row0 + 4 * R <= Dv) {
+    float* dst = Sg + (long long)(row0 + rg) * Dk + cg * 4;
+#pragma unroll
+    for (int r = 0; r < R; r++)
+#pragma unroll
+      for (int j = 0; j < CPL / 4; j++) *reinterpret_cast<ulonglong2*>(dst + r * 4 * CPL * 8 + j * 32) = make_ulonglong2(S[r][2 * j], S[r][2 * j + 1]);
+    return;
+  }
   const bool vec = (Dk & 3) == 0;
 #pragma unroll
   for (int r = 0; r < R; r++) {
@@ -229,27 +255,33 @@ __device__ __forceinline__ void ld_up4(const T* p, int c, int n, bool vec, float
   for (int e = 0; e < 4; e++) o[e] = c + e < n ? ldg_(p + c + e) : 0.f;
 }
 
-// Single tokens (a sequence may bring a few): grid (H, B), one CTA holds a head in warps of 16 rows; warp 0 makes the token's vectors while the
-// state is on its way.
-template <int CPL, typename T, bool VEC>
-__global__ void __launch_bounds__(256, 2) general_delta_step_kernel(const GdArgs a) {
+__device__ __forceinline__ void st_cluster(uint32_t addr, float v) { asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
+
+// arrive / wait of the cluster's barrier
+__device__ __forceinline__ void cluster_arrive_() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait_() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
+// Single tokens (a sequence may bring a few): grid (H CL, B), a cluster of CL CTAs holds a head in warps of 16 rows (small CTAs: more of them
+// are at different stages of fetching, computing and storing on an SM); warp 0 makes the token's vectors while the state is on its way.
+template <int CPL, int CL, typename T, bool VEC>
+__global__ void __cluster_dims__(CL, 1, 1) __launch_bounds__(256 / CL, 2 * CL) general_delta_step_kernel(const GdArgs a) {
   constexpr int DKP = CPL * 8, R = 4;
   constexpr float kRate = 0.60653065971263342f;      // exp(-1/2)
   __shared__ float4 s_vec4[DKP];             // u | w | a u | r w
   __shared__ float4 s_kv4[32], s_out4[32];   // v; norm weight * sigmoid(g)
-  __shared__ float s_scal[3], s_red[8];      // r.u, r.(a u), |k|
+  __shared__ float s_scal[3], s_red[2][8];   // r.u, r.(a u), |k|; sums of squares of every warp of the cluster
   float *s_vec = reinterpret_cast<float*>(s_vec4), *s_kv = reinterpret_cast<float*>(s_kv4), *s_out = reinterpret_cast<float*>(s_out4);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cg = lane & 7, rg = lane >> 3, nw = blockDim.x >> 5;
-  const int h = blockIdx.x, seq = blockIdx.y, Dk = a.Dk, Dv = a.Dv, hk = a.H * Dk, c = lane * 4;
+  const int h = blockIdx.x / CL, part = blockIdx.x % CL, row0 = part * nw * 16 + warp * 16, seq = blockIdx.y, Dk = a.Dk, Dv = a.Dv, hk = a.H * Dk, c = lane * 4;
   // The step's tables and the state are older than the kernel in front (every kernel triggers behind its own wait): fetched while it runs.
   const int start = a.cu[seq], n = a.cu[seq + 1] - start, slot = a.slots[seq];
   if (n <= 0 || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 48, __LINE__)) { pdl_wait(); return; }
   float* Sg = a.state + (((long long)slot * a.H + h) * Dv) * Dk;
   const bool fresh = a.fresh[seq] != 0;
   f2 S[R][CPL / 2];
-  if (warp != 0) load_state<CPL, R>(S, Sg, warp * 16, rg, cg, Dv, Dk, fresh);
+  if (warp != 0) load_state<CPL, R>(S, Sg, row0, rg, cg, Dv, Dk, fresh);
   pdl_wait(); pdl_trigger();
-  const int orow = out_row<R>(cg), lrow = warp * 16 + max(orow, 0) * 4 + rg;
+  const int orow = out_row<R>(cg), lrow = row0 + max(orow, 0) * 4 + rg;
   for (int i = 0; i < n; i++) {
     const long long t = start + i;
     if (warp == 0) {                         // the vectors' loads in front of the state's
@@ -257,7 +289,7 @@ __global__ void __launch_bounds__(256, 2) general_delta_step_kernel(const GdArgs
       float r[4], k[4], s[4], z[4], w0[4], ab[4];
       ld_up4(p + hk, c, Dk, VEC, k); ld_up4(a.decay + t * a.decay_ld + h * Dk, c, Dk, VEC, z); ld_up4(p + 2 * hk, c, Dk, VEC, s); ld_up4(p, c, Dk, VEC, r);
       ld_up4(a.w0 + h * Dk, c, Dk, VEC, w0); ld_up4(a.a_bias + h * Dk, c, Dk, VEC, ab);
-      if (i == 0) load_state<CPL, R>(S, Sg, 0, rg, cg, Dv, Dk, fresh);
+      if (i == 0) load_state<CPL, R>(S, Sg, row0, rg, cg, Dv, Dk, fresh);
       const float kk = warp_sum(k[0] * k[0] + k[1] * k[1] + k[2] * k[2] + k[3] * k[3]) + 1e-6f;
       const float inv = rsqrtf(kk);
       float ru = 0.f, rau = 0.f, o[4][4];
@@ -284,17 +316,19 @@ __global__ void __launch_bounds__(256, 2) general_delta_step_kernel(const GdArgs
     const float kn = s_scal[2];
     float kv[R];
 #pragma unroll
-    for (int r = 0; r < R; r++) kv[r] = kn * s_kv[warp * 16 + r * 4 + rg];
+    for (int r = 0; r < R; r++) kv[r] = kn * s_kv[row0 + r * 4 + rg];
     const float o = delta_token<CPL, R, false>(S, s_vec, DKP, cg, kv, kn * s_kv[lrow], s_scal[0], s_scal[1]);
     const bool mine = orow >= 0 && lrow < Dv;
     const float ss = warp_sum(mine ? o * o : 0.f);
-    if (lane == 0) s_red[warp] = ss;
-    if (i + 1 == n) store_state<CPL, R>(S, Sg, warp * 16, rg, cg, Dv, Dk);
-    __syncthreads();
+    if (CL > 1) { if (lane < CL) st_cluster(mapa_shared(smem_u32(&s_red[i & 1][part * nw + warp]), lane), ss); }
+    else if (lane == 0) s_red[i & 1][warp] = ss;
+    if (CL > 1) cluster_arrive_();
+    if (i + 1 == n) store_state<CPL, R>(S, Sg, row0, rg, cg, Dv, Dk);
+    if (CL > 1) cluster_wait_(); else __syncthreads();
     float tot = 0.f;
-    for (int w = 0; w < nw; w++) tot += s_red[w];
+    for (int w = 0; w < CL * nw; w++) tot += s_red[i & 1][w];
     if (mine) stg_(reinterpret_cast<T*>(a.out) + (t * a.H + h) * Dv + lrow, o * rsqrtf(tot / (float)Dv + a.eps) * s_out[lrow]);
-    if (i + 1 < n) __syncthreads();          // the vectors and sums are read by now
+    if (i + 1 < n) __syncthreads();          // the vectors are read by now (and the sums of the token before the next)
   }
 }
 
@@ -304,13 +338,14 @@ __device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_
 }
 constexpr int kKernelGd = 15;
 
-// grid = (H * splits, B), 4 warps of 4 R rows; `splits` CTAs share a head's Dv rows.  CH tokens are staged at a time, two buffers; warp 0 issues the
-// copies of a token's vectors, one bulk copy each.
+// grid = (H * splits, B), 4 warps of 4 R rows; `splits` CTAs share a head's Dv rows.  CH tokens are staged at a time, three buffers; every
+// warp issues the bulk copies of a quarter of them, and the warps drift apart by up to a chunk (full and empty barriers, no CTA-wide one).
 template <int CPL, int R, int CH>
 __global__ void __launch_bounds__(128, CPL * R >= 64 ? 3 : CPL * R >= 32 ? 4 : 6) general_delta_scan_kernel(const GdArgs a) {
   constexpr int DKP = CPL * 8, rows = 16 * R, kBuf = CH * (4 * DKP + rows + 4);
   extern __shared__ __align__(128) float sm[];                    // per buffer: vectors [CH][4][DKP] | |k| v [CH][rows] | r.u, r.(a u) [CH][4]
-  __shared__ uint64_t bars[2];
+  constexpr int NB = 3;
+  __shared__ uint64_t bars[2 * NB];                                // full | empty
   __shared__ int abort_word;
   volatile int* abort_flag = &abort_word;
   const int splits = gridDim.x / a.H, h = blockIdx.x / splits, row0 = (blockIdx.x % splits) * rows;
@@ -318,24 +353,29 @@ __global__ void __launch_bounds__(128, CPL * R >= 64 ? 3 : CPL * R >= 32 ? 4 : 6
   const int Dk = a.Dk, Dv = a.Dv, seq = blockIdx.y;
   const int start = a.cu[seq], n = a.cu[seq + 1] - start, slot = a.slots[seq];
   if (n <= 0 || !NE_INDEX_OK(slot, BK_STATE_SLOTS, 49, __LINE__)) return;
-  if (threadIdx.x == 0) { mbar_init(smem_u32(bars), 1); mbar_init(smem_u32(bars + 1), 1); abort_word = 0; mbar_fence_init(); }
+  if (threadIdx.x == 0) {
+    for (int b = 0; b < NB; b++) { mbar_init(smem_u32(bars + b), 4); mbar_init(smem_u32(bars + NB + b), 4); }
+    abort_word = 0;
+    mbar_fence_init();
+  }
   __syncthreads();
   const int vrows = min(rows, a.DvP - row0);                       // a multiple of 4; rows past Dv read whatever their scratch holds and are not kept
-  auto stage = [&](int buf, int i0) {                              // warp 0
-    const int m = min(CH, n - i0);
+  static_assert(CH % 4 == 0 && CH <= 32, "a warp's share of a chunk is whole tokens, one copy per lane");
+  auto stage = [&](int buf, int i0) {
+    const int first = warp * (CH / 4), m = max(0, min(CH / 4, n - i0 - first));       // this warp's tokens of the chunk
     float* base = sm + buf * kBuf;
     const uint32_t bar = smem_u32(bars + buf);
-    if (lane == 0) mbar_expect_tx(bar, m * (4 * DKP + vrows + 4) * 4);
+    if (lane == 0) { if (m) mbar_expect_tx(bar, m * (4 * DKP + vrows + 4) * 4); else mbar_arrive(bar); }
     __syncwarp();
-    for (int i = lane; i < 3 * m; i += 32) {
-      const int tok = i / 3, which = i - 3 * tok;
+    if (lane < 3 * m) {
+      const int tok = first + lane / 3, which = lane % 3;
       const long long th = (long long)(start + i0 + tok) * a.H + h;
       if (which == 0) bulk_load(smem_u32(base + tok * 4 * DKP), a.vec + th * 4 * DKP, 16 * DKP, bar);
       else if (which == 1) bulk_load(smem_u32(base + CH * 4 * DKP + tok * rows), a.val + th * a.DvP + row0, vrows * 4, bar);
       else bulk_load(smem_u32(base + CH * (4 * DKP + rows) + tok * 4), a.scal + th * 4, 16, bar);
     }
   };
-  if (warp == 0) stage(0, 0);
+  for (int c = 0; c < NB - 1 && c * CH < n; c++) stage(c, c * CH);
   float* Sg = a.state + (((long long)slot * a.H + h) * Dv) * Dk;
   f2 S[R][CPL / 2];
   const int wrow = warp * 4 * R;
@@ -344,9 +384,13 @@ __global__ void __launch_bounds__(128, CPL * R >= 64 ? 3 : CPL * R >= 32 ? 4 : 6
   const bool keep = orow >= 0 && row0 + lrow < Dv;
   bool ok = true;
   for (int i0 = 0, it = 0; i0 < n; i0 += CH, it++) {
-    const int m = min(CH, n - i0), buf = it & 1;
-    if (warp == 0 && i0 + CH < n) stage(buf ^ 1, i0 + CH);
-    if (!mbar_wait(smem_u32(bars + buf), (it >> 1) & 1, abort_flag, kKernelGd, 400 + buf)) { ok = false; *abort_flag = 1; }
+    const int m = min(CH, n - i0), buf = it % NB;
+    if (i0 + (NB - 1) * CH < n) {                                // chunk it + 2 goes where chunk it - 1 was
+      const int nb = (it + NB - 1) % NB;
+      if (it > 0 && !mbar_wait(smem_u32(bars + NB + nb), ((it - 1) / NB) & 1, abort_flag, kKernelGd, 410 + nb)) { ok = false; break; }
+      stage(nb, i0 + (NB - 1) * CH);
+    }
+    if (!mbar_wait(smem_u32(bars + buf), (it / NB) & 1, abort_flag, kKernelGd, 400 + buf)) { ok = false; break; }
     const float* vec = sm + buf * kBuf;
     const float *sv = vec + CH * 4 * DKP, *sg = sv + CH * rows;
     float* ov = a.val + ((long long)(start + i0) * a.H + h) * a.DvP + row0 + lrow;       // |k| v of these places has been read
@@ -359,14 +403,11 @@ __global__ void __launch_bounds__(128, CPL * R >= 64 ? 3 : CPL * R >= 32 ? 4 : 6
       const float o = delta_token<CPL, R, (CPL <= 16)>(S, vec + i * 4 * DKP, DKP, cg, kv, sv[i * rows + lrow], gt.x, gt.y);
       if (keep) ov[(long long)i * a.H * a.DvP] = o;
     }
-    __syncthreads();          // everyone is done with this buffer before the next-but-one chunk is copied into it
-    if (*abort_flag) break;
+    __syncwarp();
+    if (lane == 0) mbar_arrive(smem_u32(bars + NB + buf));
   }
-  if (*abort_flag) {          // a wait gave up (reported): copies in flight land before the CTA goes; the state is left as it was
-    if (threadIdx.x == 0) for (int i = 0; i < 2000; i++) __nanosleep(1000);
-    __syncthreads();
-    return;
-  }
+  // a wait gave up (reported): copies in flight land before the CTA goes, and the warp's rows stay as they were
+  if (!ok) for (int i = 0; i < 2000; i++) __nanosleep(1000);
   if (ok) store_state<CPL, R>(S, Sg, row0 + wrow, rg, cg, Dv, Dk);
 }
 
@@ -407,7 +448,7 @@ __global__ void __launch_bounds__(256) general_delta_norm_kernel(const GdArgs a)
 template <int CPL, int R>
 static int gd_scan(const GdArgs& a, cudaStream_t st) {
   constexpr int CH = CPL <= 32 ? 8 : 4, rows = 16 * R;
-  const size_t smem = sizeof(float) * 2 * CH * (4 * CPL * 8 + rows + 4);
+  const size_t smem = sizeof(float) * 3 * CH * (4 * CPL * 8 + rows + 4);
   auto k = general_delta_scan_kernel<CPL, R, CH>;
   cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
@@ -425,9 +466,11 @@ static int general_delta_t(const GdArgs& a, int max_q, cudaStream_t st) {
   const bool fours = a.Dk % 4 == 0 && a.Dv % 4 == 0 && a.proj_ld % 4 == 0 && a.decay_ld % 4 == 0 &&
                      ((uintptr_t)a.proj | (uintptr_t)a.decay | (uintptr_t)a.w0 | (uintptr_t)a.a_bias | (uintptr_t)a.norm_w | (uintptr_t)a.out) % 16 == 0;
   if (gd_whole(a.Dk, a.Dv, max_q)) {
-    const dim3 grid((unsigned)a.H, (unsigned)a.B), block((unsigned)((a.Dv + 15) / 16 * 32));
-#define NE_STEP(CPL_) (int)launch_pdl(fours ? general_delta_step_kernel<CPL_, T, true> : general_delta_step_kernel<CPL_, T, false>, grid, block, 0, st, a)
-    return a.Dk <= 32 ? NE_STEP(4) : a.Dk <= 64 ? NE_STEP(8) : a.Dk <= 96 ? NE_STEP(12) : NE_STEP(16);
+    const int cl = a.Dv > 64 ? 2 : 1;
+    const dim3 grid((unsigned)(a.H * cl), (unsigned)a.B), block((unsigned)(((a.Dv + cl - 1) / cl + 15) / 16 * 32));
+#define NE_STEP(CPL_, CL_) (int)launch_pdl(fours ? general_delta_step_kernel<CPL_, CL_, T, true> : general_delta_step_kernel<CPL_, CL_, T, false>, grid, block, 0, st, a)
+    if (cl == 2) return a.Dk <= 32 ? NE_STEP(4, 2) : a.Dk <= 64 ? NE_STEP(8, 2) : a.Dk <= 96 ? NE_STEP(12, 2) : NE_STEP(16, 2);
+    return a.Dk <= 32 ? NE_STEP(4, 1) : a.Dk <= 64 ? NE_STEP(8, 1) : a.Dk <= 96 ? NE_STEP(12, 1) : NE_STEP(16, 1);
 #undef NE_STEP
   }
   const dim3 wgrid((unsigned)(((long long)a.T * a.H + 7) / 8));

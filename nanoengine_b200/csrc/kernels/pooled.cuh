@@ -5,6 +5,11 @@
 namespace ne {
 
 __host__ __device__ __forceinline__ void pooled_group(int g, int pool, int block_size, int& page, int& row) {
+  if (block_size == 64) {                     // in 32 bits: g * pool is an eighth of a position
+    page = (g * pool) >> 3;
+    row = pool >= 8 ? 0 : (g - (page * 8 + pool - 1) / pool) * 8;
+    return;
+  }
   page = (int)((8ll * g * pool) / block_size);
   const long long first = ((long long)page * block_size + 8ll * pool - 1) / (8ll * pool);       // first group of that page
   row = (int)(g - first) * 8;

@@ -203,8 +203,8 @@ def linear_fp32(x, w: torch.Tensor) -> torch.Tensor:
     return linear(x, w, out_fp32=True)
 
 
-def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None, out_fp32: bool = False, act: Optional[str] = None,
-           act_from: int = 0) -> torch.Tensor:
+def linear(x, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None, bias=None, act: Optional[str] = None, act_from: int = 0,
+           out_fp32: bool = False) -> torch.Tensor:
     N, K = w.shape
     assert act is None or (w.dtype != FP8 and bias is None and isinstance(x, torch.Tensor))
     if isinstance(x, PrequantizedActivation):

@@ -292,9 +292,12 @@ def test_long_decoding(name, tmp_path):
 
 
 def test_pool_sized_from_the_free_memory(tmp_path):
+    import gc
+    gc.collect()                                # what earlier tests hold counts as used
+    torch.cuda.empty_cache()
     from nanoengine_b200 import LLM, Config, SamplingParams
     cfg, W, path = build("odd", tmp_path)
-    llm = LLM(Config(model=path, dtype="bfloat16", device=DEV, max_num_seqs=4, max_num_batched_tokens=1000, max_model_len=4096, gpu_memory_utilization=0.05,
+    llm = LLM(Config(model=path, dtype="bfloat16", device=DEV, max_num_seqs=4, max_num_batched_tokens=1000, max_model_len=4096, gpu_memory_utilization=0.15,
                      executor_backend="inproc", enable_prefix_caching=False, status_log_interval_s=0))
     assert llm.engine.scheduler.num_free_blocks(0) > 100
     out = llm.generate([tokens(70, cfg["vocab"], 1)], SamplingParams(temperature=0.0, max_tokens=4, ignore_eos=True))
