@@ -388,6 +388,17 @@ def case_pooled_prepare(B, q_len, H=32, G=8, D=128, dims=64, pool=16, at=4096, b
     return fn, T * W * 2 * 2 + means, 0.0
 
 
+def case_qkv_prepare(B, q_len, H=32, G=8, D=128, bs=64):
+    """The like front end of the Qwen3 family: norm per head, rotation of whole heads, key and value rows."""
+    T, W = B * q_len, H * D + 2 * G * D
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    qkv, w = torch.randn(T, W, **bf), torch.ones(D, **bf)
+    kc, vc = (torch.zeros(T // bs + 2, bs, G, D, **bf) for _ in range(2))
+    pos, table = torch.arange(T, device="cuda") % q_len, torch.rand(max(q_len, 1), D, device="cuda")
+    slots = torch.arange(T, device="cuda")
+    return lambda: sm100.gqa_qkv_prepare(qkv, H, G, D, w, w, 1e-6, False, pos, table, kc, vc, slots), T * W * 2 * 2, 0.0
+
+
 def case_postnorm(T, W=4096):
     y, w, x = torch.randn(T, W, device="cuda", dtype=torch.bfloat16), torch.ones(W, device="cuda", dtype=torch.bfloat16), torch.randn(T, W, device="cuda")
     return lambda: sm100.postnorm(y, x, 2.0, w, 1e-6), T * W * (2 + 4 + 4 + 2), 0.0
@@ -542,6 +553,8 @@ def build_cases(args):
         "pooled_prefill": lambda: case_pooled(1, 8192, 8192, 32, 8, 1024, 16),
         "pooled_prefill_nopool": lambda: case_pooled(1, 8192, 8192, 32, 8, 8192, 0),
         "pooled_prefill_w1024": lambda: case_pooled(1, 8192, 8192, 32, 8, 1024, 0),
+        "qkv_prepare_decode": lambda: case_qkv_prepare(128, 1),
+        "qkv_prepare_prefill": lambda: case_qkv_prepare(4, 2048),
         "pooled_prepare_decode": lambda: case_pooled_prepare(128, 1),
         "pooled_prepare_prefill": lambda: case_pooled_prepare(4, 2048),
         "postnorm_decode": lambda: case_postnorm(128),

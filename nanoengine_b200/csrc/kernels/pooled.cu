@@ -22,6 +22,8 @@ __device__ __forceinline__ float4 pl_ld4(const __nv_bfloat16* p) {
 __device__ __forceinline__ void pl_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void pl_st4(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
 
+__device__ __forceinline__ void cp_async8(uint32_t dst, const void* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(dst), "l"(src) : "memory"); }
+
 struct PoolArgs {
   void* qkv; long long ld;                   // [T, H D | G D | G Dv]
   const void* q_norm; const void* k_norm; float eps;
@@ -102,29 +104,49 @@ __device__ __forceinline__ void pool_block(const PoolArgs& a, long long p, long 
 template <typename T, int V>
 __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, const int pool_here) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
-  extern __shared__ __align__(16) float sm[];       // the row (fp32) | key table | value table
+  extern __shared__ __align__(16) float sm[];       // key table | value table | the row
   __shared__ float red[2][16];
   __shared__ long long offs[kOffs];
   const int t = blockIdx.x, nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.Dv, W = nq + nk + nv, D = a.D, Dv = a.Dv, dims = a.dims;
-  float* s_kt = sm + (W + 3) / 4 * 4;
-  float* s_vt = s_kt + (dims + 3) / 4 * 4;
+  float *s_kt = sm, *s_vt = sm + (dims + 3) / 4 * 4;
+  T* x0 = reinterpret_cast<T*>(s_vt + (Dv + 3) / 4 * 4);
   T* row = reinterpret_cast<T*>(a.qkv) + (long long)t * a.ld;
   long long p = a.positions[t];
   const long long slot = a.slots[t];
+  // the row is on its way while the position, and the tables' rows that it names, are looked up
+  constexpr int PE = V == 4 ? 16 / (int)sizeof(T) : 1;
+  const int step = V == 4 ? (W % PE == 0 && a.ld % PE == 0 ? PE : 4) : 1;
+  for (int i = threadIdx.x * step; i < W; i += blockDim.x * step) {
+    if constexpr (V == 4) {
+      if (step == PE) cp_async16(smem_u32(x0 + i), row + i, 16);
+      else cp_async8(smem_u32(x0 + i), row + i);
+    } else x0[i] = row[i];
+  }
   if (p < 0 || p >= a.n_pos) { if (threadIdx.x == 0) report(ST_BAD_INDEX, 52, t, (int)p); p = 0; }
+  if constexpr (V == 4) {
+    for (int i = threadIdx.x * 4; i < dims; i += blockDim.x * 4) cp_async16(smem_u32(s_kt + i), a.k_table + p * dims + i, 16);
+    for (int i = threadIdx.x * 4; i < Dv; i += blockDim.x * 4) cp_async16(smem_u32(s_vt + i), a.v_table + p * Dv + i, 16);
+  } else {
+    for (int i = threadIdx.x; i < dims; i += blockDim.x) s_kt[i] = a.k_table[p * dims + i];
+    for (int i = threadIdx.x; i < Dv; i += blockDim.x) s_vt[i] = a.v_table[p * Dv + i];
+  }
   const int* bt = nullptr;
   const long long place = pool_here ? block_place(a, t, p, bt) : -1;
-  for (int i = threadIdx.x; i < dims; i += blockDim.x) s_kt[i] = a.k_table[p * dims + i];
-  for (int i = threadIdx.x; i < Dv; i += blockDim.x) s_vt[i] = a.v_table[p * Dv + i];
+  if constexpr (V == 4) { cp_async_commit(); cp_async_wait<0>(); }
   float qq = 0.f, kk = 0.f;
-  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {             // V divides nq and nk
-    float s;
+  for (int i = threadIdx.x * step; i < W; i += blockDim.x * step) {       // what the thread copied itself
     if constexpr (V == 4) {
-      const float4 v = pl_ld4(row + i);
-      *reinterpret_cast<float4*>(sm + i) = v;
-      s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-    } else { const float v = pl_ld(row + i); sm[i] = v; s = v * v; }
-    if (i < nq) qq += s; else if (i < nq + nk) kk += s;
+#pragma unroll
+      for (int e = 0; e < PE; e += 4) {
+        if (e >= step) break;
+        const float4 v = pl_ld4(x0 + i + e);
+        const float s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        if (i + e < nq) qq += s; else if (i + e < nq + nk) kk += s;       // 4 divides nq and nk
+      }
+    } else {
+      const float v = pl_ld(x0 + i);
+      if (i < nq) qq += v * v; else if (i < nq + nk) kk += v * v;
+    }
   }
   qq = warp_sum(qq); kk = warp_sum(kk);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -132,7 +154,7 @@ __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, c
   __syncthreads();
   const float rq = rsqrtf(warp_sum(lane < nw ? red[0][lane] : 0.f) / (float)nq + a.eps), rk = rsqrtf(warp_sum(lane < nw ? red[1][lane] : 0.f) / (float)nk + a.eps);
   const bool store = slot >= 0 && NE_INDEX_OK(slot, BK_CACHE_ROWS, 53, __LINE__);
-  const float* x0 = sm;                              // one warp per head; V divides the head sizes and the halves of the rotations
+  // one warp per head; V divides the head sizes and the halves of the rotations
   for (int u = warp; u < a.H + 2 * a.G; u += nw) {
     const int part = u < a.H ? 0 : u < a.H + a.G ? 1 : 2;
     if (part && !store) break;
@@ -142,26 +164,30 @@ __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, c
     const T* w = reinterpret_cast<const T*>(part == 0 ? a.q_norm : a.k_norm) + j0;
     const float r = part == 0 ? rq : rk;
     T* dst = part == 0 ? row + j0 : part == 1 ? reinterpret_cast<T*>(a.k_cache) + slot * nk + j0 : reinterpret_cast<T*>(a.v_cache) + slot * nv + j0;
-    for (int d = lane * V; d < width; d += 32 * V) {
-      const int other = d < half ? d + half : d - half, ti = d < half ? d : d - half;
-      const float sign = d < half ? -1.f : 1.f;
+    // items of V columns: the pairs of a rotation (columns d and d + half), then the columns that pass
+    const int pairs = half / V, items = pairs + (width - turned) / V;
+    for (int item = lane; item < items; item += 32) {
+      const int d = item < pairs ? item * V : turned + (item - pairs) * V;
       if constexpr (V == 4) {
-        float4 x = *reinterpret_cast<const float4*>(x0 + i0 + d);
+        float4 x = pl_ld4(x0 + i0 + d);
         if (part < 2) { const float4 g = pl_ld4(w + d); x.x *= r * g.x; x.y *= r * g.y; x.z *= r * g.z; x.w *= r * g.w; }
-        if (d < turned) {
-          float4 y = *reinterpret_cast<const float4*>(x0 + i0 + other);
-          if (part < 2) { const float4 g = pl_ld4(w + other); y.x *= r * g.x; y.y *= r * g.y; y.z *= r * g.z; y.w *= r * g.w; }
-          const float4 c = *reinterpret_cast<const float4*>(tab + ti), s = *reinterpret_cast<const float4*>(tab + half + ti);
-          x.x = x.x * c.x + sign * y.x * s.x; x.y = x.y * c.y + sign * y.y * s.y; x.z = x.z * c.z + sign * y.z * s.z; x.w = x.w * c.w + sign * y.w * s.w;
+        if (item < pairs) {
+          float4 y = pl_ld4(x0 + i0 + d + half);
+          if (part < 2) { const float4 g = pl_ld4(w + d + half); y.x *= r * g.x; y.y *= r * g.y; y.z *= r * g.z; y.w *= r * g.w; }
+          const float4 c = *reinterpret_cast<const float4*>(tab + d), s = *reinterpret_cast<const float4*>(tab + half + d);
+          pl_st4(dst + d + half, make_float4(y.x * c.x + x.x * s.x, y.y * c.y + x.y * s.y, y.z * c.z + x.z * s.z, y.w * c.w + x.w * s.w));
+          x = make_float4(x.x * c.x - y.x * s.x, x.y * c.y - y.y * s.y, x.z * c.z - y.z * s.z, x.w * c.w - y.w * s.w);
         }
         pl_st4(dst + d, x);
       } else {
-        float x = x0[i0 + d];
+        float x = pl_ld(x0 + i0 + d);
         if (part < 2) x *= r * pl_ld(w + d);
-        if (d < turned) {
-          float y = x0[i0 + other];
-          if (part < 2) y *= r * pl_ld(w + other);
-          x = x * tab[ti] + sign * y * tab[half + ti];
+        if (item < pairs) {
+          float y = pl_ld(x0 + i0 + d + half);
+          if (part < 2) y *= r * pl_ld(w + d + half);
+          const float c = tab[d], s = tab[half + d];
+          pl_st(dst + d + half, y * c + x * s);
+          x = x * c - y * s;
         }
         pl_st(dst + d, x);
       }
@@ -172,13 +198,45 @@ __global__ void __launch_bounds__(512) pooled_prepare_kernel(const PoolArgs a, c
   pool_block<T, V>(a, p, place, bt, offs);
 }
 
+// One CTA per block completed in this call: CTA i takes the i-th, counted over the sequences.
 template <typename T, int V>
 __global__ void __launch_bounds__(256) pooled_means_kernel(const PoolArgs a) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   __shared__ long long offs[kOffs];
-  const long long p = a.positions[blockIdx.x];
+  __shared__ int s_tok;
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    int rem = blockIdx.x, tok = -1;
+    for (int s0 = 0; s0 < a.B && tok < 0; s0 += 32) {
+      const int s = s0 + lane;
+      int t0 = 0, n = 0, done = 0;
+      long long p0 = 0;
+      if (s < a.B) {
+        t0 = a.cu[s];
+        n = a.cu[s + 1] - t0;
+        if (n > 0) { p0 = a.positions[t0]; done = (int)((p0 + n) / a.pool - p0 / a.pool); }
+      }
+      int incl = done;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xffffffffu, incl, o); if (lane >= o) incl += v; }
+      const unsigned hit = __ballot_sync(0xffffffffu, rem < incl);
+      if (hit) {
+        const int l = __ffs(hit) - 1;
+        // the token at the end of the block
+        const long long mine = t0 + (p0 / a.pool + 1 + rem - (incl - done)) * a.pool - 1 - p0;
+        tok = __shfl_sync(0xffffffffu, (int)mine, l);
+      } else {
+        rem -= __shfl_sync(0xffffffffu, incl, 31);
+      }
+    }
+    if (lane == 0) s_tok = tok;
+  }
+  __syncthreads();
+  const int t = s_tok;
+  if (t < 0 || t >= a.T) return;
+  const long long p = a.positions[t];
   const int* bt = nullptr;
-  const long long place = block_place(a, blockIdx.x, p, bt);
+  const long long place = block_place(a, t, p, bt);
   if (place >= 0) pool_block<T, V>(a, p, place, bt, offs);
 }
 
@@ -186,12 +244,12 @@ template <typename T>
 static int pooled_t(const PoolArgs& a, int max_q, cudaStream_t st) {
   const int W = a.H * a.D + a.G * (a.D + a.Dv);
   const uintptr_t al = (uintptr_t)a.qkv | (uintptr_t)a.q_norm | (uintptr_t)a.k_norm | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache | (uintptr_t)a.k_pool | (uintptr_t)a.v_pool;
-  const bool vec = a.D % 4 == 0 && a.Dv % 8 == 0 && a.dims % 8 == 0 && a.ld % 4 == 0 && al % 16 == 0;
+  const bool vec = (uintptr_t)a.k_table % 16 == 0 && (uintptr_t)a.v_table % 16 == 0 && a.D % 4 == 0 && a.Dv % 8 == 0 && a.dims % 8 == 0 && a.ld % 4 == 0 && al % 16 == 0;
   const int per = vec ? 4 : 1;
   int threads = ((W + per - 1) / per + 31) / 32 * 32;
   const int most = max_q == 1 ? 512 : 256;           // few CTAs: wide ones
   threads = threads > most ? most : threads < 64 ? 64 : threads;
-  const size_t smem = sizeof(float) * ((size_t)(W + 3) / 4 * 4 + (a.dims + 3) / 4 * 4 + a.Dv);
+  const size_t smem = sizeof(float) * ((a.dims + 3) / 4 * 4 + (a.Dv + 3) / 4 * 4) + sizeof(T) * (size_t)W;
   auto k = vec ? pooled_prepare_kernel<T, 4> : pooled_prepare_kernel<T, 1>;
   if (smem > 40 * 1024) {
     if (smem > 227 * 1024) return 1001;
@@ -200,9 +258,10 @@ static int pooled_t(const PoolArgs& a, int max_q, cudaStream_t st) {
   }
   cudaError_t e = launch_pdl(k, dim3((unsigned)a.T), dim3((unsigned)threads), smem, st, a, max_q == 1 ? 1 : 0);
   if (e != cudaSuccess || max_q == 1) return (int)e;
+  const long long blocks = (long long)a.T / a.pool + a.B, most_blocks = blocks < a.T ? blocks : a.T;
   int mt = (a.G * (a.D + a.Dv) / per + 31) / 32 * 32;
   mt = mt > 256 ? 256 : mt < 64 ? 64 : mt;           // at least kOffs threads
-  return (int)launch_pdl(vec ? pooled_means_kernel<T, 4> : pooled_means_kernel<T, 1>, dim3((unsigned)a.T), dim3((unsigned)mt), 0, st, a);
+  return (int)launch_pdl(vec ? pooled_means_kernel<T, 4> : pooled_means_kernel<T, 1>, dim3((unsigned)most_blocks), dim3((unsigned)mt), 0, st, a);
 }
 
 }  // namespace ne
