@@ -69,7 +69,7 @@ def sapanex_model(width, heads, groups, ff, vocab):
     layers = []
     for _ in range(groups):
         layers += [_general_delta_spec(heads, 128, 64, ff=3 * ff // 2) for _ in range(3)]
-        layers.append(_pooled_attention_spec(heads, heads // 4, 128, 128, 1024, 16, 64, ff=3 * ff // 2, base=5e5, scaling=yarn))
+        layers.append(_pooled_attention_spec(heads, heads // 4, 128, 128, 1024, 16, 64, ff=3 * ff // 2, base=1e6, scaling=yarn))
     return ModelConfig.from_dict({"architecture": "Sapanex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "postln_alpha": 2.0,
                                   "max_position_embeddings": 16384, "layers": layers})
 

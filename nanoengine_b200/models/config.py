@@ -757,7 +757,7 @@ def sapanex_7b(**over) -> ModelConfig:
     yarn = {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}
     layers = []
     for _ in range(8):
-        layers += [_general_delta_spec(32, 128, 64, ff=16384) for _ in range(3)] + [_pooled_attention_spec(32, 8, 128, 128, 4096, 16, 64, ff=16384, base=5e5, scaling=yarn)]
+        layers += [_general_delta_spec(32, 128, 64, ff=16384) for _ in range(3)] + [_pooled_attention_spec(32, 8, 128, 128, 4096, 16, 64, ff=16384, base=1e6, scaling=yarn)]
     c = ModelConfig.from_dict({"architecture": "Sapanex", "vocab": 131072, "width": 4096, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "postln_alpha": 2.0,
                                "layers": layers})
     for k, v in over.items():

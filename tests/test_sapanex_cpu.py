@@ -66,7 +66,7 @@ def test_engine_config_refuses_layouts_it_does_not_run():
 
 
 # ---- operators against the oracle ------------------------------------------------------------------------------------
-@pytest.mark.parametrize("dims,base,sc", [(16, 10000.0, YARN), (6, 500000.0, {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}), (80, 500.0, YARN),
+@pytest.mark.parametrize("dims,base,sc", [(16, 10000.0, YARN), (6, 200000.0, {"factor": 5.0, "original": 2048, "fast": 24.0, "slow": 1.0}), (80, 500.0, YARN),
                                           (2, 100.0, {"factor": 2.0, "original": 7, "fast": 3.0, "slow": 2.9}), (24, 1000.0, None)])
 def test_rotary_tables(dims, base, sc):
     freq, factor = oracle.yarn_frequencies(dims, base, sc)

@@ -87,7 +87,7 @@ def _paged(q_lens, ctx, G, D, Dv, pool, dtype, g, page=64):
     return rnd(page, D), rnd(page, Dv), rnd(rows, D), rnd(rows, Dv), bt, _cu(q_lens), torch.tensor(ctx, dtype=torch.int32, device=DEV)
 
 
-@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 56, 40), (6, 2, 80, 24), (8, 8, 128, 128), (32, 4, 128, 64), (5, 1, 64, 256), (24, 2, 256, 200), (128, 1, 72, 8), (16, 16, 64, 80),
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 56, 40), (6, 2, 80, 24), (8, 8, 128, 128), (32, 4, 128, 64), (5, 1, 64, 256), (24, 2, 256, 200), (128, 1, 72, 8), (16, 16, 64, 72),
                                       (3, 1, 12, 20), (10, 2, 17, 6)])
 @pytest.mark.parametrize("window,pool,turned", [(70, 5, True), (64, 64, True), (1, 1, False), (33, 16, True), (200, 130, False), (5, 3, True)])
 @pytest.mark.parametrize("q_lens,ctx", [([1, 1, 1], [1, 64, 700]), ([5, 130, 1, 33], [5, 200, 129, 1095])])
@@ -127,7 +127,7 @@ def test_window_and_pooled_blocks(H, G, D, Dv, window, pool, turned, q_lens, ctx
     assert _k().kernel_status()[0] == 0
 
 
-@pytest.mark.parametrize("H,G,D,Dv,rot,pool", [(4, 2, 64, 80, 16, 12), (6, 2, 12, 10, 6, 7), (5, 1, 9, 14, 8, 23), (8, 8, 40, 56, 24, 3), (32, 8, 128, 128, 64, 16),
+@pytest.mark.parametrize("H,G,D,Dv,rot,pool", [(4, 2, 48, 72, 24, 11), (6, 2, 12, 10, 6, 7), (5, 1, 9, 14, 8, 23), (8, 8, 40, 56, 24, 3), (32, 8, 128, 128, 64, 16),
                                                (2, 2, 16, 40, 16, 70), (1, 1, 8, 8, 2, 1)])
 @pytest.mark.parametrize("starts,lens,page", [([0, 63, 200], [1, 1, 1], 64), ([0, 100, 37, 69], [130, 1, 2, 90], 64), ([11, 5], [60, 1], 16)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
