@@ -203,6 +203,8 @@ class Config:
         if mc.layer_specs:
             if self.attention_tp != 1 or self.pp != 1:
                 raise ValueError("models with listed layers run with attention_tp = pp = 1")
+            if self.ffn_ep != 1 and any((s["mlp"] or {}).get("kind") == "moe" for s in mc.layer_specs):
+                raise ValueError("mixture-of-experts layers of listed models run with ffn_ep = 1")
             if mc.learned_positions:
                 if self.max_model_len > mc.max_position_embeddings:
                     raise ValueError(f"max_model_len {self.max_model_len} is past the model's {mc.max_position_embeddings} learned positions")

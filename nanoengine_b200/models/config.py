@@ -109,11 +109,12 @@ class ModelConfig:
     o_groups: int = 0
     num_hash_layers: int = 0                 # the first this-many MoE layers pick experts from a token-id table
     # families that list every layer with its own mixer, the mixer's sizes and its feed-forward (Tuvutar: "latent_attention" | "delta",
-    # Filasun: "mamba2" | "parallel", Sapanex: "attention" | "general_delta"); the fields above describe one such layer only in the form `layer_config` derives for it
+    # Filasun: "mamba2" | "parallel", Sapanex: "attention" | "general_delta", Gipozen: "attention"); the fields above describe one such layer only in the form `layer_config` derives for it
     layer_specs: Optional[List[Dict[str, Any]]] = None
     attn_scale: float = 0.0                  # > 0: softmax scale of the latent-attention layer (0: from the head dim)
     embedding_scale: float = 1.0             # token embeddings enter the residual stream times this
     postnorm_alpha: float = 0.0              # > 0: x <- norm(alpha x + sublayer(x)), the norm behind the sum
+    logit_scale: float = 1.0                 # the logits are multiplied by this
     learned_positions: bool = False          # a learned vector per position, max_position_embeddings of them: a hard context limit
     # MTP
     num_nextn_predict_layers: int = 0
@@ -144,7 +145,7 @@ class ModelConfig:
     @property
     def is_hybrid_gdn(self) -> bool:
         if self.layer_specs:
-            return any(s["type"] in _STATE_MIXERS for s in self.layer_specs)
+            return any(self.keeps_state(i) for i in range(len(self.layer_specs)))
         return self.linear_num_value_heads > 0
 
     def layer_config(self, layer_idx: int) -> "ModelConfig":
@@ -206,8 +207,10 @@ class ModelConfig:
         return t in _ROW_MIXERS and self.kv_source_layer(layer_idx) == layer_idx
 
     def keeps_state(self, layer_idx: int) -> bool:
-        """Does the listed layer own a slot of recurrent state per sequence?  A "parallel" layer owns both."""
-        return self.layer_specs[layer_idx]["type"] in _STATE_MIXERS
+        """Does the listed layer own a slot of recurrent state per sequence?  A "parallel" layer owns both, an attention layer behind short
+        convolutions a window of their last inputs."""
+        s = self.layer_specs[layer_idx]
+        return s["type"] in _STATE_MIXERS or int(s["mixer"].get("conv", 1)) > 1
 
     def cache_rank(self, layer_idx: int) -> int:
         return sum(1 for i in range(layer_idx) if self.keeps_rows(i))
@@ -294,6 +297,8 @@ class ModelConfig:
             d = _filasun_fields(d)
         if arch == "Sapanex" and "layers" in d:
             d = _sapanex_fields(d)
+        if arch == "Gipozen" and "layers" in d:
+            d = _gipozen_fields(d)
         la = d.pop("linear_attn_config", None)
         if isinstance(la, dict):                          # Kimi delta attention block of GLM5-next / Kimi-K3
             d["linear_kind"] = "kda"
@@ -507,6 +512,50 @@ def _sapanex_fields(d: Dict[str, Any]) -> Dict[str, Any]:
            "num_attention_heads": 1, "num_key_value_heads": 1, "max_position_embeddings": int(d.get("max_position_embeddings") or 131072),
            "embedding_scale": float(d["embedding"]["scale"]), "postnorm_alpha": float(d["postln_alpha"]),
            "layer_specs": [{"type": s["type"], "mixer": dict(s["mixer"]), "mlp": dict(s["mlp"]) if s.get("mlp") is not None else None} for s in d["layers"]]}
+    for k in ("eos_token_id", "bos_token_id"):
+        if d.get(k) is not None:
+            out[k] = d[k]
+    return out
+
+
+def _gipozen_fields(d: Dict[str, Any]) -> Dict[str, Any]:
+    """config.json of a Gipozen model ({architecture, layers, logit_scale, norm, vocab, width}) as ModelConfig fields.  The design has no
+    positions in its scores and no context limit."""
+    def need(ok, i, what):
+        if not ok:
+            raise ValueError(f"layer {i}: {what}")
+
+    layers = []
+    for i, s in enumerate(d["layers"]):
+        need(s["type"] == "attention", i, f"unknown mixer type {s['type']!r}")
+        m, f = dict(s["mixer"]), s.get("mlp")
+        m["mask"] = dict(m.get("mask") or {})
+        m["conv"] = int(m.get("conv") or 1)
+        size, keep = m["mask"].get("size"), m["mask"].get("keep_first")
+        need(int(m["heads"]) % int(m["kv_heads"]) == 0, i, "heads must be a multiple of kv_heads")
+        need(size is None or int(size) >= 1, i, "the window holds at least the token itself")
+        need(keep is None or int(keep) >= 0, i, "keep_first cannot be negative")
+        need(1 <= m["conv"] <= 16, i, "1 to 16 convolution taps")
+        src = m.get("kv_from")
+        if src is None:
+            m.pop("kv_from", None)
+        else:
+            need(0 <= int(src) < i and layers[int(src)]["mixer"].get("kv_from") is None, i, "kv_from must name an earlier layer that keeps its own rows")
+            need(all(layers[int(src)]["mixer"][k] == m[k] for k in ("kv_heads", "dim", "vdim")), i, f"kv_heads, dim and vdim must equal those of layer {src}")
+        if f is not None:
+            need(f["kind"] in ("dense", "moe"), i, f"unknown feed-forward kind {f['kind']!r}")
+            f = dict(f)
+        if f is not None and f["kind"] == "moe":
+            r = f["router"] = dict(f["router"], identity=int(f["router"].get("identity") or 0))
+            need(int(r["experts"]) >= 1 and 0 <= r["identity"], i, "at least one expert")
+            need(1 <= int(r["top"]) <= min(64, int(r["experts"]) + r["identity"]) and int(r["experts"]) + r["identity"] <= 1024, i, "1 to 64 of at most 1024 experts")
+            for e in [f["expert"]] + ([f["shared"]] if f.get("shared") else []):
+                need(float(e["limit"]) > 0, i, "limit must be positive")
+        layers.append({"type": s["type"], "mixer": m, "mlp": f})
+    out = {"architecture": d["architecture"], "vocab_size": int(d["vocab"]), "hidden_size": int(d["width"]), "num_hidden_layers": len(layers),
+           "rms_norm_eps": float(d["norm"]["eps"]), "q_lora_rank": None, "n_routed_experts": 0, "n_shared_experts": 0, "tie_word_embeddings": False,
+           "num_attention_heads": 1, "num_key_value_heads": 1, "max_position_embeddings": int(d.get("max_position_embeddings") or 131072),
+           "logit_scale": float(d["logit_scale"]), "layer_specs": layers}
     for k in ("eos_token_id", "bos_token_id"):
         if d.get(k) is not None:
             out[k] = d[k]
@@ -766,3 +815,43 @@ def sapanex_7b(**over) -> ModelConfig:
 
 
 PRESETS["tiny-sapanex"], PRESETS["sapanex-7b"] = tiny_sapanex, sapanex_7b
+
+
+def _differential_spec(heads, kv_heads, dim, vdim, window, keep, conv, diff, ff=0, kv_from=None, experts=None):
+    """`ff`: a dense feed-forward; `experts` = (count, identity, top, ff, shared ff, limit): a mixture."""
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "conv": conv, "diff": diff, "mask": {"size": window, "keep_first": keep}}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    mlp = {"kind": "dense", "ff": ff} if ff else None
+    if experts:
+        n, identity, top, eff, shared, limit = experts
+        mlp = {"kind": "moe", "expert": {"ff": eff, "limit": limit}, "router": {"experts": n, "identity": identity, "top": top}}
+        if shared:
+            mlp["shared"] = {"ff": shared, "limit": limit}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def tiny_gipozen(**over) -> ModelConfig:
+    """CPU-sized Gipozen shape: two layers with rows of their own and one that reads the first one's, a dense feed-forward, a mixture, none."""
+    c = ModelConfig.from_dict({"architecture": "Gipozen", "vocab": 512, "width": 128, "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": [
+        _differential_spec(4, 2, 16, 24, 30, 4, 4, 0.3, ff=192), _differential_spec(4, 2, 16, 24, 50, 0, 4, 0.4, kv_from=0, experts=(8, 2, 3, 48, 64, 5.0)),
+        _differential_spec(6, 1, 24, 16, 20, 9, 2, 0.5)]})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+def gipozen_7b(**over) -> ModelConfig:
+    """A Gipozen shape of a real model's layer sizes (7B class, 2B active): width 2048, 16 / 4 heads of two 64-wide maps over 128-wide values, a
+    4096-token window behind 16 kept tokens, every second layer reading its predecessor's rows, dense and mixture layers in turn."""
+    layers = []
+    for i in range(12):
+        layers += [_differential_spec(16, 4, 64, 128, 4096, 16, 4, 0.3 + 0.02 * i, ff=8192),
+                   _differential_spec(16, 4, 64, 128, 4096, 16, 4, 0.3 + 0.02 * i, kv_from=2 * i, experts=(64, 4, 6, 1024, 2048, 7.0))]
+    c = ModelConfig.from_dict({"architecture": "Gipozen", "vocab": 131072, "width": 2048, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "layers": layers})
+    for k, v in over.items():
+        setattr(c, k, v)
+    return c
+
+
+PRESETS["tiny-gipozen"], PRESETS["gipozen-7b"] = tiny_gipozen, gipozen_7b

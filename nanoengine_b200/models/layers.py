@@ -117,6 +117,18 @@ class DenseMLP(nn.Module):
         return self.down_proj(self.up_proj(x, act=self.act))
 
 
+class PolyNormMLP(nn.Module):
+    """Two linears around a weighted sum of the normed first three powers of the inner values and a constant; coef = (a, b, c, e)."""
+
+    def __init__(self, hidden: int, inter: int, eps: float, dtype, device):
+        super().__init__()
+        self.up_proj, self.down_proj, self.eps = QLinear(hidden, inter, dtype, device), QLinear(inter, hidden, dtype, device), eps
+        self.coef = nn.Parameter(torch.zeros(4, dtype=torch.float32, device=device), requires_grad=False)
+
+    def forward(self, x):
+        return self.down_proj(ops.poly_norm(self.up_proj(x), self.coef, self.eps))
+
+
 class TPSwiGLUMLP(nn.Module):
     """Dense gated MLP sharded over the tensor-parallel group: gate / up column-parallel, down row-parallel.  Takes this
     rank's slice of the tokens and returns its slice of the result: all-gather -> GEMM and GEMM -> reduce-scatter, each one
@@ -344,9 +356,13 @@ class RoutedExperts(nn.Module):
             self.set_expert(s, which, w, scale_inv)
         return bool(slots)
 
-    def forward(self, x, topk_idx, topk_w, add_in=None):
+    def forward(self, x, topk_idx, topk_w, add_in=None, add_gate=None, identity_from=None):
         """Local part of the routed output for the tokens given (weights applied, zero rows where no expert is local);
-        `add_in` (the shared-expert output) is summed in by the same gather pass."""
+        `add_in` (the shared-expert output) is summed in by the same gather pass, times sigmoid(add_gate) per token where that is given.
+        Ids from `identity_from` on stand for experts whose output is their input."""
+        if add_gate is not None or identity_from is not None:
+            return ops.moe_experts(x, topk_idx, topk_w, self.gate_up_proj, self.down_proj, self.gate_up_scale, self.down_scale, self.expert_offset, add_in,
+                                   act=self.act, add_gate=add_gate, identity_from=identity_from)
         if self.quant == "nvfp4":
             if not self._nvfp4_ready:
                 self._prepare_nvfp4()
@@ -393,3 +409,23 @@ class RoutedExperts(nn.Module):
             for which, shape in (("gate", (self.inter, self.hidden)), ("up", (self.inter, self.hidden)), ("down", (self.hidden, self.inter))):
                 w = torch.empty(*shape, dtype=torch.float32, device=dev).normal_(0.0, std, generator=gen)
                 self.set_expert(e, which, w)
+
+
+class GatedSharedMoE(nn.Module):
+    """Softmax-routed experts, some of which may be the identity, beside a shared expert behind a sigmoid gate per token.  A token's choice
+    goes by score + correction, its weights are the plain scores of the chosen.  Router and gate are one fp32 product: the gate's row
+    is the last one.  `act`: gated activation of the routed experts, shared_act of the shared one (see ops.reference.glu_act)."""
+
+    def __init__(self, hidden: int, experts: int, identity: int, top: int, inter: int, act, shared_inter: int, shared_act, dtype, device):
+        super().__init__()
+        assert get_dist_context().ep_size == 1, "identity experts are not sharded"
+        self.num_experts, self.num_scores, self.top = experts, experts + identity, top
+        self.router_weight = nn.Parameter(torch.zeros(self.num_scores + (1 if shared_inter else 0), hidden, dtype=torch.float32, device=device), requires_grad=False)
+        self.correction = nn.Parameter(torch.zeros(self.num_scores, dtype=torch.float32, device=device), requires_grad=False)
+        self.experts = RoutedExperts(experts, hidden, inter, dtype, device, act=act)
+        self.shared = SwiGLUMLP(hidden, shared_inter, dtype, device, None, act=shared_act) if shared_inter else None
+
+    def forward(self, x):
+        logits = ops.router_logits(x, self.router_weight)
+        idx, w, gate = ops.moe_route(logits, self.correction, self.top, norm_topk_prob=False, scoring="softmax", gate_cols=1 if self.shared is not None else 0, split_gate=True)
+        return self.experts(x, idx, w, None if self.shared is None else self.shared(x), gate, self.num_experts)

@@ -10,10 +10,13 @@ PooledAttentionMixer   grouped-query attention over a window of tokens and the m
                 normed over all heads at once, partly rotated, and values that are cached rotated and whose sums are turned back
                 (`ops.pooled_attention_prepare`, `ops.gqa_attention_biased`).
 GeneralDeltaMixer   delta rule with a decay and a removal rate per key channel; everything from one GEMM, the decay's second, low-rank
-                factor from another one with an fp32 result; recurrence, norm and gate are `ops.general_delta`."""
+                factor from another one with an fp32 result; recurrence, norm and gate are `ops.general_delta`.
+DifferentialAttentionMixer   two softmax maps per head over the same values, their difference normed and gated, over a window and the first tokens,
+                with a short convolution behind the projections (`ops.conv_rows`, `ops.differential_attention`); a layer may read the rows
+                of an earlier one."""
 from __future__ import annotations
 
-from typing import Dict, Sequence
+from typing import Dict, Optional, Sequence
 
 import torch
 import torch.nn as nn
@@ -186,3 +189,48 @@ class GeneralDeltaMixer(nn.Module):
         self.out_proj.set_weight(w["o"])
         for p, n in ((self.w0, "w0"), (self.a_bias, "a.b"), (self.norm_weight, "norm")):
             p.copy_(w[n])
+
+
+class DifferentialAttentionMixer(nn.Module):
+    """`reads_only`: the layer has no keys and values of its own and reads cache layer `cache_idx` as an earlier layer left it.  `window` 0: all
+    earlier tokens.  `diff`: the constant part of the weight of the second map."""
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, keep_first: int, diff: float, conv: int, eps: float,
+                 cache_idx: int, reads_only: bool, state_idx: Optional[int], dtype, device):
+        super().__init__()
+        self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = hidden, heads, kv_heads, dim, vdim
+        self.scale, self.window, self.keep_first, self.diff, self.eps = scale, window, keep_first, diff, eps
+        self.cache_idx, self.reads_only, self.state_idx = cache_idx, reads_only, state_idx
+        self.rows = {"q": heads * 2 * dim} if reads_only else {"q": heads * 2 * dim, "k": kv_heads * 2 * dim, "v": kv_heads * vdim}
+        self.channels = sum(self.rows.values())
+        self.in_proj = QLinear(hidden, self.channels + heads * vdim, dtype, device)          # rows: q, k, v, output gate
+        self.out_proj = QLinear(heads * vdim, hidden, dtype, device)
+        self.conv_weight = _const(conv, self.channels, dtype=dtype, device=device)           # newest token's weights last
+        self.mixing = _const(1, device=device)                                               # weight of the second map
+
+    def forward(self, h, ctx: ForwardContext):
+        T = h.shape[0]
+        proj = self.in_proj(h)
+        kc, vc = ctx.kv_caches[self.cache_idx]
+        own = (None, None) if self.reads_only else (kc, vc)
+        q = ops.conv_rows(proj, self.conv_weight, self.rows["q"], *own, ctx.slot_mapping, None if self.state_idx is None else ctx.conv_states[self.state_idx],
+                          ctx.state_slots, ctx.cu_seqlens_q, ctx.seq_fresh, ctx.max_seqlen_q)
+        o = ops.differential_attention(q.view(T, self.heads, 2, self.dim), kc, vc, ctx.block_tables, ctx.cu_seqlens_q, ctx.context_lens, self.scale, self.window,
+                                       self.keep_first, self.mixing, 1.0 - self.diff, self.eps, proj[:, self.channels:], ctx.max_seqlen_q)
+        return self.out_proj(o)
+
+    def parts(self):
+        D, inner = self.hidden, self.heads * self.vdim
+        out = {}
+        for n, r in self.rows.items():
+            out[n], out[n + ".conv"] = (r, D), (r, self.conv_weight.shape[0])
+        out.update({n: (self.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        out["g"], out["o"] = (inner, D), (D, inner)
+        return out
+
+    def load(self, w: Dict[str, torch.Tensor]) -> None:
+        self.in_proj.set_weight(torch.cat([w[n] for n in (*self.rows, "g")], 0))
+        self.out_proj.set_weight(w["o"])
+        self.conv_weight.copy_(torch.cat([w[n + ".conv"] for n in self.rows], 0).t())
+        e = lambda i: (w["lq" + i].double() * w["lk" + i].double()).sum().exp()
+        self.mixing.fill_(float(e("1") - e("2")) + self.diff)

@@ -64,10 +64,16 @@ def _sapanex():
     return SapanexForCausalLM
 
 
+def _gipozen():
+    from .gipozen import GipozenForCausalLM
+    return GipozenForCausalLM
+
+
 # kernel sources (stems under csrc/) of the architectures that can be served from a partial build; None = all of them
 _KERNELS = {"Tuvutar": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_bf16", "mla_bf16", "delta"),
             "Filasun": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "linattn", "linattn_tc"),
-            "Sapanex": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "pooled", "general_delta")}
+            "Sapanex": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "pooled", "general_delta"),
+            "Gipozen": ("gemm", "gemm_simt", "residual", "elementwise", "attn_generic", "gqa_biased", "shortconv", "moe")}
 
 
 def kernel_sources(architecture: str):
@@ -75,7 +81,7 @@ def kernel_sources(architecture: str):
 
 
 _LAZY = {
-    "Tuvutar": _tuvutar, "Filasun": _filasun, "Sapanex": _sapanex,
+    "Tuvutar": _tuvutar, "Filasun": _filasun, "Sapanex": _sapanex, "Gipozen": _gipozen,
     "Gemma4ForCausalLM": _gemma4, "Gemma4ForConditionalGeneration": _gemma4,
     "Glm5NextForConditionalGeneration": _glm5_next, "KimiK3ForConditionalGeneration": _kimi_k3,
     "DeepseekV4ForCausalLM": _deepseek_v4,

@@ -78,6 +78,9 @@ def hf_param_shapes(cfg: ModelConfig, include_mtp: bool = False) -> Dict[str, Tu
     if cfg.architecture.startswith("Gemma4"):
         return _gemma4_param_shapes(cfg, out)
     if cfg.layer_specs:
+        if cfg.architecture == "Gipozen":
+            from .gipozen import gipozen_param_shapes
+            return gipozen_param_shapes(cfg)
         if cfg.architecture == "Sapanex":
             from .sapanex import sapanex_param_shapes
             return sapanex_param_shapes(cfg)
@@ -255,6 +258,10 @@ def random_hf_weights(cfg: ModelConfig, seed: int = 0, device="cpu", keep: Optio
         g.manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
         if cfg.layer_specs:                     # rows scaled by their fan-in, norm weights around zero or one
             leaf = name.rsplit(".", 1)[-1]
+            if cfg.architecture == "Gipozen":
+                from .gipozen import gipozen_random_tensor
+                yield name, gipozen_random_tensor(name, shape, g, dev)
+                continue
             if cfg.architecture == "Sapanex":
                 from .sapanex import sapanex_random_tensor
                 yield name, sapanex_random_tensor(name, shape, g, dev)

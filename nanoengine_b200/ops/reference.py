@@ -130,6 +130,34 @@ def postnorm(y: torch.Tensor, x: torch.Tensor, alpha: float, w: torch.Tensor, ep
     return out.to(y.dtype), x
 
 
+def depth_mix(y: torch.Tensor, x: torch.Tensor, g: torch.Tensor, eps: float, bank: Optional[torch.Tensor] = None, at: int = 0, w: Optional[torch.Tensor] = None,
+              last: bool = False):
+    """The sum behind a sublayer and the norm in front of the next one, around a 32-bit residual stream that may be averaged over the depth: x <- x + y;
+    with `bank` [layers + 1, T, W] fp32, bank[at] = x and x <- sum_{j <= at} w[j] bank[j]; the next input rmsnorm(x) g in y's dtype.  y [T, W]
+    (rows may be strided), x [T, W] fp32, g fp32 [1], w fp32 [at + 1].  Returns (input, x); the CUDA body updates x in place, and with
+    `last` it leaves both x and bank[at] as they are."""
+    x = x + y.float()
+    if bank is not None:
+        bank[at] = x
+        x = torch.einsum("j,jtw->tw", w.float(), bank[: at + 1])
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * g).to(y.dtype), x
+
+
+def depth_embed(ids: torch.Tensor, table: torch.Tensor, g: torch.Tensor, eps: float, layers: int):
+    """The start of such a stream: x = table[ids] in fp32, a bank of `layers` rows with x as its first, and the first input.  Returns (input, x, bank)."""
+    x = table[ids.long()].float()
+    bank = torch.empty(layers, *x.shape, dtype=torch.float32, device=x.device)
+    bank[0] = x
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * g).to(table.dtype), x, bank
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    """a N(z) + b N(z^2) + c N(z^3) + e over rows [T, F] in fp32, N dividing a row by its root mean square; coef fp32 [4] = (a, b, c, e)."""
+    f = z.float()
+    n = lambda p: p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)
+    return (coef[0] * n(f) + coef[1] * n(f * f) + coef[2] * n(f * f * f) + coef[3]).to(z.dtype)
+
+
 def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float):
     """The start of such a stream: x = scale * table[ids] in fp32, and its copy in the table's dtype.  Returns (input, x)."""
     x = scale * table[ids.long()].float()
@@ -325,6 +353,34 @@ def kv_rows(k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Te
     slots = slot_mapping[keep].long()
     for cache, t in ((k_cache, k), (v_cache, v)):
         cache.view(-1, cache.shape[2] * cache.shape[3])[slots] = t[keep].to(cache.dtype)
+
+
+def conv_rows(proj: torch.Tensor, w: torch.Tensor, q_width: int, k_cache, v_cache, slot_mapping: torch.Tensor, window, slots, cu_seqlens: torch.Tensor, fresh,
+              max_q_len: int = 0) -> torch.Tensor:
+    """Short causal convolution over time on the first C columns of proj [T, >= C] (q | k | v, or q alone when the caches are None), w [taps, C] with the
+    newest token's weights last: y_t = sum_j w[j] u_{t - taps + 1 + j}.  `window` [S, taps - 1, C] carries the last inputs of each sequence (zeros for a
+    `fresh` one; None for a single tap) and is updated.  The results of the key and value columns go to rows `slot_mapping` of the paged caches,
+    those of the first q_width columns are returned, [T, q_width] in proj's dtype.  `max_q_len`: planning hint of the CUDA body."""
+    taps, C = w.shape
+    T = proj.shape[0]
+    y = torch.empty(T, C, dtype=torch.float32, device=proj.device)
+    cu = cu_seqlens.tolist()
+    for i in range(len(cu) - 1):
+        s, e = cu[i], cu[i + 1]
+        if e <= s:
+            continue
+        full = proj[s:e, :C]
+        if taps > 1:
+            slot = int(slots[i])
+            win = torch.zeros_like(window[slot]) if int(fresh[i]) else window[slot]
+            full = torch.cat([win, full.to(window.dtype)], 0)
+            window[slot] = full[full.shape[0] - (taps - 1):]
+        y[s:e] = sum(full[j: j + e - s].float() * w[j].float() for j in range(taps))
+    y = y.to(proj.dtype)
+    if k_cache is not None:
+        kw = k_cache.shape[2] * k_cache.shape[3]
+        kv_rows(k_cache, v_cache, slot_mapping, y[:, q_width: q_width + kw], y[:, q_width + kw:])
+    return y[:, :q_width].contiguous()
 
 
 def gqa_qkv_prepare(qkv: torch.Tensor, hq: int, hkv: int, hd: int, q_norm_w, k_norm_w, eps: float, unit_offset: bool, positions,
@@ -526,6 +582,33 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
     return out
 
 
+def differential_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int, keep_first: int, mixing: torch.Tensor,
+                           out_scale: float, eps: float, gate: torch.Tensor, max_q_len: int = 0) -> torch.Tensor:
+    """Differential attention over paged caches.  q [T, Hq, 2, D], k_cache [blocks, block_size, Hkv, 2 D] (the keys of both maps side by side), v_cache
+    [..., Dv]: each map is a softmax of its own over the same values; a query at position i sees position j <= i when i - j < window (window 0: always)
+    or j < keep_first.  o = a1 - mixing a2 (fp32 [1]), divided by its root mean square over the head, times out_scale and, element by element,
+    sigmoid(gate [T, Hq Dv]).  Returns [T, Hq Dv] in q's dtype.  `max_q_len`: planning hint of the CUDA body."""
+    T, Hq, _, D = q.shape
+    Hkv, Dv = k_cache.shape[2], v_cache.shape[3]
+    o = torch.zeros(T, Hq, Dv, dtype=torch.float32, device=q.device)
+    for i in range(cu_seqlens_q.numel() - 1):
+        lo, hi = int(cu_seqlens_q[i]), int(cu_seqlens_q[i + 1])
+        if hi == lo:
+            continue
+        n, ql = int(context_lens[i]), hi - lo
+        k = _gather_rows(k_cache, block_tables[i], n).view(n, Hkv, 2, D).repeat_interleave(Hq // Hkv, 1)
+        v = _gather_rows(v_cache, block_tables[i], n).repeat_interleave(Hq // Hkv, 1)
+        s = torch.einsum("thmd,nhmd->tmhn", q[lo:hi].float(), k) * scale
+        pos, key = torch.arange(n - ql, n, device=q.device).view(ql, 1, 1, 1), torch.arange(n, device=q.device).view(1, 1, 1, n)
+        seen = key <= pos
+        if window > 0:
+            seen = seen & ((pos - key < window) | (key < keep_first))
+        a = torch.einsum("tmhn,nhd->tmhd", torch.softmax(s.masked_fill(~seen, float("-inf")), -1), v)
+        o[lo:hi] = a[:, 0] - mixing * a[:, 1]
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * out_scale
+    return (o.reshape(T, Hq * Dv) * torch.sigmoid(gate.float())).to(q.dtype)
+
+
 def attention_varlen(q, k, v, cu_seqlens, scale, causal: bool = False) -> torch.Tensor:
     """Attention over ragged sequences: q, k, v [T, H, D]; sequence i owns rows [cu[i], cu[i+1]).  Non-causal by default (the
     vision encoder, reference vl/vision/encoder.py:154-198)."""
@@ -577,7 +660,7 @@ def merge_attention_states(o1, lse1, o2, lse2):
 # ---- MoE -----------------------------------------------------------------------------------------
 def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, n_group: int = 1, topk_group: int = 1,
               norm_topk_prob: bool = True, routed_scaling_factor: float = 1.0, scoring: str = "sigmoid",
-              balance_ranks: int = 0, log2phy: Optional[torch.Tensor] = None, logcnt: Optional[torch.Tensor] = None):
+              balance_ranks: int = 0, log2phy: Optional[torch.Tensor] = None, logcnt: Optional[torch.Tensor] = None, gate_cols: int = 0, split_gate: bool = False):
     """DeepSeek ``noaux_tc`` routing and Qwen3 softmax routing.
 
     scores = sigmoid|softmax|sqrt(softplus) (logits fp32; the last is DeepSeek-V4's, reference models/deepseek_v4/deepseek_v4.py:40-47); choice = scores + bias; with n_group > 1 only the
@@ -589,10 +672,14 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, n_
     ids dealt evenly over that many expert-parallel ranks (a load-balance stand-in for random-init routers, reference
     layers/backends/experts/deep_gemm.py:47-67); `log2phy [E, R]` / `logcnt [E]` map every logical id to one of its
     physical replicas, picked by (row, k) hash so replicas share the load (reference experts/eplb.py, triton/generic/moe.py:561).
+
+    `split_gate`: the last `gate_cols` (0 or 1) columns of the logits are not scores; returns (idx, weights, that column [T] or None).
     """
     lf = logits.float()
     if lf.dim() == 3:          # partial sums of a split-K router product
         lf = lf.sum(0)
+    gate = lf[:, -1].contiguous() if gate_cols else None
+    lf = lf[:, : lf.shape[1] - gate_cols]
     scores = (torch.sigmoid(lf) if scoring == "sigmoid" else F.softplus(lf).sqrt() if scoring == "sqrtsoftplus" else torch.softmax(lf, -1))
     choice = scores + bias.float() if bias is not None else scores
     T, E = choice.shape
@@ -616,7 +703,8 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, n_
         k = torch.arange(top_k, device=idx.device).view(1, top_k)
         h = (((t * 2654435761 + k * 40503) & 0xFFFFFFFF) >> 8) % cnt
         idx = log2phy.to(idx.device).long()[idx, h]
-    return idx.to(torch.int32), (w * routed_scaling_factor).float()
+    idx, w = idx.to(torch.int32), (w * routed_scaling_factor).float()
+    return (idx, w, gate) if split_gate else (idx, w)
 
 
 _E2M1 = (0.0, 0.5, 1.0, 1.5, 2.0, 3.0, 4.0, 6.0)
@@ -677,9 +765,11 @@ def silu_and_mul(x: torch.Tensor, quant: bool = False, act=None) -> torch.Tensor
     return glu_act(a, b, act).to(x.dtype)
 
 
-def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, expert_offset: int = 0, add_in=None, act=None) -> torch.Tensor:
+def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, expert_offset: int = 0, add_in=None, act=None, add_gate=None,
+                identity_from: Optional[int] = None) -> torch.Tensor:
     """Routed experts held locally: ids [expert_offset, expert_offset + E_local).  w13 [E, 2I, H], w2 [E, H, I].
-    Returns the weighted sum over the local experts of each token (zeros where none is local).  `act`: see `glu_act`."""
+    Returns the weighted sum over the local experts of each token (zeros where none is local).  `act`: see `glu_act`.  Ids from `identity_from` on
+    are experts whose output is the token's own row.  `add_gate` fp32 [T]: `add_in` enters times its sigmoid, and the sum is rounded once."""
     if callable(add_in):
         add_in = add_in()
     T, H = x.shape
@@ -695,6 +785,10 @@ def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, exp
         h = silu_and_mul(h, act=act)
         y = linear(h, w2[e], None if w2_scale is None else w2_scale[e])
         out.index_add_(0, tok, y.float() * topk_w[tok, slot].unsqueeze(-1))
+    if identity_from is not None:
+        out = out + (topk_w * (topk_idx >= identity_from)).sum(-1, keepdim=True) * x.float()
+    if add_gate is not None and add_in is not None:
+        return (out + torch.sigmoid(add_gate)[:, None] * add_in.float()).to(x.dtype)
     out = out.to(x.dtype)
     return out if add_in is None else out + add_in
 

@@ -14,12 +14,12 @@ DeepSeek-V4        one shared key / value row per token and layer in the latent-
                    compressor's carry [c * ratio, c * head_dim] fp32 twice (values and scores; c = 2 for ratio 4).  With an fp8 cache a row
                    is 584 packed bytes (448 e4m3 values, 64 bf16 rotated dims, 7 scale bytes + pad) instead of head_dim values.
 
-listed layers      families that list their layers one by one (Tuvutar, Filasun, Sapanex) may give every layer its own row widths and state shape:
+listed layers      families that list their layers one by one (Tuvutar, Filasun, Sapanex, Gipozen) may give every layer its own row widths and state shape:
                    one tensor per layer instead of the stacked ones - latent rows [blocks, block_size, D_l], or keys [blocks, block_size,
                    G_l, D_l] and values [.., G_l, Dv_l]; states [slots, Hv_l, Dv_l, Dk_l] fp32 and convolution windows [slots, K_l - 1,
                    conv_dim_l].  Page families `latent_<n>` or `key_<n>` / `value_<n>` (and `pooled_key_<n>` / `pooled_value_<n>`), slot families `delta_state_<n>` / `delta_conv_<n>`.  A
                    layer may own rows, a state, both (attention and linear attention side by side) or neither (it reads an earlier layer's
-                   rows); rows and states are numbered separately.  A layer that pools adds the means of blocks of P tokens, keys
+                   rows); rows and states are numbered separately.  A state may be a convolution window alone (0 heads).  A layer that pools adds the means of blocks of P tokens, keys
                    [blocks, R, G_l, D_l] and values [blocks, R, G_l, Dv_l]: eight neighbouring pooled rows sit together in the page of the
                    first token of their first block (`ops.reference.pooled_rows_per_page`), so R = 8 for P >= 8.
 
@@ -201,12 +201,16 @@ def _make_cache_plan(mc: ModelConfig, kv_dtype_name: str, block_size: int, attn_
         if not mc.is_mla:
             mixers = [mc.layer_specs[i] for i in range(n)]
             rows = [mixers[i]["mixer"].get("left", mixers[i]["mixer"]) for i in own]
-            kv = [(int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])) for m in rows]
+            maps = lambda m: 2 if "diff" in m else 1          # differential attention keeps the keys of both maps side by side
+            kv = [(int(m["kv_heads"]), maps(m) * int(m["dim"]), int(m["vdim"])) for m in rows]
             pools = [int(m["mask"].get("pool") or 0) for m in rows]
             shapes = []
-            for s in mixers:
+            for i, s in enumerate(mixers):
                 m = s["mixer"]
-                if s["type"] == "mamba2":
+                if s["type"] == "attention" and mc.keeps_state(i):      # no recurrent state, the window of the short convolutions only
+                    own_rows = int(m["kv_heads"]) * (maps(m) * int(m["dim"]) + int(m["vdim"])) if mc.keeps_rows(i) else 0
+                    shapes.append((0, 0, 0, int(m["conv"]), int(m["heads"]) * maps(m) * int(m["dim"]) + own_rows))
+                elif s["type"] == "mamba2":
                     shapes.append((int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["conv"]), int(m["heads"]) * int(m["vdim"]) + 2 * int(m["groups"]) * int(m["state"])))
                 elif s["type"] == "parallel":
                     r = m["right"]
