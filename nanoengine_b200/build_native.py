@@ -35,7 +35,7 @@ GENCODE = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
               "-Xptxas", "-v", "-DNDEBUG", "-rdc=true"] + GENCODE
 # translation units whose 32-bit results are held to 32-bit accuracy (gates of a recurrence, tanh): no approximate functions there
-PRECISE = {"delta", "residual", "gemm_simt", "attn_generic", "linattn", "pooled", "general_delta"}
+PRECISE = {"delta", "residual", "gemm_simt", "attn_generic", "linattn", "pooled", "general_delta", "shortconv", "moe"}
 
 
 def nvcc_flags(stem: str):

@@ -10,7 +10,9 @@
 // output fp32 too: runs in true 32-bit).  Options: a window of the last keys, scores capped as cap tanh(s / cap), a distance bias
 // -slope[head] (query position - key position) after the cap, the output of a head times sigmoid(gate[token, head]) and a constant.
 // With pooled rows (pooled.cuh) a query also sees the blocks wholly in front of its window, in the same softmax; an output may be rotated back by
-// its position (pairs of columns d, d + Dv / 2).
+// its position (pairs of columns d, d + Dv / 2).  Behind a window the first `keep` tokens of the sequence stay visible.
+// Differential form (maps = 2): a head has two query vectors, a key / value head two key vectors side by side; two warps take the two maps of a head
+// over the same values, and o = a1 - mixing a2 is divided by its root mean square, scaled, and multiplied by sigmoid(egate) element by element.
 //
 // Replaces in the reference: attention/base.py:451-525 (SDPA reference), flash_mla sparse decode call sites
 // (layers/backends/mla/flash_mla.py:22-121) for the sparse case, flashinfer / FA paged GQA wrappers.
@@ -42,6 +44,9 @@ struct AttnArgs {
   const void* gate; long long gate_ld; float out_scale;      // gate null: none
   const void* k_pool; const void* v_pool; int pool, pool_rows;      // pool 0: none
   const float* turn; int n_pos;                              // [n_pos, Dv] cos | sin, or null
+  int keep;                                                  // > 0, with a window: the first keys that stay visible
+  int maps;                                                  // 1, or 2 for the differential form: H, the strides of q and kv_group then count maps
+  const float* mixing; float eps; const void* egate; long long egate_ld;
 };
 
 // kind: 0 bf16, 1 e4m3, 2 fp32
@@ -54,10 +59,10 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   extern __shared__ float sm[];
   // layout: q [4][Dk] | ktile [32][Dk+1] | vtile [32][Dv+1] (only when V is separate)
-  const int Dk = a.Dk, Dv = a.Dv;
+  const int Dk = a.Dk, Dv = a.Dv, Dks = Dk * a.maps;          // a staged key row holds the keys of all maps
   float* sq = sm;
   float* sk = sq + kHeadsPerCta * Dk;
-  float* sv = a.v_cache ? sk + kKeysPerTile * (Dk + 1) : nullptr;
+  float* sv = a.v_cache ? sk + kKeysPerTile * (Dks + 1) : nullptr;
   const int t = blockIdx.x, h0 = blockIdx.y * a.heads_per_cta;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = h0 + warp;
@@ -91,10 +96,12 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
   const int* bt = a.block_tables + (long long)seq * a.bt_stride;
 
   const int n_pool = a.pool ? pooled_visible(limit, a.window, a.pool) : 0, pool_tiles = (n_pool + kKeysPerTile - 1) / kKeysPerTile;
-  const int tile0 = first_key / kKeysPerTile, tiles = pool_tiles + max(0, (n_keys + kKeysPerTile - 1) / kKeysPerTile - tile0);
+  const int keep_tiles = (min(a.keep, first_key) + kKeysPerTile - 1) / kKeysPerTile;          // of kept keys in front of the window
+  const int tile0 = max(first_key / kKeysPerTile, keep_tiles), tiles = pool_tiles + keep_tiles + max(0, (n_keys + kKeysPerTile - 1) / kKeysPerTile - tile0);
   for (int it = 0; it < tiles; it++) {
     const bool pooled = it < pool_tiles;
-    const int k0 = (pooled ? it : it - pool_tiles + tile0) * kKeysPerTile, k_end = pooled ? n_pool : n_keys, k_first = pooled ? 0 : first_key;
+    const int at = it - pool_tiles;
+    const int k0 = (pooled ? it : at < keep_tiles ? at : at - keep_tiles + tile0) * kKeysPerTile, k_end = pooled ? n_pool : n_keys, k_first = pooled ? 0 : first_key;
     const void *kbase = pooled ? a.k_pool : a.k_cache, *vbase = pooled ? a.v_pool : a.v_cache;
     __syncthreads();
     // stage 32 key rows (and value rows) as fp32
@@ -113,20 +120,21 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
           slot = (a.block_size == 1 || NE_INDEX_OK(page, BK_CACHE_PAGES, 23, __LINE__)) ? (long long)page * a.block_size + kidx % a.block_size : -1;
         }
       }
-      for (int d = lane; d < Dk; d += 32)
-        sk[r * (Dk + 1) + d] = slot >= 0 ? load_kv(kbase, slot * a.kv_slot_stride + (long long)kvh * a.kv_head_stride + d, a.fp8) : 0.f;
+      for (int d = lane; d < Dks; d += 32)
+        sk[r * (Dks + 1) + d] = slot >= 0 ? load_kv(kbase, slot * a.kv_slot_stride + (long long)kvh * a.kv_head_stride + d, a.fp8) : 0.f;
       if (sv) for (int d = lane; d < Dv; d += 32)
         sv[r * (Dv + 1) + d] = slot >= 0 ? load_kv(vbase, slot * a.v_slot_stride + (long long)kvh * a.v_head_stride + d, a.fp8) : 0.f;
-      if (lane == 0) sk[r * (Dk + 1) + Dk] = slot >= 0 ? 1.f : 0.f;   // validity marker in the padding column
+      if (lane == 0) sk[r * (Dks + 1) + Dks] = slot >= 0 ? 1.f : 0.f;   // validity marker in the padding column
     }
     __syncthreads();
     if (!head_ok) continue;
     // lane scores key `lane`
-    const float* kr = sk + lane * (Dk + 1);
+    const float* kr = sk + lane * (Dks + 1);
     const float* qr = sq + warp * Dk;
+    const float* km = a.maps == 2 ? kr + (h & 1) * Dk : kr;
     float s = 0.f;
-    for (int d = 0; d < Dk; d++) s = fmaf(qr[d], kr[d], s);
-    bool valid = (k0 + lane < k_end) && (k0 + lane >= k_first) && kr[Dk] != 0.f;
+    for (int d = 0; d < Dk; d++) s = fmaf(qr[d], km[d], s);
+    bool valid = (k0 + lane < k_end) && (k0 + lane >= k_first || k0 + lane < a.keep) && kr[Dks] != 0.f;
     float tl = s * c;
     if (a.softcap > 0.f) tl = a.softcap * tanhf(s * a.scale / a.softcap) * kLog2e;
     if (a.slopes) tl -= slope * (float)(limit - (k0 + lane)) * kLog2e;
@@ -138,7 +146,7 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
     l_run = l_run * alpha + warp_sum(p);
     m_run = m_new;
     const float* vt = sv ? sv : sk;
-    const int vstride = sv ? Dv + 1 : Dk + 1;
+    const int vstride = sv ? Dv + 1 : Dks + 1;
 #pragma unroll
     for (int j = 0; j < 20; j++) acc[j] *= alpha;
     for (int kk = 0; kk < kKeysPerTile; kk++) {
@@ -151,7 +159,29 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(const AttnArgs a) {
       }
     }
   }
-  if (a.turn) __syncthreads();                 // the tiles' memory is free
+  if (a.turn || a.maps == 2) __syncthreads();  // the tiles' memory is free
+  if (a.maps == 2) {
+    if (head_ok) {
+      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+#pragma unroll
+      for (int j = 0; j < 20; j++) { const int d = lane + 32 * j; if (j < per_lane && d < Dv) sk[warp * Dv + d] = acc[j] * inv; }
+    }
+    __syncthreads();
+    const int hr = h0 / 2 + warp;              // the head whose maps the warps 2 w and 2 w + 1 took
+    if (2 * warp >= a.heads_per_cta || h0 + 2 * warp >= a.H) return;
+    const float* so = sk + 2 * warp * Dv;
+    const float lam = *a.mixing;
+    float ss = 0.f;
+    for (int d = lane; d < Dv; d += 32) { const float o = so[d] - lam * so[Dv + d]; ss += o * o; }
+    const float r = rsqrtf(warp_sum(ss) / (float)Dv + a.eps) * a.out_scale;
+    for (int d = lane; d < Dv; d += 32) {
+      const float o = (so[d] - lam * so[Dv + d]) * r / (1.f + expf(-load_kv(a.egate, (long long)t * a.egate_ld + (long long)hr * Dv + d, a.fp8 == 2 ? 2 : 0)));
+      const long long at = (long long)t * a.o_tok_stride + (long long)hr * a.o_head_stride + d;
+      if (a.fp8 == 2) reinterpret_cast<float*>(a.out)[at] = o;
+      else reinterpret_cast<__nv_bfloat16*>(a.out)[at] = __float2bfloat16(o);
+    }
+    return;
+  }
   if (!head_ok) return;
   float inv = (l_run > 0.f ? 1.f / l_run : 0.f) * a.out_scale;
   if (a.gate) inv /= 1.f + expf(-load_kv(a.gate, (long long)t * a.gate_ld + h, a.fp8 == 2 ? 2 : 0));
@@ -266,7 +296,7 @@ using namespace ne;
 
 static int attn_generic_launch(AttnArgs& a, cudaStream_t st) {
   // (the way out of a rotated output, kHeadsPerCta rows of Dv, fits in the tiles of 32 keys and values)
-  const size_t smem = sizeof(float) * ((size_t)kHeadsPerCta * a.Dk + (size_t)kKeysPerTile * (a.Dk + 1) + (a.v_cache ? (size_t)kKeysPerTile * (a.Dv + 1) : 0));
+  const size_t smem = sizeof(float) * ((size_t)kHeadsPerCta * a.Dk + (size_t)kKeysPerTile * (a.Dk * a.maps + 1) + (a.v_cache ? (size_t)kKeysPerTile * (a.Dv + 1) : 0));
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
     cudaError_t e = cudaFuncSetAttribute(attn_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -282,8 +312,9 @@ static int attn_generic_launch(AttnArgs& a, cudaStream_t st) {
 extern "C" int ne_attn_biased(const void* q, long long q_ld, const void* k_cache, const void* v_cache, const int* block_tables, int bt_stride, int block_size,
                               const int* cu_seqlens_q, const int* context_lens, int num_seqs, void* out, long long o_ld, int T, int H, int Hkv, int D, int Dv,
                               float scale, float softcap, const float* slopes, int window, const void* gate, long long gate_ld, float out_scale, int fp32,
-                              const void* k_pool, const void* v_pool, int pool, int pool_rows, const float* turn, int n_pos, cudaStream_t st) {
+                              const void* k_pool, const void* v_pool, int pool, int pool_rows, const float* turn, int n_pos, int keep, cudaStream_t st) {
   if (T <= 0) return 0;
+  if (keep > 0 && pool > 0) return 1004;
   if (pool > 0 && (window < 1 || softcap > 0.f || slopes || !k_pool || !v_pool || pool_rows < (block_size + 8 * pool - 1) / (8 * pool) * 8)) return 1004;
   if (turn && (n_pos < 1 || Dv % 2)) return 1005;
   if (Hkv < 1 || H % Hkv || Dv < 1 || Dv > 640 || D < 1 || D > 640) return 1001;
@@ -294,8 +325,27 @@ extern "C" int ne_attn_biased(const void* q, long long q_ld, const void* k_cache
   a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs; a.out = out; a.o_tok_stride = o_ld;
   a.o_head_stride = Dv; a.T = T; a.H = H; a.Dk = D; a.Dv = Dv; a.scale = scale; a.fp8 = fp32 ? 2 : 0; a.window = window; a.softcap = softcap; a.slopes = slopes;
   a.gate = gate; a.gate_ld = gate_ld; a.out_scale = out_scale; a.k_pool = k_pool; a.v_pool = v_pool; a.pool = pool > 0 ? pool : 0; a.pool_rows = pool_rows;
-  a.turn = turn; a.n_pos = n_pos;
+  a.turn = turn; a.n_pos = n_pos; a.keep = window > 0 && keep > 0 ? keep : 0; a.maps = 1;
   for (a.heads_per_cta = kHeadsPerCta; a.kv_group % a.heads_per_cta; a.heads_per_cta--) {}
+  return attn_generic_launch(a, st);
+}
+
+// Differential form: q [T, H, 2, D] (row stride q_ld), k_cache [slots, Hkv, 2 D], v_cache [slots, Hkv, Dv], mixing fp32 [1], gate [T, H Dv] (row stride
+// gate_ld), out [T, H Dv] with row stride o_ld.  window 0: all earlier keys; keep: the first keys stay visible behind the window.
+extern "C" int ne_attn_diff(const void* q, long long q_ld, const void* k_cache, const void* v_cache, const int* block_tables, int bt_stride, int block_size,
+                            const int* cu_seqlens_q, const int* context_lens, int num_seqs, void* out, long long o_ld, int T, int H, int Hkv, int D, int Dv,
+                            float scale, int window, int keep, const float* mixing, float out_scale, float eps, const void* gate, long long gate_ld, int fp32,
+                            cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (Hkv < 1 || H % Hkv || Dv < 1 || Dv > 640 || D < 1 || 2 * D > 640 || !mixing || !gate) return 1001;
+  AttnArgs a;
+  memset(&a, 0, sizeof(a));
+  a.q = q; a.q_tok_stride = q_ld; a.q_head_stride = D; a.k_cache = k_cache; a.v_cache = v_cache; a.kv_slot_stride = (long long)Hkv * 2 * D; a.kv_head_stride = 2 * D;
+  a.v_slot_stride = (long long)Hkv * Dv; a.v_head_stride = Dv; a.kv_group = 2 * (H / Hkv); a.block_tables = block_tables; a.bt_stride = bt_stride;
+  a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs; a.out = out; a.o_tok_stride = o_ld;
+  a.o_head_stride = Dv; a.T = T; a.H = 2 * H; a.Dk = D; a.Dv = Dv; a.scale = scale; a.fp8 = fp32 ? 2 : 0; a.window = window; a.keep = window > 0 && keep > 0 ? keep : 0;
+  a.maps = 2; a.mixing = mixing; a.out_scale = out_scale; a.eps = eps; a.egate = gate; a.egate_ld = gate_ld;
+  a.heads_per_cta = a.kv_group % 4 ? 2 : 4;
   return attn_generic_launch(a, st);
 }
 
@@ -313,7 +363,7 @@ extern "C" int ne_attn_generic(const void* q, long long q_tok_stride, int q_head
   a.bt_stride = bt_stride; a.block_size = block_size; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs;
   a.sparse = sparse; a.topk = topk; a.out = out; a.o_tok_stride = o_tok_stride; a.o_head_stride = o_head_stride; a.lse = lse;
   a.T = T; a.H = H; a.Dk = Dk; a.Dv = Dv; a.scale = scale; a.fp8 = fp8; a.window = window; a.noncausal = noncausal;
-  a.v_slot_stride = kv_slot_stride; a.v_head_stride = kv_head_stride; a.out_scale = 1.f;
+  a.v_slot_stride = kv_slot_stride; a.v_head_stride = kv_head_stride; a.out_scale = 1.f; a.maps = 1;
   // multi-head attention proper (one kv head per query head, separate V): the four query heads of a CTA would need four
   // different key tiles, so a CTA serves one head there
   a.heads_per_cta = (kv_group == 1 && kv_head_stride != 0 && v_cache != nullptr) ? 1 : kHeadsPerCta;

@@ -1,6 +1,6 @@
 // Plain tiled matrix product on CUDA cores: D[b] = A[b] B[b]^T with fp32 accumulation in the order of K.  Serves what the
 // tensor-core GEMM does not take: true 32-bit operands (fp32 runs, no TF32) and bf16 operands whose sizes or strides TMA cannot
-// address (K or N not a multiple of 8, unaligned rows).  The result of a row does not depend on the other rows of the call.
+// address (K or N not a multiple of 8, unaligned rows), also over the expert-major rows of a mixture.  The result of a row does not depend on the other rows of the call.
 #include "ptx.cuh"
 
 namespace ne {
@@ -16,11 +16,20 @@ constexpr int kTile = 64, kTileK = 16;
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* __restrict__ A, long long lda, long long a_bs, const TI* __restrict__ B, long long ldb,
                                                        long long b_bs, TO* __restrict__ D, long long ldd, long long d_bs, int M, int N, int K,
-                                                       const float* __restrict__ bias, int act, int act_from) {
+                                                       const float* __restrict__ bias, int act, int act_from, const int* __restrict__ counts,
+                                                       const int* __restrict__ row_start, int groups) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   __shared__ float sA[kTileK][kTile + 4], sB[kTileK][kTile + 4];
   A += blockIdx.z * a_bs; B += blockIdx.z * b_bs; D += blockIdx.z * d_bs;
   const int m0 = blockIdx.y * kTile, n0 = blockIdx.x * kTile;
+  if (row_start) {                  // rows of group g start at a multiple of the tile; a tile belongs to the last group that starts at or before it
+    if (m0 >= row_start[groups]) return;
+    int lo = 0, hi = groups - 1;
+    while (lo < hi) { const int mid = (lo + hi + 1) >> 1; if (row_start[mid] <= m0) lo = mid; else hi = mid - 1; }
+    M = min(M, row_start[lo] + counts[lo]);
+    if (m0 >= M) return;
+    B += lo * b_bs;
+  }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kTileK) {
@@ -55,9 +64,11 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* __restrict__ A
 
 template <typename TI, typename TO>
 static int simt(const void* A, long long lda, long long a_bs, const void* B, long long ldb, long long b_bs, void* D, long long ldd, long long d_bs,
-                int M, int N, int K, int batch, const float* bias, int act, int act_from, cudaStream_t st) {
+                int M, int N, int K, int batch, const float* bias, int act, int act_from, cudaStream_t st, const int* counts = nullptr, const int* row_start = nullptr,
+                int groups = 0) {
   const dim3 grid((unsigned)((N + kTile - 1) / kTile), (unsigned)((M + kTile - 1) / kTile), (unsigned)batch);
-  return (int)launch_pdl(gemm_simt_kernel<TI, TO>, grid, dim3(256), 0, st, (const TI*)A, lda, a_bs, (const TI*)B, ldb, b_bs, (TO*)D, ldd, d_bs, M, N, K, bias, act, act_from);
+  return (int)launch_pdl(gemm_simt_kernel<TI, TO>, grid, dim3(256), 0, st, (const TI*)A, lda, a_bs, (const TI*)B, ldb, b_bs, (TO*)D, ldd, d_bs, M, N, K, bias, act, act_from,
+                         counts, row_start, groups);
 }
 
 }  // namespace ne
@@ -74,4 +85,14 @@ extern "C" int ne_gemm_simt(const void* A, long long lda, long long a_bs, const 
   if (in_fp32) return out_fp32 ? simt<float, float>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, act, act_from, st) : 1002;
   return out_fp32 ? simt<__nv_bfloat16, float>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, act, act_from, st)
                   : simt<__nv_bfloat16, __nv_bfloat16>(A, lda, a_bs, B, ldb, b_bs, D, ldd, d_bs, M, N, K, batch, bias, act, act_from, st);
+}
+
+// Grouped form: rows [row_start[g], row_start[g] + counts[g]) of A [M, K] times B[g] [N, K]; group starts are multiples of 64, D [M, N] as A.
+extern "C" int ne_gemm_simt_groups(const void* A, const void* B, void* D, int M, int N, int K, int groups, const int* counts, const int* row_start, int fp32,
+                                   cudaStream_t st) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K < 0 || groups < 1 || (M + kTile - 1) / kTile > 65535 || !counts || !row_start) return 1001;
+  const long long b_bs = (long long)N * K;
+  return fp32 ? simt<float, float>(A, K, 0, B, K, b_bs, D, N, 0, M, N, K, 1, nullptr, 0, 0, st, counts, row_start, groups)
+              : simt<__nv_bfloat16, __nv_bfloat16>(A, K, 0, B, K, b_bs, D, N, 0, M, N, K, 1, nullptr, 0, 0, st, counts, row_start, groups);
 }

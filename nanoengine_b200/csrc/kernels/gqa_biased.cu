@@ -19,6 +19,11 @@
 // kExt: (1) beside the window a row sees the pooled rows (pooled.cuh) of blocks wholly in front of it: tiles of 64 pooled rows, fetched as eight
 // groups of eight, come before the window's pages, in one softmax; (2) a row's output is rotated back by its position (pairs of columns m, m + Dv / 2)
 // on its way out, through shared memory.
+// keep: the first tokens of a sequence stay visible behind the window; their pages come in front of the window's.
+// kDiff: differential attention.  A head has two query vectors and a key / value head two key vectors side by side; the two maps of a (token, head) pair
+// are two rows of the tile (the maps in halves of the rows), with zeros where the other map's query would be, so that one pass over keys and values
+// serves both.  A pair's rows meet in shared memory (or in the merge kernel): o = a1 - mixing a2, divided by its root mean square, scaled, gated element
+// by element.
 // With more than one slice the CTA writes a normalised partial result and its log2-sum-exp; gqa_biased_merge folds them and applies the gate.
 #include "ptx.cuh"
 #include "pooled.cuh"
@@ -47,13 +52,17 @@ struct GbArgs {
   int pool;                                    // kExt: tokens per pooled row (0: none)
   const float* turn; int n_pos;                // kExt: [n_pos, Dv] cos | sin, or null
   int bar_off;                                 // where the barriers lie in shared memory
+  int keep;                                    // first keys that stay visible behind the window
+  const float* mixing; float eps; const __nv_bfloat16* egate; long long egate_ld;      // kDiff; out_scale is part of it
 };
 
 __device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ld, long long t, int h, float scale) {
   return gate ? scale / (1.f + __expf(-__bfloat162float(gate[t * ld + h]))) : scale;
 }
 
-template <bool kCap, bool kRep, bool kExt>
+__device__ __forceinline__ float sigmoid_of(float x) { return 1.f / (1.f + __expf(-x)); }
+
+template <bool kCap, bool kRep, bool kExt, bool kDiff = false>
 __global__ void __launch_bounds__(kGbThreads, 2)
 gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                   const __grid_constant__ CUtensorMap kp_map, const __grid_constant__ CUtensorMap vp_map, const GbArgs a) {
@@ -75,7 +84,15 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 
   const int warp = threadIdx.x >> 5;
   const int hkv = blockIdx.y, split = blockIdx.z;
-  const int live_warps = kRep ? 4 : (a.g * a.tq + 31) / 32;         // softmax warps with rows of the tile
+  const int pairs = a.g * a.tq, half_rows = a.rows8 >> 1;           // kDiff: rows [0, pairs) are the first maps, [half_rows, half_rows + pairs) the second
+  const int live_warps = kRep ? 4 : ((kDiff ? half_rows + pairs : pairs) + 31) / 32;         // softmax warps with rows of the tile
+  if constexpr (kDiff) {
+    for (int i = threadIdx.x; i < a.nc * half_rows * 8; i += kGbThreads) {
+      const int c = i / (half_rows * 8), r = i - c * half_rows * 8;
+      reinterpret_cast<uint4*>(sQ + c * q_chunk + (c < a.nc >> 1 ? half_rows * 128 : 0))[r] = make_uint4(0, 0, 0, 0);      // the other map's rows
+    }
+    fence_proxy_async_smem();
+  }
   if (warp == 0) {
     int seq, tok;
     find_seq_tile(a.cu_seqlens_q, a.num_seqs, a.tq, blockIdx.x, seq, tok);
@@ -98,7 +115,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   const uint32_t tmem_base = *tmem_slot, tmem_o = tmem_base + 128;
   const int seq = s_tile[0], tok0 = s_tile[1];
 
-  int n_tiles = 0, pg_begin = 0, n_tok = 0, base_limit = -1;
+  int n_tiles = 0, pg0 = 0, kept = 0, skip = 0, n_tok = 0, base_limit = -1;       // tile i that is no tile of pooled rows: page_of(i)
   int n_pt = 0, n_pool = 0, pt_first = 0;                // tiles of pooled rows in front of the pages, pooled rows visible to the tile's last token
   const int* bt = a.block_tables;
   if (seq >= 0) {
@@ -108,19 +125,29 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int max_limit = base_limit + n_tok - 1;
     const int first = a.window > 0 ? max(0, base_limit - a.window + 1) / kBPage : 0;
     if (kExt && a.pool) { n_pool = pooled_visible(max_limit, a.window, a.pool); n_pt = (n_pool + kBPage - 1) / kBPage; }
-    const int pages = max_limit >= 0 ? max_limit / kBPage + 1 - first : 0, total = pages + n_pt;
+    kept = min((a.keep + kBPage - 1) / kBPage, first);                      // pages of kept keys in front of the window's
+    skip = first - kept;
+    const int pages = max_limit >= 0 ? max_limit / kBPage + 1 - skip : 0, total = pages + n_pt;
     const int per_split = (total + a.splits - 1) / a.splits;
-    pg_begin = first - n_pt + split * per_split;                            // tiles of pooled rows count as the n_pt pages in front of the first one
-    n_tiles = max(0, min(first + pages, pg_begin + per_split) - pg_begin);
-    n_pt = max(0, first - pg_begin);                                        // those of this slice
     pt_first = split * per_split;
+    n_tiles = max(0, min(total, pt_first + per_split) - pt_first);
+    pg0 = pt_first - n_pt;                                                  // tiles of pooled rows come first
+    n_pt = max(0, -pg0);                                                    // those of this slice
     bt = a.block_tables + (long long)seq * a.bt_stride;
   }
 
+  auto page_of = [&](int i) { const int l = pg0 + i; return l < kept ? l : l + skip; };
   if (warp == 0) {
     if (n_tiles > 0 && elect_one()) {
       constexpr int kCopies = kRep ? 4 : 1;
       mbar_expect_tx(b_qfull, kCopies * a.nc * a.g * a.tq * 128);
+      const int nc1 = a.nc >> 1;                              // kDiff: chunks per map
+      if constexpr (kDiff) {
+        for (int c = 0; c < a.nc; c++) {
+          const int m = c >= nc1;
+          tma_load_4d(smem_u32(sQ + c * q_chunk + m * half_rows * 128), &q_map, b_qfull, (c - m * nc1) * 64, m, hkv * a.g, tok0);
+        }
+      } else
       for (int r = 0; r < kCopies; r++)
         for (int c = 0; c < a.nc; c++) tma_load_3d(smem_u32(sQ + c * q_chunk + r * 32 * 128), &q_map, b_qfull, c * 64, hkv * a.g, tok0);
       for (int i = 0; i < n_tiles; i++) {
@@ -142,9 +169,15 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
             for (int j = 0; j < 8; j++) tma_load_4d(smem_u32(dst + (a.nc + c) * kBChunk + j * 1024), &vp_map, b_kvfull + 8 * s, c * 64, hkv, prow[j], page[j]);
           continue;
         }
-        int block = bt[pg_begin + i];
+        int block = bt[page_of(i)];
         if (!NE_INDEX_OK(block, BK_CACHE_PAGES, kKernelGb, __LINE__)) block = 0;      // a bad page id reads page 0
         mbar_expect_tx(b_kvfull + 8 * s, stage_bytes);
+        if constexpr (kDiff) {
+          for (int c = 0; c < a.nc; c++) {
+            const int m = c >= nc1;
+            tma_load_4d(smem_u32(dst + c * kBChunk), &k_map, b_kvfull + 8 * s, (c - m * nc1) * 64, 2 * hkv + m, 0, block);
+          }
+        } else
         for (int c = 0; c < a.nc; c++) tma_load_4d(smem_u32(dst + c * kBChunk), &k_map, b_kvfull + 8 * s, c * 64, hkv, 0, block);
         for (int c = 0; c < a.nv; c++) tma_load_4d(smem_u32(dst + (a.nc + c) * kBChunk), &v_map, b_kvfull + 8 * s, c * 64, hkv, 0, block);
       }
@@ -197,9 +230,10 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int wq = warp & 3;
     const int row = wq * 32 + (int)lane_id();
     const uint32_t lane_addr = (uint32_t)(wq * 32) << 16;
-    const int trow = kRep ? (int)lane_id() : row;             // row of the tile
+    const int map = kDiff && row >= half_rows;
+    const int trow = kRep ? (int)lane_id() : kDiff ? row - map * half_rows : row;             // row of the tile (kDiff: pair)
     const int tl = trow / a.g, head = hkv * a.g + trow % a.g;
-    const bool row_ok = trow < a.g * a.tq && tl < n_tok;
+    const bool row_ok = trow < pairs && tl < n_tok;
     constexpr int kKeys = kRep ? 16 : 64;                     // keys of a page this thread scores, from kfirst on
     const int kfirst = kRep ? wq * 16 : 0;
     const int limit = row_ok ? base_limit + tl : -1;          // this row's last visible key
@@ -227,7 +261,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       __syncwarp();
       if (lane_id() == 0) mbar_arrive(b_sempty + 8 * sb);
       const bool pooled = kExt && i < n_pt;
-      const int key0 = (pooled ? pt_first + i : pg_begin + i) * kBPage + kfirst;
+      const int key0 = (pooled ? pt_first + i : page_of(i)) * kBPage + kfirst;
       const int hi = pooled ? pool_last : limit, lo = pooled ? 0 : lowest;
       const bool p_free = i < a.pbufs || mbar_test(b_pempty + 8 * pb, ((i - a.pbufs) / a.pbufs) & 1);     // needed only after the math
       // score in the log2 domain: cap and bias
@@ -253,7 +287,7 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       if (key0 + kKeys - 1 > hi || key0 < lo) {
 #pragma unroll
         for (int j = 0; j < kKeys; j++)
-          if (key0 + j > hi || key0 + j < lo) r[j] = 0xff800000u;
+          if (key0 + j > hi || (key0 + j < lo && key0 + j >= a.keep)) r[j] = 0xff800000u;
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -304,7 +338,8 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       if (lane_id() == 0) mbar_arrive(b_pfull + 8 * pb);
     }
     if (ok && n_tiles > 0) ok = mbar_wait(b_pempty + 8 * ((n_tiles - 1) % a.pbufs), ((n_tiles - 1) / a.pbufs) & 1, abort_flag, kKernelGb, 320);
-    const long long tok = tok0 + tl, orow = row_ok ? tok * a.H + head : 0;
+    const long long all_rows = (long long)a.T * a.H * (kDiff ? 2 : 1);
+    const long long tok = tok0 + tl, orow = row_ok ? (kDiff ? (tok * a.H + head) * 2 + map : tok * a.H + head) : 0;
     const bool have = ok && n_tiles > 0;
     if (have) tc_fence_after();
     if constexpr (kRep) {
@@ -357,6 +392,59 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           *reinterpret_cast<float4*>(dst) = make_float4(f[0] * inv, f[1] * inv, f[2] * inv, f[3] * inv);
           *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4] * inv, f[5] * inv, f[6] * inv, f[7] * inv);
           if (col == 0) a.lse2[o] = den > 0.f ? m + log2f(den) : -INFINITY;
+        }
+      }
+    } else if (kDiff && a.splits == 1) {
+      // rows into shared memory (nothing else uses it any more); one warp per pair from there
+      float* fold = reinterpret_cast<float*>(smem);
+      const int ld = a.Dv + 4;
+      const float inv = (have && l_run > 0.f) ? 1.f / l_run : 0.f;
+#pragma unroll 1
+      for (int cblk = 0; cblk < a.nv * 2; cblk++) {
+        uint32_t o[32];
+        __syncwarp();                          // the lanes of rows outside the tile skip the stores below
+        if (have) {
+          tmem_ld_32x32b_x32(tmem_o + lane_addr + cblk * 32, o);
+          tc_wait_ld();
+        }
+        if (!row_ok) continue;
+#pragma unroll
+        for (int v = 0; v < 8; v++) {
+          const int col = cblk * 32 + v * 4;
+          if (col >= a.Dv) continue;
+          *reinterpret_cast<float4*>(fold + (map * pairs + trow) * ld + col) =
+              have ? make_float4(__uint_as_float(o[4 * v]) * inv, __uint_as_float(o[4 * v + 1]) * inv, __uint_as_float(o[4 * v + 2]) * inv, __uint_as_float(o[4 * v + 3]) * inv)
+                   : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      }
+      named_bar_sync(1, live_warps * 32);
+      const float lam = *a.mixing;
+      const int lane = (int)lane_id();
+      for (int p = wq; p < n_tok * a.g; p += live_warps) {
+        const long long tk = tok0 + p / a.g;
+        const int hd = hkv * a.g + p % a.g;
+        float f[8], ss = 0.f;
+        uint2 gv[2];
+#pragma unroll
+        for (int it = 0; it < 2; it++) {
+          const int col = lane * 4 + it * 128;
+          f[4 * it] = f[4 * it + 1] = f[4 * it + 2] = f[4 * it + 3] = 0.f;
+          gv[it] = make_uint2(0, 0);
+          if (col >= a.Dv) continue;
+          gv[it] = *reinterpret_cast<const uint2*>(a.egate + tk * a.egate_ld + (long long)hd * a.Dv + col);
+          const float4 x = *reinterpret_cast<const float4*>(fold + p * ld + col), y = *reinterpret_cast<const float4*>(fold + (pairs + p) * ld + col);
+          f[4 * it] = x.x - lam * y.x; f[4 * it + 1] = x.y - lam * y.y; f[4 * it + 2] = x.z - lam * y.z; f[4 * it + 3] = x.w - lam * y.w;
+          ss += f[4 * it] * f[4 * it] + f[4 * it + 1] * f[4 * it + 1] + f[4 * it + 2] * f[4 * it + 2] + f[4 * it + 3] * f[4 * it + 3];
+        }
+        const float r = rsqrtf(warp_sum(ss) / (float)a.Dv + a.eps) * a.out_scale;
+#pragma unroll
+        for (int it = 0; it < 2; it++) {
+          const int col = lane * 4 + it * 128;
+          if (col >= a.Dv) continue;
+          const float2 g0 = unpack_bf16x2(gv[it].x), g1 = unpack_bf16x2(gv[it].y);
+          *reinterpret_cast<uint2*>(a.out + tk * a.o_ld + (long long)hd * a.Dv + col) =
+              make_uint2(pack_bf16x2(f[4 * it] * r * sigmoid_of(g0.x), f[4 * it + 1] * r * sigmoid_of(g0.y)),
+                         pack_bf16x2(f[4 * it + 2] * r * sigmoid_of(g1.x), f[4 * it + 3] * r * sigmoid_of(g1.y)));
         }
       }
     } else if (kExt && a.turn && a.splits == 1) {
@@ -418,14 +506,14 @@ gqa_biased_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
             *reinterpret_cast<uint4*>(a.out + tok * a.o_ld + (long long)head * a.Dv + col) =
                 make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
           } else {
-            float* dst = a.part + ((long long)split * a.T * a.H + orow) * a.Dv + col;
+            float* dst = a.part + (split * all_rows + orow) * a.Dv + col;
             *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
             *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
           }
         }
       }
       if (a.splits > 1 && row_ok)
-        a.lse2[(long long)split * a.T * a.H + orow] = (have && l_run > 0.f) ? m_run + log2f(l_run) : -INFINITY;
+        a.lse2[split * all_rows + orow] = (have && l_run > 0.f) ? m_run + log2f(l_run) : -INFINITY;
     }
   }
 
@@ -470,15 +558,60 @@ __global__ void __launch_bounds__(128) gqa_biased_merge_kernel(const GbArgs a) {
   for (int d = threadIdx.x; d < a.Dv; d += blockDim.x) out[d] = __float2bfloat16(column(d));
 }
 
+// kDiff: the slices of both maps, their difference, norm and gate; one warp per (token, head), at most 32 slices
+__global__ void __launch_bounds__(128) gqa_diff_merge_kernel(const GbArgs a) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const long long pair = (long long)blockIdx.x * 4 + (threadIdx.x >> 5), rows = (long long)a.T * a.H * 2;
+  const int lane = (int)lane_id();
+  if (pair >= (long long)a.T * a.H) return;
+  const long long t = pair / a.H;
+  const int h = (int)(pair - t * a.H);
+  const float lam = *a.mixing;
+  float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int m = 0; m < 2; m++) {
+    const long long row = pair * 2 + m;
+    const float l = lane < a.splits ? a.lse2[lane * rows + row] : -INFINITY, mx = warp_max(l);
+    const float e = l == -INFINITY ? 0.f : exp2f(l - mx), den = warp_sum(e), w = den > 0.f ? (m ? -lam : 1.f) * e / den : 0.f;
+#pragma unroll 4
+    for (int s = 0; s < a.splits; s++) {
+      const float ws = __shfl_sync(0xffffffffu, w, s);
+#pragma unroll
+      for (int it = 0; it < 2; it++) {
+        const int col = lane * 4 + it * 128;
+        if (col >= a.Dv || ws == 0.f) continue;
+        const float4 v = *reinterpret_cast<const float4*>(a.part + (s * rows + row) * a.Dv + col);
+        f[4 * it] = fmaf(ws, v.x, f[4 * it]); f[4 * it + 1] = fmaf(ws, v.y, f[4 * it + 1]);
+        f[4 * it + 2] = fmaf(ws, v.z, f[4 * it + 2]); f[4 * it + 3] = fmaf(ws, v.w, f[4 * it + 3]);
+      }
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; e++) ss += f[e] * f[e];
+  const float r = rsqrtf(warp_sum(ss) / (float)a.Dv + a.eps) * a.out_scale;
+#pragma unroll
+  for (int it = 0; it < 2; it++) {
+    const int col = lane * 4 + it * 128;
+    if (col >= a.Dv) continue;
+    const uint2 gv = *reinterpret_cast<const uint2*>(a.egate + t * a.egate_ld + (long long)h * a.Dv + col);
+    const float2 g0 = unpack_bf16x2(gv.x), g1 = unpack_bf16x2(gv.y);
+    *reinterpret_cast<uint2*>(a.out + t * a.o_ld + (long long)h * a.Dv + col) =
+        make_uint2(pack_bf16x2(f[4 * it] * r * sigmoid_of(g0.x), f[4 * it + 1] * r * sigmoid_of(g0.y)),
+                   pack_bf16x2(f[4 * it + 2] * r * sigmoid_of(g1.x), f[4 * it + 3] * r * sigmoid_of(g1.y)));
+  }
+}
+
 struct GbPlan { int nc, nv, tq, rep, rows8, stages, pbufs, bar_off, smem; };
 
 // Tile geometry for groups of g heads, head sizes D / Dv and sequences of at most max_q new tokens; false: not covered.
-static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, bool ext, GbPlan* p) {
-  if (g < 1 || g > 128 || D < 8 || D % 8 || D > 256 || Dv < 8 || Dv % 8 || Dv > 256 || max_q < 1) return false;
-  p->nc = (D + 63) / 64; p->nv = (Dv + 63) / 64;
-  p->tq = 128 / g < max_q ? 128 / g : max_q;
+// maps = 2: kDiff, D the size of one map.
+static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, bool ext, GbPlan* p, int maps = 1) {
+  if (g < 1 || g * maps > 128 || D < 8 || D % 8 || D * maps > 256 || Dv < 8 || Dv % 8 || Dv > 256 || max_q < 1) return false;
+  p->nc = (D + 63) / 64 * maps; p->nv = (Dv + 63) / 64;
+  p->tq = 128 / (g * maps) < max_q ? 128 / (g * maps) : max_q;
   p->rep = rep && g * p->tq <= 32;
-  p->rows8 = p->rep ? 128 : (g * p->tq + 7) / 8 * 8;
+  p->rows8 = p->rep ? 128 : (g * p->tq + 7) / 8 * 8 * maps;
   const int kv = (p->nc + p->nv) * kBChunk, pb = p->rows8 * 128, q = p->nc * pb;
   // two CTAs per SM where half of its shared memory (and of its TMEM columns) holds a tile and two stages, else one with more stages
   const int half = (233472 / 2 - 1024) - 256, whole = 232448 - 256;
@@ -488,7 +621,7 @@ static bool gb_plan(int g, int D, int Dv, int max_q, bool rep, bool ext, GbPlan*
   if (p->stages > 4) p->stages = 4;
   if (p->stages < 2) return false;
   const int used = q + p->pbufs * pb + p->stages * kv;
-  const int rows_out = ext ? g * p->tq * (Dv + 4) * 4 : 0;              // kExt's way out
+  const int rows_out = ext || maps == 2 ? g * maps * p->tq * (Dv + 4) * 4 : 0;              // the way out of kExt and kDiff
   p->bar_off = ((rows_out > used ? rows_out : used) + 15) / 16 * 16;
   p->smem = p->bar_off + 256;
   if (p->smem > 232448) return false;
@@ -516,8 +649,9 @@ extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache,
                              const int* cu_seqlens_q, const int* context_lens, int num_seqs, int T, int H, int Hkv, int D, int Dv, int max_q, int max_tiles,
                              int splits, float scale, float softcap, const float* slopes, int window, const void* gate, long long gate_ld, float out_scale,
                              void* out, long long o_ld, float* part, float* lse2, const void* k_pool, const void* v_pool, int pool, int pool_rows,
-                             const float* turn, int n_pos, cudaStream_t st) {
+                             const float* turn, int n_pos, int keep, cudaStream_t st) {
   if (T <= 0) return 0;
+  if (keep > 0 && pool > 0) return 1004;
   GbPlan p;
   const bool ext = pool > 0 || turn;
   if (ext && (softcap > 0.f || slopes || (turn && n_pos < 1))) return 1003;
@@ -562,8 +696,60 @@ extern "C" int ne_gqa_biased(const void* q, long long q_ld, const void* k_cache,
   a.T = T; a.H = H; a.Dv = Dv; a.g = g; a.tq = p.tq; a.splits = splits; a.nc = p.nc; a.nv = p.nv; a.rows8 = p.rows8; a.stages = p.stages; a.pbufs = p.pbufs;
   a.window = window; a.tmem_cols = p.nv <= 2 ? 256 : 512; a.scale = scale; a.softcap = softcap; a.slopes = slopes; a.gate = (const __nv_bfloat16*)gate;
   a.gate_ld = gate_ld; a.out_scale = out_scale; a.out = (__nv_bfloat16*)out; a.o_ld = o_ld; a.part = part; a.lse2 = lse2;
-  a.pool = pool > 0 ? pool : 0; a.turn = turn; a.n_pos = n_pos; a.bar_off = p.bar_off;
+  a.pool = pool > 0 ? pool : 0; a.turn = turn; a.n_pos = n_pos; a.bar_off = p.bar_off; a.keep = window > 0 && keep > 0 ? keep : 0;
+  a.mixing = nullptr; a.eps = 0.f; a.egate = nullptr; a.egate_ld = 0;
   cudaError_t e = launch_pdl(kern, dim3((unsigned)max_tiles, (unsigned)Hkv, (unsigned)splits), dim3(kGbThreads), (size_t)p.smem, st, mq, mk, mv, mkp, mvp, a);
   if (e != cudaSuccess || splits == 1) return (int)e;
   return (int)launch_pdl(gqa_biased_merge_kernel, dim3((unsigned)((long long)T * H)), dim3(128), 0, st, a);
+}
+
+// Pairs of (token, head) tokens per tile of the differential form (0: the shape is not covered); D: size of one map
+extern "C" int ne_gqa_diff_plan(int H, int Hkv, int D, int Dv, int max_q) {
+  GbPlan p;
+  return Hkv >= 1 && H % Hkv == 0 && gb_plan(H / Hkv, D, Dv, max_q, false, false, &p, 2) ? p.tq : 0;
+}
+
+// q bf16 [T, H, 2, D] (row stride q_ld elements), k_cache bf16 [num_blocks, 64, Hkv, 2 D], v_cache bf16 [num_blocks, 64, Hkv, Dv]; mixing fp32 [1], gate bf16
+// [T, H Dv] (row stride gate_ld), out bf16 [T, H Dv] (row stride o_ld).  window 0: all earlier keys; keep: the first keys stay visible behind the window.
+// splits > 1 (at most 32): part fp32 [splits, T, H, 2, Dv], lse2 [splits, T, H, 2]; the merge kernel is launched too.
+extern "C" int ne_gqa_diff(const void* q, long long q_ld, const void* k_cache, const void* v_cache, int num_blocks, const int* block_tables, int bt_stride,
+                           const int* cu_seqlens_q, const int* context_lens, int num_seqs, int T, int H, int Hkv, int D, int Dv, int max_q, int max_tiles, int splits,
+                           float scale, int window, int keep, const float* mixing, float out_scale, float eps, const void* gate, long long gate_ld, void* out,
+                           long long o_ld, float* part, float* lse2, cudaStream_t st) {
+  if (T <= 0) return 0;
+  GbPlan p;
+  if (Hkv < 1 || H % Hkv || splits < 1 || splits > 32 || (splits > 1 && (!part || !lse2)) || max_tiles < 1 || !mixing || !gate) return 1001;
+  if (!gb_plan(H / Hkv, D, Dv, max_q, false, false, &p, 2)) return 1001;
+  if (q_ld % 8 || o_ld % 4 || gate_ld % 4 || q_ld < (long long)H * 2 * D || ((uintptr_t)q & 15) || (((uintptr_t)out | (uintptr_t)gate) & 7)) return 1002;
+  const int g = H / Hkv;
+  CUtensorMap mq, mk, mv;
+  int rc;
+  {
+    uint64_t dims[4] = {(uint64_t)D, 2, (uint64_t)H, (uint64_t)T}; uint64_t strides[3] = {(uint64_t)D * 2, (uint64_t)D * 4, (uint64_t)q_ld * 2};
+    uint32_t box[4] = {64, 1, (uint32_t)g, (uint32_t)p.tq};
+    rc = make_tmap(&mq, q, TMA_BF16, 4, dims, strides, box, TMA_SW_128); if (rc) return 2000 + rc;
+  }
+  for (int which = 0; which < 2; which++) {
+    const uint64_t w = which ? Dv : D, heads = which ? Hkv : 2 * Hkv;
+    uint64_t dims[4] = {w, heads, (uint64_t)kBPage, (uint64_t)num_blocks};
+    uint64_t strides[3] = {w * 2, heads * w * 2, (uint64_t)kBPage * heads * w * 2};
+    uint32_t box[4] = {64, 1, kBPage, 1};
+    rc = make_tmap(which ? &mv : &mk, which ? v_cache : k_cache, TMA_BF16, 4, dims, strides, box, TMA_SW_128); if (rc) return 2100 + rc;
+  }
+  auto kern = gqa_biased_kernel<false, false, false, true>;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  GbArgs a = {};
+  a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu_seqlens_q = cu_seqlens_q; a.context_lens = context_lens; a.num_seqs = num_seqs;
+  a.T = T; a.H = H; a.Dv = Dv; a.g = g; a.tq = p.tq; a.splits = splits; a.nc = p.nc; a.nv = p.nv; a.rows8 = p.rows8; a.stages = p.stages; a.pbufs = p.pbufs;
+  a.window = window; a.tmem_cols = p.nv <= 2 ? 256 : 512; a.scale = scale; a.out_scale = out_scale; a.out = (__nv_bfloat16*)out; a.o_ld = o_ld; a.part = part;
+  a.lse2 = lse2; a.bar_off = p.bar_off; a.keep = window > 0 && keep > 0 ? keep : 0; a.mixing = mixing; a.eps = eps; a.egate = (const __nv_bfloat16*)gate;
+  a.egate_ld = gate_ld;
+  cudaError_t e = launch_pdl(kern, dim3((unsigned)max_tiles, (unsigned)Hkv, (unsigned)splits), dim3(kGbThreads), (size_t)p.smem, st, mq, mk, mv, mk, mv, a);
+  if (e != cudaSuccess || splits == 1) return (int)e;
+  return (int)launch_pdl(gqa_diff_merge_kernel, dim3((unsigned)(((long long)T * H + 3) / 4)), dim3(128), 0, st, a);
 }

@@ -19,7 +19,8 @@ constexpr int kMaxExperts = 1024;
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ idx_out,
                                                        float* __restrict__ w_out, int T, int E, int top_k, int n_group, int topk_group,
                                                        int norm, float scale, int softmax, int planes, int balance_ranks,
-                                                       const int* __restrict__ log2phy, const int* __restrict__ logcnt, int max_rep) {
+                                                       const int* __restrict__ log2phy, const int* __restrict__ logcnt, int max_rep, int ld,
+                                                       float* __restrict__ gate_out) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   __shared__ float s_choice[4][kMaxExperts];
   __shared__ float s_score[4][kMaxExperts];
@@ -28,11 +29,16 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
   const int t = blockIdx.x * 4 + wl;
   if (t >= T) return;
   float* choice = s_choice[wl]; float* score = s_score[wl]; float* gsc = s_group[wl];
-  // the logits may arrive as `planes` partial sums [planes, T, E] (split-K router product)
+  // the logits may arrive as `planes` partial sums [planes, T, ld] (split-K router product); column E may hold a gate that is no score
   for (int e = lane; e < E; e += 32) {
     float v = 0.f;
-    for (int p = 0; p < planes; p++) v += logits[((long long)p * T + t) * E + e];
+    for (int p = 0; p < planes; p++) v += logits[((long long)p * T + t) * ld + e];
     choice[e] = v;
+  }
+  if (gate_out && lane == 0) {
+    float v = 0.f;
+    for (int p = 0; p < planes; p++) v += logits[((long long)p * T + t) * ld + E];
+    gate_out[t] = v;
   }
   const float* lr = choice;
   if (softmax == 1) {
@@ -40,7 +46,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     for (int e = lane; e < E; e += 32) m = fmaxf(m, lr[e]);
     m = warp_max(m);
     float s = 0.f;
-    for (int e = lane; e < E; e += 32) { float v = __expf(lr[e] - m); score[e] = v; s += v; }
+    for (int e = lane; e < E; e += 32) { float v = expf(lr[e] - m); score[e] = v; s += v; }
     s = warp_sum(s);
     float inv = 1.f / s;
     for (int e = lane; e < E; e += 32) { score[e] *= inv; choice[e] = score[e] + (bias ? bias[e] : 0.f); }
@@ -48,7 +54,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     // softmax == 2: sqrt(softplus(x)) (DeepSeek-V4), else sigmoid
     for (int e = lane; e < E; e += 32) {
       const float x = lr[e];
-      float v = softmax == 2 ? sqrtf(x > 20.f ? x : log1pf(__expf(x))) : 1.f / (1.f + __expf(-x));
+      float v = softmax == 2 ? sqrtf(x > 20.f ? x : log1pf(expf(x))) : 1.f / (1.f + expf(-x));
       score[e] = v; choice[e] = v + (bias ? bias[e] : 0.f);
     }
   }
@@ -213,7 +219,7 @@ __global__ void __launch_bounds__(256) router_gemv_kernel(const __nv_bfloat16* _
   __shared__ __align__(16) __nv_bfloat16 s_x[8][kRouterCols];
   const int t0 = blockIdx.x * 8, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h0 = blockIdx.z * kRouterCols;
-  const int hc = min(kRouterCols, H - h0);                                // multiple of 128
+  const int hc = min(kRouterCols, H - h0);                                // multiple of 8
   for (int i = threadIdx.x * 8; i < 8 * kRouterCols; i += 256 * 8) {
     const int tt = i / kRouterCols, c = i % kRouterCols;
     *reinterpret_cast<uint4*>(&s_x[tt][c]) = (t0 + tt < T && c < hc) ? *reinterpret_cast<const uint4*>(x + (long long)(t0 + tt) * H + h0 + c)
@@ -250,49 +256,124 @@ __global__ void __launch_bounds__(256) router_gemv_kernel(const __nv_bfloat16* _
   }
 }
 
-// one CTA per token
-__global__ void __launch_bounds__(256) moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ w,
-                                                         const __nv_bfloat16* __restrict__ add_in, __nv_bfloat16* __restrict__ out, int top_k, int H) {
+// The row of every token to each of its local experts, in units of U (any row width and element type): see moe_scatter_kernel
+template <typename U>
+__global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const U* __restrict__ x, const int* __restrict__ idx, const int* __restrict__ slot,
+                                                              const int* __restrict__ row_start, int* __restrict__ pos, U* __restrict__ dst, int top_k, int units,
+                                                              int expert_offset, int E_local, int max_rows) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  __shared__ int s_row[64];
+  const int t = blockIdx.x;
+  if ((int)threadIdx.x < top_k) {
+    const int i = t * top_k + threadIdx.x;
+    const int e = idx[i] - expert_offset, sl = slot[i];
+    int row = -1;
+    if (e >= 0 && e < E_local && sl >= 0) { row = row_start[e] + sl; if (row >= max_rows) row = -1; }
+    pos[i] = row; s_row[threadIdx.x] = row;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < units; c += blockDim.x) {
+    const U v = x[(long long)t * units + c];
+    for (int k = 0; k < top_k; k++) if (s_row[k] >= 0) dst[(long long)s_row[k] * units + c] = v;
+  }
+}
+
+// V values of type T
+template <typename T, int V> struct RowPiece;
+template <> struct RowPiece<__nv_bfloat16, 8> {
+  uint4 r;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void zero() { r = make_uint4(0, 0, 0, 0); }
+  __device__ __forceinline__ void add_to(float* acc, float w) const {
+    const uint32_t u[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int j = 0; j < 4; j++) { const float2 f = unpack_bf16x2(u[j]); acc[2 * j] += w * f.x; acc[2 * j + 1] += w * f.y; }
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* a) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]), pack_bf16x2(a[6], a[7]));
+  }
+};
+template <> struct RowPiece<float, 4> {
+  float4 r;
+  __device__ __forceinline__ void load(const float* p) { r = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void zero() { r = make_float4(0.f, 0.f, 0.f, 0.f); }
+  __device__ __forceinline__ void add_to(float* acc, float w) const { acc[0] += w * r.x; acc[1] += w * r.y; acc[2] += w * r.z; acc[3] += w * r.w; }
+  static __device__ __forceinline__ void store(float* p, const float* a) { *reinterpret_cast<float4*>(p) = make_float4(a[0], a[1], a[2], a[3]); }
+};
+template <> struct RowPiece<float, 1> {
+  float r;
+  __device__ __forceinline__ void load(const float* p) { r = *p; }
+  __device__ __forceinline__ void zero() { r = 0.f; }
+  __device__ __forceinline__ void add_to(float* acc, float w) const { acc[0] += w * r; }
+  static __device__ __forceinline__ void store(float* p, const float* a) { *p = a[0]; }
+};
+template <> struct RowPiece<__nv_bfloat16, 1> {
+  __nv_bfloat16 r;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = *p; }
+  __device__ __forceinline__ void zero() { r = __float2bfloat16(0.f); }
+  __device__ __forceinline__ void add_to(float* acc, float w) const { acc[0] += w * __bfloat162float(r); }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* a) { *p = __float2bfloat16(a[0]); }
+};
+__device__ __forceinline__ float round_as(float v, const __nv_bfloat16*) { return __bfloat162float(__float2bfloat16(v)); }
+__device__ __forceinline__ float round_as(float v, const float*) { return v; }
+
+// One CTA per token (and column slice).  x given: the pairs with ids from identity_from on add their weight times the token's own row x.  gate given:
+// add_in enters times sigmoid(gate[t]) and the sum is rounded once.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ w,
+                                                         const T* __restrict__ add_in, const float* __restrict__ gate, const T* __restrict__ x,
+                                                         const int* __restrict__ idx, int identity_from, T* __restrict__ out, int top_k, int H) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   const int t = blockIdx.x;
-  __shared__ int s_pos[64]; __shared__ float s_w[64];
-  if (threadIdx.x < top_k) { s_pos[threadIdx.x] = pos[(long long)t * top_k + threadIdx.x]; s_w[threadIdx.x] = w[(long long)t * top_k + threadIdx.x]; }
+  __shared__ int s_pos[64]; __shared__ float s_w[64]; __shared__ float s_own[64];
+  if (threadIdx.x < top_k) {
+    const long long i = (long long)t * top_k + threadIdx.x;
+    s_pos[threadIdx.x] = pos[i]; s_w[threadIdx.x] = w[i];
+    s_own[threadIdx.x] = x && idx[i] >= identity_from ? w[i] : 0.f;
+  }
   __syncthreads();
+  float own = 0.f;
+  if (x) for (int k = 0; k < top_k; k++) own += s_own[k];
+  const float gt = gate ? 1.f / (1.f + expf(-gate[t])) : 1.f;
   // blockIdx.y splits the row into column slices: with one CTA per token a decode batch would occupy fewer CTAs than there
   // are SMs, each with 32 KB of loads in flight, a fraction of what it takes to keep HBM busy
-  const int slice = (((H + 7) / 8 + gridDim.y - 1) / gridDim.y) * 8;
+  const int slice = (((H + V - 1) / V + gridDim.y - 1) / gridDim.y) * V;
   const int c_end = min(H, ((int)blockIdx.y + 1) * slice);
-  for (int c = blockIdx.y * slice + threadIdx.x * 8; c < c_end; c += blockDim.x * 8) {
-    float acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+  for (int c = blockIdx.y * slice + threadIdx.x * V; c < c_end; c += blockDim.x * V) {
+    float acc[V];
+#pragma unroll
+    for (int j = 0; j < V; j++) acc[j] = 0.f;
     // eight expert rows are fetched before any is used: the loads are independent and the kernel is latency-bound
     for (int k0 = 0; k0 < top_k; k0 += 8) {
-      uint4 v[8];
+      RowPiece<T, V> v[8];
 #pragma unroll
       for (int q = 0; q < 8; q++) {
         const int r = k0 + q < top_k ? s_pos[k0 + q] : -1;
-        v[q] = r >= 0 ? *reinterpret_cast<const uint4*>(y + (long long)r * H + c) : make_uint4(0, 0, 0, 0);
+        if (r >= 0) v[q].load(y + (long long)r * H + c); else v[q].zero();
       }
 #pragma unroll
-      for (int q = 0; q < 8; q++) {
-        const float wk = k0 + q < top_k ? s_w[k0 + q] : 0.f;
-        const uint32_t u[4] = {v[q].x, v[q].y, v[q].z, v[q].w};
-#pragma unroll
-        for (int j = 0; j < 4; j++) { float2 f = unpack_bf16x2(u[j]); acc[2 * j] += wk * f.x; acc[2 * j + 1] += wk * f.y; }
-      }
+      for (int q = 0; q < 8; q++) v[q].add_to(acc, k0 + q < top_k ? s_w[k0 + q] : 0.f);
     }
+    if (own != 0.f) { RowPiece<T, V> v; v.load(x + (long long)t * H + c); v.add_to(acc, own); }
     if (add_in) {
-      // the routed sum is rounded to bf16 before the shared-expert output is added, as in the unfused form
-      uint4 v = *reinterpret_cast<const uint4*>(add_in + (long long)t * H + c);
-      uint32_t u[4] = {v.x, v.y, v.z, v.w};
+      // without a gate the routed sum is rounded before the shared-expert output is added, as in the unfused form
+      if (!gate)
 #pragma unroll
-      for (int j = 0; j < 4; j++) {
-        float2 f = unpack_bf16x2(u[j]); float2 r = unpack_bf16x2(pack_bf16x2(acc[2 * j], acc[2 * j + 1]));
-        acc[2 * j] = r.x + f.x; acc[2 * j + 1] = r.y + f.y;
-      }
+        for (int j = 0; j < V; j++) acc[j] = round_as(acc[j], y);
+      RowPiece<T, V> v;
+      v.load(add_in + (long long)t * H + c);
+      v.add_to(acc, gt);
     }
-    *reinterpret_cast<uint4*>(out + (long long)t * H + c) =
-        make_uint4(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[2], acc[3]), pack_bf16x2(acc[4], acc[5]), pack_bf16x2(acc[6], acc[7]));
+    RowPiece<T, V>::store(out + (long long)t * H + c, acc);
   }
+}
+
+template <typename T, int V>
+static int moe_combine_t(const void* y, const int* pos, const float* w, const void* add_in, const float* gate, const void* x, const int* idx, int identity_from, void* out,
+                         int T_, int top_k, int H, cudaStream_t st) {
+  const int slices = T_ >= 2048 ? 1 : (T_ >= 512 ? 2 : 4);      // enough CTAs per SM at decode sizes, one pass over the tables per token otherwise
+  return (int)launch_pdl(moe_combine_kernel<T, V>, dim3(T_, slices), dim3(256), 0, st, (const T*)y, pos, w, (const T*)add_in, gate, (const T*)x, idx, identity_from, (T*)out,
+                         top_k, H);
 }
 
 }  // namespace ne
@@ -300,15 +381,17 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const __nv_bfloat16* _
 using namespace ne;
 
 // balance_ranks > 0: replace the chosen ids by ids dealt evenly over that many EP ranks (weights kept).  log2phy [E, max_rep] /
-// logcnt [E] (device int32, optional): remap every logical id to one of its physical replicas.
+// logcnt [E] (device int32, optional): remap every logical id to one of its physical replicas.  ld: row stride of the logits; gate_out [T] (or
+// null) takes column E as it is.
 extern "C" int ne_moe_route(const float* logits, const float* bias, int* idx, float* w, int T, int E, int top_k, int n_group,
                             int topk_group, int norm, float scale, int softmax, int planes, int balance_ranks, const int* log2phy,
-                            const int* logcnt, int max_rep, cudaStream_t st) {
+                            const int* logcnt, int max_rep, int ld, float* gate_out, cudaStream_t st) {
   if (T <= 0) return 0;
+  if (ld < E + (gate_out ? 1 : 0)) return 1001;
   if (E > kMaxExperts || top_k > 64 || n_group > 64 || (n_group > 1 && E % n_group) || planes < 1) return 1001;
   if (balance_ranks < 0 || (balance_ranks > 0 && E % balance_ranks) || (log2phy && (!logcnt || max_rep < 1))) return 1001;
   return (int)launch_pdl(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, idx, w, T, E, top_k, n_group, topk_group, norm, scale, softmax,
-                         planes, balance_ranks, log2phy, logcnt, max_rep);
+                         planes, balance_ranks, log2phy, logcnt, max_rep, ld, gate_out);
 }
 
 // Outputs: counts [E_local], slot [T*K] (scratch), row_start [E_local+1], pos [T*K], and the
@@ -317,7 +400,7 @@ extern "C" int ne_moe_dispatch_local(const void* x, const int* idx, int* counts,
                                      void* a_q, float* a_s, int s_ld, int T, int top_k, int H, int expert_offset, int E_local,
                                      int max_rows, int align, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (E_local > kMaxExperts || H % 128) return 1001;
+  if (E_local > kMaxExperts || H % (a_q ? 128 : 8)) return 1001;
   int n = T * top_k;
   if (top_k > 64) return 1001;
   cudaError_t e = launch_pdl(moe_count_scan_kernel, dim3(1), dim3(1024), 0, st, idx, counts, slot, row_start, n, expert_offset, E_local, align);
@@ -326,18 +409,37 @@ extern "C" int ne_moe_dispatch_local(const void* x, const int* idx, int* counts,
                          (__nv_bfloat16*)a_bf16, (uint8_t*)a_q, a_s, s_ld, top_k, H, expert_offset, E_local, max_rows, g_scale_pow2);
 }
 
-extern "C" int ne_moe_combine_local(const void* y, const int* pos, const float* w, const void* add_in, void* out, int T, int top_k, int H,
-                                    cudaStream_t st) {
+// The same for rows of any width, row_bytes a multiple of 2: no quantisation.
+extern "C" int ne_moe_dispatch_rows(const void* x, int row_bytes, const int* idx, int* counts, int* slot, int* row_start, int* pos, void* dst, int T, int top_k,
+                                    int expert_offset, int E_local, int max_rows, int align, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (H % 8 || top_k > 64) return 1001;
-  const int slices = T >= 2048 ? 1 : (T >= 512 ? 2 : 4);      // enough CTAs per SM at decode sizes, one pass over the tables per token otherwise
-  return (int)launch_pdl(moe_combine_kernel, dim3(dim3(T, slices)), dim3(256), 0, st, (const __nv_bfloat16*)y, pos, w, (const __nv_bfloat16*)add_in, (__nv_bfloat16*)out, top_k, H);
+  if (E_local > kMaxExperts || top_k > 64 || row_bytes <= 0 || row_bytes % 2) return 1001;
+  cudaError_t e = launch_pdl(moe_count_scan_kernel, dim3(1), dim3(1024), 0, st, idx, counts, slot, row_start, T * top_k, expert_offset, E_local, align);
+  if (e != cudaSuccess) return (int)e;
+  const bool vec = row_bytes % 16 == 0 && ((uintptr_t)x | (uintptr_t)dst) % 16 == 0;
+  if (vec) return (int)launch_pdl(moe_scatter_rows_kernel<uint4>, dim3(T), dim3(128), 0, st, (const uint4*)x, idx, slot, row_start, pos, (uint4*)dst, top_k, row_bytes / 16,
+                                  expert_offset, E_local, max_rows);
+  return (int)launch_pdl(moe_scatter_rows_kernel<uint16_t>, dim3(T), dim3(128), 0, st, (const uint16_t*)x, idx, slot, row_start, pos, (uint16_t*)dst, top_k, row_bytes / 2,
+                         expert_offset, E_local, max_rows);
+}
+
+// out [T, H] = the weighted rows pos [T, top_k] of y + add_in.  gate fp32 [T], x [T, H] with idx [T, top_k]: see moe_combine_kernel; null: without.
+extern "C" int ne_moe_combine_local(const void* y, const int* pos, const float* w, const void* add_in, const float* gate, const void* x, const int* idx,
+                                    int identity_from, void* out, int T, int top_k, int H, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (H < 1 || top_k > 64 || (x && !idx) || (gate && !add_in)) return 1001;
+  const int per = fp32 ? 4 : 8;
+  const bool vec = H % per == 0 && ((uintptr_t)y | (uintptr_t)add_in | (uintptr_t)x | (uintptr_t)out) % 16 == 0;
+  if (fp32) return vec ? moe_combine_t<float, 4>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st)
+                       : moe_combine_t<float, 1>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st);
+  return vec ? moe_combine_t<__nv_bfloat16, 8>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st)
+             : moe_combine_t<__nv_bfloat16, 1>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st);
 }
 
 // x bf16 [T, H], w fp32 [E, H] -> partial logits fp32 [ne_router_planes(H), T, E]; their sum over the first axis is x . w^T
 extern "C" int ne_router_planes(int H) { return (H + kRouterCols - 1) / kRouterCols; }
 extern "C" int ne_router_gemv(const void* x, const float* w, float* planes, int T, int E, int H, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (H % 128) return 1001;
+  if (H % 8) return 1001;
   return (int)launch_pdl(router_gemv_kernel, dim3(dim3((T + 7) / 8, (E + 31) / 32, ne_router_planes(H))), dim3(256), 0, st, (const __nv_bfloat16*)x, w, planes, T, E, H);
 }

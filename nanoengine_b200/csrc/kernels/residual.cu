@@ -6,6 +6,8 @@
 //   * latent_prepare: rotary part of every query head in place, and the latent cache row [rmsnorm(kv[:R]) | rope(kv[R:])]
 //   * gather of cache rows
 //   * stream_mix: constant hyper-connections - the streams of a token mixed with a sublayer's output, the next sublayer's normed input
+//   * depth_mix: the sum behind a sublayer, behind a layer the weighted sum of all layers' results so far, and the next norm (one number as weight)
+//   * poly_norm: weighted sum of the normed first three powers of a row
 //   * kv_rows: new key and value rows of any width into paged caches;  cap_rows: cap * tanh(x / cap) in place
 #include "ptx.cuh"
 
@@ -425,6 +427,179 @@ static int stream_mix_t(const StreamArgs& a, int rows, cudaStream_t st) {
   return (int)launch_pdl(k, dim3((unsigned)rows), dim3((unsigned)threads), smem, st, a);
 }
 
+// ---- averages over the depth ------------------------------------------------------------------------------------------------
+// v = x + y (ids given: v = table[id], at = 0).  With a bank of [.., rows, W] fp32: bank[at] = v and, behind a layer (w given), v = sum_{j <= at} w[j] bank[j].
+// x = v, out = rmsnorm(v) * g.  `last`: neither x nor the bank is written.  One CTA per row.
+struct DepthArgs {
+  const void* y; long long y_ld; float* x; float* bank; long long bank_ld; const float* w; const float* g; void* out; const long long* ids; const void* table;
+  int at, W, vocab, last; float eps;
+};
+template <typename T, int V>
+__global__ void __launch_bounds__(512) depth_mix_kernel(const DepthArgs a) {
+  extern __shared__ float srow[];            // W floats, then at + 1 weights
+  __shared__ float red[2][32];
+  const int W = a.W;
+  float* sw = srow + (W + 3) / 4 * 4;
+  // the coefficients are weights: they may be read before the kernel in front has finished
+  if (a.w) for (int j = threadIdx.x; j <= a.at; j += blockDim.x) sw[j] = a.w[j];
+  const float g = *a.g;
+  pdl_wait(); pdl_trigger();
+  __syncthreads();
+  const long long row = blockIdx.x;
+  float* xr = a.x + row * W;
+  float* br = a.bank ? a.bank + row * W : nullptr;
+  const T* yr = nullptr;
+  bool ok = true;
+  if (a.ids) {
+    const long long id = a.ids[row];
+    ok = id >= 0 && id < a.vocab;
+    if (!ok && threadIdx.x == 0) report(ST_BAD_INDEX, 49, (int)row, (int)id);
+    yr = reinterpret_cast<const T*>(a.table) + (ok ? id : 0) * W;
+  } else {
+    yr = reinterpret_cast<const T*>(a.y) + row * a.y_ld;
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    float v[V];
+    if constexpr (V == 4) { const float4 t = Vec4<T>::load(yr + i); v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w; }
+    else v[0] = ldx(yr + i);
+    if (a.ids) {
+      if (!ok) for (int e = 0; e < V; e++) v[e] = 0.f;
+    } else if constexpr (V == 4) {
+      const float4 t = *reinterpret_cast<const float4*>(xr + i);
+      v[0] += t.x; v[1] += t.y; v[2] += t.z; v[3] += t.w;
+    } else v[0] += xr[i];
+    if (br && !a.last) {
+      if constexpr (V == 4) *reinterpret_cast<float4*>(br + a.at * a.bank_ld + i) = make_float4(v[0], v[1], v[2], v[3]);
+      else br[a.at * a.bank_ld + i] = v[0];
+    }
+    if (a.w) {
+      const float wn = sw[a.at];
+#pragma unroll
+      for (int e = 0; e < V; e++) v[e] *= wn;
+#pragma unroll 8
+      for (int j = 0; j < a.at; j++) {
+        const float wj = sw[j];
+        if constexpr (V == 4) {
+          const float4 t = __ldcs(reinterpret_cast<const float4*>(br + j * a.bank_ld + i));
+          v[0] = fmaf(wj, t.x, v[0]); v[1] = fmaf(wj, t.y, v[1]); v[2] = fmaf(wj, t.z, v[2]); v[3] = fmaf(wj, t.w, v[3]);
+        } else v[0] = fmaf(wj, br[j * a.bank_ld + i], v[0]);
+      }
+    }
+    if constexpr (V == 4) {
+      const float4 t = make_float4(v[0], v[1], v[2], v[3]);
+      if (!a.last) *reinterpret_cast<float4*>(xr + i) = t;
+      *reinterpret_cast<float4*>(srow + i) = t;
+    } else { if (!a.last) xr[i] = v[0]; srow[i] = v[0]; }
+#pragma unroll
+    for (int e = 0; e < V; e++) ss += v[e] * v[e];
+  }
+  const float r = rsqrtf(cta_sum(ss, red, 0) / (float)W + a.eps) * g;
+  T* out = reinterpret_cast<T*>(a.out) + row * W;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {        // a thread rereads only what it stored itself
+    if constexpr (V == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(srow + i);
+      Vec4<T>::store(out + i, make_float4(v.x * r, v.y * r, v.z * r, v.w * r));
+    } else stx(out + i, srow[i] * r);
+  }
+}
+
+template <typename T>
+static int depth_mix_t(const DepthArgs& a, int rows, cudaStream_t st) {
+  const size_t smem = ((size_t)(a.W + 3) / 4 * 4 + (a.w ? a.at + 1 : 0)) * sizeof(float);
+  const uintptr_t al = (uintptr_t)a.y | (uintptr_t)a.x | (uintptr_t)a.out | (uintptr_t)a.table | (uintptr_t)a.bank;
+  const bool vec = a.W % 4 == 0 && a.y_ld % 4 == 0 && al % 16 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((a.W + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+  auto k = vec ? depth_mix_kernel<T, 4> : depth_mix_kernel<T, 1>;
+  if (smem > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl(k, dim3((unsigned)rows), dim3((unsigned)threads), smem, st, a);
+}
+
+// ---- normed powers ------------------------------------------------------------------------------------------------------------
+// out = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over rows of F; coef = (a, b, c, e).  One CTA per row, the row in shared memory.
+template <typename T, int V>
+__global__ void __launch_bounds__(512) poly_norm_kernel(const T* __restrict__ z, long long ld, T* __restrict__ out, int F, const float* __restrict__ coef, float eps) {
+  extern __shared__ float srow[];            // F floats
+  __shared__ float red[3][32];
+  const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];      // weights: they may be read before the kernel in front has finished
+  pdl_wait(); pdl_trigger();
+  const long long row = blockIdx.x;
+  const T* zr = z + row * ld;
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto add = [&](float v) { const float p = v * v; s2 += p; s4 = fmaf(p, p, s4); s6 = fmaf(p * p, p, s6); };
+  for (int i = threadIdx.x * V; i < F; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 t = Vec4<T>::load(zr + i);
+      *reinterpret_cast<float4*>(srow + i) = t;
+      add(t.x); add(t.y); add(t.z); add(t.w);
+    } else { const float t = ldx(zr + i); srow[i] = t; add(t); }
+  }
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
+  s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
+  if (l == 0) { red[0][w] = s2; red[1][w] = s4; red[2][w] = s6; }
+  __syncthreads();
+  const float n = (float)F;
+  const float r1 = ca * rsqrtf(warp_sum(l < nw ? red[0][l] : 0.f) / n + eps), r2 = cb * rsqrtf(warp_sum(l < nw ? red[1][l] : 0.f) / n + eps),
+              r3 = cc * rsqrtf(warp_sum(l < nw ? red[2][l] : 0.f) / n + eps);
+  auto f = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, r3, r2), r1), ce); };
+  T* o = out + row * F;
+  for (int i = threadIdx.x * V; i < F; i += blockDim.x * V) {        // a thread rereads only what it stored itself
+    if constexpr (V == 4) {
+      const float4 t = *reinterpret_cast<const float4*>(srow + i);
+      Vec4<T>::store(o + i, make_float4(f(t.x), f(t.y), f(t.z), f(t.w)));
+    } else stx(o + i, f(srow[i]));
+  }
+}
+
+template <typename T>
+static int poly_norm_t(const void* z, long long ld, void* out, int rows, int F, const float* coef, float eps, cudaStream_t st) {
+  const size_t smem = (size_t)F * sizeof(float);
+  const bool vec = F % 4 == 0 && ld % 4 == 0 && ((uintptr_t)z | (uintptr_t)out) % 16 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((F + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+  auto k = vec ? poly_norm_kernel<T, 4> : poly_norm_kernel<T, 1>;
+  if (smem > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl(k, dim3((unsigned)rows), dim3((unsigned)threads), smem, st, (const T*)z, ld, (T*)out, F, coef, eps);
+}
+
+// Gated activation of the valid rows of an expert-major layout: rows [row_start[g], row_start[g] + counts[g]) of x [rows, 2I] -> y [rows, I].
+// blockIdx.x: a row; rows of no group are left as they are.
+template <typename T, int V>
+__global__ void __launch_bounds__(128) glu_groups_kernel(const T* __restrict__ x, T* __restrict__ y, const int* __restrict__ counts, const int* __restrict__ row_start,
+                                                         int groups, int I, int act, float p0, float p1) {
+  pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
+  const int row = blockIdx.x;
+  if (row >= row_start[groups]) return;
+  int lo = 0, hi = groups - 1;              // the last group that starts at or before the row
+  while (lo < hi) { const int mid = (lo + hi + 1) >> 1; if (row_start[mid] <= row) lo = mid; else hi = mid - 1; }
+  if (row >= row_start[lo] + counts[lo]) return;
+  const T* g = x + (long long)row * 2 * I;
+  T* o = y + (long long)row * I;
+  for (int c = threadIdx.x * V; c < I; c += 128 * V) {
+    if constexpr (V == 4) {
+      const float4 a = Vec4<T>::load(g + c), b = Vec4<T>::load(g + I + c);
+      Vec4<T>::store(o + c, make_float4(glu_exact(a.x, b.x, act, p0, p1), glu_exact(a.y, b.y, act, p0, p1), glu_exact(a.z, b.z, act, p0, p1),
+                                        glu_exact(a.w, b.w, act, p0, p1)));
+    } else stx(o + c, glu_exact(ldx(g + c), ldx(g + I + c), act, p0, p1));
+  }
+}
+
+template <typename T>
+static int glu_groups_t(const void* x, void* y, const int* counts, const int* row_start, int groups, int rows, int I, int act, float p0, float p1, cudaStream_t st) {
+  const bool vec = I % 4 == 0 && ((uintptr_t)x | (uintptr_t)y) % 16 == 0;
+  return (int)launch_pdl(vec ? glu_groups_kernel<T, 4> : glu_groups_kernel<T, 1>, dim3((unsigned)rows), dim3(128), 0, st, (const T*)x, (T*)y, counts, row_start, groups, I,
+                         act, p0, p1);
+}
+
 // ---- key / value rows into paged caches -------------------------------------------------------------------------------------
 // Row t of k (kw elements, row stride k_ld) goes to cache row slots[t], the same for v.  U: the access unit (uint4 where everything is
 // 16-byte aligned, else one element); widths and strides in units.
@@ -568,4 +743,31 @@ extern "C" int ne_cap_rows(float* x, long long n, float cap, cudaStream_t st) {
   if (n <= 0) return 0;
   if (!(cap > 0.f)) return 1001;
   return (int)launch_pdl(cap_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, x, n, cap);
+}
+
+// See DepthArgs.  y [T, W] (row stride y_ld), x [T, W], bank [layers, T, W] or null, w [at + 1] or null (then at is the bank row to fill), g [1] fp32, out [T, W]
+extern "C" int ne_depth_mix(const void* y, long long y_ld, float* x, float* bank, int at, const float* w, const float* g, void* out, const long long* ids,
+                            const void* table, int vocab, int T, int W, float eps, int last, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (W <= 0 || W > 48 * 1024 || at < 0 || at > 1024 || !g || (w && !bank) || (!ids && !y) || (ids && (!table || w || last))) return 1001;
+  DepthArgs a;
+  a.y = ids ? nullptr : y; a.y_ld = ids ? 0 : y_ld; a.x = x; a.bank = bank; a.bank_ld = (long long)T * W; a.w = w; a.g = g; a.out = out; a.ids = ids;
+  a.table = ids ? table : nullptr; a.at = at; a.W = W; a.vocab = vocab; a.last = last; a.eps = eps;
+  return fp32 ? depth_mix_t<float>(a, T, st) : depth_mix_t<__nv_bfloat16>(a, T, st);
+}
+
+// z [T, F] (row stride ld) -> out [T, F]; coef fp32 [4]
+extern "C" int ne_poly_norm(const void* z, long long ld, void* out, int T, int F, const float* coef, float eps, int fp32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (F <= 0 || F > 48 * 1024 || ld < F) return 1001;
+  return fp32 ? poly_norm_t<float>(z, ld, out, T, F, coef, eps, st) : poly_norm_t<__nv_bfloat16>(z, ld, out, T, F, coef, eps, st);
+}
+
+// x [rows, 2I] -> y [rows, I] for the rows of `groups` experts (counts [groups], row_start [groups + 1])
+extern "C" int ne_glu_groups(const void* x, void* y, const int* counts, const int* row_start, int groups, int rows, int I, int act, float p0, float p1, int fp32,
+                             cudaStream_t st) {
+  if (rows <= 0 || I <= 0) return 0;
+  if (act < 0 || act > 4 || groups < 1) return 1001;
+  return fp32 ? glu_groups_t<float>(x, y, counts, row_start, groups, rows, I, act, p0, p1, st)
+              : glu_groups_t<__nv_bfloat16>(x, y, counts, row_start, groups, rows, I, act, p0, p1, st);
 }

@@ -260,6 +260,8 @@ def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
     Returns partial logits [P, T, E] (the hidden dimension is split into P slices so enough CTAs pull the weight at
     once); `moe_route` adds the planes up, any other consumer calls `.sum(0)`."""
+    if x.dtype == torch.float32 or x.shape[-1] % 8:
+        return linear(x, w)                # plain product in 32-bit
     x2 = _as_bf16_2d(x)
     T, H = x2.shape
     E = w.shape[0]
@@ -419,6 +421,64 @@ def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float):
     assert table.is_contiguous()
     x = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
     return _postnorm(None, x, scale, None, 0.0, None, _i64c(ids), table, table.dtype)
+
+
+def _depth_mix(y, x, g, eps, bank, at, w, last, ids, table, dt):
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and g.dtype == torch.float32
+    assert bank is None or (bank.dtype == torch.float32 and bank.is_contiguous() and bank.shape[1:] == (T, W) and at < bank.shape[0])
+    assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == at + 1)
+    out = torch.empty(T, W, dtype=dt, device=x.device)
+    _ck(lib().ne_depth_mix(_p(y), _c.c_longlong(0 if y is None else y.stride(0)), _p(x), _p(bank), _c.c_int(at), _p(w), _p(g), _p(out), _p(ids), _p(table),
+                           _c.c_int(0 if table is None else table.shape[0]), _c.c_int(T), _c.c_int(W), _c.c_float(eps), _c.c_int(int(last)),
+                           _c.c_int(int(dt == torch.float32)), _st()), "ne_depth_mix")
+    return out, x
+
+
+def depth_mix(y: torch.Tensor, x: torch.Tensor, g: torch.Tensor, eps: float, bank: Optional[torch.Tensor] = None, at: int = 0, w: Optional[torch.Tensor] = None,
+              last: bool = False):
+    """Sum, average over the depth and norm: one kernel, one CTA per row; x is updated in place."""
+    assert y.stride(1) == 1
+    return _depth_mix(y, x, g, eps, bank, at, w, last, None, None, y.dtype)
+
+
+def depth_embed(ids: torch.Tensor, table: torch.Tensor, g: torch.Tensor, eps: float, layers: int):
+    assert table.is_contiguous()
+    T, W = ids.numel(), table.shape[1]
+    x = torch.empty(T, W, dtype=torch.float32, device=table.device)
+    bank = torch.empty(layers, T, W, dtype=torch.float32, device=table.device)
+    return (*_depth_mix(None, x, g, eps, bank, 0, None, False, _i64c(ids), table, table.dtype), bank)
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    T, F = z.shape
+    assert z.stride(1) == 1 and coef.dtype == torch.float32 and coef.numel() == 4
+    out = torch.empty(T, F, dtype=z.dtype, device=z.device)
+    _ck(lib().ne_poly_norm(_p(z), _c.c_longlong(z.stride(0)), _p(out), _c.c_int(T), _c.c_int(F), _p(coef), _c.c_float(eps), _c.c_int(int(z.dtype == torch.float32)), _st()),
+        "ne_poly_norm")
+    return out
+
+
+def conv_rows(proj: torch.Tensor, w: torch.Tensor, q_width: int, k_cache, v_cache, slot_mapping: torch.Tensor, window, slots, cu_seqlens: torch.Tensor, fresh,
+              max_q_len: int = 0) -> torch.Tensor:
+    """One kernel: convolution, query rows, key and value rows into the caches, the sequences' windows."""
+    T, (taps, C) = proj.shape[0], w.shape
+    dt = proj.dtype
+    kw, vw = (0, 0) if k_cache is None else (k_cache.shape[2] * k_cache.shape[3], v_cache.shape[2] * v_cache.shape[3])
+    assert C == q_width + kw + vw and proj.stride(1) == 1 and w.dtype == dt and w.is_contiguous()
+    assert k_cache is None or (k_cache.dtype == v_cache.dtype == dt and k_cache.is_contiguous() and v_cache.is_contiguous())
+    assert taps == 1 or (window.dtype == dt and window.is_contiguous() and window.shape[1:] == (taps - 1, C))
+    q = torch.empty(T, q_width, dtype=dt, device=proj.device)
+    if T == 0:
+        return q
+    cu = _i32(cu_seqlens)
+    B = cu.numel() - 1
+    mq = max_q_len if max_q_len else (T if T > B else 1)
+    s, f = (None, None) if taps == 1 else (_i32(slots), _i32(fresh))
+    _ck(lib().ne_shortconv(_p(proj), _c.c_longlong(proj.stride(0)), _p(w), _c.c_int(taps), _p(q), _c.c_int(q_width), _p(k_cache), _c.c_int(kw), _p(v_cache), _c.c_int(vw),
+                           _p(_i64c(slot_mapping)), _p(window), _p(s), _p(cu), _p(f), _c.c_int(T), _c.c_int(B), _c.c_int(mq), _c.c_int(int(dt == torch.float32)), _st()),
+        "ne_shortconv")
+    return q
 
 
 def layernorm(x, w, b, eps):
@@ -653,33 +713,39 @@ def gqa_qkv_prepare(qkv, hq, hkv, hd, q_norm_w, k_norm_w, eps, unit_offset, posi
 
 # ---- MoE -----------------------------------------------------------------------------------------
 def moe_route(logits, bias, top_k, n_group=1, topk_group=1, norm_topk_prob=True, routed_scaling_factor=1.0, scoring="sigmoid",
-              balance_ranks: int = 0, log2phy: Optional[torch.Tensor] = None, logcnt: Optional[torch.Tensor] = None):
+              balance_ranks: int = 0, log2phy: Optional[torch.Tensor] = None, logcnt: Optional[torch.Tensor] = None, gate_cols: int = 0, split_gate: bool = False):
     """`balance_ranks`, `log2phy` / `logcnt` (int32 device tables [E, R] / [E]): see `reference.moe_route`."""
     planes = logits.shape[0] if logits.dim() == 3 else 1
-    T, E = logits.shape[-2:]
+    T, ld = logits.shape[-2:]
+    E = ld - gate_cols
     logits = logits.float().contiguous()
+    gate = torch.empty(T, dtype=torch.float32, device=logits.device) if gate_cols else None
     idx = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     if log2phy is not None:
         assert log2phy.dtype == torch.int32 and logcnt.dtype == torch.int32 and log2phy.is_contiguous() and log2phy.shape[0] == E
     _ck(lib().ne_moe_route(_p(logits), _p(bias), _p(idx), _p(w), _c.c_int(T), _c.c_int(E), _c.c_int(top_k), _c.c_int(n_group), _c.c_int(topk_group),
                            _c.c_int(1 if norm_topk_prob else 0), _c.c_float(routed_scaling_factor), _c.c_int({"sigmoid": 0, "softmax": 1, "sqrtsoftplus": 2}[scoring]),
-                           _c.c_int(planes), _c.c_int(balance_ranks), _p(log2phy), _p(logcnt), _c.c_int(0 if log2phy is None else log2phy.shape[1]), _st()),
-        "ne_moe_route")
-    return idx, w
+                           _c.c_int(planes), _c.c_int(balance_ranks), _p(log2phy), _p(logcnt), _c.c_int(0 if log2phy is None else log2phy.shape[1]),
+                           _c.c_int(ld), _p(gate), _st()), "ne_moe_route")
+    return (idx, w, gate) if split_gate else (idx, w)
 
 
-def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, expert_offset: int = 0, add_in=None, act=None) -> torch.Tensor:
+def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, expert_offset: int = 0, add_in=None, act=None, add_gate=None,
+                identity_from: Optional[int] = None) -> torch.Tensor:
     """Local routed experts over an expert-major, 128-row-aligned layout: scatter (+fp8 quant) -> grouped GEMM ->
-    SwiGLU (+requant) -> grouped GEMM -> weighted gather.  `add_in` (e.g. the shared-expert output) is summed in the gather."""
+    SwiGLU (+requant) -> grouped GEMM -> weighted gather.  `add_in` (e.g. the shared-expert output) is summed in the gather, and so are the tokens' own
+    rows of identity experts.  32-bit runs, and sizes the tensor-core GEMM cannot address, take plain products over the same layout."""
     T, H = x.shape
     E, I2, _ = w13.shape
     I = I2 // 2
     K = topk_idx.shape[1]
     dev = x.device
     fp8 = w13.dtype == FP8
-    x = _as_bf16_2d(x)
-    out = torch.empty(T, H, dtype=torch.bfloat16, device=dev)
+    f32 = w13.dtype == torch.float32
+    simt = f32 or (not fp8 and (H % 8 or I % 8))
+    x = _as_bf16_2d(x) if not simt else x.to(w13.dtype).contiguous()
+    out = torch.empty(T, H, dtype=w13.dtype if simt else torch.bfloat16, device=dev)
     if T == 0:
         return out
     R = T * K + E * 127
@@ -694,13 +760,17 @@ def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, exp
         a_s = torch.empty(H // 128, R, dtype=torch.float32, device=dev)
         a_b = None
     else:
-        a_b = torch.empty(R, H, dtype=torch.bfloat16, device=dev)
+        a_b = torch.empty(R, H, dtype=x.dtype, device=dev)
         a_q = a_s = None
-    _ck(lib().ne_moe_dispatch_local(_p(x), _p(idx), _p(counts), _p(slot), _p(row_start), _p(pos), _p(a_b), _p(a_q), _p(a_s), _c.c_int(R),
-                                    _c.c_int(T), _c.c_int(K), _c.c_int(H), _c.c_int(expert_offset), _c.c_int(E), _c.c_int(R), _c.c_int(128), _st()),
-        "ne_moe_dispatch_local")
-    g = torch.empty(R, I2, dtype=torch.bfloat16, device=dev)
-    y = torch.empty(R, H, dtype=torch.bfloat16, device=dev)
+    if simt:
+        _ck(lib().ne_moe_dispatch_rows(_p(x), _c.c_int(H * x.element_size()), _p(idx), _p(counts), _p(slot), _p(row_start), _p(pos), _p(a_b), _c.c_int(T), _c.c_int(K),
+                                       _c.c_int(expert_offset), _c.c_int(E), _c.c_int(R), _c.c_int(128), _st()), "ne_moe_dispatch_rows")
+    else:
+        _ck(lib().ne_moe_dispatch_local(_p(x), _p(idx), _p(counts), _p(slot), _p(row_start), _p(pos), _p(a_b), _p(a_q), _p(a_s), _c.c_int(R),
+                                        _c.c_int(T), _c.c_int(K), _c.c_int(H), _c.c_int(expert_offset), _c.c_int(E), _c.c_int(R), _c.c_int(128), _st()),
+            "ne_moe_dispatch_local")
+    g = torch.empty(R, I2, dtype=x.dtype, device=dev)
+    y = torch.empty(R, H, dtype=x.dtype, device=dev)
     if fp8:
         _gemm(a_q, H, 0, w13, g, I2, 0, R, I2, H, E, counts, row_start, True, a_s, R, 0, w13_scale, False)
         h_q = torch.empty(R, I, dtype=FP8, device=dev)
@@ -709,15 +779,35 @@ def moe_experts(x, topk_idx, topk_w, w13, w2, w13_scale=None, w2_scale=None, exp
                              *_act_args(act), _st()), "ne_act_mul")
         _gemm(h_q, I, 0, w2, y, H, 0, R, H, I, E, counts, row_start, True, h_s, R, 0, w2_scale, False)
     else:
-        _gemm(a_b, H, 0, w13, g, I2, 0, R, I2, H, E, counts, row_start, False, None, 0, 0, None, False)
-        h = torch.empty(R, I, dtype=torch.bfloat16, device=dev)
-        _ck(lib().ne_act_mul(_p(g), _p(h), _p(None), _p(None), _c.c_int(0), _c.c_longlong(0), _p(counts), _p(row_start), _c.c_int(E), _c.c_int(R), _c.c_int(I),
-                             *_act_args(act), _st()), "ne_act_mul")
-        _gemm(h, I, 0, w2, y, H, 0, R, H, I, E, counts, row_start, False, None, 0, 0, None, False)
+        def product(a, b, d, N, K_):
+            if simt:
+                _ck(lib().ne_gemm_simt_groups(_p(a), _p(b), _p(d), _c.c_int(R), _c.c_int(N), _c.c_int(K_), _c.c_int(E), _p(counts), _p(row_start), _c.c_int(int(f32)),
+                                              _st()), "ne_gemm_simt_groups")
+            else:
+                _gemm(a, K_, 0, b, d, N, 0, R, N, K_, E, counts, row_start, False, None, 0, 0, None, False)
+        product(a_b, w13, g, I2, H)
+        h = torch.empty(R, I, dtype=x.dtype, device=dev)
+        if simt or I % 128:
+            _ck(lib().ne_glu_groups(_p(g), _p(h), _p(counts), _p(row_start), _c.c_int(E), _c.c_int(R), _c.c_int(I), *_act_args(act), _c.c_int(int(f32)), _st()),
+                "ne_glu_groups")
+        else:
+            _ck(lib().ne_act_mul(_p(g), _p(h), _p(None), _p(None), _c.c_int(0), _c.c_longlong(0), _p(counts), _p(row_start), _c.c_int(E), _c.c_int(R), _c.c_int(I),
+                                 *_act_args(act), _st()), "ne_act_mul")
+        product(h, w2, y, H, I)
     if callable(add_in):
         add_in = add_in()          # produced on another stream: the callable joins that stream as late as possible
-    _ck(lib().ne_moe_combine_local(_p(y), _p(pos), _p(w), _p(add_in), _p(out), _c.c_int(T), _c.c_int(K), _c.c_int(H), _st()), "ne_moe_combine_local")
+    _moe_combine(y, pos, w, add_in, add_gate, x if identity_from is not None else None, idx, identity_from or 0, out)
     return out
+
+
+def _moe_combine(y, pos, w, add_in, add_gate, x, idx, identity_from, out):
+    T, H = out.shape
+    if add_in is None:
+        add_gate = None
+    assert add_in is None or (add_in.dtype == out.dtype and add_in.is_contiguous())
+    assert add_gate is None or (add_gate.dtype == torch.float32 and add_gate.is_contiguous())
+    _ck(lib().ne_moe_combine_local(_p(y), _p(pos), _p(w), _p(add_in), _p(add_gate), _p(x), _p(idx), _c.c_int(identity_from), _p(out), _c.c_int(T),
+                                   _c.c_int(w.shape[1]), _c.c_int(H), _c.c_int(int(out.dtype == torch.float32)), _st()), "ne_moe_combine_local")
 
 
 # ---- NVFP4 -------------------------------------------------------------------------------------------------------
@@ -794,7 +884,7 @@ def moe_experts_nvfp4(x, topk_idx, topk_w, w13_q, w13_sf, alpha1, a1_gscale, w2_
     y = nvfp4_gemm(hq, hsf, w2_q, w2_sf, alpha2, counts, row_start)
     if callable(add_in):
         add_in = add_in()
-    _ck(lib().ne_moe_combine_local(_p(y), _p(pos), _p(w), _p(add_in), _p(out), _c.c_int(T), _c.c_int(K), _c.c_int(H), _st()), "ne_moe_combine_local")
+    _moe_combine(y, pos, w, add_in, None, None, idx, 0, out)
     return out
 
 
@@ -842,6 +932,13 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
     from . import sm100_attn
     return sm100_attn.gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window, softcap, slopes, gate, out_scale, out,
                                            max_q_len, pooled, pool, turn_back)
+
+
+def differential_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int, keep_first: int, mixing: torch.Tensor,
+                           out_scale: float, eps: float, gate: torch.Tensor, max_q_len: int = 0) -> torch.Tensor:
+    from . import sm100_attn
+    return sm100_attn.differential_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window, keep_first, mixing, out_scale, eps, gate,
+                                             max_q_len)
 
 
 def gqa_attention_paged(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window: int = 0):

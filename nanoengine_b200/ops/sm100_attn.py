@@ -253,7 +253,7 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
         _k._ck(lib.ne_gqa_biased(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _c.c_int(k_cache.shape[0]), _k._p(bt), _c.c_int(bt.stride(0)),
                                  _k._p(cu), _k._p(cl), _c.c_int(B), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq),
                                  _c.c_int(tiles), _c.c_int(S), _c.c_float(scale), _c.c_float(softcap), _k._p(slopes), _c.c_int(int(window)), _k._p(gate),
-                                 _c.c_longlong(gate_ld), _c.c_float(out_scale), _k._p(out), _c.c_longlong(out.stride(0)), _k._p(part), _k._p(lse2), *extra, _k._st()),
+                                 _c.c_longlong(gate_ld), _c.c_float(out_scale), _k._p(out), _c.c_longlong(out.stride(0)), _k._p(part), _k._p(lse2), *extra, _c.c_int(0), _k._st()),
                "ne_gqa_biased")
         BIASED_TC_CALLS[0] += 1
         _k.LAUNCHES[0] += int(S > 1)
@@ -261,7 +261,56 @@ def gqa_attention_biased(q, k_cache, v_cache, block_tables, cu_seqlens_q, contex
     _k._ck(lib.ne_attn_biased(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _k._p(bt), _c.c_int(bt.stride(0)), _c.c_int(k_cache.shape[1]),
                               _k._p(cu), _k._p(cl), _c.c_int(B), _k._p(out), _c.c_longlong(out.stride(0)), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D),
                               _c.c_int(Dv), _c.c_float(scale), _c.c_float(softcap), _k._p(slopes), _c.c_int(int(window)), _k._p(gate), _c.c_longlong(gate_ld),
-                              _c.c_float(out_scale), _c.c_int(int(q.dtype == torch.float32)), *extra, _k._st()), "ne_attn_biased")
+                              _c.c_float(out_scale), _c.c_int(int(q.dtype == torch.float32)), *extra, _c.c_int(0), _k._st()), "ne_attn_biased")
+    return out
+
+
+DIFF_TC_CALLS = [0]          # launches of the tensor-core kernel of differential_attention
+
+
+def differential_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, context_lens, scale, window, keep_first, mixing, out_scale, eps, gate, max_q_len=0,
+                           splits=None):
+    """bf16 with maps of up to 128 and values of up to 256 in multiples of 8 and 64-token pages: tensor cores; other shapes and 32-bit runs: the generic kernel."""
+    T, Hq, _, D = q.shape
+    Hkv, Dv = k_cache.shape[2], v_cache.shape[3]
+    lib = _k.lib()
+    bt, cu, cl = _i32(block_tables), _i32(cu_seqlens_q), _i32(context_lens)
+    B = cl.numel()
+    assert q.dtype == k_cache.dtype == v_cache.dtype == gate.dtype and q.dtype in (torch.bfloat16, torch.float32) and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert q[0].is_contiguous() if T else True
+    assert k_cache.shape[3] == 2 * D and Hq % Hkv == 0 and gate.stride(1) == 1 and gate.shape == (T, Hq * Dv) and mixing.dtype == torch.float32
+    out = torch.empty(T, Hq * Dv, dtype=q.dtype, device=q.device)
+    if T == 0:
+        return out
+    mq = max_q_len if max_q_len else (1 if T <= B else T)
+    tq = 0
+    if (q.dtype == torch.bfloat16 and k_cache.shape[1] == 64 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and gate.stride(0) % 4 == 0
+            and gate.data_ptr() % 8 == 0 and D % 8 == 0 and Dv % 8 == 0):
+        tq = lib.ne_gqa_diff_plan(_c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq))
+    if tq:
+        tiles = min(T, T // tq + B)
+        S = splits
+        if S is None:
+            pages = bt.shape[1] if window <= 0 else min(bt.shape[1], (window + tq + 62) // 64 + 1 + (keep_first + 63) // 64)
+            S = 1
+            slots = _sms() * (2 if Dv <= 128 and D <= 64 else 1)      # resident CTAs
+            if tiles * Hkv * 2 <= slots:               # few CTAs (small decode batches): slice the keys
+                S = max(1, min(slots // (tiles * Hkv), max(1, pages // 4), 16))
+        part = lse2 = None
+        if S > 1:
+            part = torch.empty(S, T, Hq, 2, Dv, dtype=torch.float32, device=q.device)
+            lse2 = torch.empty(S, T, Hq, 2, dtype=torch.float32, device=q.device)
+        _k._ck(lib.ne_gqa_diff(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _c.c_int(k_cache.shape[0]), _k._p(bt), _c.c_int(bt.stride(0)),
+                               _k._p(cu), _k._p(cl), _c.c_int(B), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D), _c.c_int(Dv), _c.c_int(mq), _c.c_int(tiles),
+                               _c.c_int(S), _c.c_float(scale), _c.c_int(int(window)), _c.c_int(int(keep_first)), _k._p(mixing), _c.c_float(out_scale), _c.c_float(eps),
+                               _k._p(gate), _c.c_longlong(gate.stride(0)), _k._p(out), _c.c_longlong(out.stride(0)), _k._p(part), _k._p(lse2), _k._st()), "ne_gqa_diff")
+        DIFF_TC_CALLS[0] += 1
+        _k.LAUNCHES[0] += int(S > 1)
+        return out
+    _k._ck(lib.ne_attn_diff(_k._p(q), _c.c_longlong(q.stride(0)), _k._p(k_cache), _k._p(v_cache), _k._p(bt), _c.c_int(bt.stride(0)), _c.c_int(k_cache.shape[1]),
+                            _k._p(cu), _k._p(cl), _c.c_int(B), _k._p(out), _c.c_longlong(out.stride(0)), _c.c_int(T), _c.c_int(Hq), _c.c_int(Hkv), _c.c_int(D),
+                            _c.c_int(Dv), _c.c_float(scale), _c.c_int(int(window)), _c.c_int(int(keep_first)), _k._p(mixing), _c.c_float(out_scale), _c.c_float(eps),
+                            _k._p(gate), _c.c_longlong(gate.stride(0)), _c.c_int(int(q.dtype == torch.float32)), _k._st()), "ne_attn_diff")
     return out
 
 
