@@ -93,13 +93,13 @@ def main():
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours")
-    ap.add_argument("--model", default="deepseek-v3", choices=["deepseek-v3", "deepseek-v32", "qwen3-235b", "tuvutar", "filasun", "sapanex"],
+    ap.add_argument("--model", default="deepseek-v3", choices=["deepseek-v3", "deepseek-v32", "qwen3-235b", "tuvutar", "filasun", "sapanex", "gipozen"],
                     help="deepseek-v3: the headline (fp8, attention-DP + EP); deepseek-v32: the same body with the DSA indexer and sparse "
                          "attention (long-context decode, see --synthetic-context); qwen3-235b: bf16 GQA MoE with tensor-parallel attention + "
-                         "EP (the batch is shared by the TP ranks: --seqs-per-gpu is then the size of the whole batch); tuvutar, filasun, sapanex: prefill and "
+                         "EP (the batch is shared by the TP ranks: --seqs-per-gpu is then the size of the whole batch); tuvutar, filasun, sapanex, gipozen: prefill and "
                          "decode of that design at the sizes of --sizes beside the closest model at equal sizes (one GPU, benchmarks/hybrid_bench.py)")
-    ap.add_argument("--sizes", default="small,medium", help="tuvutar, filasun, sapanex: small (width 2048), medium (4096), large (7168)")
-    ap.add_argument("--skip-closest", action="store_true", help="tuvutar, filasun, sapanex: leave the closest model out")
+    ap.add_argument("--sizes", default="small,medium", help="tuvutar, filasun, sapanex, gipozen: small (width 2048), medium (4096), large (7168)")
+    ap.add_argument("--skip-closest", action="store_true", help="tuvutar, filasun, sapanex, gipozen: leave the closest model out")
     ap.add_argument("--synthetic-context", action="store_true",
                     help="decode-only: sequences are admitted with --prompt-len tokens of context whose cache rows are random bytes (no "
                          "prefill pass; a 64 x 65,536-token prefill would take minutes).  The decode step does all of its work.")
@@ -123,7 +123,7 @@ def main():
         return reference_arm(args)
     if args.warmup < 3:
         args.warmup = 3
-    if args.model in ("tuvutar", "filasun", "sapanex"):
+    if args.model in ("tuvutar", "filasun", "sapanex", "gipozen"):
         from benchmarks.hybrid_bench import main as hybrid_main
         return hybrid_main(args)
 

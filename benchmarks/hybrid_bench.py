@@ -1,5 +1,5 @@
 """Prefill and decode throughput of a model with listed layers beside the closest model of this package at equal sizes (`bench.py --model
-tuvutar`, `--model filasun`, `--model sapanex`).
+tuvutar`, `--model filasun`, `--model sapanex`, `--model gipozen`).
 
 Tuvutar: the closest model is Kimi-K3's layer stack without experts and with a plain residual: latent attention between delta-rule layers and
 dense gated MLPs in bf16 (its delta layers decay per key channel, its latent layers carry an output gate).  Both get the same width,
@@ -14,6 +14,11 @@ feed-forward weights, width and vocabulary; the attention window is the longest 
 Sapanex: the closest model is the dense Qwen3.5 stack again, an attention layer after every three delta layers in both, the same head counts, head
 sizes, state sizes, width and vocabulary; a feed-forward of two matrices of 3 ff / 2 stands against a gated one of three of ff.  Sapanex's attention
 layers see a window of 1024 tokens and blocks of 16, Qwen3.5's the whole context.
+
+Gipozen: the closest model is the Qwen3.5-MoE stack with attention in every layer: grouped-query attention with an output gate against two maps of half the
+head size over the same values (equal projections and rows), dense and mixture layers in turn, the same experts, shared expert behind a gate, head
+counts, width and vocabulary; a dense feed-forward of two matrices of 3 ff / 2 stands against a gated one of three of ff.  Gipozen's layers see a window
+of 4096 tokens behind 16 kept ones, route over 4 identity experts more, and keep their own rows (`kv_from` is left out); Qwen3.5's see the whole context.
 
 `prefill` is the device time of the scheduler's prompt steps (CUDA events around
 LLM.step), `decode` the replay of one decode step on resident inputs (graph + lm_head + sampling)."""
@@ -82,7 +87,26 @@ def qwen_3to1_model(width, heads, groups, ff, vocab):
                         linear_value_head_dim=128, max_position_embeddings=16384)
 
 
-DESIGNS = {"sapanex": ("Sapanex", sapanex_model, "qwen3_5_stack", qwen_3to1_model),
+def gipozen_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import ModelConfig, _differential_spec
+    layers = []
+    for i in range(2 * groups):
+        layers += [_differential_spec(heads, heads // 4, 64, 128, 4096, 16, 4, 0.4, ff=3 * ff // 2),
+                   _differential_spec(heads, heads // 4, 64, 128, 4096, 16, 4, 0.4, experts=(64, 4, 8, ff // 8, ff // 4, 7.0))]
+    return ModelConfig.from_dict({"architecture": "Gipozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "layers": layers})
+
+
+def qwen_moe_model(width, heads, groups, ff, vocab):
+    from nanoengine_b200.models.config import tiny_qwen3_5
+    n = 4 * groups
+    return tiny_qwen3_5(True, vocab_size=vocab, hidden_size=width, num_hidden_layers=n, layer_types=["full_attention"] * n, linear_num_value_heads=0,
+                        linear_num_key_heads=0, num_attention_heads=heads, num_key_value_heads=heads // 4, head_dim=128, intermediate_size=ff, n_routed_experts=64,
+                        num_experts_per_tok=8, moe_intermediate_size=ff // 8, shared_expert_intermediate_size=ff // 4, mlp_layer_types=["dense", "sparse"] * (n // 2),
+                        max_position_embeddings=16384)
+
+
+DESIGNS = {"gipozen": ("Gipozen", gipozen_model, "qwen3_5_moe_stack", qwen_moe_model),
+           "sapanex": ("Sapanex", sapanex_model, "qwen3_5_stack", qwen_3to1_model),
            "tuvutar": ("Tuvutar", tuvutar_model, "kimi_k3_stack", kimi_model),
            "filasun": ("Filasun", filasun_model, "qwen3_5_stack", qwen_model)}
 

@@ -404,6 +404,85 @@ def case_postnorm(T, W=4096):
     return lambda: sm100.postnorm(y, x, 2.0, w, 1e-6), T * W * (2 + 4 + 4 + 2), 0.0
 
 
+def case_differential(B, ctx, q_len, H=32, G=8, window=0, keep=0, D=64, Dv=128, bs=64):
+    """Differential attention (two maps of D per head over values of Dv), norm and gate included.  Bytes and FLOPs of the keys that are seen."""
+    nb = (ctx + bs - 1) // bs
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    k, v = torch.randn(B * nb + 1, bs, G, 2 * D, **bf), torch.randn(B * nb + 1, bs, G, Dv, **bf)
+    bt = torch.randperm(B * nb, device="cuda").view(B, nb).to(torch.int32)
+    T = B * q_len
+    q, gate, mixing = torch.randn(T, H, 2, D, **bf), torch.randn(T, H * Dv, **bf), torch.tensor([0.4], device="cuda")
+    cu = (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    cl = torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    fn = lambda: sm100_attn.differential_attention(q, k, v, bt, cu, cl, D ** -0.5, window, keep, mixing, 0.6, 1e-6, gate, q_len)
+    w = window or ctx
+    pairs = B * sum(min(w + (keep if window else 0), ctx - q_len + i + 1) for i in range(q_len))
+    seen = min(ctx, w + (keep if window else 0) + q_len - 1)
+    return fn, B * seen * G * (2 * D + Dv) * 2 + T * H * (2 * D + 2 * Dv) * 2, 4.0 * pairs * H * (D + Dv)
+
+
+def case_shortconv(B, q_len, H=32, G=8, D=64, Dv=128, taps=4, bs=64):
+    """Short convolution of queries, keys and values, key and value rows, windows."""
+    T, qw = B * q_len, H * 2 * D
+    C = qw + G * (2 * D + Dv)
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    proj, w, win = torch.randn(T, C + H * Dv, **bf), torch.randn(taps, C, **bf), torch.randn(B + 1, taps - 1, C, **bf)
+    kc, vc = torch.zeros(T // bs + 2, bs, G, 2 * D, **bf), torch.zeros(T // bs + 2, bs, G, Dv, **bf)
+    rows, slots, cu = torch.arange(T, device="cuda"), torch.arange(B, device="cuda", dtype=torch.int32), (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32)
+    fresh = torch.zeros(B, dtype=torch.int32, device="cuda")
+    return lambda: sm100.conv_rows(proj, w, qw, kc, vc, rows, win, slots, cu, fresh, q_len), (T * 2 + B * 2 * (taps - 1)) * C * 2, 0.0
+
+
+def case_gdn_conv(B, q_len, C=6144, taps=4):
+    """The like front end of the Qwen3.5 delta layers: convolution and silu, windows."""
+    T = B * q_len
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    x, w, win = torch.randn(T, C + 4096, **bf)[:, :C], torch.randn(C, taps, **bf), torch.randn(B + 1, taps - 1, C, **bf)
+    slots, cu, fresh = torch.arange(B, device="cuda", dtype=torch.int32), (torch.arange(B + 1, device="cuda") * q_len).to(torch.int32), torch.zeros(B, dtype=torch.int32, device="cuda")
+    return lambda: sm100.gdn_conv(x, w, win, slots, cu, fresh, q_len == 1), (T * 2 + B * 2 * (taps - 1)) * C * 2, 0.0
+
+
+def case_depth(T, at, W=4096):
+    """Sum, average over `at` + 1 layers' results, norm; at 0: sum and norm alone."""
+    y, x, g = torch.randn(T, W, device="cuda", dtype=torch.bfloat16), torch.randn(T, W, device="cuda"), torch.ones(1, device="cuda")
+    if not at:
+        return lambda: sm100.depth_mix(y, x, g, 1e-6), T * W * (2 + 4 + 4 + 2), 0.0
+    bank, w = torch.randn(at + 1, T, W, device="cuda"), torch.full((at + 1,), 1.0 / (at + 1), device="cuda")
+    return lambda: sm100.depth_mix(y, x, g, 1e-6, bank, at, w), T * W * (2 + 4 + 4 + 4 + 4 * at + 2), 0.0
+
+
+def case_poly_norm(T, F=12288):
+    z, c = torch.randn(T, F, device="cuda", dtype=torch.bfloat16), torch.ones(4, device="cuda")
+    return lambda: sm100.poly_norm(z, c, 1e-6), T * F * 4, 0.0
+
+
+def case_glu(T, F=12288):
+    x = torch.randn(T, 2 * F, device="cuda", dtype=torch.bfloat16)
+    return lambda: sm100.silu_and_mul(x), T * F * 6, 0.0
+
+
+def case_mixture(T, design, W=4096, E=64, identity=0, top=8, I=1536, shared=1536):
+    """A whole mixture block with a gated shared expert, router to weighted sum: this design's or Qwen3.5's.  Bytes of the weights and the activations
+    between the steps."""
+    from nanoengine_b200.models.config import tiny_qwen3_5
+    from nanoengine_b200.models.layers import GatedSharedMoE
+    from nanoengine_b200.models.qwen3_5 import Qwen35MoE
+    if design == "gipozen":
+        act = ("clamp_linear", 7.0, 1.702)
+        M = GatedSharedMoE(W, E, identity, top, I, act, shared, act, torch.bfloat16, "cuda")
+        run = lambda: M(x)
+    else:
+        M = Qwen35MoE(tiny_qwen3_5(True, hidden_size=W, n_routed_experts=E, num_experts_per_tok=top, moe_intermediate_size=I, shared_expert_intermediate_size=shared),
+                      torch.bfloat16, "cuda")
+        run = lambda: M(x, None)
+    with torch.no_grad():
+        for p in M.parameters():
+            p.normal_(0.0, 0.02)
+    x = torch.randn(T, W, device="cuda", dtype=torch.bfloat16)
+    rows = T * top * E // (E + identity)
+    return run, (E * I + shared) * 3 * W * 2 + rows * (4 * W + 6 * I) + T * (4 * W + 6 * shared + 2 * W * 2), 6.0 * W * (rows * I + T * shared)
+
+
 def case_streams(T, S=2, W=4096):
     y = torch.randn(T, W, device="cuda", dtype=torch.bfloat16)
     x = torch.randn(T, S, W, device="cuda")
@@ -547,6 +626,35 @@ def build_cases(args):
         "general_delta_decode_16": lambda: case_general_delta(16),
         "general_delta_prefill_4x2048": lambda: case_general_delta(4, q_len=2048),
         "general_delta_prefill_1x8192": lambda: case_general_delta(1, q_len=8192),
+        "differential_decode": lambda: case_differential(128, 8192, 1, window=4096, keep=16),
+        "differential_decode_nowindow": lambda: case_differential(128, 4096, 1),
+        "differential_decode_16": lambda: case_differential(16, 8192, 1, window=4096, keep=16),
+        "differential_decode_small_window": lambda: case_differential(128, 8192, 1, window=512, keep=16),
+        "differential_prefill": lambda: case_differential(1, 8192, 8192, window=4096, keep=16),
+        "differential_prefill_w1024": lambda: case_differential(1, 8192, 8192, window=1024, keep=16),
+        "differential_prefill_nowindow": lambda: case_differential(1, 8192, 8192),
+        "differential_prefill_d128": lambda: case_differential(1, 8192, 8192, H=16, G=4, D=128, Dv=256),
+        "differential_decode_d128": lambda: case_differential(128, 4096, 1, H=16, G=4, D=128, Dv=256),
+        "shortconv_decode": lambda: case_shortconv(128, 1),
+        "shortconv_prefill": lambda: case_shortconv(4, 2048),
+        "gdn_conv_decode": lambda: case_gdn_conv(128, 1),
+        "gdn_conv_prefill": lambda: case_gdn_conv(4, 2048),
+        "depth_sum_decode": lambda: case_depth(128, 0),
+        "depth_sum_prefill": lambda: case_depth(8192, 0),
+        "depth_mix8_decode": lambda: case_depth(128, 8),
+        "depth_mix8_prefill": lambda: case_depth(8192, 8),
+        "depth_mix24_decode": lambda: case_depth(128, 24),
+        "poly_norm_decode": lambda: case_poly_norm(128),
+        "poly_norm_prefill": lambda: case_poly_norm(8192),
+        "glu_decode": lambda: case_glu(128),
+        "glu_prefill": lambda: case_glu(8192),
+        "mixture_decode": lambda: case_mixture(128, "gipozen"),
+        "mixture_decode_16": lambda: case_mixture(16, "gipozen"),
+        "mixture_identity_decode": lambda: case_mixture(128, "gipozen", identity=8),
+        "mixture_prefill": lambda: case_mixture(8192, "gipozen"),
+        "qwen_mixture_decode": lambda: case_mixture(128, "qwen"),
+        "qwen_mixture_decode_16": lambda: case_mixture(16, "qwen"),
+        "qwen_mixture_prefill": lambda: case_mixture(8192, "qwen"),
         "pooled_decode": lambda: case_pooled(128, 8192, 1, 32, 8, 4096, 16),
         "pooled_decode_16": lambda: case_pooled(16, 8192, 1, 32, 8, 4096, 16),
         "pooled_decode_small_window": lambda: case_pooled(128, 8192, 1, 32, 8, 512, 16),

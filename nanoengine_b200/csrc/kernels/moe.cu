@@ -321,7 +321,7 @@ __device__ __forceinline__ float round_as(float v, const float*) { return v; }
 // add_in enters times sigmoid(gate[t]) and the sum is rounded once.
 template <typename T, int V>
 __global__ void __launch_bounds__(256) moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ w,
-                                                         const T* __restrict__ add_in, const float* __restrict__ gate, const T* __restrict__ x,
+                                                         const T* __restrict__ add_in, long long add_ld, const float* __restrict__ gate, const T* __restrict__ x,
                                                          const int* __restrict__ idx, int identity_from, T* __restrict__ out, int top_k, int H) {
   pdl_wait(); pdl_trigger();      // dependent launch: nothing above this line touches global memory
   const int t = blockIdx.x;
@@ -361,7 +361,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const T* __restrict__ 
 #pragma unroll
         for (int j = 0; j < V; j++) acc[j] = round_as(acc[j], y);
       RowPiece<T, V> v;
-      v.load(add_in + (long long)t * H + c);
+      v.load(add_in + t * add_ld + c);
       v.add_to(acc, gt);
     }
     RowPiece<T, V>::store(out + (long long)t * H + c, acc);
@@ -369,10 +369,10 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const T* __restrict__ 
 }
 
 template <typename T, int V>
-static int moe_combine_t(const void* y, const int* pos, const float* w, const void* add_in, const float* gate, const void* x, const int* idx, int identity_from, void* out,
-                         int T_, int top_k, int H, cudaStream_t st) {
+static int moe_combine_t(const void* y, const int* pos, const float* w, const void* add_in, long long add_ld, const float* gate, const void* x, const int* idx, int identity_from,
+                         void* out, int T_, int top_k, int H, cudaStream_t st) {
   const int slices = T_ >= 2048 ? 1 : (T_ >= 512 ? 2 : 4);      // enough CTAs per SM at decode sizes, one pass over the tables per token otherwise
-  return (int)launch_pdl(moe_combine_kernel<T, V>, dim3(T_, slices), dim3(256), 0, st, (const T*)y, pos, w, (const T*)add_in, gate, (const T*)x, idx, identity_from, (T*)out,
+  return (int)launch_pdl(moe_combine_kernel<T, V>, dim3(T_, slices), dim3(256), 0, st, (const T*)y, pos, w, (const T*)add_in, add_ld, gate, (const T*)x, idx, identity_from, (T*)out,
                          top_k, H);
 }
 
@@ -423,17 +423,17 @@ extern "C" int ne_moe_dispatch_rows(const void* x, int row_bytes, const int* idx
                          expert_offset, E_local, max_rows);
 }
 
-// out [T, H] = the weighted rows pos [T, top_k] of y + add_in.  gate fp32 [T], x [T, H] with idx [T, top_k]: see moe_combine_kernel; null: without.
-extern "C" int ne_moe_combine_local(const void* y, const int* pos, const float* w, const void* add_in, const float* gate, const void* x, const int* idx,
-                                    int identity_from, void* out, int T, int top_k, int H, int fp32, cudaStream_t st) {
+// out [T, H] = the weighted rows pos [T, top_k] of y + add_in (row stride add_ld).  gate fp32 [T], x [T, H] with idx [T, top_k]: see moe_combine_kernel; null: without.
+extern "C" int ne_moe_combine_local(const void* y, const int* pos, const float* w, const void* add_in, long long add_ld, const float* gate, const void* x,
+                                    const int* idx, int identity_from, void* out, int T, int top_k, int H, int fp32, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (H < 1 || top_k > 64 || (x && !idx) || (gate && !add_in)) return 1001;
+  if (H < 1 || top_k > 64 || (x && !idx) || (gate && !add_in) || (add_in && add_ld < H)) return 1001;
   const int per = fp32 ? 4 : 8;
-  const bool vec = H % per == 0 && ((uintptr_t)y | (uintptr_t)add_in | (uintptr_t)x | (uintptr_t)out) % 16 == 0;
-  if (fp32) return vec ? moe_combine_t<float, 4>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st)
-                       : moe_combine_t<float, 1>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st);
-  return vec ? moe_combine_t<__nv_bfloat16, 8>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st)
-             : moe_combine_t<__nv_bfloat16, 1>(y, pos, w, add_in, gate, x, idx, identity_from, out, T, top_k, H, st);
+  const bool vec = H % per == 0 && add_ld % per == 0 && ((uintptr_t)y | (uintptr_t)add_in | (uintptr_t)x | (uintptr_t)out) % 16 == 0;
+  if (fp32) return vec ? moe_combine_t<float, 4>(y, pos, w, add_in, add_ld, gate, x, idx, identity_from, out, T, top_k, H, st)
+                       : moe_combine_t<float, 1>(y, pos, w, add_in, add_ld, gate, x, idx, identity_from, out, T, top_k, H, st);
+  return vec ? moe_combine_t<__nv_bfloat16, 8>(y, pos, w, add_in, add_ld, gate, x, idx, identity_from, out, T, top_k, H, st)
+             : moe_combine_t<__nv_bfloat16, 1>(y, pos, w, add_in, add_ld, gate, x, idx, identity_from, out, T, top_k, H, st);
 }
 
 // x bf16 [T, H], w fp32 [E, H] -> partial logits fp32 [ne_router_planes(H), T, E]; their sum over the first axis is x . w^T

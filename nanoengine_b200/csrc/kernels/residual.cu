@@ -434,17 +434,17 @@ struct DepthArgs {
   const void* y; long long y_ld; float* x; float* bank; long long bank_ld; const float* w; const float* g; void* out; const long long* ids; const void* table;
   int at, W, vocab, last; float eps;
 };
-template <typename T, int V>
-__global__ void __launch_bounds__(512) depth_mix_kernel(const DepthArgs a) {
+template <typename T, int V, bool kMix>
+__global__ void __launch_bounds__(512, kMix ? 2 : 3) depth_mix_kernel(const DepthArgs a) {
   extern __shared__ float srow[];            // W floats, then at + 1 weights
   __shared__ float red[2][32];
   const int W = a.W;
   float* sw = srow + (W + 3) / 4 * 4;
   // the coefficients are weights: they may be read before the kernel in front has finished
-  if (a.w) for (int j = threadIdx.x; j <= a.at; j += blockDim.x) sw[j] = a.w[j];
+  if (kMix) for (int j = threadIdx.x; j <= a.at; j += blockDim.x) sw[j] = a.w[j];
   const float g = *a.g;
   pdl_wait(); pdl_trigger();
-  __syncthreads();
+  if (kMix) __syncthreads();
   const long long row = blockIdx.x;
   float* xr = a.x + row * W;
   float* br = a.bank ? a.bank + row * W : nullptr;
@@ -473,11 +473,11 @@ __global__ void __launch_bounds__(512) depth_mix_kernel(const DepthArgs a) {
       if constexpr (V == 4) *reinterpret_cast<float4*>(br + a.at * a.bank_ld + i) = make_float4(v[0], v[1], v[2], v[3]);
       else br[a.at * a.bank_ld + i] = v[0];
     }
-    if (a.w) {
+    if constexpr (kMix) {
       const float wn = sw[a.at];
 #pragma unroll
       for (int e = 0; e < V; e++) v[e] *= wn;
-#pragma unroll 8
+#pragma unroll 4
       for (int j = 0; j < a.at; j++) {
         const float wj = sw[j];
         if constexpr (V == 4) {
@@ -512,7 +512,7 @@ static int depth_mix_t(const DepthArgs& a, int rows, cudaStream_t st) {
   const int per = vec ? 4 : 1;
   int threads = ((a.W + per - 1) / per + 31) / 32 * 32;
   threads = threads > 512 ? 512 : threads;
-  auto k = vec ? depth_mix_kernel<T, 4> : depth_mix_kernel<T, 1>;
+  auto k = a.w ? (vec ? depth_mix_kernel<T, 4, true> : depth_mix_kernel<T, 1, true>) : vec ? depth_mix_kernel<T, 4, false> : depth_mix_kernel<T, 1, false>;
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;

@@ -19,48 +19,44 @@ struct ShortConvArgs {
   int num_seqs, C, qw, kw, vw, taps;
 };
 
-// V values of type T as they lie in memory
+// V values of type T as they lie in memory, in 32-bit words
 template <typename T, int V> struct Pack;
 template <> struct Pack<__nv_bfloat16, 8> {
-  uint4 r;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = *reinterpret_cast<const uint4*>(p); }
-  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint4*>(p) = r; }
-  __device__ __forceinline__ void zero() { r = make_uint4(0, 0, 0, 0); }
-  __device__ __forceinline__ void get(float* f) const {
-    const float2 a = unpack_bf16x2(r.x), b = unpack_bf16x2(r.y), c = unpack_bf16x2(r.z), d = unpack_bf16x2(r.w);
-    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
-  }
-  __device__ __forceinline__ void set(const float* f) { r = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7])); }
+  static constexpr int kWords = 4;
+  uint32_t w[4];
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { const uint4 r = *reinterpret_cast<const uint4*>(p); w[0] = r.x; w[1] = r.y; w[2] = r.z; w[3] = r.w; }
+  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]); }
 };
 template <> struct Pack<float, 4> {
-  float4 r;
-  __device__ __forceinline__ void load(const float* p) { r = *reinterpret_cast<const float4*>(p); }
-  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = r; }
-  __device__ __forceinline__ void zero() { r = make_float4(0.f, 0.f, 0.f, 0.f); }
-  __device__ __forceinline__ void get(float* f) const { f[0] = r.x; f[1] = r.y; f[2] = r.z; f[3] = r.w; }
-  __device__ __forceinline__ void set(const float* f) { r = make_float4(f[0], f[1], f[2], f[3]); }
+  static constexpr int kWords = 4;
+  uint32_t w[4];
+  __device__ __forceinline__ void load(const float* p) { const uint4 r = *reinterpret_cast<const uint4*>(p); w[0] = r.x; w[1] = r.y; w[2] = r.z; w[3] = r.w; }
+  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]); }
 };
 template <> struct Pack<__nv_bfloat16, 1> {
-  __nv_bfloat16 r;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = *p; }
-  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *p = r; }
-  __device__ __forceinline__ void zero() { r = __float2bfloat16(0.f); }
-  __device__ __forceinline__ void get(float* f) const { f[0] = __bfloat162float(r); }
-  __device__ __forceinline__ void set(const float* f) { r = __float2bfloat16(f[0]); }
+  static constexpr int kWords = 1;
+  uint32_t w[1];
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { w[0] = *reinterpret_cast<const uint16_t*>(p); }
+  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint16_t*>(p) = (uint16_t)w[0]; }
 };
 template <> struct Pack<float, 1> {
-  float r;
-  __device__ __forceinline__ void load(const float* p) { r = *p; }
-  __device__ __forceinline__ void store(float* p) const { *p = r; }
-  __device__ __forceinline__ void zero() { r = 0.f; }
-  __device__ __forceinline__ void get(float* f) const { f[0] = r; }
-  __device__ __forceinline__ void set(const float* f) { r = f[0]; }
+  static constexpr int kWords = 1;
+  uint32_t w[1];
+  __device__ __forceinline__ void load(const float* p) { w[0] = *reinterpret_cast<const uint32_t*>(p); }
+  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<uint32_t*>(p) = w[0]; }
 };
+// the values of one word: a pair of bf16 (the upper one unused in a pack of one), or a float
+__device__ __forceinline__ float2 word_get(uint32_t w, const __nv_bfloat16*) { return unpack_bf16x2(w); }
+__device__ __forceinline__ float2 word_get(uint32_t w, const float*) { return make_float2(__uint_as_float(w), 0.f); }
+__device__ __forceinline__ uint32_t word_put(float2 f, const __nv_bfloat16*) { return pack_bf16x2(f.x, f.y); }
+__device__ __forceinline__ uint32_t word_put(float2 f, const float*) { return __float_as_uint(f.x); }
 
 // kTaps = 0: any number up to kMaxTaps, with the inputs read again for every tap
 template <typename T, int V, int kTaps, int kTile>
-__global__ void __launch_bounds__(128) shortconv_kernel(const ShortConvArgs a) {
+__global__ void __launch_bounds__(128, kTile == 8 ? 5 : 6) shortconv_kernel(const ShortConvArgs a) {
   const int c = (int)(blockIdx.y * 128 + threadIdx.x) * V, taps = kTaps ? kTaps : a.taps;
+  constexpr int kW = Pack<T, V>::kWords;
+  const T* kind = nullptr;           // picks the word functions
   const bool live = c < a.C;
   const T* w = reinterpret_cast<const T*>(a.w) + c;
   Pack<T, V> wv[kTaps ? kTaps : 1];
@@ -80,12 +76,13 @@ __global__ void __launch_bounds__(128) shortconv_kernel(const ShortConvArgs a) {
   // input s of the sequence, counted from the first token of this step
   auto input = [&](int s, Pack<T, V>& p) {
     if (s >= 0) p.load(u + (long long)s * a.ld);
-    else if (fresh) p.zero();
+    else if (fresh) {
+#pragma unroll
+      for (int e = 0; e < kW; e++) p.w[e] = 0;
+    }
     else p.load(win + (long long)(back + s) * a.C);
   };
-  auto put = [&](int t, const float* f) {
-    Pack<T, V> o;
-    o.set(f);
+  auto put = [&](int t, const Pack<T, V>& o) {
     const long long tok = tok0 + t;
     if (c < a.qw) { o.store(reinterpret_cast<T*>(a.q) + tok * a.qw + c); return; }
     const long long row = a.rows[tok];
@@ -97,38 +94,51 @@ __global__ void __launch_bounds__(128) shortconv_kernel(const ShortConvArgs a) {
     Pack<T, V> in[kTile + kTaps - 1];
 #pragma unroll
     for (int j = 0; j < kTile + kTaps - 1; j++)
-      if (j < n + kTaps - 1) input(r0 - (kTaps - 1) + j, in[j]);
-    float wf[kTaps][V];
+      if (j < kTaps - 1) input(r0 - (kTaps - 1) + j, in[j]);
+      else if (j < n + kTaps - 1) in[j].load(u + (long long)(r0 - (kTaps - 1) + j) * a.ld);
+      else {
 #pragma unroll
-    for (int j = 0; j < kTaps; j++) wv[j].get(wf[j]);
-#pragma unroll
-    for (int t = 0; t < kTile; t++) {
-      if (t >= n) break;
-      float y[V], f[V];
-#pragma unroll
-      for (int e = 0; e < V; e++) y[e] = 0.f;
-#pragma unroll
-      for (int j = 0; j < kTaps; j++) {
-        in[t + j].get(f);
-#pragma unroll
-        for (int e = 0; e < V; e++) y[e] = fmaf(wf[j][e], f[e], y[e]);
+        for (int e = 0; e < kW; e++) in[j].w[e] = 0;
       }
-      put(t, y);
+    // word by word, the results in place of the oldest input of each
+#pragma unroll
+    for (int e = 0; e < kW; e++) {
+      float2 f[kTaps + 1], wf[kTaps];
+#pragma unroll
+      for (int j = 0; j < kTaps; j++) { wf[j] = word_get(wv[j].w[e], kind); f[j] = word_get(in[j].w[e], kind); }
+#pragma unroll
+      for (int t = 0; t < kTile; t++) {
+        float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < kTaps; j++) { y.x = fmaf(wf[j].x, f[j].x, y.x); y.y = fmaf(wf[j].y, f[j].y, y.y); }
+        in[t].w[e] = word_put(y, kind);
+#pragma unroll
+        for (int j = 0; j + 1 < kTaps; j++) f[j] = f[j + 1];
+        if (t + 1 < kTile) f[kTaps - 1] = word_get(in[t + kTaps].w[e], kind);
+      }
     }
+#pragma unroll
+    for (int t = 0; t < kTile; t++)
+      if (t < n) put(t, in[t]);
   } else {
     for (int t = 0; t < n; t++) {
-      float y[V], f[V], g[V];
+      float2 y[kW];
 #pragma unroll
-      for (int e = 0; e < V; e++) y[e] = 0.f;
+      for (int e = 0; e < kW; e++) y[e] = make_float2(0.f, 0.f);
       for (int j = 0; j < taps; j++) {
         Pack<T, V> p, q;
         input(r0 + t - back + j, p);
         q.load(w + (long long)j * a.C);
-        p.get(f); q.get(g);
 #pragma unroll
-        for (int e = 0; e < V; e++) y[e] = fmaf(g[e], f[e], y[e]);
+        for (int e = 0; e < kW; e++) {
+          const float2 f = word_get(p.w[e], kind), g = word_get(q.w[e], kind);
+          y[e].x = fmaf(g.x, f.x, y[e].x); y[e].y = fmaf(g.y, f.y, y[e].y);
+        }
       }
-      put(t, y);
+      Pack<T, V> o;
+#pragma unroll
+      for (int e = 0; e < kW; e++) o.w[e] = word_put(y[e], kind);
+      put(t, o);
     }
   }
   if (r0 == 0)                       // the next window; a short portion keeps the end of the old one, which lies behind the row being written

@@ -804,9 +804,9 @@ def _moe_combine(y, pos, w, add_in, add_gate, x, idx, identity_from, out):
     T, H = out.shape
     if add_in is None:
         add_gate = None
-    assert add_in is None or (add_in.dtype == out.dtype and add_in.is_contiguous())
+    assert add_in is None or (add_in.dtype == out.dtype and add_in.stride(1) == 1 and add_in.shape == out.shape)
     assert add_gate is None or (add_gate.dtype == torch.float32 and add_gate.is_contiguous())
-    _ck(lib().ne_moe_combine_local(_p(y), _p(pos), _p(w), _p(add_in), _p(add_gate), _p(x), _p(idx), _c.c_int(identity_from), _p(out), _c.c_int(T),
+    _ck(lib().ne_moe_combine_local(_p(y), _p(pos), _p(w), _p(add_in), _c.c_longlong(0 if add_in is None else add_in.stride(0)), _p(add_gate), _p(x), _p(idx), _c.c_int(identity_from), _p(out), _c.c_int(T),
                                    _c.c_int(w.shape[1]), _c.c_int(H), _c.c_int(int(out.dtype == torch.float32)), _st()), "ne_moe_combine_local")
 
 

@@ -50,16 +50,16 @@ def visible(i, size, keep_first):
 
 def one_map(q, k, v, scale, size, keep_first, hide=None):
     """q [n, d], k [n, d], v [n, dv] of one head -> [n, dv].  `hide` plants a mistake: hide(i) gives the positions query i leaves out."""
-    out = torch.zeros(q.shape[0], v.shape[1], dtype=q.dtype)
+    s = torch.full((q.shape[0], q.shape[0]), float("-inf"), dtype=q.dtype)
+    scores = q @ k.T * scale
     for i in range(q.shape[0]):
         at = visible(i, size, keep_first)
         if hide is not None:
             no = hide(i)
             at = [j for j in at if j not in no or j == i]
-        s = k[at] @ q[i] * scale
-        e = torch.exp(s - s.max())
-        out[i] = (e / e.sum()) @ v[at]
-    return out
+        s[i, at] = scores[i, at]
+    e = torch.exp(s - s.max(-1, keepdim=True).values)
+    return (e / e.sum(-1, keepdim=True)) @ v
 
 
 def mixing_factor(W, diff):
