@@ -15,6 +15,7 @@ buffers, shared pool, capture per size, run).
 """
 from __future__ import annotations
 
+import contextlib
 import gc
 from typing import Dict, List
 
@@ -29,6 +30,19 @@ def make_bs_list(max_bs: int) -> List[int]:
     if max_bs not in out:
         out.append(max_bs)
     return sorted(set(out))
+
+
+@contextlib.contextmanager
+def no_cycle_collection():
+    """Around a capture: an engine that died earlier in this process would free its graphs and caches in a cycle collection, which invalidates the
+    capture."""
+    collecting = gc.isenabled()
+    gc.disable()
+    try:
+        yield
+    finally:
+        if collecting:
+            gc.enable()
 
 
 class DecodeGraphRunner:
@@ -123,16 +137,8 @@ class DecodeGraphRunner:
         torch.cuda.current_stream().wait_stream(s)
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
-        # no cycle collection inside a capture: an engine that died earlier in this process would free its graphs and caches there,
-        # which invalidates the capture
-        collecting = gc.isenabled()
-        gc.disable()
-        try:
-            with torch.cuda.graph(g, pool=self.pool):
-                out = self.r.model(ids, pos, sctx)
-        finally:
-            if collecting:
-                gc.enable()
+        with no_cycle_collection(), torch.cuda.graph(g, pool=self.pool):
+            out = self.r.model(ids, pos, sctx)
         if self.pool is None:
             self.pool = g.pool()
         self.graphs[b], self.outputs[b] = g, out

@@ -29,6 +29,7 @@ import torch
 
 from .._native import _core as C
 from .context import ForwardContext
+from .graph_runner import no_cycle_collection
 
 
 from ..ops.reference import mtp_greedy_verify as linear_greedy_verify          # noqa: E402  (the numerics live with the operators;
@@ -293,7 +294,7 @@ class MTPGraphRunner:
         torch.cuda.current_stream().wait_stream(s)
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g, pool=self.pool):
+        with no_cycle_collection(), torch.cuda.graph(g, pool=self.pool):
             out = self._step(b)
         if self.pool is None:
             self.pool = g.pool()
