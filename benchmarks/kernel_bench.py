@@ -462,8 +462,8 @@ def case_glu(T, F=12288):
 
 
 def case_mixture(T, design, W=4096, E=64, identity=0, top=8, I=1536, shared=1536):
-    """A whole mixture block with a gated shared expert, router to weighted sum: this design's or Qwen3.5's.  Bytes of the weights and the activations
-    between the steps."""
+    """A whole mixture block with a gated shared expert, router to weighted sum: this design's or Qwen3.5's.  Bytes of the weights of the experts that
+    are chosen (under even choices) and of the activations between the steps."""
     from nanoengine_b200.models.config import tiny_qwen3_5
     from nanoengine_b200.models.layers import GatedSharedMoE
     from nanoengine_b200.models.qwen3_5 import Qwen35MoE
@@ -480,7 +480,8 @@ def case_mixture(T, design, W=4096, E=64, identity=0, top=8, I=1536, shared=1536
             p.normal_(0.0, 0.02)
     x = torch.randn(T, W, device="cuda", dtype=torch.bfloat16)
     rows = T * top * E // (E + identity)
-    return run, (E * I + shared) * 3 * W * 2 + rows * (4 * W + 6 * I) + T * (4 * W + 6 * shared + 2 * W * 2), 6.0 * W * (rows * I + T * shared)
+    hit = E * (1.0 - (1.0 - top / (E + identity)) ** T)
+    return run, (hit * I + shared) * 3 * W * 2 + rows * (4 * W + 6 * I) + T * (4 * W + 6 * shared + 2 * W * 2), 6.0 * W * (rows * I + T * shared)
 
 
 def case_streams(T, S=2, W=4096):
